@@ -212,10 +212,11 @@ TQ_API int tq_sample(tq_ctx* ctx, const float* logits_dev, size_t slices, size_t
  * tokens in out_tokens[row][*step], makes them the next step's input, adds one to every position, to *step and
  * (when given) to every entry of lens_io -- the per-sequence count of past tokens that tq_sample's repetition
  * penalty reads when out_tokens is the sequences' whole history and *step starts at the prompt length.
+ * step_io = NULL: row i is stored at column lens_io[i] instead (prompts of different lengths).
  * With the decode step and tq_argmax_rows / tq_sample in front of it, one captured graph generates a token per
  * replay and no logits leave the device.  rows <= 1024. */
 TQ_API int tq_generate_advance(tq_ctx* ctx, const int* chosen_dev, size_t rows, int* tokens_io_dev, int* positions_io_dev,
-                               int* out_tokens_dev, size_t out_ld, int* step_io_dev, int* lens_io_dev_or_null);
+                               int* out_tokens_dev, size_t out_ld, int* step_io_dev_or_null, int* lens_io_dev_or_null);
 
 /* ---- attention -------------------------------------------------------------------------------
  * ComputeDevice::kv_attention (device.rs:161-180; cpu.rs:257-315) on f32 buffers, exactly the
@@ -429,6 +430,94 @@ TQ_API int tq_mla_create(tq_ctx* ctx, const tq_mla_config* cfg, const tq_qweight
 TQ_API int tq_mla_destroy(tq_mla* layer);
 TQ_API int tq_mla_layer_decode(tq_mla* layer, const void* h_bf16_dev, const void* cache_bf16_dev, const int* lens_dev, size_t batch,
                                size_t seq_stride, size_t max_len, tq_comm* comm_or_null, float* out_dev);
+
+/* ---- dense (unquantised) linear layers ---------------------------------------------------------
+ * y[m, rows] = x[m, cols] . W^T with W in bf16 (tensor cores, f32 accumulation: a GEMV kernel up to 8 rows, tcgen05
+ * above) or in f32 (x and every operation f32, no reduced-precision mode); Linear::forward_2d,
+ * crates/tang-compute/src/modules.rs:56-70, on an unquantised weight.  A handle owns its storage, zero when created;
+ * tq_dweight_put copies a [rows, cols] block (bf16 or f32, host or device memory) to (row0, col0), so that several
+ * projections of one input can share a handle.  interleave = 1 / 2 places the rows as the gate / up halves of 16-row
+ * blocks (eight gate rows, then the eight up rows of the same outputs). */
+typedef struct tq_dweight tq_dweight;
+TQ_API int tq_dweight_create(tq_ctx* ctx, size_t rows, size_t cols, int dtype, tq_dweight** out);
+TQ_API int tq_dweight_put(tq_ctx* ctx, tq_dweight* w, const void* src, int src_dtype, size_t rows, size_t cols, size_t row0,
+                          size_t col0, int interleave);
+TQ_API int tq_dweight_free(tq_ctx* ctx, tq_dweight* w);
+/* The stored matrix: [rows_padded][cols_padded] of the handle's dtype. */
+TQ_API int tq_dweight_data(const tq_dweight* w, void** dev, size_t* rows_padded, size_t* cols_padded);
+/* x has the weight's dtype, 16-byte aligned rows for bf16; y f32 or bf16; ldx / ldy row strides (0 = dense). */
+TQ_API int tq_dlinear(tq_ctx* ctx, const tq_dweight* w, const void* x_dev, size_t ldx, size_t m, void* y_dev, int y_dtype, size_t ldy);
+/* out = g * sigmoid(alpha g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit); no reference counterpart. */
+TQ_API int tq_clamped_glu(tq_ctx* ctx, const void* gate_dev, const void* up_dev, int in_dtype, size_t n, float limit, float alpha,
+                          void* out_dev, int out_dtype);
+
+/* ---- steps over ragged batches ------------------------------------------------------------------
+ * No reference counterpart.  A step's rows are the next tokens of n_seqs sequences, packed: sequence b's are rows
+ * seq_rows[b] .. seq_rows[b+1]-1 (seq_rows = NULL: row b), its first one sits at position starts[b], and its cache is
+ * slot slots[b] (NULL: b) of max_seq rows.  tq_embedding_pos forms out[m, :] = table[id] + pos_table[position] (f32)
+ * and leaves each row's position and cache row (slot * max_seq + position; -1 outside the cache, which tq_sync reports). */
+TQ_API int tq_embedding_pos(tq_ctx* ctx, const void* table_dev, const void* pos_table_dev, int dtype, const int* ids_dev,
+                            const int* seq_rows_dev_or_null, const int* starts_dev, const int* slots_dev_or_null, size_t n_seqs,
+                            size_t rows, size_t dim, size_t vocab, size_t n_pos, size_t max_seq, size_t n_slots, float* out_dev,
+                            int* row_pos_dev, int* cache_row_dev);
+/* Differential attention: two softmax maps per head over the same values, o = a1 - lambda a2, then
+ * o / sqrt(mean(o^2) + eps) * out_scale over the head's vdim values.  The query at position i sees key j when j <= i and
+ * (i - j < window or j < keep_first).  q [rows][ldq]: head h's map m at column (2h + m) * dim.  Caches: key row
+ * [kv_heads][2][dim rounded up to 8], value row [kv_heads][vdim rounded up to 8], padding zero; the step's own rows are
+ * in them already.  out [rows][ldo], head h at column h * vdim.  dtype (TQ_BF16 or TQ_F32) is that of all four.  max_q
+ * bounds the rows a sequence brings, max_len every position + 1.  bf16: f32 scores and weights, weights into the tensor
+ * core as two bf16 terms. */
+typedef struct tq_diff_attn_config {
+  uint32_t heads, kv_heads, dim, vdim;
+  uint32_t window, keep_first;
+  float scale, lambda, out_scale, eps;
+} tq_diff_attn_config;
+TQ_API int tq_diff_attention(tq_ctx* ctx, const tq_diff_attn_config* cfg, int dtype, const void* q_dev, size_t ldq, const void* k_cache_dev,
+                             const void* v_cache_dev, size_t cache_rows, const int* seq_rows_dev_or_null, const int* row_pos_dev,
+                             const int* cache_row_dev, size_t n_seqs, size_t rows, size_t max_q, size_t max_len, void* out_dev,
+                             size_t ldo);
+
+/* ---- Tofazen ------------------------------------------------------------------------------------
+ * No reference counterpart.  A decoder with learned absolute positions and parallel layers,
+ *   h = rms_norm(x);  x <- x + residual_mult * (W_o attention(h) + W_down glu(W_gate h, W_up h)),
+ * with the differential attention above, layers that read an earlier layer's keys and values (kv_from) and the clamped
+ * GLU (sigmoid factor 1.702).  The model owns weights, caches (one per layer with keys of its own, [max_slots][max_seq])
+ * and workspaces.  dtype TQ_BF16: bf16 weights, activations and caches, f32 stream, norms and scores; TQ_F32: everything f32. */
+typedef struct tq_tofazen tq_tofazen;
+typedef struct tq_tofazen_config {
+  uint32_t n_layers, width, vocab;
+  uint32_t max_positions;  /* rows of the position table */
+  uint32_t max_seq;        /* cache rows per slot (<= max_positions) */
+  uint32_t max_slots;
+  int dtype;
+  float eps, residual_mult;
+} tq_tofazen_config;
+typedef struct tq_tofazen_layer {
+  uint32_t heads, kv_heads, dim, vdim;
+  uint32_t ff;             /* 0: no feed-forward */
+  int kv_from;             /* -1: keys and values of its own */
+  uint32_t window, keep_first;
+  float scale, lambda, out_scale, limit;
+} tq_tofazen_layer;
+typedef enum tq_tofazen_tensor {
+  TQ_TZ_EMBED = 0, TQ_TZ_POS = 1, TQ_TZ_FINAL_NORM = 2, TQ_TZ_HEAD = 3,
+  TQ_TZ_NORM = 4, TQ_TZ_Q = 5, TQ_TZ_K = 6, TQ_TZ_V = 7, TQ_TZ_O = 8, TQ_TZ_GATE = 9, TQ_TZ_UP = 10, TQ_TZ_DOWN = 11
+} tq_tofazen_tensor;
+TQ_API int tq_tofazen_create(tq_ctx* ctx, const tq_tofazen_config* cfg, const tq_tofazen_layer* layers, tq_tofazen** out);
+TQ_API int tq_tofazen_destroy(tq_tofazen* model);
+/* Copies one tensor (row-major [rows, cols], bf16 or f32, host or device memory; a vector is [1, n]) into the model. */
+TQ_API int tq_tofazen_put(tq_tofazen* model, int tensor, size_t layer, const void* src, int src_dtype, size_t rows, size_t cols);
+/* One step over a ragged batch (see tq_embedding_pos): appends the rows' keys and values, attends, and writes f32 logits
+ * [n_logits, vocab] of the rows listed in logit_rows (NULL: every row, n_logits = rows); n_logits = 0 skips the head.
+ * Decoding (one row per sequence) and prompt portions of any size are the same call.  Asynchronous; capturable once run
+ * eagerly with the same sizes. */
+TQ_API int tq_tofazen_step(tq_tofazen* model, const int* token_ids_dev, size_t rows, const int* seq_rows_dev_or_null, const int* starts_dev,
+                           const int* slots_dev_or_null, size_t n_seqs, size_t max_q, size_t max_len, const int* logit_rows_dev_or_null,
+                           size_t n_logits, float* logits_dev);
+/* The f32 stream [rows, width] after the last step's layers. */
+TQ_API int tq_tofazen_hidden(tq_tofazen* model, float** hidden_dev);
+/* While set, every step also copies the stream after each layer to streams [n_layers][rows][width] (NULL turns it off). */
+TQ_API int tq_tofazen_trace(tq_tofazen* model, float* streams_dev_or_null);
 
 /* ---- CUDA graphs ------------------------------------------------------------------------------
  * CudaComputeDevice::begin_capture / end_capture (crates/tang-compute/src/cuda.rs:344-356): every

@@ -98,6 +98,20 @@ PROTOTYPES = {
     "tq_mla_create": (_i, [_p, _p, _p, _p, _p, _p, _p, _p, _p, _p, _pp]),
     "tq_mla_destroy": (_i, [_p]),
     "tq_mla_layer_decode": (_i, [_p, _p, _p, _p, _sz, _sz, _sz, _p, _p]),
+    "tq_dweight_create": (_i, [_p, _sz, _sz, _i, _pp]),
+    "tq_dweight_put": (_i, [_p, _p, _p, _i, _sz, _sz, _sz, _sz, _i]),
+    "tq_dweight_free": (_i, [_p, _p]),
+    "tq_dweight_data": (_i, [_p, _pp, C.POINTER(_sz), C.POINTER(_sz)]),
+    "tq_dlinear": (_i, [_p, _p, _p, _sz, _sz, _p, _i, _sz]),
+    "tq_clamped_glu": (_i, [_p, _p, _p, _i, _sz, C.c_float, C.c_float, _p, _i]),
+    "tq_embedding_pos": (_i, [_p, _p, _p, _i, _p, _p, _p, _p, _sz, _sz, _sz, _sz, _sz, _sz, _sz, _p, _p, _p]),
+    "tq_diff_attention": (_i, [_p, _p, _i, _p, _sz, _p, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _sz, _p, _sz]),
+    "tq_tofazen_create": (_i, [_p, _p, _p, _pp]),
+    "tq_tofazen_destroy": (_i, [_p]),
+    "tq_tofazen_put": (_i, [_p, _i, _sz, _p, _i, _sz, _sz]),
+    "tq_tofazen_step": (_i, [_p, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _p, _sz, _p]),
+    "tq_tofazen_hidden": (_i, [_p, _pp]),
+    "tq_tofazen_trace": (_i, [_p, _p]),
     "tq_graph_begin": (_i, [_p]),
     "tq_graph_end": (_i, [_p, _pp]),
     "tq_graph_launch": (_i, [_p, _p]),
@@ -108,16 +122,21 @@ PROTOTYPES = {
 _lib = None
 
 
-def load() -> C.CDLL:
-    """Loads the shared library and binds every prototype.  Raises if it has not been built."""
+def load(path: str | None = None) -> C.CDLL:
+    """Loads the shared library and binds every prototype.  Raises if it has not been built.  `path` names a partial
+    library (``_build.ensure``); entry points it does not have stay unbound and fail when they are called."""
     global _lib
     if _lib is None:
-        if not os.path.exists(LIB_PATH):
+        full = path is None or os.path.abspath(path) == LIB_PATH
+        path = path or LIB_PATH
+        if not os.path.exists(path):
             raise TangqError(TQ_EUNSUPPORTED,
-                             f"{LIB_PATH} is missing; build it with `python -m tang_b200._build` (needs nvcc). "
+                             f"{path} is missing; build it with `python -m tang_b200._build` (needs nvcc). "
                              "There is no CPU fallback.")
-        lib = C.CDLL(LIB_PATH)
+        lib = C.CDLL(path)
         for name, (res, args) in PROTOTYPES.items():
+            if not full and not hasattr(lib, name):
+                continue
             fn = getattr(lib, name)
             fn.restype, fn.argtypes = res, args
         _lib = lib

@@ -1,0 +1,791 @@
+// Dense linear layers (see dense.cuh): GEMV for few rows, tcgen05 GEMM for many, f32 GEMM, weight handles and the
+// C entry points tq_dweight_* / tq_dlinear / tq_clamped_glu.
+#include "dense.cuh"
+
+#include <cstring>
+#include <new>
+#include <vector>
+
+#include "qgemm_umma.cuh"
+#include "tensormap.h"
+
+namespace tq {
+
+// ------------------------------------------------------------------------------------------------ GEMV, 1..8 rows
+constexpr int kGvWarps = 8;
+constexpr int kGvThreads = 32 * kGvWarps;
+constexpr int kGvPad = 128;         // weight rows are padded to this many columns
+
+struct GemvParams {
+  const __nv_bfloat16* w;
+  int kpad, n_rb;                   // n_rb: 16-row blocks
+  const __nv_bfloat16* x;
+  long long ldx;
+  int m, cols;
+  const float* h;                   // RMSNorm prologue (x is null then)
+  long long ldh;
+  const int* h_rows;
+  const __nv_bfloat16* gain;
+  float eps;
+  DenseEpilogue epi;
+};
+
+// 32 bytes of a weight row: read once, not kept in L1, first to leave L2.
+struct Frag32 {
+  uint32_t v[8];
+};
+__device__ __forceinline__ Frag32 ldg_stream(const void* p) {
+  Frag32 f;
+  asm volatile("ld.global.nc.L1::no_allocate.L2::evict_first.v8.b32 {%0,%1,%2,%3,%4,%5,%6,%7}, [%8];"
+               : "=r"(f.v[0]), "=r"(f.v[1]), "=r"(f.v[2]), "=r"(f.v[3]), "=r"(f.v[4]), "=r"(f.v[5]), "=r"(f.v[6]), "=r"(f.v[7])
+               : "l"(p));
+  return f;
+}
+
+// The first n (at most 8) of eight bf16 values, zeros behind them.
+__device__ __forceinline__ uint4 x_tail(const void* src, int n) {
+  const uint16_t* e = static_cast<const uint16_t*>(src);
+  uint32_t w[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) w[j] = (2 * j < n ? (uint32_t)e[2 * j] : 0u) | (2 * j + 1 < n ? (uint32_t)e[2 * j + 1] << 16 : 0u);
+  return make_uint4(w[0], w[1], w[2], w[3]);
+}
+
+// A CTA walks groups of RB 16-row blocks (grid-stride); its eight warps take the k chunks of a group in turn and meet
+// in shared memory.  Lane 4g + t holds bytes 32t .. 32t + 31 of rows g and g + 8 of every 64-k step (a row's four lanes
+// read one 128-byte line): words 2i, 2i + 1 are the two k halves of MMA i; the activations are read the same way.  The loads of
+// the next step -- of the next group too -- are issued before the current step is multiplied, and the first ones before
+// the kernel waits for its predecessor (weights do not change).  XS: activations in shared memory, else from global.
+template <int RB, bool XS>
+__global__ void __launch_bounds__(kGvThreads, 2) dgemv_kernel(const __grid_constant__ GemvParams p) {
+  extern __shared__ __align__(16) uint8_t gv_smem[];
+  __shared__ float red[2][kGvWarps][RB][128];
+  __shared__ float ssq[kGvWarps];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const int n_groups = (p.n_rb + RB - 1) / RB;
+  constexpr int U = RB == 1 ? 2 : 1;                 // 64-k loads per row and step: about 32 registers in flight
+  constexpr int kGvChunk = 64 * U;                   // k per warp step
+  const int n_ch = p.kpad / kGvChunk;
+  const size_t row_bytes = (size_t)p.kpad * 2;
+  const uint8_t* wb = reinterpret_cast<const uint8_t*>(p.w);
+
+  Frag32 nxt[RB][U][2];
+  auto load = [&](int grp, int c) {
+#pragma unroll
+    for (int r = 0; r < RB; ++r) {
+      const int rb = min(grp * RB + r, p.n_rb - 1);
+      const uint8_t* src = wb + (size_t)(rb * 16 + g) * row_bytes + (size_t)c * (kGvChunk * 2) + 32 * t;
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        nxt[r][u][0] = ldg_stream(src + 128 * u);
+        nxt[r][u][1] = ldg_stream(src + 8 * row_bytes + 128 * u);
+      }
+    }
+  };
+  int grp = blockIdx.x;
+  const bool any = warp < n_ch;
+  if (grp < n_groups && any) load(grp, warp);
+
+  pdl_wait();
+  pdl_launch_dependents();
+
+  const size_t xs_stride = row_bytes + 16;   // bytes; 16 mod 32: two rows' reads, 32 bytes apart, do not meet in a bank
+  if constexpr (XS) {
+    if (p.h) {
+      int wpr = kGvWarps;                        // warps per row
+      while (wpr * p.m > kGvWarps) wpr >>= 1;
+      const int row = warp / wpr, part = warp % wpr;
+      const bool mine = row < p.m;
+      const float* src = p.h + (size_t)(mine ? (p.h_rows ? p.h_rows[row] : row) : 0) * p.ldh;
+      const bool vec = (p.cols & 3) == 0 && (p.ldh & 3) == 0;
+      float sq = 0.f;
+      if (mine) {
+        if (vec) {
+#pragma unroll 4
+          for (int d = 4 * (part * 32 + lane); d < p.cols; d += 128 * wpr) {
+            const float4 v = *reinterpret_cast<const float4*>(src + d);
+            sq += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+          }
+        } else {
+          for (int d = part * 32 + lane; d < p.cols; d += 32 * wpr) sq += src[d] * src[d];
+        }
+      }
+      sq = warp_sum(sq);
+      if (lane == 0) ssq[warp] = sq;
+      __syncthreads();
+      if (mine) {
+        float tot = 0.f;
+        for (int i = 0; i < wpr; ++i) tot += ssq[row * wpr + i];
+        const float inv = 1.0f / sqrtf(tot / (float)p.cols + p.eps);
+        __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(gv_smem + row * xs_stride);
+        if (vec) {
+#pragma unroll 4
+          for (int d = 4 * (part * 32 + lane); d < p.cols; d += 128 * wpr) {
+            const float4 v = *reinterpret_cast<const float4*>(src + d);
+            const uint2 gr = *reinterpret_cast<const uint2*>(p.gain + d);
+            const __nv_bfloat162 a = __floats2bfloat162_rn(v.x * inv * bf16_bits_to_float(gr.x & 0xFFFFu), v.y * inv * bf16_bits_to_float(gr.x >> 16));
+            const __nv_bfloat162 b = __floats2bfloat162_rn(v.z * inv * bf16_bits_to_float(gr.y & 0xFFFFu), v.w * inv * bf16_bits_to_float(gr.y >> 16));
+            *reinterpret_cast<uint2*>(dst + d) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+          }
+        } else {
+          for (int d = part * 32 + lane; d < p.cols; d += 32 * wpr) dst[d] = __float2bfloat16_rn(src[d] * inv * __bfloat162float(p.gain[d]));
+        }
+        for (int d = p.cols + part * 32 + lane; d < p.kpad; d += 32 * wpr) dst[d] = __float2bfloat16_rn(0.f);
+      }
+    } else {
+      const int vpr = p.kpad / 8;
+      for (int i = threadIdx.x; i < p.m * vpr; i += kGvThreads) {
+        const int row = i / vpr, c = i % vpr;
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        const __nv_bfloat16* src = p.x + (size_t)row * p.ldx + 8 * c;
+        if (8 * c + 8 <= p.cols) v = *reinterpret_cast<const uint4*>(src);
+        else if (8 * c < p.cols) v = x_tail(src, p.cols - 8 * c);
+        *reinterpret_cast<uint4*>(gv_smem + row * xs_stride + 16 * c) = v;
+      }
+    }
+    __syncthreads();
+  }
+  const bool live = g < p.m;
+  const uint8_t* xrow = XS ? gv_smem + (live ? g : 0) * xs_stride + 32 * t
+                           : reinterpret_cast<const uint8_t*>(p.x + (size_t)(live ? g : 0) * p.ldx) + 32 * t;
+
+  int buf = 0;
+  for (; grp < n_groups; grp += gridDim.x) {
+    float acc[RB][4];
+#pragma unroll
+    for (int r = 0; r < RB; ++r) acc[r][0] = acc[r][1] = acc[r][2] = acc[r][3] = 0.f;
+    for (int c = warp; c < n_ch; c += kGvWarps) {
+      Frag32 cur[RB][U][2];
+#pragma unroll
+      for (int r = 0; r < RB; ++r)
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          cur[r][u][0] = nxt[r][u][0];
+          cur[r][u][1] = nxt[r][u][1];
+        }
+      const bool more = c + kGvWarps < n_ch;
+      if (more || grp + (int)gridDim.x < n_groups) load(more ? grp : grp + gridDim.x, more ? c + kGvWarps : warp);
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        uint4 xa = make_uint4(0u, 0u, 0u, 0u), xb = xa;
+        if (live) {
+          const int k = c * kGvChunk + 64 * u + 16 * t;       // (shared memory is padded with zeros, global memory is not)
+          const uint8_t* xp = xrow + (size_t)c * (kGvChunk * 2) + 128 * u;
+          if (XS || k + 16 <= p.cols) {
+            xa = *reinterpret_cast<const uint4*>(xp);
+            xb = *reinterpret_cast<const uint4*>(xp + 16);
+          } else if (k < p.cols) {
+            xa = x_tail(xp, p.cols - k);
+            if (k + 8 < p.cols) xb = x_tail(xp + 16, p.cols - k - 8);
+          }
+        }
+        const uint32_t xw[8] = {xa.x, xa.y, xa.z, xa.w, xb.x, xb.y, xb.z, xb.w};
+#pragma unroll
+        for (int r = 0; r < RB; ++r)
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            mma_bf16_16816(acc[r], cur[r][u][0].v[2 * i], cur[r][u][1].v[2 * i], cur[r][u][0].v[2 * i + 1], cur[r][u][1].v[2 * i + 1],
+                           xw[2 * i], xw[2 * i + 1]);
+      }
+    }
+    // rows g, g + 8 x activation rows 2t, 2t + 1
+#pragma unroll
+    for (int r = 0; r < RB; ++r) {
+      float* d = red[buf][warp][r];
+      d[g * 8 + 2 * t] = acc[r][0];
+      d[g * 8 + 2 * t + 1] = acc[r][1];
+      d[(g + 8) * 8 + 2 * t] = acc[r][2];
+      d[(g + 8) * 8 + 2 * t + 1] = acc[r][3];
+    }
+    __syncthreads();
+    if (threadIdx.x < RB * 128) {
+      const int r = threadIdx.x >> 7, row = (threadIdx.x >> 3) & 15, m = threadIdx.x & 7;
+      const int rb = grp * RB + r;
+      if (rb < p.n_rb && m < p.m) {
+        const DenseDst d = dense_dst(p.epi, rb * 16 + row);
+        if (d.kind != DENSE_GLU || row < 8) {
+          float v = 0.f;
+#pragma unroll
+          for (int w = 0; w < kGvWarps; ++w) v += red[buf][w][r][row * 8 + m];
+          if (d.kind == DENSE_GLU) {
+            float up = 0.f;
+#pragma unroll
+            for (int w = 0; w < kGvWarps; ++w) up += red[buf][w][r][(row + 8) * 8 + m];
+            v = clamped_glu(v, up, p.epi.glu_limit, p.epi.glu_alpha);
+          }
+          dense_store(p.epi, d, m, v);
+        }
+      }
+    }
+    buf ^= 1;
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ tcgen05 GEMM
+// The weights are the UMMA M operand (128 features per tile), the activation rows the N operand (16..256), both K-major
+// in the 128-byte swizzle; D[128 x rows] in tensor memory.  Warp 0 copies, warp 1 multiplies, warps 4..11 store.
+constexpr int kDuThreads = 384;
+constexpr int kDuEpiWarp0 = 4, kDuEpiWarps = 8;
+constexpr int kDuMaxStages = 12;
+constexpr int kDuHeader = 1024;
+
+struct DUmmaParams {
+  int m, ntok, stages;
+  int n_ft, n_tt, splits, n_tiles;   // feature tiles, row tiles, K splits; n_tiles = product
+  int kb_total, kb_per_split;        // 64-k steps
+  int n_acc, acc_stride, tmem_cols;
+  float* partial;                    // [splits][m][n_ft * 128], splits > 1
+  int* counters;                     // one per (feature tile, row tile), zero between launches
+  DenseEpilogue epi;
+  int* err;
+};
+
+__global__ void __launch_bounds__(kDuThreads, 1)
+dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_constant__ CUtensorMap x_map, const __grid_constant__ DUmmaParams p) {
+  extern __shared__ uint8_t du_smem[];
+  uint64_t* full = reinterpret_cast<uint64_t*>(du_smem);
+  uint64_t* empty = full + kDuMaxStages;
+  uint64_t* acc_full = empty + kDuMaxStages;
+  uint64_t* acc_empty = acc_full + 2;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(acc_empty + 2);
+  volatile int* failed = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  volatile int* last_flag = failed + 1;
+  const uint32_t base_u32 = smem_u32(du_smem);
+  uint8_t* tiles_s = du_smem + kDuHeader + ((1024 - ((base_u32 + kDuHeader) & 1023)) & 1023);
+  const uint32_t stage_bytes = (uint32_t)(kUmmaRows + p.ntok) * 128u;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int S = p.stages;
+
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < S; ++s) {
+      mbar_init(&full[s], 1);
+      mbar_init(&empty[s], 1);
+    }
+    for (int a = 0; a < 2; ++a) {
+      mbar_init(&acc_full[a], 1);
+      mbar_init(&acc_empty[a], kDuEpiWarps);
+    }
+    *failed = 0;
+    mbar_init_fence();
+  }
+  if (warp == 2) tmem_alloc(tmem_slot, (uint32_t)p.tmem_cols);
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_d = *tmem_slot;
+
+  auto give_up = [&](int code) {
+    *failed = 1;
+    atomicCAS(p.err, 0, code);
+  };
+  // tile -> (feature tile, row tile, K split): splits fastest, then row tiles, so that the CTAs of a wave share weights
+  auto coords = [&](int tile, int& ft, int& tt, int& kb0, int& kbn, int& z) {
+    z = tile % p.splits;
+    const int q = tile / p.splits;
+    tt = q % p.n_tt;
+    ft = q / p.n_tt;
+    kb0 = z * p.kb_per_split;
+    kbn = min(p.kb_per_split, p.kb_total - kb0);
+  };
+
+  if (warp == 0) {
+    if (lane == 0) {
+      // The weights of the first stages do not depend on the previous kernel: their copies start before the wait.
+      int ft, tt, kb0, kbn, z;
+      int pre = 0;
+      if ((int)blockIdx.x < p.n_tiles) {
+        coords(blockIdx.x, ft, tt, kb0, kbn, z);
+        pre = min(S, kbn);
+        for (int s = 0; s < pre; ++s) {
+          mbar_arrive_expect_tx(&full[s], stage_bytes);
+          tma_load_2d(tiles_s + (size_t)s * stage_bytes, &w_map, (kb0 + s) * kUmmaK, ft * kUmmaRows, &full[s]);
+        }
+      }
+      pdl_wait();
+      int s = 0;
+      uint32_t ph = 0;
+      bool ok = true;
+      for (int tile = blockIdx.x; tile < p.n_tiles && ok; tile += gridDim.x) {
+        coords(tile, ft, tt, kb0, kbn, z);
+        for (int kb = 0; kb < kbn; ++kb) {
+          uint8_t* st = tiles_s + (size_t)s * stage_bytes;
+          if (pre > 0) {
+            --pre;
+          } else {
+            ok = !*failed && mbar_wait_spin(&empty[s], ph ^ 1u);
+            if (!ok) { give_up(DERR_EMPTY_WAIT); break; }
+            mbar_arrive_expect_tx(&full[s], stage_bytes);
+            tma_load_2d(st, &w_map, (kb0 + kb) * kUmmaK, ft * kUmmaRows, &full[s]);
+          }
+          tma_load_2d(st + kUmmaRows * 128, &x_map, (kb0 + kb) * kUmmaK, tt * p.ntok, &full[s]);
+          if (++s == S) {
+            s = 0;
+            ph ^= 1u;
+          }
+        }
+      }
+    }
+    __syncwarp();
+  } else if (warp == 1) {
+    const bool leader = elect_one();
+    const uint32_t idesc = umma_idesc_bf16(p.ntok);
+    const uint64_t desc0 = umma_desc_sw128(tiles_s);
+    const uint32_t stage_u = stage_bytes >> 4, b_off = (uint32_t)(kUmmaRows * 128) >> 4;
+    int s = 0, a = 0;
+    uint32_t ph = 0, aph = 0;
+    bool ok = true;
+    for (int tile = blockIdx.x; tile < p.n_tiles && ok; tile += gridDim.x) {
+      int ft, tt, kb0, kbn, z;
+      coords(tile, ft, tt, kb0, kbn, z);
+      ok = !*failed && mbar_wait_spin(&acc_empty[a], aph ^ 1u);
+      if (!ok) { give_up(DERR_TMEM); break; }
+      tc_fence_after();
+      const uint32_t acc = tmem_d + (uint32_t)(a * p.acc_stride);
+      for (int kb = 0; kb < kbn; ++kb) {
+        ok = !*failed && mbar_wait_spin(&full[s], ph);
+        if (!ok) { give_up(DERR_FULL_WAIT); break; }
+        tc_fence_after();
+        if (leader) {
+          const uint64_t ad = desc0 + (uint64_t)((uint32_t)s * stage_u);
+#pragma unroll
+          for (int k16 = 0; k16 < kUmmaK / 16; ++k16) umma_f16(acc, ad + 2 * k16, ad + b_off + 2 * k16, idesc, (kb | k16) != 0);
+          umma_commit(&empty[s]);
+        }
+        __syncwarp();
+        if (++s == S) {
+          s = 0;
+          ph ^= 1u;
+        }
+      }
+      if (!ok) break;
+      if (leader) umma_commit(&acc_full[a]);
+      __syncwarp();
+      if (++a == p.n_acc) {
+        a = 0;
+        aph ^= 1u;
+      }
+    }
+  } else if (warp >= kDuEpiWarp0) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int q = warp & 3, half = (warp - kDuEpiWarp0) >> 2;
+    const int et = threadIdx.x - 32 * kDuEpiWarp0;     // 0..255
+    int a = 0;
+    uint32_t aph = 0;
+    const int n_pad = p.n_ft * kUmmaRows;
+    for (int tile = blockIdx.x; tile < p.n_tiles; tile += gridDim.x) {
+      int ft, tt, kb0, kbn, z;
+      coords(tile, ft, tt, kb0, kbn, z);
+      // (after a failure every warp still walks all tiles, without touching memory: the named barriers below stay matched)
+      const bool good = __all_sync(0xffffffffu, !*failed && mbar_wait_spin(&acc_full[a], aph));
+      if (!good) give_up(DERR_TMEM);
+      tc_fence_after();
+      const int row = ft * kUmmaRows + 32 * q + lane;
+      const int m0 = tt * p.ntok, m_n = good ? min(p.ntok, p.m - m0) : 0;
+      const uint32_t t_addr = tmem_d + (uint32_t)(a * p.acc_stride) + ((uint32_t)(32 * q) << 16);
+      const DenseDst dst = dense_dst(p.epi, row);
+      for (int c0 = 16 * half; c0 < m_n; c0 += 32) {
+        float v[16];
+        tmem_ld16(t_addr + (uint32_t)c0, v);
+        const int n = min(16, m_n - c0), mb = m0 + c0;
+        if (p.splits > 1) {
+          float* pp = p.partial + ((size_t)z * p.m + mb) * n_pad + row;
+#pragma unroll
+          for (int j = 0; j < 16; ++j)
+            if (j < n) __stcg(pp + (size_t)j * n_pad, v[j]);
+          continue;
+        }
+        // a half-warp's rows share a section, so the shuffles below are only ever needed by lanes that agree on the kind
+        const bool glu = dst.kind == DENSE_GLU;
+        if (__any_sync(0xffffffffu, glu)) {
+          // lanes with (row & 8) == 0 hold gates, the others the matching ups: of every two columns the gate lanes
+          // finish the first and the up lanes the second
+          const bool upper = lane & 8;
+#pragma unroll
+          for (int j = 0; j < 16; j += 2) {
+            const float give = upper ? v[j] : v[j + 1];
+            const float got = __shfl_xor_sync(0xffffffffu, give, 8);
+            if (glu) {
+              const float val = upper ? clamped_glu(got, v[j + 1], p.epi.glu_limit, p.epi.glu_alpha)
+                                      : clamped_glu(v[j], got, p.epi.glu_limit, p.epi.glu_alpha);
+              const int jj = upper ? j + 1 : j;
+              if (jj < n) dense_store(p.epi, dst, mb + jj, val);
+            }
+          }
+          if (glu) continue;
+        }
+        if (dst.kind == DENSE_RESID) {
+          if (dst.base) {
+            float old[16];
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              if (j < n) old[j] = *reinterpret_cast<const float*>(dst.base + (long long)(mb + j) * dst.ld);
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              if (j < n) *reinterpret_cast<float*>(dst.base + (long long)(mb + j) * dst.ld) = old[j] + p.epi.mult * v[j];
+          }
+        } else {
+#pragma unroll
+          for (int j = 0; j < 16; ++j)
+            if (j < n) dense_store(p.epi, dst, mb + j, v[j]);
+        }
+      }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&acc_empty[a]);
+      if (++a == p.n_acc) {
+        a = 0;
+        aph ^= 1u;
+      }
+      if (p.splits > 1) {
+        // the CTA that counts in last adds the tile's partials in split order (the same bits whichever CTA that is)
+        __threadfence();
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        if (et == 0) {
+          int* c = p.counters + ft * p.n_tt + tt;
+          const int seen = atomicAdd(c, 1);
+          *last_flag = seen == p.splits - 1;
+          if (seen == p.splits - 1) *c = 0;
+          __threadfence();
+        }
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        if (*last_flag) {
+          __threadfence();
+          const size_t plane = (size_t)p.m * n_pad;
+          // warp (q, half): features 32q.., every other pair of rows
+          const bool upper = lane & 8;
+          for (int c0 = 4 * half; c0 < m_n; c0 += 8) {
+            float v[4] = {0.f, 0.f, 0.f, 0.f};
+            const int n = min(4, m_n - c0), mb = m0 + c0;
+            const float* src = p.partial + (size_t)mb * n_pad + row;
+            for (int zz = 0; zz < p.splits; ++zz) {
+#pragma unroll
+              for (int j = 0; j < 4; ++j)
+                if (j < n) v[j] += __ldcg(src + (size_t)zz * plane + (size_t)j * n_pad);
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+              const float other = __shfl_xor_sync(0xffffffffu, v[j], 8);
+              if (j >= n) continue;
+              if (dst.kind == DENSE_GLU) {
+                if (!upper) dense_store(p.epi, dst, mb + j, clamped_glu(v[j], other, p.epi.glu_limit, p.epi.glu_alpha));
+              } else {
+                dense_store(p.epi, dst, mb + j, v[j]);
+              }
+            }
+          }
+        }
+        asm volatile("bar.sync 1, 256;" ::: "memory");     // last_flag is read before the next tile rewrites it
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (*failed && threadIdx.x == 0) {
+    // copies and products that are still in flight target this CTA's memories: give them time to land before leaving
+    for (int i = 0; i < 10000; ++i) __nanosleep(1000);
+  }
+  __syncthreads();
+  if (warp == 2) tmem_dealloc(tmem_d, (uint32_t)p.tmem_cols);
+}
+
+// ------------------------------------------------------------------------------------------------ f32 GEMM
+// 64 activation rows x 64 features per CTA, 16 k per step; every operation is an f32 FMA in ascending k.
+constexpr int kDfTile = 64, kDfK = 16;
+
+__global__ void __launch_bounds__(256) dgemm_f32_kernel(const float* w, int kpad, int rpad, const float* x, long long ldx, int m, int cols,
+                                                        const __grid_constant__ DenseEpilogue epi) {
+  __shared__ __align__(16) float xs[kDfK][kDfTile + 4], ws[kDfK][kDfTile + 4];
+  __shared__ float ys[kDfTile][kDfTile + 1];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int n0 = blockIdx.x * kDfTile, m0 = blockIdx.y * kDfTile;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;      // features 4 tx.., rows 4 ty..
+  const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4; // this thread's share of the loads
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < cols; k0 += kDfK) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int k = k0 + lk + i;
+      xs[lk + i][lr] = m0 + lr < m && k < cols ? x[(size_t)(m0 + lr) * ldx + k] : 0.f;
+      ws[lk + i][lr] = n0 + lr < rpad && k < cols ? w[(size_t)(n0 + lr) * kpad + k] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kDfK; ++k) {
+      const float4 a = *reinterpret_cast<const float4*>(&xs[k][4 * ty]), b = *reinterpret_cast<const float4*>(&ws[k][4 * tx]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) ys[4 * ty + i][4 * tx + j] = acc[i][j];
+  __syncthreads();
+  const int n = threadIdx.x & 63;
+  const DenseDst d = dense_dst(epi, n0 + n);
+  if (d.kind == DENSE_GLU && (n & 8)) return;
+  for (int r = threadIdx.x >> 6; r < kDfTile && m0 + r < m; r += 4) {
+    float v = ys[r][n];
+    if (d.kind == DENSE_GLU) v = clamped_glu(v, ys[r][n + 8], epi.glu_limit, epi.glu_alpha);
+    dense_store(epi, d, m0 + r, v);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ launches
+constexpr size_t kGvSmemMax = 100 * 1024;   // activations of the GEMV in shared memory (two CTAs per SM)
+constexpr size_t kGvRows = 8;
+
+template <typename K>
+static int set_smem(tq_ctx* ctx, K kern, size_t bytes) {
+  if (bytes > 48 * 1024) TQ_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes));
+  return TQ_OK;
+}
+
+static int launch_gemv(tq_ctx* ctx, const tq_dweight* w, const DenseInput& in, size_t m, const DenseEpilogue& epi, bool xs) {
+  GemvParams p;
+  p.w = static_cast<const __nv_bfloat16*>(w->data);
+  p.kpad = (int)w->kpad;
+  p.n_rb = (int)(w->rpad / 16);
+  p.x = static_cast<const __nv_bfloat16*>(in.x);
+  p.ldx = (long long)in.ldx;
+  p.m = (int)m;
+  p.cols = (int)w->cols;
+  p.h = in.h;
+  p.ldh = (long long)in.ldh;
+  p.h_rows = in.h_rows;
+  p.gain = static_cast<const __nv_bfloat16*>(in.gain);
+  p.eps = in.eps;
+  p.epi = epi;
+  const size_t smem = xs ? m * (w->kpad * 2 + 16) : 0;
+  const int rb = xs ? 1 : 2;
+  int per_sm = 2;
+  while (per_sm > 1 && per_sm * (smem + 10 * 1024 * rb) > 220 * 1024) --per_sm;
+  const int groups = (p.n_rb + rb - 1) / rb;
+  int grid = ctx->sm_count * per_sm;
+  if (grid > groups) grid = groups;
+  if (xs) {
+    if (int st = set_smem(ctx, dgemv_kernel<1, true>, smem)) return st;
+    TQ_CUDA(ctx, launch_k(ctx, dgemv_kernel<1, true>, dim3((unsigned)grid), dim3(kGvThreads), smem, p));
+  } else {
+    TQ_CUDA(ctx, launch_k(ctx, dgemv_kernel<2, false>, dim3((unsigned)grid), dim3(kGvThreads), 0, p));
+  }
+  return TQ_OK;
+}
+
+static int launch_umma(tq_ctx* ctx, const tq_dweight* w, const void* x, size_t ldx, size_t m, const DenseEpilogue& epi) {
+  if (!w->has_map) return fail(ctx, TQ_EUNSUPPORTED, "cuTensorMapEncodeTiled is not available from this driver");
+  TQ_REQUIRE(ctx, ((uintptr_t)x & 15) == 0 && ldx % 8 == 0, "dense linear: activation rows must be 16-byte aligned");
+  DUmmaParams p;
+  p.m = (int)m;
+  p.n_ft = (int)((w->rpad + kUmmaRows - 1) / kUmmaRows);
+  p.kb_total = (int)((w->cols + kUmmaK - 1) / kUmmaK);
+  // Row tile: the width that makes (waves of CTAs) x (width) smallest; the wider one on a tie.
+  int ntok = 16;
+  long long best = 0;
+  for (int cand = 256; cand >= 16; cand -= 16) {
+    if (cand > 16 && (size_t)(cand - 15) > m && cand - 16 >= (int)m) continue;     // wider than the rows need
+    const long long tiles = (long long)p.n_ft * (long long)((m + cand - 1) / cand);
+    const long long waves = (tiles + ctx->sm_count - 1) / ctx->sm_count;
+    const long long cost = waves * (cand < 96 ? 96 : cand);   // (below about 96 rows a step costs the same)
+    if (best == 0 || cost < best) {
+      best = cost;
+      ntok = cand;
+    }
+  }
+  p.ntok = ntok;
+  p.n_tt = (int)((m + ntok - 1) / ntok);
+  const int base = p.n_ft * p.n_tt;
+  int splits = 1;
+  if (base <= ctx->sm_count / 2 && base <= kTileCounters) {
+    splits = ctx->sm_count / base;
+    if (splits > p.kb_total / 4) splits = p.kb_total / 4;    // at least four 64-k steps each
+    if (splits > 16) splits = 16;
+    if (splits < 1) splits = 1;
+  }
+  p.kb_per_split = (p.kb_total + splits - 1) / splits;
+  p.splits = (p.kb_total + p.kb_per_split - 1) / p.kb_per_split;
+  p.n_tiles = base * p.splits;
+  p.acc_stride = ntok <= 32 ? 32 : ntok <= 64 ? 64 : ntok <= 128 ? 128 : 256;
+  p.n_acc = 2;
+  p.tmem_cols = 2 * p.acc_stride;
+  const size_t stage = (size_t)(kUmmaRows + ntok) * 128, budget = 227 * 1024 - kDuHeader - 1024;
+  p.stages = (int)(budget / stage);
+  if (p.stages > kDuMaxStages) p.stages = kDuMaxStages;
+  p.epi = epi;
+  p.err = ctx->dev_err;
+  p.counters = ctx->dev_err + 1;
+  p.partial = nullptr;
+  if (p.splits > 1) {
+    if (int st = ensure_splitk(ctx, (size_t)p.splits * m * p.n_ft * kUmmaRows * sizeof(float))) return st;
+    p.partial = static_cast<float*>(ctx->splitk);
+  }
+  CUtensorMap xmap;
+  if (!encode_bf16_k64(&xmap, x, m, w->cols, ldx, (unsigned)ntok)) return fail(ctx, TQ_ECUDA, "cuTensorMapEncodeTiled failed");
+  const size_t smem = kDuHeader + 1024 + (size_t)p.stages * stage;
+  if (int st = set_smem(ctx, dgemm_umma_kernel, smem)) return st;
+  const int grid = p.n_tiles < ctx->sm_count ? p.n_tiles : ctx->sm_count;
+  TQ_CUDA(ctx, launch_k(ctx, dgemm_umma_kernel, dim3((unsigned)grid), dim3(kDuThreads), smem, w->map, xmap, p));
+  return TQ_OK;
+}
+
+int launch_dense(tq_ctx* ctx, const tq_dweight* w, const DenseInput& in, size_t m, const DenseEpilogue& epi) {
+  if (m == 0) return TQ_OK;
+  TQ_REQUIRE(ctx, epi.n >= 1 && epi.n <= kDenseMaxSections && epi.s[epi.n - 1].row_end <= (int)w->rpad, "dense linear: bad output sections");
+  const bool bf = w->dtype == TQ_BF16;
+  const bool fits = m <= kGvRows && m * (w->kpad * 2 + 16) <= kGvSmemMax;
+  DenseInput x = in;
+  if (in.h && !(bf && fits)) {
+    TQ_REQUIRE(ctx, in.xn_tmp != nullptr, "dense linear: no buffer for the normalised rows");
+    if (int st = launch_rms_norm_rows(ctx, in.h, in.ldh, in.h_rows, in.gain, in.gain_dtype, m, w->cols, in.eps, in.xn_tmp,
+                                      bf ? TQ_BF16 : TQ_F32, w->kpad)) return st;
+    x = DenseInput();
+    x.x = in.xn_tmp;
+    x.ldx = w->kpad;
+  }
+  if (!bf) {
+    TQ_CUDA(ctx, launch_k(ctx, dgemm_f32_kernel, dim3((unsigned)((w->rpad + kDfTile - 1) / kDfTile), (unsigned)((m + kDfTile - 1) / kDfTile)),
+                          dim3(256), 0, static_cast<const float*>(w->data), (int)w->kpad, (int)w->rpad, static_cast<const float*>(x.x),
+                          (long long)x.ldx, (int)m, (int)w->cols, epi));
+    return TQ_OK;
+  }
+  if (x.h && !(w->dtype == x.gain_dtype)) return fail(ctx, TQ_EINVAL, "dense linear: the norm's gain must have the weight's dtype");
+  if (!x.h) TQ_REQUIRE(ctx, ((uintptr_t)x.x & 15) == 0 && x.ldx % 8 == 0, "dense linear: activation rows must be 16-byte aligned");
+  if (fits) return launch_gemv(ctx, w, x, m, epi, true);
+  if (m <= kGvRows) return launch_gemv(ctx, w, x, m, epi, false);
+  return launch_umma(ctx, w, x.x, x.ldx, m, epi);
+}
+
+__global__ void dweight_put_kernel(const void* src, int s_dt, void* dst, int d_dt, size_t rows, size_t cols, size_t kpad, size_t row0,
+                                   size_t col0, int interleave) {
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= rows * cols) return;
+  const size_t r = i / cols, c = i % cols;
+  const float v = s_dt == TQ_F32 ? reinterpret_cast<const float*>(src)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(src)[i]);
+  const size_t dr = row0 + (interleave ? (r / 8) * 16 + (interleave == 2 ? 8 : 0) + r % 8 : r);
+  const size_t o = dr * kpad + col0 + c;
+  if (d_dt == TQ_F32) reinterpret_cast<float*>(dst)[o] = v;
+  else reinterpret_cast<__nv_bfloat16*>(dst)[o] = __float2bfloat16_rn(v);
+}
+
+__global__ void clamped_glu_kernel(const void* gate, const void* up, int dt, size_t n, float limit, float alpha, void* out, int out_dt) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const float g = dt == TQ_F32 ? reinterpret_cast<const float*>(gate)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(gate)[i]);
+  const float u = dt == TQ_F32 ? reinterpret_cast<const float*>(up)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(up)[i]);
+  const float v = clamped_glu(g, u, limit, alpha);
+  if (out_dt == TQ_F32) reinterpret_cast<float*>(out)[i] = v;
+  else reinterpret_cast<__nv_bfloat16*>(out)[i] = __float2bfloat16_rn(v);
+}
+
+}  // namespace tq
+
+using namespace tq;
+
+extern "C" {
+
+int tq_dweight_create(tq_ctx* ctx, size_t rows, size_t cols, int dtype, tq_dweight** out) {
+  if (int st = bind(ctx)) return st;
+  TQ_REQUIRE(ctx, out && rows > 0 && cols > 0, "tq_dweight_create: empty weight");
+  *out = nullptr;
+  TQ_REQUIRE(ctx, dtype == TQ_BF16 || dtype == TQ_F32, "tq_dweight_create: dtype must be bf16 or f32");
+  TQ_REQUIRE(ctx, rows < (1ull << 30) && cols < (1ull << 30), "tq_dweight_create: weight too large");
+  tq_dweight* w = new (std::nothrow) tq_dweight();
+  if (!w) return fail(ctx, TQ_ENOMEM, "out of host memory");
+  w->dtype = dtype;
+  w->rows = rows;
+  w->cols = cols;
+  w->rpad = (rows + 15) / 16 * 16;
+  w->kpad = (cols + kGvPad - 1) / kGvPad * kGvPad;
+  const size_t bytes = w->rpad * w->kpad * dtype_size(dtype);
+  cudaError_t e = cudaMalloc(&w->data, bytes);
+  if (e == cudaSuccess) e = cudaMemsetAsync(w->data, 0, bytes, ctx->stream);
+  if (e != cudaSuccess) {
+    if (w->data) cudaFree(w->data);
+    delete w;
+    cudaGetLastError();
+    return fail(ctx, e == cudaErrorMemoryAllocation ? TQ_ENOMEM : TQ_ECUDA, "tq_dweight_create: %s", cudaGetErrorString(e));
+  }
+  if (dtype == TQ_BF16) w->has_map = encode_bf16_k64(&w->map, w->data, w->rpad, w->kpad, w->kpad, kUmmaRows);
+  *out = w;
+  return TQ_OK;
+}
+
+int tq_dweight_put(tq_ctx* ctx, tq_dweight* w, const void* src, int src_dtype, size_t rows, size_t cols, size_t row0, size_t col0,
+                   int interleave) {
+  if (int st = bind(ctx)) return st;
+  TQ_REQUIRE(ctx, w && src && rows > 0 && cols > 0, "tq_dweight_put: null argument");
+  TQ_REQUIRE(ctx, src_dtype == TQ_BF16 || src_dtype == TQ_F32, "tq_dweight_put: the source must be bf16 or f32");
+  TQ_REQUIRE(ctx, interleave >= 0 && interleave <= 2 && (!interleave || row0 % 16 == 0), "tq_dweight_put: bad row order");
+  const size_t last = interleave ? ((rows - 1) / 8) * 16 + 8 * (interleave - 1) + (rows - 1) % 8 : rows - 1;
+  TQ_REQUIRE(ctx, row0 + last < w->rpad && col0 + cols <= w->kpad, "tq_dweight_put: block outside the weight");
+  const size_t bytes = rows * cols * dtype_size(src_dtype);
+  void* tmp = nullptr;
+  TQ_CUDA(ctx, cudaMalloc(&tmp, bytes));
+  cudaError_t e = cudaMemcpyAsync(tmp, src, bytes, cudaMemcpyDefault, ctx->stream);
+  if (e == cudaSuccess) {
+    dweight_put_kernel<<<(unsigned)((rows * cols + 255) / 256), 256, 0, ctx->stream>>>(tmp, src_dtype, w->data, w->dtype, rows, cols, w->kpad,
+                                                                                      row0, col0, interleave);
+    ctx->launches++;
+    e = cudaGetLastError();
+  }
+  if (e == cudaSuccess) e = cudaStreamSynchronize(ctx->stream);
+  cudaFree(tmp);
+  TQ_CUDA(ctx, e);
+  return TQ_OK;
+}
+
+int tq_dweight_free(tq_ctx* ctx, tq_dweight* w) {
+  if (!w) return TQ_OK;
+  if (int st = bind(ctx)) return st;
+  cudaStreamSynchronize(ctx->stream);
+  cudaFree(w->data);
+  delete w;
+  return TQ_OK;
+}
+
+int tq_dweight_data(const tq_dweight* w, void** dev, size_t* rows_padded, size_t* cols_padded) {
+  if (!w) return TQ_EINVAL;
+  if (dev) *dev = w->data;
+  if (rows_padded) *rows_padded = w->rpad;
+  if (cols_padded) *cols_padded = w->kpad;
+  return TQ_OK;
+}
+
+int tq_dlinear(tq_ctx* ctx, const tq_dweight* w, const void* x_dev, size_t ldx, size_t m, void* y_dev, int y_dtype, size_t ldy) {
+  if (int st = bind(ctx)) return st;
+  TQ_REQUIRE(ctx, w && x_dev && y_dev, "tq_dlinear: null pointer");
+  TQ_REQUIRE(ctx, y_dtype == TQ_F32 || y_dtype == TQ_BF16, "tq_dlinear: y must be f32 or bf16");
+  DenseInput in;
+  in.x = x_dev;
+  in.ldx = ldx ? ldx : w->cols;
+  DenseEpilogue e;
+  e.n = 1;
+  e.s[0].row_end = (int)w->rpad;
+  e.s[0].rows = (int)w->rows;
+  e.s[0].f32 = y_dtype == TQ_F32;
+  e.s[0].ld = (long long)(ldy ? ldy : w->rows);
+  e.s[0].out = y_dev;
+  return launch_dense(ctx, w, in, m, e);
+}
+
+int tq_clamped_glu(tq_ctx* ctx, const void* gate_dev, const void* up_dev, int in_dtype, size_t n, float limit, float alpha, void* out_dev,
+                   int out_dtype) {
+  if (int st = bind(ctx)) return st;
+  TQ_REQUIRE(ctx, (in_dtype == TQ_F32 || in_dtype == TQ_BF16) && (out_dtype == TQ_F32 || out_dtype == TQ_BF16),
+             "tq_clamped_glu: dtypes must be f32 or bf16");
+  if (n == 0) return TQ_OK;
+  TQ_REQUIRE(ctx, gate_dev && up_dev && out_dev, "tq_clamped_glu: null pointer");
+  TQ_CUDA(ctx, launch_k(ctx, clamped_glu_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, gate_dev, up_dev, in_dtype, n, limit, alpha,
+                        out_dev, out_dtype));
+  return TQ_OK;
+}
+
+}  // extern "C"

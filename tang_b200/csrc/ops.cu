@@ -61,11 +61,13 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, size_t i, float4 v) {
 // dim % 4 == 0 and 16-byte aligned rows.
 template <typename XT, typename WT, typename OT>
 __global__ void __launch_bounds__(kNormThreads) rms_norm_vec_kernel(const XT* x, const float* residual, const WT* w, int dim,
-                                                                    float eps, OT* out, float* sum_out) {
+                                                                    float eps, OT* out, float* sum_out, const int* rows,
+                                                                    size_t ld_in, size_t ld_out) {
   __shared__ float red[kNormThreads / 32];
   pdl_wait();
   pdl_launch_dependents();
-  const size_t base = (size_t)blockIdx.x * dim;
+  // (`rows`: the input row of each output row; only the rows form has strides that differ from dim)
+  const size_t base = (size_t)(rows ? rows[blockIdx.x] : (int)blockIdx.x) * ld_in, obase = (size_t)blockIdx.x * ld_out;
   const bool has_res = residual != nullptr;
   float4 v[kNormVecs], r[kNormVecs], g[kNormVecs];
 #pragma unroll
@@ -95,7 +97,7 @@ __global__ void __launch_bounds__(kNormThreads) rms_norm_vec_kernel(const XT* x,
   for (int i = 0; i < kNormVecs; ++i) {
     const int d = 4 * (threadIdx.x + i * kNormThreads);
     if (d < dim) {
-      store4(out, base + d, make_float4(v[i].x * inv * g[i].x, v[i].y * inv * g[i].y, v[i].z * inv * g[i].z, v[i].w * inv * g[i].w));
+      store4(out, obase + d, make_float4(v[i].x * inv * g[i].x, v[i].y * inv * g[i].y, v[i].z * inv * g[i].z, v[i].w * inv * g[i].w));
       if (sum_out) store4(sum_out, base + d, v[i]);
     }
   }
@@ -104,12 +106,13 @@ __global__ void __launch_bounds__(kNormThreads) rms_norm_vec_kernel(const XT* x,
 // Any dim <= 8192, any alignment: one element per step (the rarely used fallback).
 __global__ void __launch_bounds__(kNormThreads) rms_norm_kernel(const void* x, int x_dt, const float* residual,
                                                                 const void* w, int w_dt, int dim, float eps, void* out,
-                                                                int out_dt, float* sum_out) {
+                                                                int out_dt, float* sum_out, const int* rows, size_t ld_in,
+                                                                size_t ld_out) {
   __shared__ float red[kNormThreads / 32];
   __shared__ float row_s[8192];
   pdl_wait();
   pdl_launch_dependents();
-  const size_t base = (size_t)blockIdx.x * dim;
+  const size_t base = (size_t)(rows ? rows[blockIdx.x] : (int)blockIdx.x) * ld_in, obase = (size_t)blockIdx.x * ld_out;
   float sq = 0.f;
   for (int d = threadIdx.x; d < dim; d += kNormThreads) {
     float t = load_as_float(x, x_dt, base + d);
@@ -120,7 +123,7 @@ __global__ void __launch_bounds__(kNormThreads) rms_norm_kernel(const void* x, i
   const float total = block_sum(sq, red);
   const float inv = 1.0f / sqrtf(total / (float)dim + eps);
   for (int d = threadIdx.x; d < dim; d += kNormThreads) {
-    store_from_float(out, out_dt, base + d, row_s[d] * inv * load_as_float(w, w_dt, d));
+    store_from_float(out, out_dt, obase + d, row_s[d] * inv * load_as_float(w, w_dt, d));
     if (sum_out) sum_out[base + d] = row_s[d];
   }
 }
@@ -221,6 +224,77 @@ __global__ void qkv_post_kernel(const float* qkv, const float* cos_t, const floa
   }
 }
 
+int launch_rms_norm_rows(tq_ctx* ctx, const float* x, size_t ldx, const int* rows, const void* gain, int gain_dtype, size_t n,
+                         size_t dim, float eps, void* out, int out_dtype, size_t ld_out) {
+  TQ_REQUIRE(ctx, dim > 0 && dim <= 8192, "rms_norm: dim must be in 1..8192");
+  if (n == 0) return TQ_OK;
+  const bool vec = dim % 4 == 0 && ldx % 4 == 0 && ld_out % 4 == 0 && (((uintptr_t)x | (uintptr_t)gain | (uintptr_t)out) & 15) == 0;
+  using bf = __nv_bfloat16;
+  const dim3 grid((unsigned)n), block(kNormThreads);
+  const float* none = nullptr;
+  float* no_sum = nullptr;
+  if (!vec) {
+    TQ_CUDA(ctx, launch_k(ctx, rms_norm_kernel, grid, block, 0, (const void*)x, (int)TQ_F32, none, gain, gain_dtype, (int)dim, eps, out,
+                          out_dtype, no_sum, rows, ldx, ld_out));
+  } else if (gain_dtype == TQ_BF16 && out_dtype == TQ_BF16) {
+    TQ_CUDA(ctx, launch_k(ctx, rms_norm_vec_kernel<float, bf, bf>, grid, block, 0, x, none, (const bf*)gain, (int)dim, eps, (bf*)out,
+                          no_sum, rows, ldx, ld_out));
+  } else if (gain_dtype == TQ_F32 && out_dtype == TQ_F32) {
+    TQ_CUDA(ctx, launch_k(ctx, rms_norm_vec_kernel<float, float, float>, grid, block, 0, x, none, (const float*)gain, (int)dim, eps,
+                          (float*)out, no_sum, rows, ldx, ld_out));
+  } else {
+    return fail(ctx, TQ_EUNSUPPORTED, "rms_norm rows: gain and output must share a dtype");
+  }
+  return TQ_OK;
+}
+
+// Token embedding plus a learned vector per absolute position, and the bookkeeping of a step over several sequences at
+// once: rows seq_rows[b] .. seq_rows[b+1]-1 (null: row b) are the next tokens of sequence b, whose first one sits at
+// position starts[b]; its cache is slot slots[b] (null: b) of `max_seq` rows.  Every row's position and cache row are
+// left for the kernels that follow; a position or slot outside the cache gives cache row -1 (nothing is stored for it)
+// and is reported through the status word.  One CTA per row.
+__global__ void __launch_bounds__(256) embedding_pos_kernel(const void* table, const void* pos_table, int dt, const int* ids, const int* seq_rows,
+                                                            const int* starts, const int* slots, int n_seqs, int dim, int vocab,
+                                                            int n_pos, int max_seq, int n_slots, float* out, int* row_pos, int* cache_row,
+                                                            int* err) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int m = blockIdx.x;
+  int b = m, off = 0;
+  if (seq_rows) {
+    int lo = 0, hi = n_seqs;          // last b with seq_rows[b] <= m (empty sequences share a boundary: take the last)
+    while (hi - lo > 1) {
+      const int mid = (lo + hi) >> 1;
+      if (seq_rows[mid] <= m) lo = mid;
+      else hi = mid;
+    }
+    b = lo;
+    off = m - seq_rows[b];
+  }
+  const int pos = starts[b] + off, slot = slots ? slots[b] : b;
+  const int id = ids[m];
+  const bool ok = pos >= 0 && pos < max_seq && pos < n_pos && slot >= 0 && slot < n_slots;
+  if (threadIdx.x == 0) {
+    row_pos[m] = ok ? pos : 0;
+    cache_row[m] = ok ? slot * max_seq + pos : -1;
+    if (!ok) atomicCAS(err, 0, (int)DERR_POSITION);
+  }
+  const bool tok_ok = id >= 0 && id < vocab;
+  for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+    float v = tok_ok ? load_as_float(table, dt, (size_t)id * dim + d) : 0.f;
+    if (ok) v += load_as_float(pos_table, dt, (size_t)pos * dim + d);
+    out[(size_t)m * dim + d] = v;
+  }
+}
+
+int launch_embedding_pos(tq_ctx* ctx, const void* table, const void* pos_table, int dt, const int* ids, const int* seq_rows,
+                         const int* starts, const int* slots, int n_seqs, size_t rows, int dim, int vocab, int n_pos, int max_seq,
+                         int n_slots, float* out, int* row_pos, int* cache_row) {
+  TQ_CUDA(ctx, launch_k(ctx, embedding_pos_kernel, dim3((unsigned)rows), dim3(256), 0, table, pos_table, dt, ids, seq_rows, starts, slots,
+                        n_seqs, dim, vocab, n_pos, max_seq, n_slots, out, row_pos, cache_row, ctx->dev_err));
+  return TQ_OK;
+}
+
 int launch_qkv_post(tq_ctx* ctx, const float* qkv, const float* cos_t, const float* sin_t, const int* positions,
                     const int* rope_positions, int B, int n_heads, int n_kv, int hd, int max_seq, void* q_out, void* k_cache,
                     void* v_cache, size_t seq_stride, int q_len) {
@@ -282,16 +356,17 @@ __global__ void generate_advance_kernel(const int* chosen, int rows, int* tokens
                                         int out_ld, int* step_io, int* lens_io) {
   pdl_wait();
   pdl_launch_dependents();
-  const int step = *step_io;
+  const int step = step_io ? *step_io : 0;
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i < rows) {
-    if (step < out_ld) out_tokens[(size_t)i * out_ld + step] = chosen[i];
+    const int col = step_io ? step : lens_io[i];    // without a common step every row appends at its own length
+    if (col >= 0 && col < out_ld) out_tokens[(size_t)i * out_ld + col] = chosen[i];
     tokens_io[i] = chosen[i];
     positions_io[i] += 1;
     if (lens_io) lens_io[i] += 1;
   }
   __syncthreads();                       // a single block (rows <= 1024): every thread has read `step`
-  if (threadIdx.x == 0) *step_io = step + 1;
+  if (step_io && threadIdx.x == 0) *step_io = step + 1;
 }
 
 }  // namespace tq
@@ -315,11 +390,12 @@ int tq_rms_norm(tq_ctx* ctx, const void* x_dev, int x_dtype, const float* residu
   using bf = __nv_bfloat16;
 #define TQ_NORM(XT, WT, OT)                                                                                           \
   TQ_CUDA(ctx, launch_k(ctx, rms_norm_vec_kernel<XT, WT, OT>, grid, block, 0, static_cast<const XT*>(x_dev), residual_dev, \
-                        static_cast<const WT*>(weight_dev), (int)dim, eps, static_cast<OT*>(out_dev), sum_out_dev))
+                        static_cast<const WT*>(weight_dev), (int)dim, eps, static_cast<OT*>(out_dev), sum_out_dev, \
+                        (const int*)nullptr, dim, dim))
   const int key = (x_dtype == TQ_BF16) * 4 + (w_dtype == TQ_BF16) * 2 + (out_dtype == TQ_BF16);
   if (!vec) {
     TQ_CUDA(ctx, launch_k(ctx, rms_norm_kernel, grid, block, 0, x_dev, x_dtype, residual_dev, weight_dev, w_dtype, (int)dim, eps,
-                          out_dev, out_dtype, sum_out_dev));
+                          out_dev, out_dtype, sum_out_dev, (const int*)nullptr, dim, dim));
   } else {
     switch (key) {
       case 0: TQ_NORM(float, float, float); break;
@@ -411,7 +487,8 @@ int tq_generate_advance(tq_ctx* ctx, const int* chosen_dev, size_t rows, int* to
                         int* out_tokens_dev, size_t out_ld, int* step_io_dev, int* lens_io_dev) {
   if (int st = bind(ctx)) return st;
   if (rows == 0) return TQ_OK;
-  TQ_REQUIRE(ctx, chosen_dev && tokens_io_dev && positions_io_dev && out_tokens_dev && step_io_dev, "tq_generate_advance: null pointer");
+  TQ_REQUIRE(ctx, chosen_dev && tokens_io_dev && positions_io_dev && out_tokens_dev && (step_io_dev || lens_io_dev),
+             "tq_generate_advance: null pointer");
   TQ_REQUIRE(ctx, rows <= 1024, "tq_generate_advance: at most 1024 sequences");
   TQ_CUDA(ctx, launch_k(ctx, generate_advance_kernel, dim3(1), dim3(1024), 0, chosen_dev, (int)rows, tokens_io_dev,
                         positions_io_dev, out_tokens_dev, (int)out_ld, step_io_dev, lens_io_dev));

@@ -4,6 +4,7 @@
 
 #include "internal.h"
 #include "qgemm_umma.cuh"
+#include "tensormap.h"
 
 namespace tq {
 
@@ -486,24 +487,6 @@ qgemm_umma_kernel(const __grid_constant__ CUtensorMap x_map, const UmmaParams p)
 }
 
 // ---- host side ------------------------------------------------------------------------------------
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-static EncodeTiledFn encode_tiled() {
-  static EncodeTiledFn fn = nullptr;
-  static bool tried = false;
-  if (!tried) {
-    tried = true;
-    void* ptr = nullptr;
-    cudaDriverEntryPointQueryResult qres;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &qres) == cudaSuccess &&
-        qres == cudaDriverEntryPointSuccess)
-      fn = reinterpret_cast<EncodeTiledFn>(ptr);
-  }
-  return fn;
-}
-
 bool umma_supported(const tq_qweight* w, size_t m) {
   return (w->kind == TQ_Q4_F16 || w->kind == TQ_Q4_F32 || w->kind == TQ_Q8_F32 || w->kind == TQ_I8_ROW) && w->rows % kUmmaRows == 0 &&
          w->cols % kTileK == 0 && m >= 1;
@@ -515,8 +498,7 @@ bool umma_supported(const tq_qweight* w, size_t m) {
 int launch_qgemm_umma(tq_ctx* ctx, const tq_qweight* w, const void* x_bf16, size_t ldx, size_t m, void* y, int y_dtype,
                       size_t ldy, int terms, const UmmaGroups* grp, bool swiglu) {
   if (w->kind == TQ_I8_ROW) terms = 1;   // exact with one term: the row scale is applied to the accumulator
-  EncodeTiledFn enc = encode_tiled();
-  if (!enc) return fail(ctx, TQ_EUNSUPPORTED, "cuTensorMapEncodeTiled is not available from this driver");
+  if (!encode_tiled()) return fail(ctx, TQ_EUNSUPPORTED, "cuTensorMapEncodeTiled is not available from this driver");
   TQ_REQUIRE(ctx, umma_supported(w, m), "tcgen05 GEMM: needs rows %% 128 == 0 and cols %% 128 == 0");
   TQ_REQUIRE(ctx, ((uintptr_t)x_bf16 & 15) == 0 && (ldx * 2) % 16 == 0, "tcgen05 GEMM: activation rows must be 16-byte aligned");
   // Ring sizes.  Two rules come from the dequant groups running ahead of one another (a parity wait
@@ -608,14 +590,7 @@ int launch_qgemm_umma(tq_ctx* ctx, const tq_qweight* w, const void* x_bf16, size
   if (raw_stages > slots_needed) raw_stages = slots_needed;
   if (stages < kUmmaGroups || raw_stages < 1) return fail(ctx, TQ_EUNSUPPORTED, "tcgen05 GEMM: ring sizes %d/%d", stages, raw_stages);
   CUtensorMap map;
-  const cuuint64_t gdim[2] = {(cuuint64_t)w->cols, (cuuint64_t)m};
-  const cuuint64_t gstride[1] = {(cuuint64_t)ldx * 2};
-  const cuuint32_t box[2] = {(cuuint32_t)kUmmaK, (cuuint32_t)ntok};
-  const cuuint32_t estr[2] = {1, 1};
-  CUresult cr = enc(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(x_bf16), gdim, gstride, box, estr,
-                    CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-                    CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  if (cr != CUDA_SUCCESS) return fail(ctx, TQ_ECUDA, "cuTensorMapEncodeTiled failed (%d)", (int)cr);
+  if (!encode_bf16_k64(&map, x_bf16, m, w->cols, ldx, (unsigned)ntok)) return fail(ctx, TQ_ECUDA, "cuTensorMapEncodeTiled failed");
   UmmaParams p;
   p.tiles = w->tiles;
   p.row_scales = w->row_scales;

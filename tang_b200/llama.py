@@ -10,6 +10,7 @@ import numpy as np
 
 from . import _lib
 from .device import Buffer, QBuffer, QuantComputeDevice
+from .generation import check_lengths, decode_loop
 
 
 class LlamaConfig(C.Structure):
@@ -135,50 +136,16 @@ class LlamaModel:
         with `seed` (as ``Sampler::with_seed`` per call of ``generate``); the repetition penalty sees the prompt and
         everything generated so far.  Returns int32 [batch, n_new]; the caller cuts at its stop token (what is
         drawn before a stop token does not depend on what follows)."""
-        from .device import SamplerConfig
-
-        dev, L = self.dev, self.dev._L
         prompts = np.asarray(prompts, np.int32)
+        check_lengths(prompts, n_new, self.cfg.max_seq)
+        dev = self.dev
         B, P = prompts.shape
-        if P < 1 or n_new < 1:
-            raise _lib.TangqError(_lib.TQ_EINVAL, "generate: need at least one prompt token and one new token")
-        if P + n_new > self.cfg.max_seq:
-            raise _lib.TangqError(_lib.TQ_EINVAL, "generate: prompt + new tokens exceed max_seq")
-        cfg = sampling if sampling is not None else SamplerConfig(0.0, 0, 1.0, 1.0)
-        vocab, ld = self.cfg.vocab, P + n_new
-        logits = dev.alloc(B * vocab, _lib.F32)
-        tok, pos = dev.alloc(B, _lib.I32), dev.alloc(B, _lib.I32)
-        chosen = dev.alloc(B, _lib.I32)
-        step = dev.upload(np.full(1, P, np.int32), _lib.I32)            # column of the history the next token goes to
-        hist = np.zeros((B, ld), np.int32)
-        hist[:, :P] = prompts
-        hist_d = dev.upload(hist, _lib.I32)                             # prompt + generated tokens: the penalty's past
-        lens = dev.upload(np.full(B, P, np.int32), _lib.I32)
-        rng = dev.upload(np.full(B, seed, np.uint64).view(np.float64), _lib.F64)
         if P > 1:                                   # all prompt tokens but the last: one prefill chunk fills the cache
+            scratch = dev.alloc(B * self.cfg.vocab, _lib.F32)
             self.prefill(dev.upload(np.ascontiguousarray(prompts[:, :P - 1]), _lib.I32), dev.upload(np.zeros(B, np.int32), _lib.I32),
-                         B, P - 1, logits)
-        dev.upload_into(tok, prompts[:, P - 1].copy())
-        dev.upload_into(pos, np.full(B, P - 1, np.int32))
-
-        def one():
-            self.decode(tok, pos, B, P + n_new, logits)
-            dev._check(L.tq_sample(dev._ctx, C.c_void_p(logits.ptr), comm_world, B, vocab // comm_world, C.byref(cfg),
-                                   C.c_void_p(rng.ptr), C.c_void_p(hist_d.ptr), C.c_void_p(lens.ptr), ld, C.c_void_p(chosen.ptr)))
-            dev._check(L.tq_generate_advance(dev._ctx, C.c_void_p(chosen.ptr), B, C.c_void_p(tok.ptr), C.c_void_p(pos.ptr),
-                                             C.c_void_p(hist_d.ptr), ld, C.c_void_p(step.ptr), C.c_void_p(lens.ptr)))
-        one()                                       # eager once (workspaces), then the remaining steps from a graph
-        if n_new > 1:
-            dev.sync()
-            dev.begin_capture()
-            one()
-            graph = dev.end_capture()
-            for _ in range(n_new - 1):
-                graph.launch()
-            dev.sync()
-            graph.free()
-        dev.sync()
-        return hist_d.to_vec().reshape(B, ld)[:, P:].copy()
+                         B, P - 1, scratch)
+        return decode_loop(dev, lambda tok, pos, logits: self.decode(tok, pos, B, P + n_new, logits), prompts, n_new,
+                           self.cfg.vocab, sampling, seed, comm_world)
 
     def generate_greedy(self, prompts, n_new: int, comm_world: int = 1) -> np.ndarray:
         """``generate`` with ``SamplingConfig::greedy()``."""
