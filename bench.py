@@ -442,10 +442,10 @@ def decode_bytes_per_gpu(batch: int, tp: int, n_layers: int) -> int:
     return (wbytes + kv) // tp
 
 
-def build_llama(dev, tb, torch, stream, comm, rank, world, n_layers, max_batch):
+def build_llama(dev, tb, torch, stream, comm, rank, world, n_layers, max_batch, c=None):
     import ctypes as C
 
-    c = LLAMA
+    c = c or LLAMA
     tp = world
     hl, kl, fl, vl = c["n_heads"] // tp, c["n_kv"] // tp, c["ffn"] // tp, c["vocab"] // tp
     d, hd = c["d"], c["hd"]
@@ -903,6 +903,213 @@ def run_sharded_extras(dev, tb, torch, stream, peak_gbs, comm, rank, world, barr
     return out
 
 
+# ----------------------------------------------------------------------------------------------
+# --tofazen: the Tofazen family (bf16, dense) beside the Llama-shaped model (int4) at equal width, head and ffn sizes,
+# random weights: decode and prefill throughput of both, and their like kernels one by one against their rooflines.
+# ----------------------------------------------------------------------------------------------
+TOFAZEN_SIZES = {
+    # heads x 2 maps x dim = the Llama model's q width; vdim = its head size, so caches and products are equal
+    "8b": {"layers": 32, "width": 4096, "heads": 32, "kv": 8, "dim": 64, "vdim": 128, "ff": 14336, "vocab": 128256},
+    "1b": {"layers": 16, "width": 2048, "heads": 16, "kv": 4, "dim": 64, "vdim": 128, "ff": 8192, "vocab": 32000},
+}
+
+
+def build_tofazen(dev, tb, torch, stream, s, ctx, max_batch, window, keep_first):
+    from tang_b200.tofazen import TofazenLayer, tensor_names
+
+    gen = torch.Generator(device="cuda").manual_seed(5)
+    layers = [TofazenLayer(s["heads"], s["kv"], s["dim"], s["vdim"], s["dim"] ** -0.5, 0.3, window, keep_first, None, s["ff"], 7.0)
+              for _ in range(s["layers"])]
+    cfg = tb.TofazenConfig(s["vocab"], s["width"], ctx + 1, 1e-6, 1.0, layers)
+    model = tb.TofazenModel(dev, cfg, [0.5] * s["layers"], tb.BF16, max_batch, ctx + 1)
+    d, qr, kr, vr = s["width"], s["heads"] * 2 * s["dim"], s["kv"] * 2 * s["dim"], s["kv"] * s["vdim"]
+    shapes = {"embed": (s["vocab"], d), "pos": (ctx + 1, d), "final.norm": (1, d), "head": (s["vocab"], d), "norm1": (1, d), "q": (qr, d), "k": (kr, d),
+              "v": (vr, d), "o": (d, s["heads"] * s["vdim"]), "gate": (s["ff"], d), "up": (s["ff"], d), "down": (d, s["ff"])}
+    for name, tensor, layer in tensor_names(cfg):
+        r, c = shapes[name if name in shapes else name.split(".")[-1]]
+        with torch.cuda.stream(stream):
+            t = (torch.randn((r, c), device="cuda", generator=gen) * (0.05 if r == 1 else c ** -0.5) + (1.0 if r == 1 else 0.0)).bfloat16()
+        stream.synchronize()
+        model.put_pointer(tensor, layer, t.data_ptr(), tb.BF16, r, c)
+        del t
+    return model
+
+
+def run_tofazen(args) -> None:
+    import ctypes as C
+
+    import torch
+
+    import tang_b200 as tb
+
+    torch.cuda.set_device(0)
+    dev = tb.QuantComputeDevice(0)
+    L_ = dev._L
+    stream = torch.cuda.ExternalStream(dev.stream, device=torch.device("cuda", 0))
+    peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")) else {}
+    hbm, tf = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    ctx = 2048
+    sampler = ClockSampler(0)
+    sampler.start()
+    t_start = time.perf_counter()
+
+    def graph_ms(fn, reps=10):
+        fn()
+        dev.sync()
+        dev.begin_capture()
+        fn()
+        g = dev.end_capture()
+        ms = _time_ms(torch, stream, dev, g.launch, reps, warm=3)
+        g.free()
+        return ms
+
+    def rand_bf16(*shape, std=1.0):
+        with torch.cuda.stream(stream):
+            t = (torch.randn(shape, device="cuda") * std).bfloat16()
+        stream.synchronize()
+        return t
+
+    def buf(t, dt):
+        return tb.Buffer(dev, t.data_ptr(), t.numel(), dt, owns=False)
+
+    out = {"metric": "tofazen_throughput", "unit": "tokens/s", "data": "synthetic", "dtype": "bf16", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf},
+           "models": [], "kernels": []}
+    batches = [1, 2, 4, 8, 16, 64]
+    for size in [x for x in args.tofazen.split(",") if x in TOFAZEN_SIZES]:
+        s = TOFAZEN_SIZES[size]
+        c = {"d": s["width"], "n_heads": s["heads"], "n_kv": s["kv"], "hd": s["vdim"], "ffn": s["ff"], "vocab": s["vocab"], "ctx": ctx}
+        w_layer = s["width"] * (s["heads"] * 2 * s["dim"] + s["kv"] * (2 * s["dim"] + s["vdim"]) + s["heads"] * s["vdim"] + 3 * s["ff"])
+        params = s["layers"] * w_layer + s["vocab"] * s["width"]
+        kv_row = s["layers"] * s["kv"] * (2 * s["dim"] + s["vdim"]) * 2
+        for label, window, keep in (("full", ctx + 1, 0), ("window512", 512, 4)):
+            model = build_tofazen(dev, tb, torch, stream, s, ctx, max(batches), window, keep)
+            row = {"size": size, "model": "tofazen", "mask": label, "decode": {}, "prefill": {}}
+            for B in batches:
+                tok = dev.upload(np.random.randint(0, s["vocab"], B).astype(np.int32), tb.I32)
+                pos = dev.upload(np.full(B, ctx, np.int32), tb.I32)
+                lg = dev.alloc(B * s["vocab"], tb.F32)
+                ms = graph_ms(lambda: model.decode(tok, pos, B, ctx + 1, lg))
+                byt = params * 2 + B * kv_row * min(ctx + 1, window + keep)
+                row["decode"][B] = {"ms": ms, "tokens_per_s": B / ms * 1e3, "frac_of_hbm": byt / ms / 1e6 / hbm}
+            tok = dev.upload(np.random.randint(0, s["vocab"], ctx).astype(np.int32), tb.I32)
+            cu, st = dev.upload(np.array([0, ctx], np.int32), tb.I32), dev.upload(np.zeros(1, np.int32), tb.I32)
+            last, lg = dev.upload(np.array([ctx - 1], np.int32), tb.I32), dev.alloc(s["vocab"], tb.F32)
+            ms = graph_ms(lambda: model.step(tok, ctx, cu, st, None, 1, ctx, ctx, last, 1, lg), 3)
+            row["prefill"] = {"tokens": ctx, "ms": ms, "tokens_per_s": ctx / ms * 1e3, "frac_of_bf16": 2.0 * ctx * s["layers"] * w_layer / ms / 1e9 / tf}
+            out["models"].append(row)
+            model.destroy()
+        if s["layers"] and not args.tofazen_only:
+            torch.cuda.empty_cache()
+            model = build_llama(dev, tb, torch, stream, None, 0, 1, s["layers"], max(batches), c)
+            row = {"size": size, "model": "llama int4", "mask": "full", "decode": {}, "prefill": {}}
+            q4 = params // 2 + params // 16
+            for B in batches:
+                tok = dev.upload(np.random.randint(0, s["vocab"], B).astype(np.int32), tb.I32)
+                pos = dev.upload(np.full(B, ctx, np.int32), tb.I32)
+                lg = dev.alloc(B * s["vocab"], tb.F32)
+                ms = graph_ms(lambda: model.decode(tok, pos, B, ctx + 1, lg))
+                row["decode"][B] = {"ms": ms, "tokens_per_s": B / ms * 1e3, "frac_of_hbm": (q4 + B * kv_row * (ctx + 1)) / ms / 1e6 / hbm}
+            tok, st = dev.upload(np.random.randint(0, s["vocab"], ctx).astype(np.int32), tb.I32), dev.upload(np.zeros(1, np.int32), tb.I32)
+            lg = dev.alloc(s["vocab"], tb.F32)
+            model.prefill(tok, st, 1, ctx, lg)
+            ms = _time_ms(torch, stream, dev, lambda: model.prefill(tok, st, 1, ctx, lg), 3)
+            row["prefill"] = {"tokens": ctx, "ms": ms, "tokens_per_s": ctx / ms * 1e3, "frac_of_bf16": 2.0 * ctx * s["layers"] * w_layer / ms / 1e9 / tf}
+            out["models"].append(row)
+            model.destroy()
+            torch.cuda.empty_cache()
+
+    # ---- like kernels: a pass over several distinct weights (> L2), one launch each, from a graph
+    def dense_handle(rows, cols):
+        t = rand_bf16(rows, cols, std=cols ** -0.5)
+        h = C.c_void_p()
+        dev._check(L_.tq_dweight_create(dev._ctx, rows, cols, tb.BF16, C.byref(h)))
+        dev._check(L_.tq_dweight_put(dev._ctx, h, C.c_void_p(t.data_ptr()), tb.BF16, rows, cols, 0, 0, 0))
+        return h
+
+    def q4_handle(rows, cols):
+        with torch.cuda.stream(stream):
+            pay = torch.randint(0, 256, (rows, cols // 2), dtype=torch.uint8, device="cuda")
+            sc = (torch.rand((rows, cols // 32), device="cuda") * 0.018 + 0.002).half()
+        stream.synchronize()
+        h = C.c_void_p()
+        dev._check(L_.tq_qweight_from_device_arrays(dev._ctx, tb.Q4_F16, C.c_void_p(pay.data_ptr()), C.c_void_p(sc.data_ptr()), rows, cols, C.byref(h)))
+        dev.sync()
+        return h
+
+    for name, rows, cols in (("in", 34816, 4096), ("out", 4096, 18432)):
+        n = 8
+        dense, quant = [dense_handle(rows, cols) for _ in range(n)], [q4_handle(rows, cols) for _ in range(n)]
+        for m in (1, 2, 4, 8, 16, 64, 256, 2048):
+            x, y = rand_bf16(m, cols), torch.empty((m, rows), dtype=torch.bfloat16, device="cuda")
+            stream.synchronize()
+            xp, yp = C.c_void_p(x.data_ptr()), C.c_void_p(y.data_ptr())
+            flops, io = 2.0 * m * rows * cols, m * (rows + cols) * 2
+            for kind, hs, wb in (("dense bf16", dense, rows * cols * 2), ("int4", quant, rows * cols // 2 + rows * cols // 16)):
+                if kind == "int4" and args.tofazen_only:
+                    continue
+                call = (lambda h: L_.tq_dlinear(dev._ctx, h, xp, cols, m, yp, tb.BF16, rows)) if hs is dense else \
+                       (lambda h: L_.tq_qlinear(dev._ctx, h, xp, tb.BF16, 0, m, yp, tb.BF16, 0, None))
+                us = graph_ms(lambda: [dev._check(call(h)) for h in hs]) / n * 1e3
+                roof = max((wb + io) / hbm / 1e3, flops / tf / 1e6)
+                out["kernels"].append({"kernel": f"linear {name} {rows}x{cols}", "kind": kind, "m": m, "us": us, "roofline_us": roof, "frac": roof / us})
+        for h in dense:
+            L_.tq_dweight_free(dev._ctx, h)
+        for h in quant:
+            L_.tq_qweight_free(dev._ctx, h)
+
+    class Attn(C.Structure):
+        _fields_ = [(k, C.c_uint32) for k in ("heads", "kv_heads", "dim", "vdim", "window", "keep_first")] + [
+            (k, C.c_float) for k in ("scale", "lam", "out_scale", "eps")]
+
+    H, G, D, V = 32, 8, 64, 128
+    for B in (1, 16, 64):
+        n = max(1, min(16, 64 // B * 2))               # distinct caches per pass
+        k, v, q = rand_bf16(n, B, ctx, G * 2 * D), rand_bf16(n, B, ctx, G * V), rand_bf16(B, H * 2 * D)
+        o = torch.empty((B, H * V), dtype=torch.bfloat16, device="cuda")
+        lens = dev.upload(np.full(B, ctx, np.int32), tb.I32)
+        rp = dev.upload(np.full(B, ctx - 1, np.int32), tb.I32)
+        cr = dev.upload((np.arange(B) * ctx + ctx - 1).astype(np.int32), tb.I32)
+        for kind, window in (("differential", ctx), ("differential window 512", 512), ("gqa", ctx)):
+            a = Attn(H, G, D, V, window, 4, D ** -0.5, 0.5, 0.7, 1e-6)
+
+            def one():
+                for i in range(n):
+                    if kind == "gqa":
+                        dev._check(L_.tq_gqa_decode(dev._ctx, C.c_void_p(q.data_ptr()), C.c_void_p(k[i].data_ptr()), C.c_void_p(v[i].data_ptr()),
+                                                    C.c_void_p(lens.ptr), B, H, G, 128, ctx * G * 128, ctx, C.c_void_p(o.data_ptr()), tb.BF16))
+                    else:
+                        dev._check(L_.tq_diff_attention(dev._ctx, C.byref(a), tb.BF16, C.c_void_p(q.data_ptr()), H * 2 * D, C.c_void_p(k[i].data_ptr()),
+                                                        C.c_void_p(v[i].data_ptr()), B * ctx, None, C.c_void_p(rp.ptr), C.c_void_p(cr.ptr), B, B, 1, ctx,
+                                                        C.c_void_p(o.data_ptr()), H * V))
+            us = graph_ms(one) / n * 1e3
+            roof = B * min(ctx, window + (4 if window < ctx else 0)) * G * (2 * D + V) * 2 / hbm / 1e3
+            out["kernels"].append({"kernel": "decode attention", "kind": kind, "m": B, "us": us, "roofline_us": roof, "frac": roof / us})
+        del k, v
+        torch.cuda.empty_cache()
+    for T in (512, 2048):
+        k, v, q = rand_bf16(T, G * 2 * D), rand_bf16(T, G * V), rand_bf16(T, H * 2 * D)
+        o = torch.empty((T, H * V), dtype=torch.bfloat16, device="cuda")
+        cu, st = dev.upload(np.array([0, T], np.int32), tb.I32), dev.upload(np.zeros(1, np.int32), tb.I32)
+        rp = dev.upload(np.arange(T, dtype=np.int32), tb.I32)
+        for kind, window in (("differential", T), ("differential window 256", 256), ("gqa", T)):
+            a = Attn(H, G, D, V, window, 4, D ** -0.5, 0.5, 0.7, 1e-6)
+            if kind == "gqa":
+                fn = lambda: dev._check(L_.tq_gqa_prefill(dev._ctx, C.c_void_p(q.data_ptr()), C.c_void_p(k.data_ptr()), C.c_void_p(v.data_ptr()),
+                                                          C.c_void_p(st.ptr), 1, T, H, G, 128, T * G * 128, C.c_void_p(o.data_ptr()), tb.BF16))
+                flops = 4.0 * H * 128 * T * (T + 1) / 2
+            else:
+                fn = lambda: dev._check(L_.tq_diff_attention(dev._ctx, C.byref(a), tb.BF16, C.c_void_p(q.data_ptr()), H * 2 * D, C.c_void_p(k.data_ptr()),
+                                                             C.c_void_p(v.data_ptr()), T, C.c_void_p(cu.ptr), C.c_void_p(rp.ptr), C.c_void_p(rp.ptr), 1, T, T, T,
+                                                             C.c_void_p(o.data_ptr()), H * V))
+                pairs = sum(min(i + 1, window + 4) for i in range(T))
+                flops = 2.0 * H * 2 * (D + V) * pairs
+            us = graph_ms(fn) * 1e3
+            out["kernels"].append({"kernel": "prefill attention", "kind": kind, "m": T, "us": us, "tflops": flops / us / 1e6, "roofline_us": flops / tf / 1e6,
+                                   "frac": flops / tf / 1e6 / us})
+    out["clocks"] = sampler.stop(t_start, time.perf_counter())
+    print(json.dumps(out))
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -919,7 +1126,12 @@ def main() -> None:
     ap.add_argument("--decode-batches", default="1,16,64")
     ap.add_argument("--decode-layers", type=int, default=32)
     ap.add_argument("--decode-steps", type=int, default=10)
+    ap.add_argument("--tofazen", nargs="?", const="8b,1b", default="", help="time the Tofazen family instead (sizes: 8b, 1b, or none: kernels only)")
+    ap.add_argument("--tofazen-only", action="store_true", help="with --tofazen: leave the int4 model out")
     args = ap.parse_args()
+    if args.tofazen:
+        run_tofazen(args)
+        return
     args.warmup = max(args.warmup, 3) if args.impl == "ours" else args.warmup
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
