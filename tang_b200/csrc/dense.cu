@@ -51,46 +51,39 @@ __device__ __forceinline__ uint4 x_tail(const void* src, int n) {
   return make_uint4(w[0], w[1], w[2], w[3]);
 }
 
-// A CTA walks groups of RB 16-row blocks (grid-stride); its eight warps take the k chunks of a group in turn and meet
+// A CTA walks 16-row blocks (grid-stride); its eight warps take the k chunks of a block in turn and meet
 // in shared memory.  Lane 4g + t holds bytes 32t .. 32t + 31 of rows g and g + 8 of every 64-k step (a row's four lanes
 // read one 128-byte line): words 2i, 2i + 1 are the two k halves of MMA i; the activations are read the same way.  The loads of
-// the next step -- of the next group too -- are issued before the current step is multiplied, and the first ones before
-// the kernel waits for its predecessor (weights do not change).  XS: activations in shared memory, else from global.
-template <int RB, bool XS>
+// the next step -- of the next block too -- are issued before the current step is multiplied, and the first ones before
+// the kernel waits for its predecessor (weights do not change).  The activations sit in shared memory.
 __global__ void __launch_bounds__(kGvThreads, 2) dgemv_kernel(const __grid_constant__ GemvParams p) {
+  constexpr int U = 2;                               // 64-k loads per row and step: 32 registers in flight
+  constexpr int kGvChunk = 64 * U;                   // k per warp step
   extern __shared__ __align__(16) uint8_t gv_smem[];
-  __shared__ float red[2][kGvWarps][RB][128];
+  __shared__ float red[2][kGvWarps][128];
   __shared__ float ssq[kGvWarps];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-  const int n_groups = (p.n_rb + RB - 1) / RB;
-  constexpr int U = RB == 1 ? 2 : 1;                 // 64-k loads per row and step: about 32 registers in flight
-  constexpr int kGvChunk = 64 * U;                   // k per warp step
   const int n_ch = p.kpad / kGvChunk;
   const size_t row_bytes = (size_t)p.kpad * 2;
-  const uint8_t* wb = reinterpret_cast<const uint8_t*>(p.w);
+  const uint8_t* wb = reinterpret_cast<const uint8_t*>(p.w) + (size_t)g * row_bytes + 32 * t;
 
-  Frag32 nxt[RB][U][2];
-  auto load = [&](int grp, int c) {
+  Frag32 nxt[U][2];
+  auto load = [&](int rb, int c) {
+    const uint8_t* src = wb + (size_t)rb * 16 * row_bytes + (size_t)c * (kGvChunk * 2);
 #pragma unroll
-    for (int r = 0; r < RB; ++r) {
-      const int rb = min(grp * RB + r, p.n_rb - 1);
-      const uint8_t* src = wb + (size_t)(rb * 16 + g) * row_bytes + (size_t)c * (kGvChunk * 2) + 32 * t;
-#pragma unroll
-      for (int u = 0; u < U; ++u) {
-        nxt[r][u][0] = ldg_stream(src + 128 * u);
-        nxt[r][u][1] = ldg_stream(src + 8 * row_bytes + 128 * u);
-      }
+    for (int u = 0; u < U; ++u) {
+      nxt[u][0] = ldg_stream(src + 128 * u);
+      nxt[u][1] = ldg_stream(src + 8 * row_bytes + 128 * u);
     }
   };
-  int grp = blockIdx.x;
-  const bool any = warp < n_ch;
-  if (grp < n_groups && any) load(grp, warp);
+  int rb = blockIdx.x;
+  if (rb < p.n_rb && warp < n_ch) load(rb, warp);
 
   pdl_wait();
   pdl_launch_dependents();
 
   const size_t xs_stride = row_bytes + 16;   // bytes; 16 mod 32: two rows' reads, 32 bytes apart, do not meet in a bank
-  if constexpr (XS) {
+  {
     if (p.h) {
       int wpr = kGvWarps;                        // warps per row
       while (wpr * p.m > kGvWarps) wpr >>= 1;
@@ -146,75 +139,55 @@ __global__ void __launch_bounds__(kGvThreads, 2) dgemv_kernel(const __grid_const
     __syncthreads();
   }
   const bool live = g < p.m;
-  const uint8_t* xrow = XS ? gv_smem + (live ? g : 0) * xs_stride + 32 * t
-                           : reinterpret_cast<const uint8_t*>(p.x + (size_t)(live ? g : 0) * p.ldx) + 32 * t;
+  const uint8_t* xrow = gv_smem + (live ? g : 0) * xs_stride + 32 * t;
 
   int buf = 0;
-  for (; grp < n_groups; grp += gridDim.x) {
-    float acc[RB][4];
-#pragma unroll
-    for (int r = 0; r < RB; ++r) acc[r][0] = acc[r][1] = acc[r][2] = acc[r][3] = 0.f;
+  for (; rb < p.n_rb; rb += gridDim.x) {
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
     for (int c = warp; c < n_ch; c += kGvWarps) {
-      Frag32 cur[RB][U][2];
+      Frag32 cur[U][2];
 #pragma unroll
-      for (int r = 0; r < RB; ++r)
-#pragma unroll
-        for (int u = 0; u < U; ++u) {
-          cur[r][u][0] = nxt[r][u][0];
-          cur[r][u][1] = nxt[r][u][1];
-        }
+      for (int u = 0; u < U; ++u) {
+        cur[u][0] = nxt[u][0];
+        cur[u][1] = nxt[u][1];
+      }
       const bool more = c + kGvWarps < n_ch;
-      if (more || grp + (int)gridDim.x < n_groups) load(more ? grp : grp + gridDim.x, more ? c + kGvWarps : warp);
+      if (more || rb + (int)gridDim.x < p.n_rb) load(more ? rb : rb + gridDim.x, more ? c + kGvWarps : warp);
 #pragma unroll
       for (int u = 0; u < U; ++u) {
         uint4 xa = make_uint4(0u, 0u, 0u, 0u), xb = xa;
         if (live) {
-          const int k = c * kGvChunk + 64 * u + 16 * t;       // (shared memory is padded with zeros, global memory is not)
           const uint8_t* xp = xrow + (size_t)c * (kGvChunk * 2) + 128 * u;
-          if (XS || k + 16 <= p.cols) {
-            xa = *reinterpret_cast<const uint4*>(xp);
-            xb = *reinterpret_cast<const uint4*>(xp + 16);
-          } else if (k < p.cols) {
-            xa = x_tail(xp, p.cols - k);
-            if (k + 8 < p.cols) xb = x_tail(xp + 16, p.cols - k - 8);
-          }
+          xa = *reinterpret_cast<const uint4*>(xp);
+          xb = *reinterpret_cast<const uint4*>(xp + 16);
         }
         const uint32_t xw[8] = {xa.x, xa.y, xa.z, xa.w, xb.x, xb.y, xb.z, xb.w};
 #pragma unroll
-        for (int r = 0; r < RB; ++r)
-#pragma unroll
-          for (int i = 0; i < 4; ++i)
-            mma_bf16_16816(acc[r], cur[r][u][0].v[2 * i], cur[r][u][1].v[2 * i], cur[r][u][0].v[2 * i + 1], cur[r][u][1].v[2 * i + 1],
-                           xw[2 * i], xw[2 * i + 1]);
+        for (int i = 0; i < 4; ++i)
+          mma_bf16_16816(acc, cur[u][0].v[2 * i], cur[u][1].v[2 * i], cur[u][0].v[2 * i + 1], cur[u][1].v[2 * i + 1], xw[2 * i], xw[2 * i + 1]);
       }
     }
     // rows g, g + 8 x activation rows 2t, 2t + 1
-#pragma unroll
-    for (int r = 0; r < RB; ++r) {
-      float* d = red[buf][warp][r];
-      d[g * 8 + 2 * t] = acc[r][0];
-      d[g * 8 + 2 * t + 1] = acc[r][1];
-      d[(g + 8) * 8 + 2 * t] = acc[r][2];
-      d[(g + 8) * 8 + 2 * t + 1] = acc[r][3];
-    }
+    float* part = red[buf][warp];
+    part[g * 8 + 2 * t] = acc[0];
+    part[g * 8 + 2 * t + 1] = acc[1];
+    part[(g + 8) * 8 + 2 * t] = acc[2];
+    part[(g + 8) * 8 + 2 * t + 1] = acc[3];
     __syncthreads();
-    if (threadIdx.x < RB * 128) {
-      const int r = threadIdx.x >> 7, row = (threadIdx.x >> 3) & 15, m = threadIdx.x & 7;
-      const int rb = grp * RB + r;
-      if (rb < p.n_rb && m < p.m) {
-        const DenseDst d = dense_dst(p.epi, rb * 16 + row);
-        if (d.kind != DENSE_GLU || row < 8) {
-          float v = 0.f;
+    const int row = threadIdx.x >> 3, m = threadIdx.x & 7;
+    if (row < 16 && m < p.m) {
+      const DenseDst d = dense_dst(p.epi, rb * 16 + row);
+      if (d.kind != DENSE_GLU || row < 8) {
+        float v = 0.f;
 #pragma unroll
-          for (int w = 0; w < kGvWarps; ++w) v += red[buf][w][r][row * 8 + m];
-          if (d.kind == DENSE_GLU) {
-            float up = 0.f;
+        for (int w = 0; w < kGvWarps; ++w) v += red[buf][w][row * 8 + m];
+        if (d.kind == DENSE_GLU) {
+          float up = 0.f;
 #pragma unroll
-            for (int w = 0; w < kGvWarps; ++w) up += red[buf][w][r][(row + 8) * 8 + m];
-            v = clamped_glu(v, up, p.epi.glu_limit, p.epi.glu_alpha);
-          }
-          dense_store(p.epi, d, m, v);
+          for (int w = 0; w < kGvWarps; ++w) up += red[buf][w][(row + 8) * 8 + m];
+          v = clamped_glu(v, up, p.epi.glu_limit, p.epi.glu_alpha);
         }
+        dense_store(p.epi, d, m, v);
       }
     }
     buf ^= 1;
@@ -547,7 +520,7 @@ static int set_smem(tq_ctx* ctx, K kern, size_t bytes) {
   return TQ_OK;
 }
 
-static int launch_gemv(tq_ctx* ctx, const tq_dweight* w, const DenseInput& in, size_t m, const DenseEpilogue& epi, bool xs) {
+static int launch_gemv(tq_ctx* ctx, const tq_dweight* w, const DenseInput& in, size_t m, const DenseEpilogue& epi) {
   GemvParams p;
   p.w = static_cast<const __nv_bfloat16*>(w->data);
   p.kpad = (int)w->kpad;
@@ -562,19 +535,11 @@ static int launch_gemv(tq_ctx* ctx, const tq_dweight* w, const DenseInput& in, s
   p.gain = static_cast<const __nv_bfloat16*>(in.gain);
   p.eps = in.eps;
   p.epi = epi;
-  const size_t smem = xs ? m * (w->kpad * 2 + 16) : 0;
-  const int rb = xs ? 1 : 2;
-  int per_sm = 2;
-  while (per_sm > 1 && per_sm * (smem + 10 * 1024 * rb) > 220 * 1024) --per_sm;
-  const int groups = (p.n_rb + rb - 1) / rb;
-  int grid = ctx->sm_count * per_sm;
-  if (grid > groups) grid = groups;
-  if (xs) {
-    if (int st = set_smem(ctx, dgemv_kernel<1, true>, smem)) return st;
-    TQ_CUDA(ctx, launch_k(ctx, dgemv_kernel<1, true>, dim3((unsigned)grid), dim3(kGvThreads), smem, p));
-  } else {
-    TQ_CUDA(ctx, launch_k(ctx, dgemv_kernel<2, false>, dim3((unsigned)grid), dim3(kGvThreads), 0, p));
-  }
+  const size_t smem = m * (w->kpad * 2 + 16);
+  int grid = ctx->sm_count * 2;
+  if (grid > p.n_rb) grid = p.n_rb;
+  if (int st = set_smem(ctx, dgemv_kernel, smem)) return st;
+  TQ_CUDA(ctx, launch_k(ctx, dgemv_kernel, dim3((unsigned)grid), dim3(kGvThreads), smem, p));
   return TQ_OK;
 }
 
@@ -656,8 +621,7 @@ int launch_dense(tq_ctx* ctx, const tq_dweight* w, const DenseInput& in, size_t 
   }
   if (x.h && !(w->dtype == x.gain_dtype)) return fail(ctx, TQ_EINVAL, "dense linear: the norm's gain must have the weight's dtype");
   if (!x.h) TQ_REQUIRE(ctx, ((uintptr_t)x.x & 15) == 0 && x.ldx % 8 == 0, "dense linear: activation rows must be 16-byte aligned");
-  if (fits) return launch_gemv(ctx, w, x, m, epi, true);
-  if (m <= kGvRows) return launch_gemv(ctx, w, x, m, epi, false);
+  if (fits) return launch_gemv(ctx, w, x, m, epi);
   return launch_umma(ctx, w, x.x, x.ldx, m, epi);
 }
 

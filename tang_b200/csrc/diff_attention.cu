@@ -66,10 +66,11 @@ __device__ __forceinline__ void da_split(float a, float b, uint32_t& hi, uint32_
 
 // DVT: value columns / 8 (padded to 16 columns, so even).
 template <int DVT, bool SPLIT>
-__global__ void __launch_bounds__(SPLIT ? 128 : 256) diff_attention_kernel(const __grid_constant__ DiffParams p) {
+__global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 2) diff_attention_kernel(const __grid_constant__ DiffParams p) {
   constexpr int kThreads = SPLIT ? 128 : 256;
   constexpr int kWarps = kThreads / 32;
-  constexpr int NT = SPLIT ? 2 : 8;                 // 8-key tiles of scores per warp and key tile
+  constexpr int NT = SPLIT ? 2 : 4;                 // 8-key tiles of scores a warp forms at a time
+  constexpr int kSub = SPLIT ? 1 : kDaKeys / (8 * NT);   // such steps per key tile
   extern __shared__ __align__(128) uint8_t da_smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const int k_row = p.dp * 4 + 16;                  // bytes: both maps of a key, then a shift of one bank group per row
@@ -88,7 +89,8 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256) diff_attention_kernel(const
   const int row0 = p.b.seq_rows ? p.b.seq_rows[b] : b;
   const int n_q = p.b.seq_rows ? p.b.seq_rows[b + 1] - row0 : 1;
   const int pos_per_cta = SPLIT ? 1 : 64 / p.gb;
-  const int i0 = SPLIT ? 0 : blockIdx.x * pos_per_cta;     // first query of this CTA inside the sequence
+  // first query of this CTA inside the sequence; the last queries see the most keys and go first
+  const int i0 = SPLIT ? 0 : ((int)gridDim.x - 1 - (int)blockIdx.x) * pos_per_cta;
   if (i0 >= n_q || row0 < 0 || row0 + n_q > p.b.rows) return;
   const int i1 = min(i0 + pos_per_cta, n_q) - 1;
   const int p0 = p.b.row_pos[row0 + i0], p1 = p0 + (i1 - i0);
@@ -121,19 +123,29 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256) diff_attention_kernel(const
     __syncthreads();
   }
   const int kcm = p.a.dim_pad / 8, vcm = p.a.vdim_pad / 8;   // 16-byte pieces per map / value row
+  const int per_row = 2 * kcm + vcm;
+  const int row_first = threadIdx.x / per_row, c_first = threadIdx.x % per_row;
+  const int row_step = kThreads / per_row, c_step = kThreads % per_row;
   auto load_tile = [&](int li, int buf) {
     const int tile = li < n_kept ? li : lo_t + li - n_kept;
     const int key0 = tile * kDaKeys;
-    const int per_row = 2 * kcm + vcm;
-    for (int i = threadIdx.x; i < kDaKeys * per_row; i += kThreads) {
-      const int row = i / per_row, c = i - row * per_row;
+    // (row, piece) of this thread's copies, without a division per copy
+    int row = row_first, c = c_first;
+    while (row < kDaKeys) {
       const int key = key0 + row;
       const bool valid = key <= p1;
+      const size_t kr = (size_t)(valid ? key : p1);
       if (c < 2 * kcm) {
         const int mp = c >= kcm;
-        da_cp16(k_s + ((size_t)buf * kDaKeys + row) * k_row + mp * p.dp * 2 + (c - mp * kcm) * 16, kb + (size_t)(valid ? key : p1) * ke + c * 8, valid);
+        da_cp16(k_s + (buf * kDaKeys + row) * k_row + mp * p.dp * 2 + (c - mp * kcm) * 16, kb + kr * ke + c * 8, valid);
       } else {
-        da_cp16(v_s + ((size_t)buf * kDaKeys + row) * v_row + (c - 2 * kcm) * 16, vb + (size_t)(valid ? key : p1) * ve + (c - 2 * kcm) * 8, valid);
+        da_cp16(v_s + (buf * kDaKeys + row) * v_row + (c - 2 * kcm) * 16, vb + kr * ve + (c - 2 * kcm) * 8, valid);
+      }
+      row += row_step;
+      c += c_step;
+      if (c >= per_row) {
+        c -= per_row;
+        ++row;
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -141,14 +153,27 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256) diff_attention_kernel(const
   if (li0 < li1) load_tile(li0, 0);
 
   // ---- queries: pair r = 8 * warp + g (prefill) or g; both maps side by side like a key row
-  for (int i = threadIdx.x; i < q_rows * 2 * p.a.dim; i += kThreads) {
-    const int r = i / (2 * p.a.dim), c = i - r * 2 * p.a.dim;
-    const int mp = c >= p.a.dim, d = c - mp * p.a.dim;
-    const int qi = SPLIT ? 0 : r / p.gb, hh = SPLIT ? r : r % p.gb;
-    __nv_bfloat16 x = __float2bfloat16_rn(0.f);
-    if (i0 + qi <= i1 && (SPLIT || r < pos_per_cta * p.gb) && hh < gb)
-      x = p.q[(size_t)(row0 + i0 + qi) * p.ldq + (size_t)(2 * (head0 + hh) + mp) * p.a.dim + d];
-    *reinterpret_cast<__nv_bfloat16*>(q_s + (size_t)r * k_row + (mp * p.dp + d) * 2) = x;
+  if ((p.a.dim & 7) == 0 && (p.ldq & 7) == 0) {
+    const int pm = p.a.dim / 8;                            // 16-byte pieces per map
+    for (int i = threadIdx.x; i < q_rows * 2 * pm; i += kThreads) {
+      const int r = i / (2 * pm), c = i - r * 2 * pm;
+      const int mp = c >= pm;
+      const int qi = SPLIT ? 0 : r / p.gb, hh = SPLIT ? r : r % p.gb;
+      uint4 x = make_uint4(0u, 0u, 0u, 0u);
+      if (i0 + qi <= i1 && (SPLIT || r < pos_per_cta * p.gb) && hh < gb)
+        x = *reinterpret_cast<const uint4*>(p.q + (size_t)(row0 + i0 + qi) * p.ldq + (size_t)2 * (head0 + hh) * p.a.dim + c * 8);
+      *reinterpret_cast<uint4*>(q_s + (size_t)r * k_row + mp * p.dp * 2 + (c - mp * pm) * 16) = x;
+    }
+  } else {
+    for (int i = threadIdx.x; i < q_rows * 2 * p.a.dim; i += kThreads) {
+      const int r = i / (2 * p.a.dim), c = i - r * 2 * p.a.dim;
+      const int mp = c >= p.a.dim, d = c - mp * p.a.dim;
+      const int qi = SPLIT ? 0 : r / p.gb, hh = SPLIT ? r : r % p.gb;
+      __nv_bfloat16 x = __float2bfloat16_rn(0.f);
+      if (i0 + qi <= i1 && (SPLIT || r < pos_per_cta * p.gb) && hh < gb)
+        x = p.q[(size_t)(row0 + i0 + qi) * p.ldq + (size_t)(2 * (head0 + hh) + mp) * p.a.dim + d];
+      *reinterpret_cast<__nv_bfloat16*>(q_s + (size_t)r * k_row + (mp * p.dp + d) * 2) = x;
+    }
   }
 
   const int pr = SPLIT ? g : 8 * warp + g;                 // this lane's pair
@@ -174,11 +199,12 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256) diff_attention_kernel(const
     }
     __syncthreads();
     const int tile = li < n_kept ? li : lo_t + li - n_kept;
-    const int w0 = SPLIT ? 16 * warp : 0;                  // first key of the tile for this warp
-    const int key0 = tile * kDaKeys + w0;
-    if (key0 <= p1) {
-      const uint8_t* kt = k_s + ((size_t)buf * kDaKeys + w0) * k_row;
-      const uint8_t* vt = v_s + ((size_t)buf * kDaKeys + w0) * v_row;
+    for (int sub = 0; sub < kSub; ++sub) {
+      const int w0 = SPLIT ? 16 * warp : 8 * NT * sub;     // first key of the tile for this warp's step
+      const int key0 = tile * kDaKeys + w0;
+      if (key0 > p1) break;
+      const uint8_t* kt = k_s + (buf * kDaKeys + w0) * k_row;
+      const uint8_t* vt = v_s + (buf * kDaKeys + w0) * v_row;
       float s[NT][4];
 #pragma unroll
       for (int n = 0; n < NT; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
@@ -187,13 +213,13 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256) diff_attention_kernel(const
       for (int ks = 0; ks < nks; ++ks) {
         const uint32_t q10 = *reinterpret_cast<const uint32_t*>(qrow + 32 * ks), q11 = *reinterpret_cast<const uint32_t*>(qrow + 32 * ks + 16);
         const uint32_t q20 = *reinterpret_cast<const uint32_t*>(qrow + p.dp * 2 + 32 * ks), q21 = *reinterpret_cast<const uint32_t*>(qrow + p.dp * 2 + 32 * ks + 16);
+        uint32_t kf[NT][4];
 #pragma unroll
-        for (int n = 0; n < NT; ++n) {
-          uint32_t kf[4];
-          da_ldm4(kf, kaddr + (size_t)(8 * n) * k_row + 32 * ks);
-          mma_bf16_16816(s[n], q10, 0u, q11, 0u, kf[0], kf[1]);
-          mma_bf16_16816(s[n], 0u, q20, 0u, q21, kf[2], kf[3]);
-        }
+        for (int n = 0; n < NT; ++n) da_ldm4(kf[n], kaddr + 8 * n * k_row + 32 * ks);
+#pragma unroll
+        for (int n = 0; n < NT; ++n) mma_bf16_16816(s[n], q10, 0u, q11, 0u, kf[n][0], kf[n][1]);
+#pragma unroll
+        for (int n = 0; n < NT; ++n) mma_bf16_16816(s[n], 0u, q20, 0u, q21, kf[n][2], kf[n][3]);
       }
       float mx[2] = {-FLT_MAX, -FLT_MAX};
 #pragma unroll
@@ -243,14 +269,16 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256) diff_attention_kernel(const
         da_split(s[2 * kk + 1][0], s[2 * kk + 1][1], h2, r2);
         da_split(s[2 * kk + 1][2], s[2 * kk + 1][3], h3, r3);
         const uint8_t* vaddr = vt + (size_t)(16 * kk + (lane & 15)) * v_row + 16 * (lane >> 4);
+        // two column pairs at a time, the four leading terms before the four residual ones: no product waits for the last
 #pragma unroll
-        for (int j = 0; j < DVT / 2; ++j) {
-          uint32_t vf[4];
-          da_ldm4t(vf, vaddr + 32 * j);
-          mma_bf16_16816(o[2 * j], h0, h1, h2, h3, vf[0], vf[1]);
-          mma_bf16_16816(o[2 * j + 1], h0, h1, h2, h3, vf[2], vf[3]);
-          mma_bf16_16816(o[2 * j], r0, r1, r2, r3, vf[0], vf[1]);
-          mma_bf16_16816(o[2 * j + 1], r0, r1, r2, r3, vf[2], vf[3]);
+        for (int j = 0; j < DVT / 2; j += 2) {
+          uint32_t vf[2][4];
+          da_ldm4t(vf[0], vaddr + 32 * j);
+          da_ldm4t(vf[1], vaddr + 32 * j + 32);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) mma_bf16_16816(o[2 * j + i], h0, h1, h2, h3, vf[i >> 1][2 * (i & 1)], vf[i >> 1][2 * (i & 1) + 1]);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) mma_bf16_16816(o[2 * j + i], r0, r1, r2, r3, vf[i >> 1][2 * (i & 1)], vf[i >> 1][2 * (i & 1) + 1]);
         }
       }
     }
@@ -367,19 +395,18 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256) diff_attention_kernel(const
   }
 }
 
-// Merges the splits of one (row, head), forms the difference and the head norm.  One warp per head.
-__global__ void __launch_bounds__(128) diff_combine_kernel(const float* part_o, const float* part_ml, int n_splits, int W, DiffAttn a, int rows,
+// Merges the splits of one (row, head), forms the difference and the head norm.  One CTA per head, a thread per column.
+__global__ void __launch_bounds__(256) diff_combine_kernel(const float* part_o, const float* part_ml, int n_splits, int W, DiffAttn a,
                                                            const int* cache_row, __nv_bfloat16* out, long long ldo) {
+  __shared__ float wgt[2][kDaMaxSplits];                   // weight of each split in the head's result, 1 / l and lambda in it
+  __shared__ float red[8];
   pdl_wait();
   pdl_launch_dependents();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const size_t rh = (size_t)blockIdx.x * 4 + warp;         // row * heads + head
-  if (rh >= (size_t)rows * a.heads) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, d = threadIdx.x;
+  const size_t rh = blockIdx.x;                            // row * heads + head
   const int row = (int)(rh / a.heads), head = (int)(rh % a.heads);
   if (cache_row[row] < 0) return;
-  float wt[2][2], L[2];                                    // lane's splits: lane, lane + 32
-#pragma unroll
-  for (int mp = 0; mp < 2; ++mp) {
+  for (int mp = warp; mp < 2; mp += (int)(blockDim.x >> 5)) {
     const float* ml = part_ml + (rh * 2 + mp) * n_splits * 2;
     float m[2], l[2];
 #pragma unroll
@@ -389,35 +416,31 @@ __global__ void __launch_bounds__(128) diff_combine_kernel(const float* part_o, 
       l[i] = s < n_splits ? ml[2 * s + 1] : 0.f;
     }
     const float M = warp_max(fmaxf(m[0], m[1]));
-#pragma unroll
-    for (int i = 0; i < 2; ++i) wt[mp][i] = exp2f(m[i] - M);
-    L[mp] = warp_sum(l[0] * wt[mp][0] + l[1] * wt[mp][1]);
+    const float w0 = exp2f(m[0] - M), w1 = exp2f(m[1] - M);
+    const float L = warp_sum(l[0] * w0 + l[1] * w1);
+    const float f = (mp ? -a.lambda : 1.0f) / L;
+    wgt[mp][lane] = w0 * f;
+    wgt[mp][lane + 32] = w1 * f;
   }
-  float acc[2][8];                                         // W <= 256
-#pragma unroll
-  for (int i = 0; i < 8; ++i) acc[0][i] = acc[1][i] = 0.f;
-  for (int s = 0; s < n_splits; ++s)
-#pragma unroll
-    for (int mp = 0; mp < 2; ++mp) {
-      const float w = __shfl_sync(0xffffffffu, s < 32 ? wt[mp][0] : wt[mp][1], s & 31);
-      const float* src = part_o + ((rh * 2 + mp) * n_splits + s) * W;
-#pragma unroll
-      for (int i = 0; i < 8; ++i)
-        if (lane + 32 * i < W) acc[mp][i] += src[lane + 32 * i] * w;
+  __syncthreads();
+  float v = 0.f;
+  if (d < a.vdim) {
+    float acc[2] = {0.f, 0.f};
+    const float* src = part_o + rh * 2 * n_splits * W + d;
+#pragma unroll 8
+    for (int s = 0; s < n_splits; ++s) {
+      acc[0] += src[(size_t)s * W] * wgt[0][s];
+      acc[1] += src[(size_t)(n_splits + s) * W] * wgt[1][s];
     }
-  const float w1 = 1.0f / L[0], w2 = a.lambda / L[1];
-  float sq = 0.f;
-#pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    acc[0][i] = acc[0][i] * w1 - acc[1][i] * w2;
-    if (lane + 32 * i < a.vdim) sq += acc[0][i] * acc[0][i];
+    v = acc[0] + acc[1];
   }
-  sq = warp_sum(sq);
-  const float inv = a.out_scale / sqrtf(sq / (float)a.vdim + a.eps);
-  __nv_bfloat16* dst = out + (size_t)row * ldo + (size_t)head * a.vdim;
-#pragma unroll
-  for (int i = 0; i < 8; ++i)
-    if (lane + 32 * i < a.vdim) dst[lane + 32 * i] = __float2bfloat16_rn(acc[0][i] * inv);
+  const float sq = warp_sum(v * v);
+  if (lane == 0) red[warp] = sq;
+  __syncthreads();
+  float tot = 0.f;
+  for (int i = 0; i < (int)(blockDim.x >> 5); ++i) tot += red[i];
+  const float inv = a.out_scale / sqrtf(tot / (float)a.vdim + a.eps);
+  if (d < a.vdim) out[(size_t)row * ldo + (size_t)head * a.vdim + d] = __float2bfloat16_rn(v * inv);
 }
 
 // ------------------------------------------------------------------------------------------------ f32 / any size
@@ -607,8 +630,8 @@ int launch_diff_attention(tq_ctx* ctx, const DiffAttn& a, const DiffAttnBatch& b
   }
   if (st != TQ_OK) return st;
   if (p.n_splits > 1)
-    TQ_CUDA(ctx, launch_k(ctx, diff_combine_kernel, dim3((unsigned)(((size_t)b.rows * a.heads + 3) / 4)), dim3(128), 0, (const float*)p.part_o,
-                          (const float*)p.part_ml, p.n_splits, W, a, b.rows, b.cache_row, p.out, p.ldo));
+    TQ_CUDA(ctx, launch_k(ctx, diff_combine_kernel, dim3((unsigned)((size_t)b.rows * a.heads)), dim3((unsigned)((a.vdim + 31) / 32 * 32)), 0,
+                          (const float*)p.part_o, (const float*)p.part_ml, p.n_splits, W, a, b.cache_row, p.out, p.ldo));
   return TQ_OK;
 }
 

@@ -67,9 +67,9 @@ def test_dlinear_bf16(dev, shape):
     lin.free()
 
 
-def test_dlinear_bf16_wide_gemv_reads_global_activations(dev):
-    """Eight rows whose activations do not fit shared memory, a ragged last k chunk, padded row stride with garbage behind
-    the columns."""
+def test_dlinear_bf16_strided_activations(dev):
+    """Few rows on both sides of what the GEMV keeps in shared memory, a ragged last k chunk, a row stride with garbage
+    behind the columns."""
     import tang_b200 as tb
 
     rng = np.random.default_rng(4)
