@@ -42,9 +42,15 @@ struct DiffParams {
   int* err;
 };
 
-__device__ __forceinline__ void da_cp16(void* dst, const void* src, bool valid) {
+__device__ __forceinline__ void da_cp16(uint32_t dst, const void* src, bool valid) {
   const uint32_t n = valid ? 16u : 0u;
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(n) : "memory");
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
+}
+// 2^x for x <= 0: results below the normal range are zero.
+__device__ __forceinline__ float da_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 __device__ __forceinline__ void da_ldm4(uint32_t (&r)[4], const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
@@ -123,29 +129,27 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
     __syncthreads();
   }
   const int kcm = p.a.dim_pad / 8, vcm = p.a.vdim_pad / 8;   // 16-byte pieces per map / value row
+  // This thread copies piece `pc` of every row_step-th row of a tile (at most 96 pieces: a row has 2 * 32 + 32).
   const int per_row = 2 * kcm + vcm;
-  const int row_first = threadIdx.x / per_row, c_first = threadIdx.x % per_row;
-  const int row_step = kThreads / per_row, c_step = kThreads % per_row;
+  const int row_step = kThreads / per_row;
+  const int row_first = threadIdx.x / per_row, pc = threadIdx.x - row_first * per_row;
+  const bool copies = row_first < row_step, is_v = pc >= 2 * kcm;
+  const int mp_c = pc >= kcm ? 1 : 0;
+  const __nv_bfloat16* src_c = is_v ? vb + (pc - 2 * kcm) * 8 : kb + pc * 8;
+  const size_t src_ld = is_v ? ve : ke;
+  const int dst_ld = is_v ? v_row : k_row;
+  const uint32_t dst_c = smem_u32(is_v ? v_s + (pc - 2 * kcm) * 16 : k_s + mp_c * p.dp * 2 + (pc - mp_c * kcm) * 16);
   auto load_tile = [&](int li, int buf) {
-    const int tile = li < n_kept ? li : lo_t + li - n_kept;
-    const int key0 = tile * kDaKeys;
-    // (row, piece) of this thread's copies, without a division per copy
-    int row = row_first, c = c_first;
-    while (row < kDaKeys) {
-      const int key = key0 + row;
-      const bool valid = key <= p1;
-      const size_t kr = (size_t)(valid ? key : p1);
-      if (c < 2 * kcm) {
-        const int mp = c >= kcm;
-        da_cp16(k_s + (buf * kDaKeys + row) * k_row + mp * p.dp * 2 + (c - mp * kcm) * 16, kb + kr * ke + c * 8, valid);
-      } else {
-        da_cp16(v_s + (buf * kDaKeys + row) * v_row + (c - 2 * kcm) * 16, vb + kr * ve + (c - 2 * kcm) * 8, valid);
-      }
-      row += row_step;
-      c += c_step;
-      if (c >= per_row) {
-        c -= per_row;
-        ++row;
+    const int key0 = (li < n_kept ? li : lo_t + li - n_kept) * kDaKeys;
+    if (copies) {
+      const __nv_bfloat16* src = src_c + (size_t)(key0 + row_first) * src_ld;
+      uint32_t dst = dst_c + (uint32_t)((buf * kDaKeys + row_first) * dst_ld);
+      const int n_valid = p1 + 1 - key0;                   // rows at or beyond it become zeros
+#pragma unroll 4
+      for (int row = row_first; row < kDaKeys; row += row_step) {
+        da_cp16(dst, row < n_valid ? src : src_c, row < n_valid);
+        src += row_step * src_ld;
+        dst += (uint32_t)(row_step * dst_ld);
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -185,7 +189,7 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
   float o[DVT][4];                                         // [columns 8j + 2t, +1] of map 1, then of map 2
 #pragma unroll
   for (int j = 0; j < DVT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-  float m_run[2] = {-FLT_MAX, -FLT_MAX}, l_run[2] = {0.f, 0.f};
+  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   const float sl2 = p.a.scale * kDaLog2e;
   const int nks = p.dp / 16;
 
@@ -221,24 +225,36 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
 #pragma unroll
         for (int n = 0; n < NT; ++n) mma_bf16_16816(s[n], 0u, q20, 0u, q21, kf[n][2], kf[n][3]);
       }
-      float mx[2] = {-FLT_MAX, -FLT_MAX};
+      // a step whose keys every query of the CTA sees needs no mask (rows without a query are never stored)
+      const bool full = key0 + 8 * NT - 1 <= p0 && (p1 - key0 < p.a.window || key0 + 8 * NT <= p.a.keep_first);
+      float mx[2] = {-INFINITY, -INFINITY};
+      if (full) {
 #pragma unroll
-      for (int n = 0; n < NT; ++n)
+        for (int n = 0; n < NT; ++n)
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          const int key = key0 + 8 * n + 2 * t + (c & 1);
-          const bool ok = live && key <= qpos && (qpos - key < p.a.window || key < p.a.keep_first);
-          const float v = ok ? s[n][c] * sl2 : -FLT_MAX;
-          s[n][c] = v;
-          mx[c >> 1] = fmaxf(mx[c >> 1], v);
-        }
-      float alpha[2];
+          for (int c = 0; c < 4; ++c) {
+            s[n][c] *= sl2;
+            mx[c >> 1] = fmaxf(mx[c >> 1], s[n][c]);
+          }
+      } else {
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            const int key = key0 + 8 * n + 2 * t + (c & 1);
+            const bool ok = live && key <= qpos && (qpos - key < p.a.window || key < p.a.keep_first);
+            s[n][c] = ok ? s[n][c] * sl2 : -INFINITY;
+            mx[c >> 1] = fmaxf(mx[c >> 1], s[n][c]);
+          }
+      }
+      float alpha[2], base[2];
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
         mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
         mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
         const float mn = fmaxf(m_run[h], mx[h]);
-        alpha[h] = exp2f(m_run[h] - mn);
+        base[h] = mn == -INFINITY ? 0.f : mn;              // (nothing seen yet: every weight below becomes zero)
+        alpha[h] = da_ex2(m_run[h] - base[h]);
         m_run[h] = mn;
       }
       float ps[2] = {0.f, 0.f};
@@ -246,9 +262,8 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
       for (int n = 0; n < NT; ++n)
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-          const float w = s[n][c] == -FLT_MAX ? 0.f : exp2f(s[n][c] - m_run[c >> 1]);
-          s[n][c] = w;
-          ps[c >> 1] += w;
+          s[n][c] = da_ex2(s[n][c] - base[c >> 1]);
+          ps[c >> 1] += s[n][c];
         }
       l_run[0] = l_run[0] * alpha[0] + ps[0];
       l_run[1] = l_run[1] * alpha[1] + ps[1];
@@ -331,9 +346,10 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
 #pragma unroll
       for (int c = 0; c < 4; ++c) mo[((size_t)warp * 16 + g + 8 * (c >> 1)) * W + 8 * j + 2 * t + (c & 1)] = o[j][c];
     if (t == 0) {
-      mml[(warp * 16 + g) * 2] = m_run[0];
+      // (a finite stand-in for "no key seen": its weight is zero beside any real maximum)
+      mml[(warp * 16 + g) * 2] = fmaxf(m_run[0], -FLT_MAX);
       mml[(warp * 16 + g) * 2 + 1] = l_run[0];
-      mml[(warp * 16 + g + 8) * 2] = m_run[1];
+      mml[(warp * 16 + g + 8) * 2] = fmaxf(m_run[1], -FLT_MAX);
       mml[(warp * 16 + g + 8) * 2 + 1] = l_run[1];
     }
     __syncthreads();
