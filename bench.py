@@ -12,6 +12,7 @@ weak and the aggregate is the sum over ranks.
     python bench.py --gpus 1 --steps 50 --warmup 5
     python -m torch.distributed.run --nnodes=1 --nproc-per-node N ... bench.py --gpus N ...
     python bench.py --impl reference        # the CPU restatement of tang-infer on the host cores
+    python bench.py --tofazen               # instead: the Tofazen family beside the int4 model (one JSON line of its own)
 
 The JSON line also carries: `e2e` (the same rate through the reference-shaped call q4_matvec with
 HOST vectors, copies inside the timed region), `roofline` (dominant kernel vs measured HBM peak),

@@ -513,6 +513,7 @@ __global__ void __launch_bounds__(256) dgemm_f32_kernel(const float* w, int kpad
 // ------------------------------------------------------------------------------------------------ launches
 constexpr size_t kGvSmemMax = 100 * 1024;   // activations of the GEMV in shared memory (two CTAs per SM)
 constexpr size_t kGvRows = 8;
+constexpr size_t kGvNormRows = 2;           // up to here every CTA of the GEMV norms the rows itself; above, a kernel of its own does
 
 template <typename K>
 static int set_smem(tq_ctx* ctx, K kern, size_t bytes) {
@@ -605,7 +606,7 @@ int launch_dense(tq_ctx* ctx, const tq_dweight* w, const DenseInput& in, size_t 
   const bool bf = w->dtype == TQ_BF16;
   const bool fits = m <= kGvRows && m * (w->kpad * 2 + 16) <= kGvSmemMax;
   DenseInput x = in;
-  if (in.h && !(bf && fits)) {
+  if (in.h && !(bf && fits && m <= kGvNormRows)) {
     TQ_REQUIRE(ctx, in.xn_tmp != nullptr, "dense linear: no buffer for the normalised rows");
     if (int st = launch_rms_norm_rows(ctx, in.h, in.ldh, in.h_rows, in.gain, in.gain_dtype, m, w->cols, in.eps, in.xn_tmp,
                                       bf ? TQ_BF16 : TQ_F32, w->kpad)) return st;
