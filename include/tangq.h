@@ -519,6 +519,97 @@ TQ_API int tq_tofazen_hidden(tq_tofazen* model, float** hidden_dev);
 /* While set, every step also copies the stream after each layer to streams [n_layers][rows][width] (NULL turns it off). */
 TQ_API int tq_tofazen_trace(tq_tofazen* model, float* streams_dev_or_null);
 
+/* ---- row operators, windowed attention, gated linear attention, routing to dense experts --------
+ * No reference counterpart.  All take the ragged rows above (row_pos and cache_row of tq_embedding_pos). */
+/* Frequencies of a rotary embedding, host arrays: base^(-2i/dims), and with factor > 0 stretched by YaRN (divided by `factor`
+ * for pairs with fewer than `slow` turns over `original` positions, kept above `fast`, blended between).  *mult: the factor
+ * on cosine and sine, 0.1 ln(factor) + 1 (1 without scaling). */
+TQ_API int tq_yarn_frequencies(size_t dims, double base, double factor, double original, double fast, double slow, float* freq_host,
+                               float* mult_host);
+/* Per row: y = sum of n_y rows of y (y_rows[m * n_y + i], negative: none; y_rows NULL: row m);  x += y / rms(y) * gain_post;
+ * out = x / rms(x) * gain_next.  f32 x, y and gains; y NULL: only the second half, gain_next NULL: only the first. */
+TQ_API int tq_add_norm(tq_ctx* ctx, float* x_dev, const float* y_dev_or_null, const int* y_rows_dev_or_null, size_t n_y,
+                       const float* gain_post_dev_or_null, const float* gain_next_dev_or_null, size_t rows, size_t width, float eps,
+                       void* out_dev_or_null, int out_dtype, size_t ld_out);
+/* Queries [rows][ldq] and the raw keys of the rows' cache rows [kv_heads][dim rounded up to 8] are divided by their root mean
+ * square over the whole projection, multiplied by the gains, and the first rot_dims dimensions of every head rotated
+ * (dimension i with i + rot_dims / 2).  Queries in place, keys to the same rows of another cache. */
+TQ_API int tq_qk_norm_rope(tq_ctx* ctx, int dtype, size_t heads, size_t kv_heads, size_t dim, void* q_dev, size_t ldq, const void* raw_dev,
+                           void* keys_dev, size_t cache_rows, const void* q_gain_dev, const void* k_gain_dev, size_t rot_dims,
+                           const float* freq_dev, float rot_mult, float eps, const int* row_pos_dev, const int* cache_row_dev, size_t rows);
+/* Grouped-query attention: s = (q . k) scale, softcap * tanh(s / softcap) unless softcap is 0; weights
+ * exp(s_j) / (exp(sink) + sum exp(s)) (sink -infinity: none); the query at position i sees j when 0 <= i - j < window; the
+ * result times sigmoid(gate).  q [rows][ldq], gate (may be NULL) [rows][ldg], caches as in tq_diff_attention with one map. */
+typedef struct tq_window_attn_config {
+  uint32_t heads, kv_heads, dim, vdim;
+  uint32_t window;
+  float scale, softcap, sink;
+} tq_window_attn_config;
+TQ_API int tq_window_attention(tq_ctx* ctx, const tq_window_attn_config* cfg, int dtype, const void* q_dev, size_t ldq,
+                               const void* gate_dev_or_null, size_t ldg, const void* k_cache_dev, const void* v_cache_dev, size_t cache_rows,
+                               const int* seq_rows_dev_or_null, const int* row_pos_dev, const int* cache_row_dev, size_t n_seqs, size_t rows,
+                               size_t max_q, size_t max_len, void* out_dev, size_t ldo);
+/* Gated linear attention: S_t = diag(alpha_t) S_(t-1) + k_t v_t^T, o_t = S_t^T (q_scale q_t), per head, with
+ * alpha_t = sigmoid(a2 a1_t + bias)^(1/tau) per key channel; out = o / sqrt(mean(o^2) + eps) * norm * silu(gate).  Rows of q, k
+ * (heads * dim), v, gate (heads * vdim) are `ld` elements apart, a1 [rows][ld_a1] and everything about the state is f32.
+ * state [slots][heads][dim][vdim], slot = cache_row / max_seq; a sequence's position 0 starts from zero. */
+typedef struct tq_gla_config {
+  uint32_t heads, dim, vdim, rank;
+  float tau, q_scale, eps;
+} tq_gla_config;
+TQ_API int tq_gla(tq_ctx* ctx, const tq_gla_config* cfg, int dtype, const void* q_dev, const void* k_dev, const void* v_dev, const void* gate_dev,
+                  size_t ld, const float* a1_dev, size_t ld_a1, const float* a2_dev, const float* a2_bias_dev, const float* norm_dev,
+                  float* state_dev, size_t max_seq, size_t cache_rows, const int* seq_rows_dev_or_null, const int* row_pos_dev,
+                  const int* cache_row_dev, size_t n_seqs, size_t rows, size_t max_q, void* out_dev, size_t ldo);
+/* The `top` experts with the largest logits [rows][experts] per row (the lower index among equals) with weights sigmoid(z)
+ * (score 0) or softmax (score 1), divided by their sum if renorm.  Pair p = row * top + i gets a slot; the slots of an expert are
+ * consecutive.  jobs int[.][4]: (expert, first slot, slots <= chunk, 0), at most min(pairs, experts + pairs / chunk). */
+TQ_API int tq_route(tq_ctx* ctx, const float* logits_dev, size_t rows, size_t experts, size_t top, int score, int renorm, size_t chunk,
+                    int* expert_dev, float* weight_dev, int* slot_dev, int* slot_row_dev, int* jobs_dev, int* n_jobs_dev);
+
+/* ---- Numuzen ------------------------------------------------------------------------------------
+ * No reference counterpart.  A decoder with a norm before and after every sublayer (weights stored around zero),
+ *   x <- x + norm1b(mixer(norm1(x)));  x <- x + norm2b(experts(norm2(x))),
+ * whose mixers are windowed attention (whole-projection query/key norm, YaRN rotation, capped scores, a sink of score 0, output
+ * gate, the raw keys as values) or gated linear attention, with sigmoid-routed experts whose weight multiplies their input,
+ * the clamped GLU (sigmoid factor 1.702) and tied embeddings.  The model owns weights, caches, states (one slot per sequence)
+ * and workspaces.  dtype TQ_BF16: bf16 weights, activations and caches; stream, norms, scores, router, recurrences f32; TQ_F32:
+ * everything f32. */
+typedef struct tq_numuzen tq_numuzen;
+typedef struct tq_numuzen_config {
+  uint32_t n_layers, width, vocab;
+  uint32_t max_seq;        /* positions per slot */
+  uint32_t max_slots;
+  int dtype;
+  float eps;
+} tq_numuzen_config;
+typedef enum tq_numuzen_mixer { TQ_NZ_ATTENTION = 0, TQ_NZ_GLA = 1 } tq_numuzen_mixer;
+typedef struct tq_numuzen_layer {
+  uint32_t kind;
+  uint32_t heads, kv_heads, dim, vdim;   /* kv_heads: attention only */
+  uint32_t window, rot_dims;             /* attention */
+  uint32_t rank;                         /* recurrent: rows of a1 */
+  uint32_t experts, top, ff;             /* experts = 0: no feed-forward */
+  float scale;                           /* attention: of the scores; recurrent: of the queries */
+  float softcap, tau, limit;
+  double rot_base, rot_factor, rot_original, rot_fast, rot_slow;   /* rot_factor = 0: no scaling */
+} tq_numuzen_layer;
+typedef enum tq_numuzen_tensor {
+  TQ_NZ_EMBED = 0, TQ_NZ_FINAL_NORM = 1, TQ_NZ_NORM1 = 2, TQ_NZ_NORM1B = 3, TQ_NZ_NORM2 = 4, TQ_NZ_NORM2B = 5, TQ_NZ_Q = 6, TQ_NZ_K = 7,
+  TQ_NZ_V = 8, TQ_NZ_G = 9, TQ_NZ_O = 10, TQ_NZ_Q_NORM = 11, TQ_NZ_K_NORM = 12, TQ_NZ_O_NORM = 13, TQ_NZ_A1 = 14, TQ_NZ_A2 = 15,
+  TQ_NZ_A2_BIAS = 16, TQ_NZ_ROUTER = 17, TQ_NZ_GATE = 18, TQ_NZ_UP = 19, TQ_NZ_DOWN = 20
+} tq_numuzen_tensor;
+TQ_API int tq_numuzen_create(tq_ctx* ctx, const tq_numuzen_config* cfg, const tq_numuzen_layer* layers, tq_numuzen** out);
+TQ_API int tq_numuzen_destroy(tq_numuzen* model);
+/* As tq_tofazen_put; `expert` counts for gate, up and down. */
+TQ_API int tq_numuzen_put(tq_numuzen* model, int tensor, size_t layer, size_t expert, const void* src, int src_dtype, size_t rows, size_t cols);
+/* As tq_tofazen_step; a sequence's recurrent states advance with its rows, and its position 0 starts them from zero. */
+TQ_API int tq_numuzen_step(tq_numuzen* model, const int* token_ids_dev, size_t rows, const int* seq_rows_dev_or_null, const int* starts_dev,
+                           const int* slots_dev_or_null, size_t n_seqs, size_t max_q, size_t max_len, const int* logit_rows_dev_or_null,
+                           size_t n_logits, float* logits_dev);
+TQ_API int tq_numuzen_hidden(tq_numuzen* model, float** hidden_dev);
+TQ_API int tq_numuzen_trace(tq_numuzen* model, float* streams_dev_or_null);
+
 /* ---- CUDA graphs ------------------------------------------------------------------------------
  * CudaComputeDevice::begin_capture / end_capture (crates/tang-compute/src/cuda.rs:344-356): every
  * asynchronous call made on the context between begin and end is recorded instead of run, and

@@ -21,7 +21,8 @@ NVCC_FLAGS = [
 
 # sources of the partial libraries (name -> csrc/*.cu stems)
 COMPONENTS = {
-    "dense": ["api_core", "graph", "ops", "sampler", "dense", "diff_attention", "tofazen"],
+    "dense": ["api_core", "graph", "ops", "sampler", "dense", "rowops", "expert_route", "diff_attention",
+              "window_attention", "gla", "tofazen", "numuzen"],
 }
 
 

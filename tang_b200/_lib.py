@@ -112,6 +112,18 @@ PROTOTYPES = {
     "tq_tofazen_step": (_i, [_p, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _p, _sz, _p]),
     "tq_tofazen_hidden": (_i, [_p, _pp]),
     "tq_tofazen_trace": (_i, [_p, _p]),
+    "tq_yarn_frequencies": (_i, [_sz] + [C.c_double] * 5 + [_p, _p]),
+    "tq_add_norm": (_i, [_p, _p, _p, _p, _sz, _p, _p, _sz, _sz, C.c_float, _p, _i, _sz]),
+    "tq_qk_norm_rope": (_i, [_p, _i, _sz, _sz, _sz, _p, _sz, _p, _p, _sz, _p, _p, _sz, _p, C.c_float, C.c_float, _p, _p, _sz]),
+    "tq_window_attention": (_i, [_p, _p, _i, _p, _sz, _p, _sz, _p, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _sz, _p, _sz]),
+    "tq_gla": (_i, [_p, _p, _i, _p, _p, _p, _p, _sz, _p, _sz, _p, _p, _p, _p, _sz, _sz, _p, _p, _p, _sz, _sz, _sz, _p, _sz]),
+    "tq_route": (_i, [_p, _p, _sz, _sz, _sz, _i, _i, _sz, _p, _p, _p, _p, _p, _p]),
+    "tq_numuzen_create": (_i, [_p, _p, _p, _pp]),
+    "tq_numuzen_destroy": (_i, [_p]),
+    "tq_numuzen_put": (_i, [_p, _i, _sz, _sz, _p, _i, _sz, _sz]),
+    "tq_numuzen_step": (_i, [_p, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _p, _sz, _p]),
+    "tq_numuzen_hidden": (_i, [_p, _pp]),
+    "tq_numuzen_trace": (_i, [_p, _p]),
     "tq_graph_begin": (_i, [_p]),
     "tq_graph_end": (_i, [_p, _pp]),
     "tq_graph_launch": (_i, [_p, _p]),

@@ -27,6 +27,7 @@ struct GemvParams {
   const int* h_rows;
   const __nv_bfloat16* gain;
   float eps;
+  DenseGroups grp;                  // GROUPED only
   DenseEpilogue epi;
 };
 
@@ -56,6 +57,8 @@ __device__ __forceinline__ uint4 x_tail(const void* src, int n) {
 // read one 128-byte line): words 2i, 2i + 1 are the two k halves of MMA i; the activations are read the same way.  The loads of
 // the next step -- of the next block too -- are issued before the current step is multiplied, and the first ones before
 // the kernel waits for its predecessor (weights do not change).  The activations sit in shared memory.
+// GROUPED: a CTA walks a contiguous range of (job, 16-row block) pairs and stages a job's activations when it comes to it.
+template <bool GROUPED>
 __global__ void __launch_bounds__(kGvThreads, 2) dgemv_kernel(const __grid_constant__ GemvParams p) {
   constexpr int U = 2;                               // 64-k loads per row and step: 32 registers in flight
   constexpr int kGvChunk = 64 * U;                   // k per warp step
@@ -76,14 +79,31 @@ __global__ void __launch_bounds__(kGvThreads, 2) dgemv_kernel(const __grid_const
       nxt[u][1] = ldg_stream(src + 8 * row_bytes + 128 * u);
     }
   };
-  int rb = blockIdx.x;
-  if (rb < p.n_rb && warp < n_ch) load(rb, warp);
+  // tile -> 16-row block of the weight
+  int tile = blockIdx.x, tile_end = p.n_rb;
+  const int tile_step = GROUPED ? 1 : gridDim.x;
+  auto row_block = [&](int tl) {
+    if constexpr (!GROUPED) return tl;
+    return p.grp.jobs[tl / p.n_rb].x * (int)(p.grp.group_rows / 16) + tl % p.n_rb;
+  };
+  if constexpr (GROUPED) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const long long n = (long long)min(*p.grp.n_jobs, p.grp.max_jobs) * p.n_rb;
+    tile = (int)(n * blockIdx.x / gridDim.x);
+    tile_end = (int)(n * (blockIdx.x + 1) / gridDim.x);
+    if (tile >= tile_end) return;
+  }
+  if (tile < tile_end && warp < n_ch) load(row_block(tile), warp);
 
-  pdl_wait();
-  pdl_launch_dependents();
+  if constexpr (!GROUPED) {
+    pdl_wait();
+    pdl_launch_dependents();
+  }
 
   const size_t xs_stride = row_bytes + 16;   // bytes; 16 mod 32: two rows' reads, 32 bytes apart, do not meet in a bank
-  {
+  int m_rows = p.m, m_first = 0, job = -1;
+  if constexpr (!GROUPED) {
     if (p.h) {
       int wpr = kGvWarps;                        // warps per row
       while (wpr * p.m > kGvWarps) wpr >>= 1;
@@ -138,11 +158,34 @@ __global__ void __launch_bounds__(kGvThreads, 2) dgemv_kernel(const __grid_const
     }
     __syncthreads();
   }
-  const bool live = g < p.m;
+  bool live = g < m_rows;
   const uint8_t* xrow = gv_smem + (live ? g : 0) * xs_stride + 32 * t;
 
   int buf = 0;
-  for (; rb < p.n_rb; rb += gridDim.x) {
+  for (; tile < tile_end; tile += tile_step) {
+    if constexpr (GROUPED) {
+      if (tile / p.n_rb != job) {                // (the barrier of the previous block was behind its last read of the activations)
+        job = tile / p.n_rb;
+        const int4 jb = p.grp.jobs[job];
+        m_first = jb.y;
+        m_rows = min(jb.z, p.grp.chunk);
+        const int vpr = p.kpad / 8;
+        for (int i = threadIdx.x; i < m_rows * vpr; i += kGvThreads) {
+          const int row = i / vpr, c = i % vpr;
+          const int xr = p.grp.x_rows ? p.grp.x_rows[m_first + row] : m_first + row;
+          uint4 v = make_uint4(0u, 0u, 0u, 0u);
+          const __nv_bfloat16* src = p.x + (size_t)xr * p.ldx + 8 * c;
+          if (8 * c + 8 <= p.cols) v = *reinterpret_cast<const uint4*>(src);
+          else if (8 * c < p.cols) v = x_tail(src, p.cols - 8 * c);
+          *reinterpret_cast<uint4*>(gv_smem + row * xs_stride + 16 * c) = v;
+        }
+        __syncthreads();
+        live = g < m_rows;
+        xrow = gv_smem + (live ? g : 0) * xs_stride + 32 * t;
+      }
+    }
+    const bool last_tile = tile + tile_step >= tile_end;
+    const int rb = row_block(tile), rb_next = last_tile ? 0 : row_block(tile + tile_step);
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
     for (int c = warp; c < n_ch; c += kGvWarps) {
       Frag32 cur[U][2];
@@ -152,7 +195,7 @@ __global__ void __launch_bounds__(kGvThreads, 2) dgemv_kernel(const __grid_const
         cur[u][1] = nxt[u][1];
       }
       const bool more = c + kGvWarps < n_ch;
-      if (more || rb + (int)gridDim.x < p.n_rb) load(more ? rb : rb + gridDim.x, more ? c + kGvWarps : warp);
+      if (more || !last_tile) load(more ? rb : rb_next, more ? c + kGvWarps : warp);
 #pragma unroll
       for (int u = 0; u < U; ++u) {
         uint4 xa = make_uint4(0u, 0u, 0u, 0u), xb = xa;
@@ -175,19 +218,21 @@ __global__ void __launch_bounds__(kGvThreads, 2) dgemv_kernel(const __grid_const
     part[(g + 8) * 8 + 2 * t + 1] = acc[3];
     __syncthreads();
     const int row = threadIdx.x >> 3, m = threadIdx.x & 7;
-    if (row < 16 && m < p.m) {
-      const DenseDst d = dense_dst(p.epi, rb * 16 + row);
+    if (row < 16 && m < m_rows) {
+      const DenseDst d = dense_dst(p.epi, (GROUPED ? tile % p.n_rb : rb) * 16 + row);
       if (d.kind != DENSE_GLU || row < 8) {
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < kGvWarps; ++w) v += red[buf][w][row * 8 + m];
+        const float scale = p.epi.row_scale ? p.epi.row_scale[m_first + m] : 1.f;
+        v *= scale;
         if (d.kind == DENSE_GLU) {
           float up = 0.f;
 #pragma unroll
           for (int w = 0; w < kGvWarps; ++w) up += red[buf][w][(row + 8) * 8 + m];
-          v = clamped_glu(v, up, p.epi.glu_limit, p.epi.glu_alpha);
+          v = clamped_glu(v, up * scale, p.epi.glu_limit, p.epi.glu_alpha);
         }
-        dense_store(p.epi, d, m, v);
+        dense_store(p.epi, d, m_first + m, v);
       }
     }
     buf ^= 1;
@@ -209,6 +254,8 @@ struct DUmmaParams {
   int n_acc, acc_stride, tmem_cols;
   float* partial;                    // [splits][m][n_ft * 128], splits > 1
   int* counters;                     // one per (feature tile, row tile), zero between launches
+  int grouped;                       // tiles are (job, feature tile), listed by grp (n_tiles bounds them)
+  DenseGroups grp;
   DenseEpilogue epi;
   int* err;
 };
@@ -252,7 +299,15 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
     atomicCAS(p.err, 0, code);
   };
   // tile -> (feature tile, row tile, K split): splits fastest, then row tiles, so that the CTAs of a wave share weights
+  // (grouped: tt is the job)
   auto coords = [&](int tile, int& ft, int& tt, int& kb0, int& kbn, int& z) {
+    if (p.grouped) {
+      z = kb0 = 0;
+      kbn = p.kb_total;
+      tt = tile / p.n_ft;
+      ft = tile % p.n_ft;
+      return;
+    }
     z = tile % p.splits;
     const int q = tile / p.splits;
     tt = q % p.n_tt;
@@ -261,12 +316,17 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
     kbn = min(p.kb_per_split, p.kb_total - kb0);
   };
 
+  // the number of tiles and a tile's first weight row / activation row; grouped: only behind the wait
+  auto tiles_total = [&]() { return p.grouped ? min(*p.grp.n_jobs, p.grp.max_jobs) * p.n_ft : p.n_tiles; };
+  auto w_row = [&](int ft, int tt) { return ft * kUmmaRows + (p.grouped ? p.grp.jobs[tt].x * (int)p.grp.group_rows : 0); };
+  auto x_row = [&](int tt) { return p.grouped ? p.grp.jobs[tt].y : tt * p.ntok; };
+
   if (warp == 0) {
     if (lane == 0) {
       // The weights of the first stages do not depend on the previous kernel: their copies start before the wait.
       int ft, tt, kb0, kbn, z;
       int pre = 0;
-      if ((int)blockIdx.x < p.n_tiles) {
+      if (!p.grouped && (int)blockIdx.x < p.n_tiles) {
         coords(blockIdx.x, ft, tt, kb0, kbn, z);
         pre = min(S, kbn);
         for (int s = 0; s < pre; ++s) {
@@ -278,8 +338,10 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
       int s = 0;
       uint32_t ph = 0;
       bool ok = true;
-      for (int tile = blockIdx.x; tile < p.n_tiles && ok; tile += gridDim.x) {
+      const int n_tiles = tiles_total();
+      for (int tile = blockIdx.x; tile < n_tiles && ok; tile += gridDim.x) {
         coords(tile, ft, tt, kb0, kbn, z);
+        const int wr = w_row(ft, tt), xr = x_row(tt);
         for (int kb = 0; kb < kbn; ++kb) {
           uint8_t* st = tiles_s + (size_t)s * stage_bytes;
           if (pre > 0) {
@@ -288,9 +350,9 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
             ok = !*failed && mbar_wait_spin(&empty[s], ph ^ 1u);
             if (!ok) { give_up(DERR_EMPTY_WAIT); break; }
             mbar_arrive_expect_tx(&full[s], stage_bytes);
-            tma_load_2d(st, &w_map, (kb0 + kb) * kUmmaK, ft * kUmmaRows, &full[s]);
+            tma_load_2d(st, &w_map, (kb0 + kb) * kUmmaK, wr, &full[s]);
           }
-          tma_load_2d(st + kUmmaRows * 128, &x_map, (kb0 + kb) * kUmmaK, tt * p.ntok, &full[s]);
+          tma_load_2d(st + kUmmaRows * 128, &x_map, (kb0 + kb) * kUmmaK, xr, &full[s]);
           if (++s == S) {
             s = 0;
             ph ^= 1u;
@@ -300,6 +362,8 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
     }
     __syncwarp();
   } else if (warp == 1) {
+    if (p.grouped) pdl_wait();
+    const int n_tiles = tiles_total();
     const bool leader = elect_one();
     const uint32_t idesc = umma_idesc_bf16(p.ntok);
     const uint64_t desc0 = umma_desc_sw128(tiles_s);
@@ -307,7 +371,7 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
     int s = 0, a = 0;
     uint32_t ph = 0, aph = 0;
     bool ok = true;
-    for (int tile = blockIdx.x; tile < p.n_tiles && ok; tile += gridDim.x) {
+    for (int tile = blockIdx.x; tile < n_tiles && ok; tile += gridDim.x) {
       int ft, tt, kb0, kbn, z;
       coords(tile, ft, tt, kb0, kbn, z);
       ok = !*failed && mbar_wait_spin(&acc_empty[a], aph ^ 1u);
@@ -346,7 +410,8 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
     int a = 0;
     uint32_t aph = 0;
     const int n_pad = p.n_ft * kUmmaRows;
-    for (int tile = blockIdx.x; tile < p.n_tiles; tile += gridDim.x) {
+    const int n_tiles = tiles_total();
+    for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x) {
       int ft, tt, kb0, kbn, z;
       coords(tile, ft, tt, kb0, kbn, z);
       // (after a failure every warp still walks all tiles, without touching memory: the named barriers below stay matched)
@@ -354,7 +419,7 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
       if (!good) give_up(DERR_TMEM);
       tc_fence_after();
       const int row = ft * kUmmaRows + 32 * q + lane;
-      const int m0 = tt * p.ntok, m_n = good ? min(p.ntok, p.m - m0) : 0;
+      const int m0 = x_row(tt), m_n = good ? min(p.ntok, p.grouped ? p.grp.jobs[tt].z : p.m - m0) : 0;
       const uint32_t t_addr = tmem_d + (uint32_t)(a * p.acc_stride) + ((uint32_t)(32 * q) << 16);
       const DenseDst dst = dense_dst(p.epi, row);
       for (int c0 = 16 * half; c0 < m_n; c0 += 32) {
@@ -367,6 +432,11 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
           for (int j = 0; j < 16; ++j)
             if (j < n) __stcg(pp + (size_t)j * n_pad, v[j]);
           continue;
+        }
+        if (p.epi.row_scale) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j)
+            if (j < n) v[j] *= p.epi.row_scale[mb + j];
         }
         // a half-warp's rows share a section, so the shuffles below are only ever needed by lanes that agree on the kind
         const bool glu = dst.kind == DENSE_GLU;
@@ -466,21 +536,31 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
 // 64 activation rows x 64 features per CTA, 16 k per step; every operation is an f32 FMA in ascending k.
 constexpr int kDfTile = 64, kDfK = 16;
 
+// Grouped (jobs given): blockIdx.y is the job, rpad a group's rows.
 __global__ void __launch_bounds__(256) dgemm_f32_kernel(const float* w, int kpad, int rpad, const float* x, long long ldx, int m, int cols,
-                                                        const __grid_constant__ DenseEpilogue epi) {
+                                                        const __grid_constant__ DenseGroups grp, const __grid_constant__ DenseEpilogue epi) {
   __shared__ __align__(16) float xs[kDfK][kDfTile + 4], ws[kDfK][kDfTile + 4];
   __shared__ float ys[kDfTile][kDfTile + 1];
   pdl_wait();
   pdl_launch_dependents();
-  const int n0 = blockIdx.x * kDfTile, m0 = blockIdx.y * kDfTile;
+  const int n0 = blockIdx.x * kDfTile;
+  int m0 = blockIdx.y * kDfTile;
+  if (grp.jobs) {
+    if ((int)blockIdx.y >= *grp.n_jobs) return;
+    const int4 job = grp.jobs[blockIdx.y];
+    w += (size_t)job.x * grp.group_rows * kpad;
+    m0 = job.y;
+    m = min(m, m0 + min(job.z, kDfTile));
+  }
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;      // features 4 tx.., rows 4 ty..
   const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4; // this thread's share of the loads
   float acc[4][4] = {};
+  const float* xrow = x + (size_t)(m0 + lr < m ? (grp.x_rows ? grp.x_rows[m0 + lr] : m0 + lr) : 0) * ldx;
   for (int k0 = 0; k0 < cols; k0 += kDfK) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int k = k0 + lk + i;
-      xs[lk + i][lr] = m0 + lr < m && k < cols ? x[(size_t)(m0 + lr) * ldx + k] : 0.f;
+      xs[lk + i][lr] = m0 + lr < m && k < cols ? xrow[k] : 0.f;
       ws[lk + i][lr] = n0 + lr < rpad && k < cols ? w[(size_t)(n0 + lr) * kpad + k] : 0.f;
     }
     __syncthreads();
@@ -504,8 +584,9 @@ __global__ void __launch_bounds__(256) dgemm_f32_kernel(const float* w, int kpad
   const DenseDst d = dense_dst(epi, n0 + n);
   if (d.kind == DENSE_GLU && (n & 8)) return;
   for (int r = threadIdx.x >> 6; r < kDfTile && m0 + r < m; r += 4) {
-    float v = ys[r][n];
-    if (d.kind == DENSE_GLU) v = clamped_glu(v, ys[r][n + 8], epi.glu_limit, epi.glu_alpha);
+    const float scale = epi.row_scale ? epi.row_scale[m0 + r] : 1.f;
+    float v = ys[r][n] * scale;
+    if (d.kind == DENSE_GLU) v = clamped_glu(v, ys[r][n + 8] * scale, epi.glu_limit, epi.glu_alpha);
     dense_store(epi, d, m0 + r, v);
   }
 }
@@ -535,48 +616,60 @@ static int launch_gemv(tq_ctx* ctx, const tq_dweight* w, const DenseInput& in, s
   p.h_rows = in.h_rows;
   p.gain = static_cast<const __nv_bfloat16*>(in.gain);
   p.eps = in.eps;
+  p.grp = DenseGroups();
   p.epi = epi;
   const size_t smem = m * (w->kpad * 2 + 16);
   int grid = ctx->sm_count * 2;
   if (grid > p.n_rb) grid = p.n_rb;
-  if (int st = set_smem(ctx, dgemv_kernel, smem)) return st;
-  TQ_CUDA(ctx, launch_k(ctx, dgemv_kernel, dim3((unsigned)grid), dim3(kGvThreads), smem, p));
+  if (int st = set_smem(ctx, dgemv_kernel<false>, smem)) return st;
+  TQ_CUDA(ctx, launch_k(ctx, dgemv_kernel<false>, dim3((unsigned)grid), dim3(kGvThreads), smem, p));
   return TQ_OK;
 }
 
-static int launch_umma(tq_ctx* ctx, const tq_dweight* w, const void* x, size_t ldx, size_t m, const DenseEpilogue& epi) {
+static int launch_umma(tq_ctx* ctx, const tq_dweight* w, const void* x, size_t ldx, size_t m, const DenseEpilogue& epi, const DenseGroups* groups = nullptr) {
   if (!w->has_map) return fail(ctx, TQ_EUNSUPPORTED, "cuTensorMapEncodeTiled is not available from this driver");
   TQ_REQUIRE(ctx, ((uintptr_t)x & 15) == 0 && ldx % 8 == 0, "dense linear: activation rows must be 16-byte aligned");
   DUmmaParams p;
   p.m = (int)m;
-  p.n_ft = (int)((w->rpad + kUmmaRows - 1) / kUmmaRows);
+  p.grouped = groups != nullptr;
+  p.grp = groups ? *groups : DenseGroups();
+  p.n_ft = (int)(((groups ? groups->group_rows : w->rpad) + kUmmaRows - 1) / kUmmaRows);
   p.kb_total = (int)((w->cols + kUmmaK - 1) / kUmmaK);
-  // Row tile: the width that makes (waves of CTAs) x (width) smallest; the wider one on a tie.
   int ntok = 16;
-  long long best = 0;
-  for (int cand = 256; cand >= 16; cand -= 16) {
-    if (cand > 16 && (size_t)(cand - 15) > m && cand - 16 >= (int)m) continue;     // wider than the rows need
-    const long long tiles = (long long)p.n_ft * (long long)((m + cand - 1) / cand);
-    const long long waves = (tiles + ctx->sm_count - 1) / ctx->sm_count;
-    const long long cost = waves * (cand < 96 ? 96 : cand);   // (below about 96 rows a step costs the same)
-    if (best == 0 || cost < best) {
-      best = cost;
-      ntok = cand;
+  if (groups) {
+    ntok = groups->chunk;
+    p.n_tt = groups->max_jobs;
+    p.splits = 1;
+    p.kb_per_split = p.kb_total;
+    TQ_REQUIRE(ctx, (long long)p.n_ft * p.n_tt < (1ll << 31), "dense linear: too many jobs");
+    p.n_tiles = p.n_ft * p.n_tt;
+  } else {
+    // Row tile: the width that makes (waves of CTAs) x (width) smallest; the wider one on a tie.
+    long long best = 0;
+    for (int cand = 256; cand >= 16; cand -= 16) {
+      if (cand > 16 && (size_t)(cand - 15) > m && cand - 16 >= (int)m) continue;     // wider than the rows need
+      const long long tiles = (long long)p.n_ft * (long long)((m + cand - 1) / cand);
+      const long long waves = (tiles + ctx->sm_count - 1) / ctx->sm_count;
+      const long long cost = waves * (cand < 96 ? 96 : cand);   // (below about 96 rows a step costs the same)
+      if (best == 0 || cost < best) {
+        best = cost;
+        ntok = cand;
+      }
     }
+    p.n_tt = (int)((m + ntok - 1) / ntok);
+    const int base = p.n_ft * p.n_tt;
+    int splits = 1;
+    if (base <= ctx->sm_count / 2 && base <= kTileCounters && !epi.row_scale) {
+      splits = ctx->sm_count / base;
+      if (splits > p.kb_total / 4) splits = p.kb_total / 4;    // at least four 64-k steps each
+      if (splits > 16) splits = 16;
+      if (splits < 1) splits = 1;
+    }
+    p.kb_per_split = (p.kb_total + splits - 1) / splits;
+    p.splits = (p.kb_total + p.kb_per_split - 1) / p.kb_per_split;
+    p.n_tiles = base * p.splits;
   }
   p.ntok = ntok;
-  p.n_tt = (int)((m + ntok - 1) / ntok);
-  const int base = p.n_ft * p.n_tt;
-  int splits = 1;
-  if (base <= ctx->sm_count / 2 && base <= kTileCounters) {
-    splits = ctx->sm_count / base;
-    if (splits > p.kb_total / 4) splits = p.kb_total / 4;    // at least four 64-k steps each
-    if (splits > 16) splits = 16;
-    if (splits < 1) splits = 1;
-  }
-  p.kb_per_split = (p.kb_total + splits - 1) / splits;
-  p.splits = (p.kb_total + p.kb_per_split - 1) / p.kb_per_split;
-  p.n_tiles = base * p.splits;
   p.acc_stride = ntok <= 32 ? 32 : ntok <= 64 ? 64 : ntok <= 128 ? 128 : 256;
   p.n_acc = 2;
   p.tmem_cols = 2 * p.acc_stride;
@@ -600,13 +693,59 @@ static int launch_umma(tq_ctx* ctx, const tq_dweight* w, const void* x, size_t l
   return TQ_OK;
 }
 
+int dense_group_chunk(int dtype, size_t kpad, size_t rows, size_t n_groups) {
+  if (dtype == TQ_F32) return kDfTile;
+  const size_t mean = (rows + n_groups - 1) / n_groups;
+  size_t gv = kGvSmemMax / (kpad * 2 + 16);
+  if (gv > kGvRows) gv = kGvRows;
+  if (mean <= 4 && gv > 0) return (int)gv;
+  const size_t want = (mean + mean / 4 + 15) / 16 * 16;      // most groups in one job each
+  return (int)(want > 256 ? 256 : want);
+}
+
+int launch_dense_grouped(tq_ctx* ctx, const tq_dweight* w, const void* x, size_t ldx, size_t rows, const DenseGroups& g, const DenseEpilogue& epi) {
+  if (rows == 0) return TQ_OK;
+  TQ_REQUIRE(ctx, g.jobs && g.n_jobs && g.max_jobs > 0 && g.chunk > 0 && g.group_rows > 0 && g.group_rows % 16 == 0, "grouped dense linear: bad groups");
+  TQ_REQUIRE(ctx, epi.n >= 1 && epi.n <= kDenseMaxSections && epi.s[epi.n - 1].row_end <= (int)g.group_rows, "grouped dense linear: bad output sections");
+  if (w->dtype == TQ_F32) {
+    TQ_REQUIRE(ctx, g.chunk == kDfTile && g.max_jobs <= 65535, "grouped dense linear: f32 jobs have up to %d rows", kDfTile);
+    TQ_CUDA(ctx, launch_k(ctx, dgemm_f32_kernel, dim3((unsigned)((g.group_rows + kDfTile - 1) / kDfTile), (unsigned)g.max_jobs), dim3(256), 0,
+                          static_cast<const float*>(w->data), (int)w->kpad, (int)g.group_rows, static_cast<const float*>(x), (long long)ldx, (int)rows,
+                          (int)w->cols, g, epi));
+    return TQ_OK;
+  }
+  TQ_REQUIRE(ctx, ((uintptr_t)x & 15) == 0 && ldx % 8 == 0, "dense linear: activation rows must be 16-byte aligned");
+  if (g.chunk > (int)kGvRows) {
+    TQ_REQUIRE(ctx, g.chunk % 16 == 0 && g.chunk <= 256 && !g.x_rows, "grouped dense linear: bad job size");
+    return launch_umma(ctx, w, x, ldx, rows, epi, &g);
+  }
+  GemvParams p = {};
+  p.w = static_cast<const __nv_bfloat16*>(w->data);
+  p.kpad = (int)w->kpad;
+  p.n_rb = (int)(g.group_rows / 16);
+  p.x = static_cast<const __nv_bfloat16*>(x);
+  p.ldx = (long long)ldx;
+  p.m = g.chunk;
+  p.cols = (int)w->cols;
+  p.grp = g;
+  p.epi = epi;
+  const size_t smem = g.chunk * (w->kpad * 2 + 16);
+  TQ_REQUIRE(ctx, smem <= kGvSmemMax, "grouped dense linear: rows too long for the job size");
+  const long long tiles = (long long)p.n_rb * g.max_jobs;
+  TQ_REQUIRE(ctx, tiles < (1ll << 31), "dense linear: too many jobs");
+  const int grid = (int)(tiles < ctx->sm_count * 2 ? tiles : ctx->sm_count * 2);
+  if (int st = set_smem(ctx, dgemv_kernel<true>, smem)) return st;
+  TQ_CUDA(ctx, launch_k(ctx, dgemv_kernel<true>, dim3((unsigned)grid), dim3(kGvThreads), smem, p));
+  return TQ_OK;
+}
+
 int launch_dense(tq_ctx* ctx, const tq_dweight* w, const DenseInput& in, size_t m, const DenseEpilogue& epi) {
   if (m == 0) return TQ_OK;
   TQ_REQUIRE(ctx, epi.n >= 1 && epi.n <= kDenseMaxSections && epi.s[epi.n - 1].row_end <= (int)w->rpad, "dense linear: bad output sections");
   const bool bf = w->dtype == TQ_BF16;
   const bool fits = m <= kGvRows && m * (w->kpad * 2 + 16) <= kGvSmemMax;
   DenseInput x = in;
-  if (in.h && !(bf && fits && m <= kGvNormRows)) {
+  if (in.h && !(bf && fits && m <= kGvNormRows && in.gain_dtype == TQ_BF16)) {
     TQ_REQUIRE(ctx, in.xn_tmp != nullptr, "dense linear: no buffer for the normalised rows");
     if (int st = launch_rms_norm_rows(ctx, in.h, in.ldh, in.h_rows, in.gain, in.gain_dtype, m, w->cols, in.eps, in.xn_tmp,
                                       bf ? TQ_BF16 : TQ_F32, w->kpad)) return st;
@@ -617,10 +756,9 @@ int launch_dense(tq_ctx* ctx, const tq_dweight* w, const DenseInput& in, size_t 
   if (!bf) {
     TQ_CUDA(ctx, launch_k(ctx, dgemm_f32_kernel, dim3((unsigned)((w->rpad + kDfTile - 1) / kDfTile), (unsigned)((m + kDfTile - 1) / kDfTile)),
                           dim3(256), 0, static_cast<const float*>(w->data), (int)w->kpad, (int)w->rpad, static_cast<const float*>(x.x),
-                          (long long)x.ldx, (int)m, (int)w->cols, epi));
+                          (long long)x.ldx, (int)m, (int)w->cols, DenseGroups(), epi));
     return TQ_OK;
   }
-  if (x.h && !(w->dtype == x.gain_dtype)) return fail(ctx, TQ_EINVAL, "dense linear: the norm's gain must have the weight's dtype");
   if (!x.h) TQ_REQUIRE(ctx, ((uintptr_t)x.x & 15) == 0 && x.ldx % 8 == 0, "dense linear: activation rows must be 16-byte aligned");
   if (fits) return launch_gemv(ctx, w, x, m, epi);
   return launch_umma(ctx, w, x.x, x.ldx, m, epi);

@@ -30,7 +30,7 @@ struct tq_dweight {
 
 namespace tq {
 
-constexpr int kDenseMaxSections = 4;
+constexpr int kDenseMaxSections = 5;
 
 enum DenseOutKind : int {
   DENSE_ROW = 0,     // out[m * ld + column]
@@ -56,6 +56,7 @@ struct DenseEpilogue {
   DenseSection s[kDenseMaxSections];
   const int* cache_row = nullptr;
   float mult = 1.f;                       // DENSE_RESID
+  const float* row_scale = nullptr;       // factor on the products of every activation row (before the GLU); not with K splits
   float glu_limit = 0.f, glu_alpha = 0.f; // DENSE_GLU
 };
 
@@ -133,6 +134,23 @@ struct DenseInput {
 };
 
 int launch_dense(tq_ctx* ctx, const tq_dweight* w, const DenseInput& in, size_t m, const DenseEpilogue& epi);
+
+// Several weights of one shape stacked by rows in one handle (experts): a job multiplies rows first .. first + n - 1 of the
+// activations with group g's rows g * group_rows ...  The job list is written on the device by an earlier kernel.
+struct DenseGroups {
+  const int4* jobs = nullptr;      // (group, first row, rows, unused); rows <= chunk
+  const int* n_jobs = nullptr;
+  int max_jobs = 0;                // bounds *n_jobs
+  int chunk = 0;                   // dense_group_chunk
+  size_t group_rows = 0;           // multiple of 16
+  const int* x_rows = nullptr;     // where activation row i is in x; null: row i.  Not with chunks above 8 of bf16 weights
+};
+
+// Rows per job that suit `rows` activation rows spread over n_groups, for weights with these padded columns: up to 8 the
+// GEMV runs, above the tcgen05 kernel; f32 weights always take 64.
+int dense_group_chunk(int dtype, size_t kpad, size_t rows, size_t n_groups);
+// The epilogue's sections describe one group's rows; its row indices are activation rows (`first` of a job onwards).
+int launch_dense_grouped(tq_ctx* ctx, const tq_dweight* w, const void* x, size_t ldx, size_t rows, const DenseGroups& groups, const DenseEpilogue& epi);
 
 // rms_norm of rows of an f32 matrix, output row stride ld_out (csrc/ops.cu).
 int launch_rms_norm_rows(tq_ctx* ctx, const float* x, size_t ldx, const int* rows, const void* gain, int gain_dtype, size_t n,

@@ -19,12 +19,12 @@
 
 #include <cfloat>
 
+#include "attn_mma.cuh"
 #include "common.cuh"
 
 namespace tq {
 
 constexpr int kDaKeys = 64;
-constexpr float kDaLog2e = 1.4426950408889634f;
 constexpr int kDaMaxSplits = 64;
 
 struct DiffParams {
@@ -32,7 +32,7 @@ struct DiffParams {
   __nv_bfloat16* out;
   long long ldq, ldo;
   DiffAttn a;
-  DiffAttnBatch b;
+  RaggedBatch b;
   int group, gb, n_hb;         // heads per KV head; heads per block; blocks per KV head
   int dp;                      // dim rounded up to 16
   int stages;
@@ -41,34 +41,6 @@ struct DiffParams {
   float* part_ml;              // [rows][heads][2][n_splits][2]
   int* err;
 };
-
-__device__ __forceinline__ void da_cp16(uint32_t dst, const void* src, bool valid) {
-  const uint32_t n = valid ? 16u : 0u;
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
-}
-// 2^x for x <= 0: results below the normal range are zero.
-__device__ __forceinline__ float da_ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-__device__ __forceinline__ void da_ldm4(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void da_ldm4t(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ uint32_t da_pack(float lo, float hi) {
-  const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-  return *reinterpret_cast<const uint32_t*>(&v);
-}
-// Splits two weights into bf16 terms: hi + lo keeps 16 significant bits.
-__device__ __forceinline__ void da_split(float a, float b, uint32_t& hi, uint32_t& lo) {
-  hi = da_pack(a, b);
-  lo = da_pack(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xFFFF0000u));
-}
 
 // DVT: value columns / 8 (padded to 16 columns, so even).
 template <int DVT, bool SPLIT>
@@ -147,7 +119,7 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
       const int n_valid = p1 + 1 - key0;                   // rows at or beyond it become zeros
 #pragma unroll 4
       for (int row = row_first; row < kDaKeys; row += row_step) {
-        da_cp16(dst, row < n_valid ? src : src_c, row < n_valid);
+        cp_async16(dst, row < n_valid ? src : src_c, row < n_valid);
         src += row_step * src_ld;
         dst += (uint32_t)(row_step * dst_ld);
       }
@@ -190,7 +162,7 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
 #pragma unroll
   for (int j = 0; j < DVT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
-  const float sl2 = p.a.scale * kDaLog2e;
+  const float sl2 = p.a.scale * kLog2e;
   const int nks = p.dp / 16;
 
   for (int li = li0; li < li1; ++li) {
@@ -219,7 +191,7 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
         const uint32_t q20 = *reinterpret_cast<const uint32_t*>(qrow + p.dp * 2 + 32 * ks), q21 = *reinterpret_cast<const uint32_t*>(qrow + p.dp * 2 + 32 * ks + 16);
         uint32_t kf[NT][4];
 #pragma unroll
-        for (int n = 0; n < NT; ++n) da_ldm4(kf[n], kaddr + 8 * n * k_row + 32 * ks);
+        for (int n = 0; n < NT; ++n) ldmatrix4(kf[n], kaddr + 8 * n * k_row + 32 * ks);
 #pragma unroll
         for (int n = 0; n < NT; ++n) mma_bf16_16816(s[n], q10, 0u, q11, 0u, kf[n][0], kf[n][1]);
 #pragma unroll
@@ -254,7 +226,7 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
         mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
         const float mn = fmaxf(m_run[h], mx[h]);
         base[h] = mn == -INFINITY ? 0.f : mn;              // (nothing seen yet: every weight below becomes zero)
-        alpha[h] = da_ex2(m_run[h] - base[h]);
+        alpha[h] = ex2_ftz(m_run[h] - base[h]);
         m_run[h] = mn;
       }
       float ps[2] = {0.f, 0.f};
@@ -262,7 +234,7 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
       for (int n = 0; n < NT; ++n)
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-          s[n][c] = da_ex2(s[n][c] - base[c >> 1]);
+          s[n][c] = ex2_ftz(s[n][c] - base[c >> 1]);
           ps[c >> 1] += s[n][c];
         }
       l_run[0] = l_run[0] * alpha[0] + ps[0];
@@ -279,17 +251,17 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
 #pragma unroll
       for (int kk = 0; kk < NT / 2; ++kk) {
         uint32_t h0, h1, h2, h3, r0, r1, r2, r3;
-        da_split(s[2 * kk][0], s[2 * kk][1], h0, r0);
-        da_split(s[2 * kk][2], s[2 * kk][3], h1, r1);
-        da_split(s[2 * kk + 1][0], s[2 * kk + 1][1], h2, r2);
-        da_split(s[2 * kk + 1][2], s[2 * kk + 1][3], h3, r3);
+        split_bf16(s[2 * kk][0], s[2 * kk][1], h0, r0);
+        split_bf16(s[2 * kk][2], s[2 * kk][3], h1, r1);
+        split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], h2, r2);
+        split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], h3, r3);
         const uint8_t* vaddr = vt + (size_t)(16 * kk + (lane & 15)) * v_row + 16 * (lane >> 4);
         // two column pairs at a time, the four leading terms before the four residual ones: no product waits for the last
 #pragma unroll
         for (int j = 0; j < DVT / 2; j += 2) {
           uint32_t vf[2][4];
-          da_ldm4t(vf[0], vaddr + 32 * j);
-          da_ldm4t(vf[1], vaddr + 32 * j + 32);
+          ldmatrix4_t(vf[0], vaddr + 32 * j);
+          ldmatrix4_t(vf[1], vaddr + 32 * j + 32);
 #pragma unroll
           for (int i = 0; i < 4; ++i) mma_bf16_16816(o[2 * j + i], h0, h1, h2, h3, vf[i >> 1][2 * (i & 1)], vf[i >> 1][2 * (i & 1) + 1]);
 #pragma unroll
@@ -329,7 +301,7 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
     for (int j = 0; j < DVT; ++j) {
       const int d = 8 * j + 2 * t;
       if (even) {
-        if (d < vd) *reinterpret_cast<uint32_t*>(dst + d) = da_pack(o[j][0] * inv, o[j][1] * inv);
+        if (d < vd) *reinterpret_cast<uint32_t*>(dst + d) = pack_bf16(o[j][0] * inv, o[j][1] * inv);
       } else {
         if (d < vd) dst[d] = __float2bfloat16_rn(o[j][0] * inv);
         if (d + 1 < vd) dst[d + 1] = __float2bfloat16_rn(o[j][1] * inv);
@@ -468,7 +440,7 @@ __device__ __forceinline__ void da_store(__nv_bfloat16* p, float v) { *p = __flo
 // One CTA per (row, head); 128 keys at a time, one per thread; then every thread owns value columns.
 template <typename T>
 __global__ void __launch_bounds__(128) diff_attention_simt_kernel(const T* q, long long ldq, const T* k, const T* v, T* out, long long ldo,
-                                                                  DiffAttn a, DiffAttnBatch b) {
+                                                                  DiffAttn a, RaggedBatch b) {
   extern __shared__ float ds_smem[];
   float* qs = ds_smem;                       // [2][dim]
   float* acc = qs + 2 * a.dim;               // [2][vdim]
@@ -544,7 +516,7 @@ __global__ void __launch_bounds__(128) diff_attention_simt_kernel(const T* q, lo
 
 // ------------------------------------------------------------------------------------------------ launch
 template <typename T>
-static int launch_simt(tq_ctx* ctx, const DiffAttn& a, const DiffAttnBatch& b, const void* q, size_t ldq, const void* k, const void* v,
+static int launch_simt(tq_ctx* ctx, const DiffAttn& a, const RaggedBatch& b, const void* q, size_t ldq, const void* k, const void* v,
                        void* out, size_t ldo) {
   const size_t smem = ((size_t)2 * a.dim + 2 * a.vdim + 256) * sizeof(float);
   if (smem > 200 * 1024) return fail(ctx, TQ_EUNSUPPORTED, "differential attention: head sizes %d / %d are too large", a.dim, a.vdim);
@@ -565,7 +537,7 @@ static int launch_mma(tq_ctx* ctx, DiffParams& p, bool split, size_t smem, dim3 
   return split ? go(diff_attention_kernel<DVT, true>, 128) : go(diff_attention_kernel<DVT, false>, 256);
 }
 
-int launch_diff_attention(tq_ctx* ctx, const DiffAttn& a, const DiffAttnBatch& b, int dtype, const void* q, size_t ldq, const void* k_cache,
+int launch_diff_attention(tq_ctx* ctx, const DiffAttn& a, const RaggedBatch& b, int dtype, const void* q, size_t ldq, const void* k_cache,
                           const void* v_cache, void* out, size_t ldo) {
   TQ_REQUIRE(ctx, a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0, "differential attention: heads must be a multiple of kv_heads");
   TQ_REQUIRE(ctx, a.dim > 0 && a.vdim > 0 && a.dim_pad >= a.dim && a.vdim_pad >= a.vdim && a.dim_pad % 8 == 0 && a.vdim_pad % 8 == 0,
@@ -616,7 +588,7 @@ int launch_diff_attention(tq_ctx* ctx, const DiffAttn& a, const DiffAttnBatch& b
     // about four CTAs per SM, at least two key tiles each
     const int kept_tiles = (a.keep_first + kDaKeys - 1) / kDaKeys;
     long long tiles = (b.max_len + kDaKeys - 1) / kDaKeys;
-    const long long win_tiles = (long long)(a.window - 1 + kDaKeys - 1) / kDaKeys + 1 + kept_tiles;
+    const long long win_tiles = ((long long)a.window - 1 + kDaKeys - 1) / kDaKeys + 1 + kept_tiles;
     if (win_tiles < tiles) tiles = win_tiles;
     const long long ctas = (long long)a.kv_heads * p.n_hb * b.n_seqs;
     long long n = (4ll * ctx->sm_count + ctas - 1) / ctas;

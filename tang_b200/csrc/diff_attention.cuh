@@ -5,6 +5,7 @@
 #pragma once
 
 #include "internal.h"
+#include "ragged.h"
 
 namespace tq {
 
@@ -16,18 +17,9 @@ struct DiffAttn {
   float scale = 0.f, lambda = 0.f, out_scale = 1.f, eps = 0.f;
 };
 
-struct DiffAttnBatch {
-  int n_seqs = 0, rows = 0, max_q = 1;   // rows of q in total; the longest sequence's rows
-  int max_len = 0;                       // bounds every position + 1
-  const int* seq_rows = nullptr;         // [n_seqs + 1] first row of each sequence; null: one row each
-  const int* row_pos = nullptr;          // [rows] position of each row
-  const int* cache_row = nullptr;        // [rows] its cache row (slot * max_seq + position); negative: the row is skipped
-  size_t cache_rows = 0;                 // rows of the cache: nothing at or beyond is read
-};
-
 // q [rows][ldq], head h's map m at column (2h + m) * dim; out [rows][ldo], head h at column h * vdim.  dtype (TQ_BF16 or
 // TQ_F32) is that of q, keys, values and out; in TQ_F32 every operation is f32.
-int launch_diff_attention(tq_ctx* ctx, const DiffAttn& a, const DiffAttnBatch& b, int dtype, const void* q, size_t ldq, const void* k_cache,
+int launch_diff_attention(tq_ctx* ctx, const DiffAttn& a, const RaggedBatch& b, int dtype, const void* q, size_t ldq, const void* k_cache,
                           const void* v_cache, void* out, size_t ldo);
 
 }  // namespace tq

@@ -164,6 +164,28 @@ inline cudaError_t launch_k(tq_ctx* ctx, void (*kern)(KArgs...), dim3 grid, dim3
   return cudaLaunchKernelEx(&cfg, kern, KArgs(args)...);
 }
 
+// The same for a kernel whose blocks form clusters of `cluster` along x.
+template <typename... KArgs, typename... Args>
+inline cudaError_t launch_k_cluster(tq_ctx* ctx, void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, int cluster, Args... args) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid;
+  cfg.blockDim = block;
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = ctx->stream;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = (unsigned)cluster;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = ctx->pdl ? 2 : 1;
+  ctx->launches++;
+  ctx->inflight_unknown = true;
+  ctx->n_inflight = 0;
+  return cudaLaunchKernelEx(&cfg, kern, KArgs(args)...);
+}
+
 // The same launch for a kernel that neither reads nor writes anything a kernel in flight touches and that waits for
 // nothing before its last instruction (the host-vector staging kernel): what the context knows about the kernels
 // in flight stays valid.

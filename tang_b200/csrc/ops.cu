@@ -8,6 +8,7 @@
 
 #include "common.cuh"
 #include "internal.h"
+#include "ragged.h"
 
 namespace tq {
 
@@ -242,18 +243,21 @@ int launch_rms_norm_rows(tq_ctx* ctx, const float* x, size_t ldx, const int* row
   } else if (gain_dtype == TQ_F32 && out_dtype == TQ_F32) {
     TQ_CUDA(ctx, launch_k(ctx, rms_norm_vec_kernel<float, float, float>, grid, block, 0, x, none, (const float*)gain, (int)dim, eps,
                           (float*)out, no_sum, rows, ldx, ld_out));
+  } else if (gain_dtype == TQ_F32 && out_dtype == TQ_BF16) {
+    TQ_CUDA(ctx, launch_k(ctx, rms_norm_vec_kernel<float, float, bf>, grid, block, 0, x, none, (const float*)gain, (int)dim, eps, (bf*)out,
+                          no_sum, rows, ldx, ld_out));
   } else {
-    return fail(ctx, TQ_EUNSUPPORTED, "rms_norm rows: gain and output must share a dtype");
+    return fail(ctx, TQ_EUNSUPPORTED, "rms_norm rows: an f32 output needs an f32 gain");
   }
   return TQ_OK;
 }
 
-// Token embedding plus a learned vector per absolute position, and the bookkeeping of a step over several sequences at
+// Token embedding (plus a learned vector per absolute position when there is a table of them), and the bookkeeping of a step over several sequences at
 // once: rows seq_rows[b] .. seq_rows[b+1]-1 (null: row b) are the next tokens of sequence b, whose first one sits at
 // position starts[b]; its cache is slot slots[b] (null: b) of `max_seq` rows.  Every row's position and cache row are
 // left for the kernels that follow; a position or slot outside the cache gives cache row -1 (nothing is stored for it)
 // and is reported through the status word.  One CTA per row.
-__global__ void __launch_bounds__(256) embedding_pos_kernel(const void* table, const void* pos_table, int dt, const int* ids, const int* seq_rows,
+__global__ void __launch_bounds__(256) embedding_pos_kernel(const void* table, size_t ld_table, const void* pos_table, int dt, const int* ids, const int* seq_rows,
                                                             const int* starts, const int* slots, int n_seqs, int dim, int vocab,
                                                             int n_pos, int max_seq, int n_slots, float* out, int* row_pos, int* cache_row,
                                                             int* err) {
@@ -281,16 +285,16 @@ __global__ void __launch_bounds__(256) embedding_pos_kernel(const void* table, c
   }
   const bool tok_ok = id >= 0 && id < vocab;
   for (int d = threadIdx.x; d < dim; d += blockDim.x) {
-    float v = tok_ok ? load_as_float(table, dt, (size_t)id * dim + d) : 0.f;
-    if (ok) v += load_as_float(pos_table, dt, (size_t)pos * dim + d);
+    float v = tok_ok ? load_as_float(table, dt, (size_t)id * ld_table + d) : 0.f;
+    if (ok && pos_table) v += load_as_float(pos_table, dt, (size_t)pos * dim + d);
     out[(size_t)m * dim + d] = v;
   }
 }
 
-int launch_embedding_pos(tq_ctx* ctx, const void* table, const void* pos_table, int dt, const int* ids, const int* seq_rows,
+int launch_embedding_pos(tq_ctx* ctx, const void* table, size_t ld_table, const void* pos_table, int dt, const int* ids, const int* seq_rows,
                          const int* starts, const int* slots, int n_seqs, size_t rows, int dim, int vocab, int n_pos, int max_seq,
                          int n_slots, float* out, int* row_pos, int* cache_row) {
-  TQ_CUDA(ctx, launch_k(ctx, embedding_pos_kernel, dim3((unsigned)rows), dim3(256), 0, table, pos_table, dt, ids, seq_rows, starts, slots,
+  TQ_CUDA(ctx, launch_k(ctx, embedding_pos_kernel, dim3((unsigned)rows), dim3(256), 0, table, ld_table, pos_table, dt, ids, seq_rows, starts, slots,
                         n_seqs, dim, vocab, n_pos, max_seq, n_slots, out, row_pos, cache_row, ctx->dev_err));
   return TQ_OK;
 }

@@ -18,12 +18,6 @@
 #include "dense.cuh"
 #include "diff_attention.cuh"
 
-namespace tq {
-int launch_embedding_pos(tq_ctx* ctx, const void* table, const void* pos_table, int dt, const int* ids, const int* seq_rows,
-                         const int* starts, const int* slots, int n_seqs, size_t rows, int dim, int vocab, int n_pos, int max_seq,
-                         int n_slots, float* out, int* row_pos, int* cache_row);
-}
-
 using namespace tq;
 
 namespace {
@@ -290,10 +284,10 @@ int tq_tofazen_step(tq_tofazen* m, const int* token_ids_dev, size_t rows, const 
   if (int st = ensure_rows(m, rows)) return st;
 #define TQ_STEP(expr) \
   if (int st = (expr)) return st;
-  TQ_STEP(launch_embedding_pos(ctx, m->embed, m->pos, c.dtype, token_ids_dev, seq_rows_dev, starts_dev, slots_dev, (int)n_seqs, rows, (int)c.width,
+  TQ_STEP(launch_embedding_pos(ctx, m->embed, c.width, m->pos, c.dtype, token_ids_dev, seq_rows_dev, starts_dev, slots_dev, (int)n_seqs, rows, (int)c.width,
                                (int)c.vocab, (int)c.max_positions, (int)c.max_seq, (int)c.max_slots, m->x, m->row_pos, m->cache_row));
   const int f32 = c.dtype == TQ_F32;
-  DiffAttnBatch batch;
+  RaggedBatch batch;
   batch.n_seqs = (int)n_seqs;
   batch.rows = (int)rows;
   batch.max_q = (int)max_q;
@@ -393,7 +387,7 @@ int tq_embedding_pos(tq_ctx* ctx, const void* table_dev, const void* pos_table_d
   if (rows == 0) return TQ_OK;
   TQ_REQUIRE(ctx, table_dev && pos_table_dev && ids_dev && starts_dev && out_dev && row_pos_dev && cache_row_dev && n_seqs > 0, "tq_embedding_pos: null pointer");
   TQ_REQUIRE(ctx, seq_rows_dev || rows == n_seqs, "tq_embedding_pos: without row offsets every sequence brings one row");
-  return launch_embedding_pos(ctx, table_dev, pos_table_dev, dtype, ids_dev, seq_rows_dev, starts_dev, slots_dev, (int)n_seqs, rows, (int)dim,
+  return launch_embedding_pos(ctx, table_dev, dim, pos_table_dev, dtype, ids_dev, seq_rows_dev, starts_dev, slots_dev, (int)n_seqs, rows, (int)dim,
                               (int)vocab, (int)n_pos, (int)max_seq, (int)n_slots, out_dev, row_pos_dev, cache_row_dev);
 }
 
@@ -418,7 +412,7 @@ int tq_diff_attention(tq_ctx* ctx, const tq_diff_attn_config* cfg, int dtype, co
   a.lambda = cfg->lambda;
   a.out_scale = cfg->out_scale;
   a.eps = cfg->eps;
-  DiffAttnBatch b;
+  RaggedBatch b;
   b.n_seqs = (int)n_seqs;
   b.rows = (int)rows;
   b.max_q = (int)max_q;

@@ -1,0 +1,25 @@
+// Grouped-query attention under a sliding window, with capped scores, a sink and an output gate:
+//     s = (q . k) * scale;  s <- softcap * tanh(s / softcap)          (softcap 0: no cap)
+//     p_j = exp(s_j) / (exp(sink) + sum exp(s))                       (sink -infinity: none; it has no value)
+//     out = (sum p_j v_j) * sigmoid(gate)                             (no gate pointer: 1)
+// Mask: the query at position i sees key j when j <= i and i - j < window.
+#pragma once
+
+#include "internal.h"
+#include "ragged.h"
+
+namespace tq {
+
+// Cache rows: keys [kv_heads][dim_pad], values [kv_heads][vdim_pad]; the padding (to 8 elements) is zero.
+struct WindowAttn {
+  int heads = 0, kv_heads = 0, dim = 0, vdim = 0, dim_pad = 0, vdim_pad = 0;
+  int window = 0;
+  float scale = 0.f, softcap = 0.f, sink = 0.f;
+};
+
+// q [rows][ldq], head h at column h * dim; gate [rows][ldg] and out [rows][ldo], head h at column h * vdim.  dtype (TQ_BF16 or
+// TQ_F32) is that of q, gate, caches and out; scores, weights and sums are f32, in TQ_F32 every operation is.
+int launch_window_attention(tq_ctx* ctx, const WindowAttn& a, const RaggedBatch& b, int dtype, const void* q, size_t ldq, const void* gate,
+                            size_t ldg, const void* k_cache, const void* v_cache, void* out, size_t ldo);
+
+}  // namespace tq

@@ -1,4 +1,4 @@
-"""Cache slots and ragged batching over a model that has ``step`` (``TofazenModel``).
+"""Cache slots and ragged batching over a model that has ``step`` (``StepModel``).
 
 Requests are named by the caller; each holds one cache slot from ``open`` (or its first ``step``) to ``close``.  A step
 takes the next tokens of any set of requests, packs them into one batch without padding -- in portions of at most

@@ -6,10 +6,13 @@ import os
 
 from . import _lib
 from .checkpoint import read_safetensors
+from .numuzen import NumuzenConfig, NumuzenModel
 from .tofazen import TofazenConfig, TofazenModel
 
 # architecture -> (configuration class, model class with ``from_tensors``)
-ARCHITECTURES = {"Tofazen": (TofazenConfig, TofazenModel)}
+ARCHITECTURES = {"Tofazen": (TofazenConfig, TofazenModel), "Numuzen": (NumuzenConfig, NumuzenModel)}
+
+DEFAULT_MAX_SEQ = 8192      # for designs without a largest position
 
 DTYPES = {"bfloat16": _lib.BF16, "float32": _lib.F32}
 
@@ -32,11 +35,13 @@ def resolve(config: dict):
 
 def load_model(dev, folder: str, dtype: int = _lib.BF16, max_slots: int = 64, max_seq: int | None = None, cache_budget: int = 64 << 30):
     """Loads config.json and model.safetensors from `folder`.  `max_slots` concurrent sequences of `max_seq` positions
-    (default: all the model has); fewer slots when they would take more than `cache_budget` bytes."""
+    (default: all the model has, or DEFAULT_MAX_SEQ when its design sets no limit); fewer slots when they would take more than `cache_budget` bytes."""
     config = read_config(folder)
     config_class, model_class = resolve(config)
     cfg = config_class.from_dict(config)
-    seq = min(max_seq or cfg.max_positions, cfg.max_positions)
-    per_slot = max(1, seq * cfg.cache_bytes_per_token(dtype))
-    max_slots = max(1, min(max_slots, cache_budget // per_slot))
+    limit = getattr(cfg, "max_positions", None)
+    seq = max_seq or limit or DEFAULT_MAX_SEQ
+    if limit:
+        seq = min(seq, limit)
+    max_slots = max(1, min(max_slots, cache_budget // max(1, cfg.bytes_per_slot(dtype, seq))))
     return model_class.from_tensors(dev, config, read_safetensors(os.path.join(folder, "model.safetensors")), dtype, max_slots, seq)

@@ -13,18 +13,12 @@ from dataclasses import dataclass
 import numpy as np
 
 from . import _lib
-from .checkpoint import SafetensorsError, TensorView
-from .device import Buffer, QuantComputeDevice
-from .generation import check_lengths, decode_loop
-
-_NO_WINDOW = 0x7FFFFFFF
+from .checkpoint import TensorView
+from .device import QuantComputeDevice
+from .stepmodel import NO_WINDOW, ConfigError, StepModel, host_array, need
 
 # tq_tofazen_tensor
 EMBED, POS, FINAL_NORM, HEAD, NORM, Q, K, V, O, GATE, UP, DOWN = range(12)
-
-
-class ConfigError(ValueError):
-    """A configuration that is not of this design."""
 
 
 class _CConfig(C.Structure):
@@ -75,7 +69,7 @@ class TofazenConfig:
                 src = m.get("kv_from")
                 layers.append(TofazenLayer(
                     int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), float(m["diff"]),
-                    int(mask.get("size", _NO_WINDOW)), int(mask.get("keep_first", 0)), None if src is None else int(src),
+                    int(mask.get("size", NO_WINDOW)), int(mask.get("keep_first", 0)), None if src is None else int(src),
                     0 if mlp is None else int(mlp["ff"]), 0.0 if mlp is None else float(mlp["limit"])))
             return cls(int(c["vocab"]), int(c["width"]), int(c["max_positions"]), float(c["norm"]["eps"]), float(c["residual_mult"]), layers)
         except (KeyError, TypeError) as e:
@@ -85,6 +79,10 @@ class TofazenConfig:
         up8 = lambda n: (n + 7) // 8 * 8
         n = sum(l.kv_heads * (2 * up8(l.dim) + up8(l.vdim)) for l in self.layers if l.kv_from is None)
         return n * (4 if dtype == _lib.F32 else 2)
+
+    def bytes_per_slot(self, dtype: int, max_seq: int) -> int:
+        """Device memory that one more concurrent sequence takes."""
+        return max_seq * self.cache_bytes_per_token(dtype)
 
 
 def tensor_names(cfg: TofazenConfig):
@@ -106,9 +104,11 @@ def map_balance(l: TofazenLayer, lq1, lk1, lq2, lk2) -> float:
     return math.exp(dot(lq1, lk1)) - math.exp(dot(lq2, lk2)) + l.diff
 
 
-class TofazenModel:
+class TofazenModel(StepModel):
     """Weights, caches and the step.  `dtype` BF16: bf16 weights, activations and caches with an f32 stream; F32: all f32.
     `lambdas`: one factor of the second map per layer (``map_balance``)."""
+
+    abi = "tq_tofazen"
 
     def __init__(self, dev: QuantComputeDevice, cfg: TofazenConfig, lambdas, dtype: int = _lib.BF16, max_slots: int = 64,
                  max_seq: int | None = None):
@@ -121,78 +121,26 @@ class TofazenModel:
         h = C.c_void_p()
         dev._check(dev._L.tq_tofazen_create(dev._ctx, C.byref(cc), cl, C.byref(h)))
         self.handle = h.value
-        self._bufs = {}
 
     @classmethod
     def from_tensors(cls, dev: QuantComputeDevice, config: dict, tensors: dict, dtype: int = _lib.BF16, max_slots: int = 64,
                      max_seq: int | None = None) -> "TofazenModel":
         """From a parsed config.json and the tensors of the checkpoint (``read_safetensors``)."""
         cfg = TofazenConfig.from_dict(config)
-
-        def need(name: str) -> TensorView:
-            if name not in tensors:
-                raise SafetensorsError(f"tensor {name!r} is missing")
-            return tensors[name]
-
-        lambdas = [map_balance(l, *(need(f"l{i}.mix.{n}").to_f32() for n in ("lq1", "lk1", "lq2", "lk2"))) for i, l in enumerate(cfg.layers)]
+        lambdas = [map_balance(l, *(need(tensors, f"l{i}.mix.{n}").to_f32() for n in ("lq1", "lk1", "lq2", "lk2"))) for i, l in enumerate(cfg.layers)]
         model = cls(dev, cfg, lambdas, dtype, max_slots, max_seq)
         try:
             for name, tensor, layer in tensor_names(cfg):
-                model.put(tensor, layer, need(name))
+                model.put(tensor, layer, need(tensors, name))
         except Exception:
             model.destroy()
             raise
         return model
 
     def put(self, tensor: int, layer: int, view: TensorView) -> None:
-        if view.dtype == "BF16":
-            a, dt = np.ascontiguousarray(view.data), _lib.BF16
-        else:
-            a, dt = np.ascontiguousarray(view.to_f32()), _lib.F32
-        rows, cols = view.shape if len(view.shape) == 2 else (1, int(np.prod(view.shape)))
+        a, dt, rows, cols = host_array(view)
         self.put_pointer(tensor, layer, a.ctypes.data, dt, rows, cols)
 
     def put_pointer(self, tensor: int, layer: int, ptr: int, dtype: int, rows: int, cols: int) -> None:
         """`ptr`: host or device address of the row-major [rows, cols] tensor."""
-        self.dev._check(self.dev._L.tq_tofazen_put(C.c_void_p(self.handle), tensor, layer, C.c_void_p(ptr), dtype, rows, cols))
-
-    # ------------------------------------------------------------------ steps
-    def step(self, tokens: Buffer, rows: int, seq_rows: Buffer | None, starts: Buffer, slots: Buffer | None, n_seqs: int, max_q: int,
-             max_len: int, logit_rows: Buffer | None, n_logits: int, logits: Buffer | None) -> None:
-        """``tq_tofazen_step``; asynchronous."""
-        ptr = lambda b: C.c_void_p(b.ptr if b is not None else 0)
-        self.dev._check(self.dev._L.tq_tofazen_step(C.c_void_p(self.handle), ptr(tokens), rows, ptr(seq_rows), ptr(starts), ptr(slots), n_seqs,
-                                                    max_q, max_len, ptr(logit_rows), n_logits, ptr(logits)))
-
-    def decode(self, token_ids: Buffer, positions: Buffer, batch: int, max_len: int, logits: Buffer, slots: Buffer | None = None) -> None:
-        """One new token for each of `batch` sequences (cache slots 0 .. batch-1 unless given)."""
-        self.step(token_ids, batch, None, positions, slots, batch, 1, max_len, None, batch, logits)
-
-    def trace(self, streams: Buffer | None) -> None:
-        """While set, every step leaves the f32 stream after each layer in `streams` [layers, rows, width]."""
-        self.dev._check(self.dev._L.tq_tofazen_trace(C.c_void_p(self.handle), C.c_void_p(streams.ptr if streams is not None else 0)))
-
-    def generate(self, prompts, n_new: int, sampling=None, seed: int = 42) -> np.ndarray:
-        """``generate`` for a batch of prompts of any lengths: the prompts run as one ragged batch (all tokens but the
-        last of each), then decode -> sample -> advance as one replayed graph.  Returns int32 [batch, n_new]."""
-        from .engine import Engine
-
-        prompts = [np.asarray(p, np.int32) for p in prompts]
-        check_lengths(prompts, n_new, self.max_seq)
-        engine = Engine(self)
-        heads = [(i, p[:-1], ()) for i, p in enumerate(prompts)]
-        slots = [engine.open(i) for i in range(len(prompts))]
-        if any(len(t) for _, t, _ in heads):
-            engine.step([h for h in heads if len(h[1])])
-        B, longest = len(prompts), max(len(p) for p in prompts)
-        slot_buf = self.dev.upload(np.array(slots, np.int32), _lib.I32)
-        return decode_loop(self.dev, lambda tok, pos, logits: self.decode(tok, pos, B, longest + n_new, logits, slot_buf), prompts, n_new,
-                           self.cfg.vocab, sampling, seed)
-
-    def generate_greedy(self, prompts, n_new: int) -> np.ndarray:
-        return self.generate(prompts, n_new, None)
-
-    def destroy(self) -> None:
-        if self.handle:
-            self.dev._L.tq_tofazen_destroy(C.c_void_p(self.handle))
-            self.handle = 0
+        self._call("put", tensor, layer, C.c_void_p(ptr), dtype, rows, cols)
