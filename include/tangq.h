@@ -451,6 +451,15 @@ TQ_API int tq_dlinear(tq_ctx* ctx, const tq_dweight* w, const void* x_dev, size_
 TQ_API int tq_clamped_glu(tq_ctx* ctx, const void* gate_dev, const void* up_dev, int in_dtype, size_t n, float limit, float alpha,
                           void* out_dev, int out_dtype);
 
+/* Several weights of one shape stacked by rows in one handle: job j (int[4]: group, first row, rows <= chunk, 0; on the device,
+ * *n_jobs <= max_jobs of them) multiplies activation rows first .. with rows group * group_rows .. of the weight.  chunk: up to
+ * 8 (GEMV), a multiple of 16 up to 256 (tcgen05), or 64 for f32 weights.  x_rows: where activation row i is in x (NULL: row i;
+ * not for tcgen05).  row_scale: a factor on every row's products.  glu_alpha = 0: y[row][group_rows] gets the products;
+ * otherwise the group's rows are interleaved gate / up halves and y[row][group_rows / 2] gets tq_clamped_glu of them. */
+TQ_API int tq_dlinear_grouped(tq_ctx* ctx, const tq_dweight* w, const void* x_dev, size_t ldx, size_t rows, const int* jobs_dev,
+                              const int* n_jobs_dev, size_t max_jobs, size_t chunk, size_t group_rows, const int* x_rows_dev_or_null,
+                              const float* row_scale_dev_or_null, float glu_limit, float glu_alpha, void* y_dev, int y_dtype, size_t ldy);
+
 /* ---- steps over ragged batches ------------------------------------------------------------------
  * No reference counterpart.  A step's rows are the next tokens of n_seqs sequences, packed: sequence b's are rows
  * seq_rows[b] .. seq_rows[b+1]-1 (seq_rows = NULL: row b), its first one sits at position starts[b], and its cache is

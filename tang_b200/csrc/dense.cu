@@ -879,6 +879,33 @@ int tq_dlinear(tq_ctx* ctx, const tq_dweight* w, const void* x_dev, size_t ldx, 
   return launch_dense(ctx, w, in, m, e);
 }
 
+int tq_dlinear_grouped(tq_ctx* ctx, const tq_dweight* w, const void* x_dev, size_t ldx, size_t rows, const int* jobs_dev, const int* n_jobs_dev,
+                       size_t max_jobs, size_t chunk, size_t group_rows, const int* x_rows_dev, const float* row_scale_dev, float glu_limit,
+                       float glu_alpha, void* y_dev, int y_dtype, size_t ldy) {
+  if (int st = bind(ctx)) return st;
+  TQ_REQUIRE(ctx, w && x_dev && y_dev && jobs_dev && n_jobs_dev, "tq_dlinear_grouped: null pointer");
+  TQ_REQUIRE(ctx, y_dtype == TQ_F32 || y_dtype == TQ_BF16, "tq_dlinear_grouped: y must be f32 or bf16");
+  DenseGroups g;
+  g.jobs = reinterpret_cast<const int4*>(jobs_dev);
+  g.n_jobs = n_jobs_dev;
+  g.max_jobs = (int)max_jobs;
+  g.chunk = (int)chunk;
+  g.group_rows = group_rows;
+  g.x_rows = x_rows_dev;
+  DenseEpilogue e;
+  e.n = 1;
+  e.s[0].row_end = (int)group_rows;
+  e.s[0].rows = (int)(glu_alpha != 0.f ? group_rows / 2 : group_rows);
+  e.s[0].kind = glu_alpha != 0.f ? DENSE_GLU : DENSE_ROW;
+  e.s[0].f32 = y_dtype == TQ_F32;
+  e.s[0].ld = (long long)(ldy ? ldy : (size_t)e.s[0].rows);
+  e.s[0].out = y_dev;
+  e.glu_limit = glu_limit;
+  e.glu_alpha = glu_alpha;
+  e.row_scale = row_scale_dev;
+  return launch_dense_grouped(ctx, w, x_dev, ldx ? ldx : w->cols, rows, g, e);
+}
+
 int tq_clamped_glu(tq_ctx* ctx, const void* gate_dev, const void* up_dev, int in_dtype, size_t n, float limit, float alpha, void* out_dev,
                    int out_dtype) {
   if (int st = bind(ctx)) return st;

@@ -30,6 +30,11 @@ struct GlaRows {
   size_t ldo = 0;
 };
 
+// Prompts in bf16 on the tensor cores (csrc/gla_chunk.cu): head sizes that are multiples of 16 up to 256, rows and sections on
+// 16-byte boundaries.
+bool gla_chunked_supported(const Gla& g, const GlaRows& r);
+int launch_gla_chunked(tq_ctx* ctx, const Gla& g, const GlaRows& r, const RaggedBatch& b);
+
 int launch_gla(tq_ctx* ctx, const Gla& g, const GlaRows& r, const RaggedBatch& b, int dtype);
 
 }  // namespace tq

@@ -55,21 +55,23 @@ def visible(i, j, size):
     return 0 <= i - j < size
 
 
-def one_query(q, keys, values, i, scale, softcap, size):
-    """One query vector at position i over keys and values at positions 0 .. i: capped scores, and a sink of score 0."""
-    js = [j for j in range(i + 1) if visible(i, j, size)]
+def one_query(q, keys, values, i, scale, softcap, size, sink=0.0):
+    """One query vector at position i over keys and values at positions 0 .. i: scores capped unless softcap is 0, and a sink
+    of the given score (None: none) in the denominator."""
+    js = [j for j in range(max(0, i - size + 1), i + 1) if visible(i, j, size)]
     s = keys[js] @ q * scale
-    s = softcap * np.tanh(s / softcap)
-    m = max(s.max(), 0.0)
+    if softcap:
+        s = softcap * np.tanh(s / softcap)
+    m = s.max() if sink is None else max(s.max(), sink)
     w = np.exp(s - m)
-    return (w / (np.exp(-m) + w.sum())) @ values[js]
+    return (w / (w.sum() + (0.0 if sink is None else np.exp(sink - m)))) @ values[js]
 
 
-def attention(q, keys, values, start, scale, softcap, size):
-    """q [n, H, dim] of positions start ..; keys, values [total, G, dim] of all positions.  Returns [n, H, dim]."""
+def attention(q, keys, values, start, scale, softcap, size, sink=0.0):
+    """q [n, H, dim] of positions start ..; keys [total, G, dim], values [total, G, vdim] of all positions.  [n, H, vdim]."""
     n, H = q.shape[:2]
     G = keys.shape[1]
-    return np.array([[one_query(q[r, h], keys[:, h // (H // G)], values[:, h // (H // G)], start + r, scale, softcap, size)
+    return np.array([[one_query(q[r, h], keys[:, h // (H // G)], values[:, h // (H // G)], start + r, scale, softcap, size, sink)
                       for h in range(H)] for r in range(n)])
 
 
