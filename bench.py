@@ -13,6 +13,7 @@ weak and the aggregate is the sum over ranks.
     python -m torch.distributed.run --nnodes=1 --nproc-per-node N ... bench.py --gpus N ...
     python bench.py --impl reference        # the CPU restatement of tang-infer on the host cores
     python bench.py --tofazen               # instead: the Tofazen family beside the int4 model (one JSON line of its own)
+    python bench.py --numuzen               # instead: the Numuzen family beside the Tofazen family (one JSON line of its own)
 
 The JSON line also carries: `e2e` (the same rate through the reference-shaped call q4_matvec with
 HOST vectors, copies inside the timed region), `roofline` (dominant kernel vs measured HBM peak),
@@ -1110,6 +1111,266 @@ def run_tofazen(args) -> None:
     out["clocks"] = sampler.stop(t_start, time.perf_counter())
     print(json.dumps(out))
 
+# ----------------------------------------------------------------------------------------------
+# --numuzen: the Numuzen family (bf16) beside the Tofazen family at equal width, head sizes, window and active feed-forward,
+# random weights: decode and prefill throughput of both, and the kernels one by one against their rooflines.
+# ----------------------------------------------------------------------------------------------
+NUMUZEN_SIZES = {
+    # alternating mixers; top experts of ff values together are as wide as the dense model's feed-forward
+    "8b": {"layers": 32, "width": 4096, "heads": 32, "kv": 8, "dim": 128, "gla": (16, 128, 256), "experts": 8, "top": 2, "ff": 7168, "vocab": 128256},
+    "1b": {"layers": 16, "width": 2048, "heads": 16, "kv": 4, "dim": 128, "gla": (8, 128, 256), "experts": 32, "top": 4, "ff": 2048, "vocab": 32000},
+}
+
+
+def build_numuzen(dev, tb, torch, stream, s, max_seq, max_batch, window):
+    from tang_b200 import numuzen as nz
+
+    gen = torch.Generator(device="cuda").manual_seed(7)
+    experts = nz.Experts(s["experts"], s["top"], s["ff"], 7.0)
+    rot = nz.Rotation(64, 500000.0, 4.0, 4096, 32.0, 1.0)
+    gh, gd, gv = s["gla"]
+    layers = [nz.NumuzenLayer(nz.ATTENTION, s["heads"], s["dim"], s["dim"], s["dim"] ** -0.5, s["kv"], window, 50.0, rot, experts=experts) if i % 2 == 0 else
+              nz.NumuzenLayer(nz.GLA, gh, gd, gv, gd ** -0.5, tau=16.0, rank=16, experts=experts) for i in range(s["layers"])]
+    cfg = tb.NumuzenConfig(s["vocab"], s["width"], 1e-6, layers)
+    model = tb.NumuzenModel(dev, cfg, tb.BF16, max_batch, max_seq)
+    pool = {}
+    for name, tensor, i, e in nz.tensor_names(cfg):
+        l, d = cfg.layers[i], s["width"]
+        qr, vr, kr = l.heads * l.dim, l.heads * l.vdim, (l.kv_heads or l.heads) * l.dim
+        r, c = {nz.EMBED: (s["vocab"], d), nz.Q: (qr, d), nz.K: (kr, d), nz.V: (vr, d), nz.G: (vr, d), nz.O: (d, vr), nz.Q_NORM: (1, qr), nz.K_NORM: (1, kr),
+                nz.O_NORM: (1, l.vdim), nz.A1: (l.rank, d), nz.A2: (qr, l.rank), nz.A2_BIAS: (1, qr), nz.ROUTER: (s["experts"], d), nz.GATE: (s["ff"], d),
+                nz.UP: (s["ff"], d), nz.DOWN: (d, s["ff"])}.get(tensor, (1, d))
+        plain = tensor in (nz.Q_NORM, nz.K_NORM, nz.O_NORM)
+        key = (r, c, plain, tensor in (nz.ROUTER,) and i)
+        if key not in pool:
+            with torch.cuda.stream(stream):
+                pool[key] = (torch.randn((r, c), device="cuda", generator=gen) * (0.05 if r == 1 else c ** -0.5) + (1.0 if plain else 0.0)).bfloat16()
+            stream.synchronize()
+        model.put_pointer(tensor, i, pool[key].data_ptr(), tb.BF16, r, c, e)
+    return model
+
+
+def run_numuzen(args) -> None:
+    import ctypes as C
+
+    import torch
+
+    import tang_b200 as tb
+
+    torch.cuda.set_device(0)
+    dev = tb.QuantComputeDevice(0)
+    L_ = dev._L
+    stream = torch.cuda.ExternalStream(dev.stream, device=torch.device("cuda", 0))
+    peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")) else {}
+    hbm, tf = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    ctx, window = 2048, 512
+    sampler = ClockSampler(0)
+    sampler.start()
+    t_start = time.perf_counter()
+
+    def graph_ms(fn, reps=10):
+        fn()
+        dev.sync()
+        dev.begin_capture()
+        fn()
+        g = dev.end_capture()
+        ms = _time_ms(torch, stream, dev, g.launch, reps, warm=3)
+        g.free()
+        return ms
+
+    def rand(*shape, std=1.0, dt=None):
+        with torch.cuda.stream(stream):
+            t = torch.randn(shape, device="cuda") * std
+            t = t if dt == tb.F32 else t.bfloat16()
+        stream.synchronize()
+        return t
+
+    P = lambda t: C.c_void_p(t.data_ptr() if hasattr(t, "data_ptr") else t.ptr)
+    ints = lambda a: dev.upload(np.asarray(a, np.int32).reshape(-1), tb.I32)
+
+    def touched(experts, top, rows):
+        """Expected number of experts that `rows` rows choose."""
+        return experts * (1 - (1 - top / experts) ** rows)
+
+    out = {"metric": "numuzen_throughput", "unit": "tokens/s", "data": "synthetic", "dtype": "bf16", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf},
+           "window": window, "models": [], "kernels": []}
+    batches = [1, 2, 4, 8, 16, 64]
+
+    def time_model(size, name, model, s, decode_bytes, prefill_params):
+        row = {"size": size, "model": name, "decode": {}, "prefill": {}}
+        for B in batches:
+            tok = ints(np.random.randint(0, s["vocab"], B))
+            pos, lg = ints(np.full(B, ctx)), dev.alloc(B * s["vocab"], tb.F32)
+            ms = graph_ms(lambda: model.decode(tok, pos, B, ctx + 1, lg))
+            row["decode"][B] = {"ms": ms, "tokens_per_s": B / ms * 1e3, "frac_of_hbm": decode_bytes(B) / ms / 1e6 / hbm}
+        tok = ints(np.random.randint(0, s["vocab"], ctx))
+        cu, st, last, lg = ints([0, ctx]), ints([0]), ints([ctx - 1]), dev.alloc(s["vocab"], tb.F32)
+        ms = graph_ms(lambda: model.step(tok, ctx, cu, st, None, 1, ctx, ctx, last, 1, lg), 3)
+        row["prefill"] = {"tokens": ctx, "ms": ms, "tokens_per_s": ctx / ms * 1e3, "frac_of_bf16": 2.0 * ctx * prefill_params / ms / 1e9 / tf}
+        out["models"].append(row)
+        model.destroy()
+        torch.cuda.empty_cache()
+
+    for size in [x for x in args.numuzen.split(",") if x in NUMUZEN_SIZES]:
+        s = NUMUZEN_SIZES[size]
+        d, (gh, gd, gv) = s["width"], s["gla"]
+        att = d * (3 * s["heads"] + s["kv"]) * s["dim"]
+        rec = d * (2 * gh * gd + 3 * gh * gv + 16)
+        mixers = s["layers"] // 2 * (att + rec)
+        one = 3 * d * s["ff"]
+        kv = s["layers"] // 2 * s["kv"] * 2 * s["dim"] * 2 * window
+        state = s["layers"] // 2 * gh * gd * gv * 4 * 2
+        fixed = 2 * (mixers + s["layers"] * s["experts"] * d + s["vocab"] * d)
+        time_model(size, "numuzen", build_numuzen(dev, tb, torch, stream, s, ctx + 1, max(batches), window), s,
+                   lambda B: fixed + 2 * s["layers"] * one * touched(s["experts"], s["top"], B) + B * (kv + state), mixers + s["layers"] * s["top"] * one)
+        if not args.numuzen_only:
+            z = dict(TOFAZEN_SIZES[size])
+            w = z["width"] * (z["heads"] * 2 * z["dim"] + z["kv"] * (2 * z["dim"] + z["vdim"]) + z["heads"] * z["vdim"] + 3 * z["ff"])
+            row_b = z["layers"] * z["kv"] * (2 * z["dim"] + z["vdim"]) * 2
+            time_model(size, "tofazen", build_tofazen(dev, tb, torch, stream, z, ctx, max(batches), window, 4), z,
+                       lambda B: 2 * (z["layers"] * w + z["vocab"] * z["width"]) + B * row_b * (window + 4), z["layers"] * w)
+
+    def kernel(name, m, us, byt=0.0, flops=0.0):
+        roof = max(byt / hbm / 1e3, flops / tf / 1e6)
+        out["kernels"].append({"kernel": name, "m": m, "us": round(us, 2), "roofline_us": round(roof, 2), "frac": round(roof / us, 3)})
+
+    # ---- linear layers: the mixers' projections, and the experts beside a dense layer of the same products
+    def handle(rows, cols):
+        t = rand(min(rows, 65536), cols, std=cols ** -0.5)
+        h = C.c_void_p()
+        dev._check(L_.tq_dweight_create(dev._ctx, rows, cols, tb.BF16, C.byref(h)))
+        for r in range(0, rows, 65536):
+            n = min(65536, rows - r)
+            dev._check(L_.tq_dweight_put(dev._ctx, h, P(t), tb.BF16, n, cols, r, 0, 0))
+        return h
+
+    d = 4096
+    for name, rows, cols in (("attention in", 9216, d), ("recurrent in", 12304, d), ("mixer out", d, 4096)):
+        hs = [handle(rows, cols) for _ in range(8)]
+        for m in (1, 8, 64, 2048):
+            x, y = rand(m, cols), torch.empty((m, rows), dtype=torch.bfloat16, device="cuda")
+            us = graph_ms(lambda: [dev._check(L_.tq_dlinear(dev._ctx, h, P(x), cols, m, P(y), tb.BF16, rows)) for h in hs]) / len(hs) * 1e3
+            kernel(f"linear {name} {rows}x{cols}", m, us, rows * cols * 2 + m * (rows + cols) * 2, 2.0 * m * rows * cols)
+        for h in hs:
+            L_.tq_dweight_free(dev._ctx, h)
+    for E, top, ff, d in ((8, 2, 7168, 4096), (32, 4, 2048, 2048)):
+        n = 2
+        gu, dn = [handle(E * 2 * ff, d) for _ in range(n)], [handle(E * d, ff) for _ in range(n)]
+        dense_gu, dense_dn = [handle(top * 2 * ff, d) for _ in range(3 * n)], [handle(d, top * ff) for _ in range(3 * n)]
+        rng = np.random.default_rng(0)
+        for m in (1, 2, 4, 8, 16, 64, 256, 2048):
+            pairs = m * top
+            chosen = np.stack([rng.permutation(E)[:top] for _ in range(m)])
+            counts = np.bincount(chosen.reshape(-1), minlength=E)
+            chunk = L_.tq_dense_group_chunk(tb.BF16, max(d, ff), pairs, E)
+            jobs, first = [], 0
+            for e in range(E):
+                jobs += [(e, first + i, min(chunk, counts[e] - i), 0) for i in range(0, counts[e], chunk)]
+                first += counts[e]
+            jd, nd = ints(jobs), ints([len(jobs)])
+            sr = ints(np.argsort(chosen.reshape(-1), kind="stable") // top) if chunk <= 8 else None
+            w = dev.upload(np.ones(pairs, np.float32), tb.F32)
+            mj = min(pairs, E + pairs // chunk)
+            x, act, y = rand(max(pairs, m), d), torch.empty((pairs, ff), dtype=torch.bfloat16, device="cuda"), torch.empty((pairs, d), device="cuda")
+            null = C.c_void_p(0)
+            live = int((counts > 0).sum())
+            for what, hs, call, wb, io in (
+                    ("gate/up", gu, lambda h: L_.tq_dlinear_grouped(dev._ctx, h, P(x), d, pairs, P(jd), P(nd), mj, chunk, 2 * ff, P(sr) if sr else null, P(w), 7.0, 1.702,
+                                                                    P(act), tb.BF16, ff), live * 2 * ff * d * 2, pairs * (d + ff) * 2),
+                    ("down", dn, lambda h: L_.tq_dlinear_grouped(dev._ctx, h, P(act), ff, pairs, P(jd), P(nd), mj, chunk, d, null, null, 0.0, 0.0, P(y), tb.F32, d),
+                     live * ff * d * 2, pairs * (ff * 2 + d * 4))):
+                us = graph_ms(lambda: [dev._check(call(h)) for h in hs]) / len(hs) * 1e3
+                kernel(f"experts {what} {E}x{ff}x{d} top {top}", m, us, wb + io, 2.0 * pairs * ff * d * (2 if what == "gate/up" else 1))
+            dx, dy = rand(m, max(d, top * ff)), torch.empty((m, max(d, top * 2 * ff)), device="cuda")
+            for what, hs, rows, cols in (("gate/up", dense_gu, top * 2 * ff, d), ("down", dense_dn, d, top * ff)):
+                us = graph_ms(lambda: [dev._check(L_.tq_dlinear(dev._ctx, h, P(dx), cols, m, P(dy), tb.BF16 if what == "gate/up" else tb.F32, rows)) for h in hs]) / len(hs) * 1e3
+                kernel(f"dense {what} {rows}x{cols}", m, us, rows * cols * 2 + m * (cols * 2 + rows * (2 if what == "gate/up" else 4)), 2.0 * m * rows * cols)
+        for h in gu + dn + dense_gu + dense_dn:
+            L_.tq_dweight_free(dev._ctx, h)
+        del x, act, y, dx, dy
+        torch.cuda.empty_cache()
+
+    # ---- attention and recurrence, one row per sequence at position ctx - 1, then one prompt
+    class Win(C.Structure):
+        _fields_ = [(k, C.c_uint32) for k in ("heads", "kv_heads", "dim", "vdim", "window")] + [(k, C.c_float) for k in ("scale", "softcap", "sink")]
+
+    class Diff(C.Structure):
+        _fields_ = [(k, C.c_uint32) for k in ("heads", "kv_heads", "dim", "vdim", "window", "keep_first")] + [
+            (k, C.c_float) for k in ("scale", "lam", "out_scale", "eps")]
+
+    class Gla(C.Structure):
+        _fields_ = [(k, C.c_uint32) for k in ("heads", "dim", "vdim", "rank")] + [(k, C.c_float) for k in ("tau", "q_scale", "eps")]
+
+    H, G, D = 32, 8, 128
+    gh, gd, gv = 16, 128, 256
+    gw = 2 * gh * gd + 2 * gh * gv
+    a2, bias, gnorm = rand(gh * gd, 16, dt=tb.F32), rand(gh * gd, dt=tb.F32), rand(gv, dt=tb.F32)
+
+    def attention(kind, w, q, k, v, gate, o, B, rows, n_seqs, cu, rp, cr, max_q):
+        if kind == "window":
+            a = Win(H, G, D, D, w, D ** -0.5, 50.0, 0.0)
+            return L_.tq_window_attention(dev._ctx, C.byref(a), tb.BF16, P(q), H * D, P(gate), H * D, P(k), P(v), B * ctx, cu, P(rp), P(cr), n_seqs, rows, max_q, ctx,
+                                          P(o), H * D)
+        a = Diff(H, G, D // 2, D, w, 4, D ** -0.5, 0.5, 0.7, 1e-6)
+        return L_.tq_diff_attention(dev._ctx, C.byref(a), tb.BF16, P(q), H * D, P(k), P(v), B * ctx, cu, P(rp), P(cr), n_seqs, rows, max_q, ctx, P(o), H * D)
+
+    def recurrence(x, a1, state, o, rows, n_seqs, cu, rp, cr, max_q):
+        g, off = Gla(gh, gd, gv, 16, 16.0, gd ** -0.5, 1e-6), lambda n: C.c_void_p(x.data_ptr() + 2 * n)
+        return L_.tq_gla(dev._ctx, C.byref(g), tb.BF16, off(0), off(gh * gd), off(2 * gh * gd), off(2 * gh * gd + gh * gv), gw, P(a1), 16, P(a2), P(bias), P(gnorm),
+                         P(state), ctx, n_seqs * ctx, cu, P(rp), P(cr), n_seqs, rows, max_q, P(o), gh * gv)
+
+    null = C.c_void_p(0)
+    for B in (1, 16, 64):
+        n = max(1, min(16, 64 // B * 2))               # distinct caches per pass
+        k, v, q, gate = rand(n, B, ctx, G * D), rand(n, B, ctx, G * D), rand(B, H * D), rand(B, H * D)
+        o = torch.empty((B, H * D), dtype=torch.bfloat16, device="cuda")
+        rp, cr = ints(np.full(B, ctx - 1)), ints(np.arange(B) * ctx + ctx - 1)
+        for kind in ("window", "differential"):
+            for w in (window, ctx):
+                us = graph_ms(lambda: [dev._check(attention(kind, w, q, k[i], v[i], gate, o, B, B, B, null, rp, cr, 1)) for i in range(n)]) / n * 1e3
+                kernel(f"decode attention {kind} {w}", B, us, B * w * G * D * 2 * 2)
+        del k, v
+        st = [rand(B, gh, gd, gv, dt=tb.F32) for _ in range(max(4, min(64, 128 // B)))]
+        x, a1, o = rand(B, gw), rand(B, 16, dt=tb.F32), torch.empty((B, gh * gv), dtype=torch.bfloat16, device="cuda")
+        us = graph_ms(lambda: [dev._check(recurrence(x, a1, t, o, B, B, null, rp, cr, 1)) for t in st]) / len(st) * 1e3
+        kernel("decode recurrence", B, us, B * gh * gd * gv * 4 * 2)
+        del st
+        torch.cuda.empty_cache()
+    for T in (512, 2048):
+        k, v, q, gate = rand(T, G * D), rand(T, G * D), rand(T, H * D), rand(T, H * D)
+        o = torch.empty((T, H * D), dtype=torch.bfloat16, device="cuda")
+        cu, rp = ints([0, T]), ints(np.arange(T))
+        for kind in ("window", "differential"):
+            for w in (256, ctx):
+                us = graph_ms(lambda: dev._check(attention(kind, w, q, k, v, gate, o, 1, T, 1, P(cu), rp, rp, T))) * 1e3
+                kernel(f"prefill attention {kind} {w}", T, us, 0, 2.0 * H * (2 * D if kind == "window" else 3 * D) * sum(min(i + 1, w) for i in range(T)))
+        x, a1, st = rand(T, gw), rand(T, 16, dt=tb.F32), rand(1, gh, gd, gv, dt=tb.F32)
+        o = torch.empty((T, gh * gv), dtype=torch.bfloat16, device="cuda")
+        us = graph_ms(lambda: dev._check(recurrence(x, a1, st, o, T, 1, P(cu), rp, rp, T))) * 1e3
+        # (chunked form with single products: 64-token pair weights and their values, contributions to and readings of the state)
+        kernel("prefill recurrence", T, us, T * (gw + gh * gv) * 2, 2.0 * T * gh * (32 * (gd + gv) + 2 * gd * gv))
+
+    # ---- row operators beside the plain norm
+    for m in (1, 64, 2048):
+        x, y, gain, h = rand(m, 4096, dt=tb.F32), rand(m * 2, 4096, dt=tb.F32), rand(4096, dt=tb.F32), torch.empty((m, 4096), dtype=torch.bfloat16, device="cuda")
+        slots = ints(np.random.permutation(2 * m))
+        n = 20
+        for name, call, byt in (
+                ("post-norm, stream, next norm", lambda: L_.tq_add_norm(dev._ctx, P(x), P(y), null, 1, P(gain), P(gain), m, 4096, 1e-6, P(h), tb.BF16, 4096), m * 4096 * 14),
+                ("the same over two experts", lambda: L_.tq_add_norm(dev._ctx, P(x), P(y), P(slots), 2, P(gain), P(gain), m, 4096, 1e-6, P(h), tb.BF16, 4096), m * 4096 * 18),
+                ("plain norm", lambda: L_.tq_rms_norm(dev._ctx, P(x), tb.F32, null, P(gain), tb.F32, m, 4096, 1e-6, P(h), tb.BF16, null), m * 4096 * 6)):
+            kernel(name, m, graph_ms(lambda: [dev._check(call()) for _ in range(n)]) / n * 1e3, byt)
+        q, raw, keys, qg, kg, fr = rand(m, H * D), rand(m, G * D), rand(m, G * D), rand(H * D), rand(G * D), rand(32, dt=tb.F32)
+        rp = ints(np.arange(m))
+        us = graph_ms(lambda: [dev._check(L_.tq_qk_norm_rope(dev._ctx, tb.BF16, H, G, D, P(q), H * D, P(raw), P(keys), m, P(qg), P(kg), 64, P(fr), 1.0, 1e-6, P(rp), P(rp), m))
+                               for _ in range(n)]) / n * 1e3
+        kernel("query/key norm and rotation", m, us, m * (H + G) * D * 4)
+        z = rand(m, 32, dt=tb.F32)
+        bufs = [ints(np.zeros(m * 4)) for _ in range(4)] + [ints(np.zeros(4 * (m * 4 + 32))), ints([0])]
+        us = graph_ms(lambda: [dev._check(L_.tq_route(dev._ctx, P(z), m, 32, 4, 0, 0, 8, *map(P, bufs))) for _ in range(n)]) / n * 1e3
+        kernel("routing, 4 of 32", m, us, m * 32 * 4)
+    out["clocks"] = sampler.stop(t_start, time.perf_counter())
+    print(json.dumps(out))
 
 def main() -> None:
     ap = argparse.ArgumentParser()
@@ -1129,7 +1390,12 @@ def main() -> None:
     ap.add_argument("--decode-steps", type=int, default=10)
     ap.add_argument("--tofazen", nargs="?", const="8b,1b", default="", help="time the Tofazen family instead (sizes: 8b, 1b, or none: kernels only)")
     ap.add_argument("--tofazen-only", action="store_true", help="with --tofazen: leave the int4 model out")
+    ap.add_argument("--numuzen", nargs="?", const="8b,1b", default="", help="time the Numuzen family instead (sizes: 8b, 1b, or none: kernels only)")
+    ap.add_argument("--numuzen-only", action="store_true", help="with --numuzen: leave the Tofazen model out")
     args = ap.parse_args()
+    if args.numuzen:
+        run_numuzen(args)
+        return
     if args.tofazen:
         run_tofazen(args)
         return

@@ -456,6 +456,8 @@ TQ_API int tq_clamped_glu(tq_ctx* ctx, const void* gate_dev, const void* up_dev,
  * 8 (GEMV), a multiple of 16 up to 256 (tcgen05), or 64 for f32 weights.  x_rows: where activation row i is in x (NULL: row i;
  * not for tcgen05).  row_scale: a factor on every row's products.  glu_alpha = 0: y[row][group_rows] gets the products;
  * otherwise the group's rows are interleaved gate / up halves and y[row][group_rows / 2] gets tq_clamped_glu of them. */
+/* The chunk the library takes for `rows` activation rows over n_groups weights of up to `cols` columns. */
+TQ_API size_t tq_dense_group_chunk(int dtype, size_t cols, size_t rows, size_t n_groups);
 TQ_API int tq_dlinear_grouped(tq_ctx* ctx, const tq_dweight* w, const void* x_dev, size_t ldx, size_t rows, const int* jobs_dev,
                               const int* n_jobs_dev, size_t max_jobs, size_t chunk, size_t group_rows, const int* x_rows_dev_or_null,
                               const float* row_scale_dev_or_null, float glu_limit, float glu_alpha, void* y_dev, int y_dtype, size_t ldy);

@@ -103,6 +103,7 @@ PROTOTYPES = {
     "tq_dweight_free": (_i, [_p, _p]),
     "tq_dweight_data": (_i, [_p, _pp, C.POINTER(_sz), C.POINTER(_sz)]),
     "tq_dlinear": (_i, [_p, _p, _p, _sz, _sz, _p, _i, _sz]),
+    "tq_dense_group_chunk": (_sz, [_i, _sz, _sz, _sz]),
     "tq_dlinear_grouped": (_i, [_p, _p, _p, _sz, _sz, _p, _p, _sz, _sz, _sz, _p, _p, C.c_float, C.c_float, _p, _i, _sz]),
     "tq_clamped_glu": (_i, [_p, _p, _p, _i, _sz, C.c_float, C.c_float, _p, _i]),
     "tq_embedding_pos": (_i, [_p, _p, _p, _i, _p, _p, _p, _p, _sz, _sz, _sz, _sz, _sz, _sz, _sz, _p, _p, _p]),

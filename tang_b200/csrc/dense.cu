@@ -879,6 +879,11 @@ int tq_dlinear(tq_ctx* ctx, const tq_dweight* w, const void* x_dev, size_t ldx, 
   return launch_dense(ctx, w, in, m, e);
 }
 
+size_t tq_dense_group_chunk(int dtype, size_t cols, size_t rows, size_t n_groups) {
+  if (cols == 0 || n_groups == 0) return 0;
+  return (size_t)dense_group_chunk(dtype, (cols + kGvPad - 1) / kGvPad * kGvPad, rows, n_groups);
+}
+
 int tq_dlinear_grouped(tq_ctx* ctx, const tq_dweight* w, const void* x_dev, size_t ldx, size_t rows, const int* jobs_dev, const int* n_jobs_dev,
                        size_t max_jobs, size_t chunk, size_t group_rows, const int* x_rows_dev, const float* row_scale_dev, float glu_limit,
                        float glu_alpha, void* y_dev, int y_dtype, size_t ldy) {
