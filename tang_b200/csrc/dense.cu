@@ -2,6 +2,7 @@
 // C entry points tq_dweight_* / tq_dlinear / tq_clamped_glu.
 #include "dense.cuh"
 
+#include <cmath>
 #include <cstring>
 #include <new>
 #include <vector>
@@ -699,8 +700,9 @@ int dense_group_chunk(int dtype, size_t kpad, size_t rows, size_t n_groups) {
   size_t gv = kGvSmemMax / (kpad * 2 + 16);
   if (gv > kGvRows) gv = kGvRows;
   if (mean <= 4 && gv > 0) return (int)gv;
-  const size_t want = (mean + mean / 4 + 15) / 16 * 16;      // most groups in one job each
-  return (int)(want > 256 ? 256 : want);
+  // a group of two standard deviations above the mean (rows spread at random) still fills its jobs: ntok is paid in full
+  const size_t need = mean + 2 * (size_t)std::ceil(std::sqrt((double)mean)), jobs = (need + 255) / 256;
+  return (int)(((need + jobs - 1) / jobs + 15) / 16 * 16);
 }
 
 int launch_dense_grouped(tq_ctx* ctx, const tq_dweight* w, const void* x, size_t ldx, size_t rows, const DenseGroups& g, const DenseEpilogue& epi) {

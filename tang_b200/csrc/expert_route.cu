@@ -2,6 +2,8 @@
 // (a warp per row), a plan kernel (one CTA: offsets and jobs) and a placement kernel that also gathers the rows.
 #include "expert_route.cuh"
 
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace tq {
@@ -10,52 +12,61 @@ constexpr int kErMaxExperts = 1024, kErMaxTop = 64;
 constexpr int kErThreads = 1024;
 constexpr int kErSmall = 2048;      // pairs of the one-CTA form
 
-// Selection of one row by a warp: lane l owns experts l, l + 32, ...  Lane 0 calls emit(i, expert, weight).
-template <typename Emit>
+// Selection of one row by a warp: lane l owns experts l, l + 32, ... (NR of them at most, in registers).  The lanes call
+// emit(i, expert, weight) for their choices.
+template <int NR, typename Emit>
 __device__ __forceinline__ void choose_experts(const float* z, int experts, int top, int score, bool renorm, Emit emit) {
   const int lane = threadIdx.x & 31;
+  float v[NR];
+  unsigned key[NR];            // order of the values as integers; 0: taken or none
+#pragma unroll
+  for (int j = 0; j < NR; ++j) {
+    const int e = lane + 32 * j;
+    v[j] = e < experts ? z[e] : -INFINITY;
+    const unsigned u = __float_as_uint(v[j]);
+    key[j] = e < experts ? max(u ^ ((u >> 31) ? 0xFFFFFFFFu : 0x80000000u), 1u) : 0u;
+  }
   float mx = -INFINITY, sum = 0.f;
   if (score == ROUTE_SOFTMAX) {
-    for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, z[e]);
+#pragma unroll
+    for (int j = 0; j < NR; ++j) mx = fmaxf(mx, v[j]);
     mx = warp_max(mx);
-    for (int e = lane; e < experts; e += 32) sum += expf(z[e] - mx);
+#pragma unroll
+    for (int j = 0; j < NR; ++j) sum += expf(v[j] - mx);
     sum = warp_sum(sum);
   }
-  auto weight = [&](float v) { return score == ROUTE_SIGMOID ? 1.0f / (1.0f + expf(-v)) : expf(v - mx) / sum; };
-  unsigned taken = 0;
-  float chosen = 0.f;
-  const int passes = renorm ? 2 : 1;
-  for (int pass = 0; pass < passes; ++pass) {
-    taken = 0;
-    float total = 0.f;
-    for (int i = 0; i < top; ++i) {
-      float bv = -INFINITY;
-      int be = -1;
-      for (int j = 0, e = lane; e < experts; ++j, e += 32) {
-        const float v = z[e];
-        if (!((taken >> j) & 1u) && (be < 0 || v > bv)) {        // ascending: '>' keeps the lower index
-          bv = v;
-          be = e;
-        }
-      }
+  float mine[kErMaxTop / 32];  // lane l keeps choices l and l + 32
+  int chosen[kErMaxTop / 32];
+  float total = 0.f;
+  for (int i = 0; i < top; ++i) {
+    unsigned best = 0u;
+    float bv = 0.f;
+    int be = 0x7FFFFFFF;
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-        const int oe = __shfl_xor_sync(0xffffffffu, be, o);
-        if (oe >= 0 && (be < 0 || ov > bv || (!(bv > ov) && oe < be))) {
-          bv = ov;
-          be = oe;
-        }
+    for (int j = 0; j < NR; ++j)
+      if (key[j] > best) {                               // ascending: '>' keeps the lower index
+        best = key[j];
+        bv = v[j];
+        be = lane + 32 * j;
       }
-      be = __shfl_sync(0xffffffffu, be, 0);                        // (a NaN has no order: all lanes go with lane 0)
-      bv = __shfl_sync(0xffffffffu, bv, 0);
-      if ((be & 31) == lane) taken |= 1u << (be >> 5);
-      const float w = weight(bv);
-      total += w;
-      if (pass == passes - 1 && lane == 0) emit(i, be, renorm ? w / chosen : w);
-    }
-    chosen = total;
+    const unsigned mxk = __reduce_max_sync(0xffffffffu, best);
+    const int e = (int)__reduce_min_sync(0xffffffffu, best == mxk ? (unsigned)be : 0x7FFFFFFFu);
+    bv = __shfl_sync(0xffffffffu, bv, e & 31);
+#pragma unroll
+    for (int j = 0; j < NR; ++j)
+      if (e == lane + 32 * j) key[j] = 0u;
+    const float w = score == ROUTE_SIGMOID ? 1.0f / (1.0f + expf(-bv)) : expf(bv - mx) / sum;
+    total += w;
+#pragma unroll
+    for (int h = 0; h < kErMaxTop / 32; ++h)
+      if (i == lane + 32 * h) {
+        mine[h] = w;
+        chosen[h] = e;
+      }
   }
+#pragma unroll
+  for (int h = 0; h < kErMaxTop / 32; ++h)
+    if (lane + 32 * h < top) emit(lane + 32 * h, chosen[h], renorm ? mine[h] / total : mine[h]);
 }
 
 // Offsets and jobs from the counts (in shared memory) of up to 1024 experts, one thread each; all threads of the CTA come here.
@@ -89,51 +100,54 @@ __device__ __forceinline__ void plan_jobs(int count, int experts, int chunk, int
   if (e == blockDim.x - 1) *n_jobs = min(bj + sj, max_jobs);
 }
 
+template <int NR>
 __global__ void __launch_bounds__(kErThreads) route_small_kernel(const float* logits, size_t ld, int rows, int experts, int top, int score, bool renorm,
                                                                  int chunk, int max_jobs, Routing r, const uint8_t* x, size_t ldx, int row_vecs,
                                                                  uint8_t* gathered, size_t ldg) {
-  __shared__ int counts[kErMaxExperts], offs[kErMaxExperts];
+  __shared__ int counts[32 * NR], offs[32 * NR];
+  __shared__ unsigned short pe[kErSmall], pk[kErSmall];   // expert of every pair and its place among the expert's
+  __shared__ float pw[kErSmall];
+  for (int e = threadIdx.x; e < experts; e += blockDim.x) counts[e] = 0;
   pdl_wait();
   pdl_launch_dependents();
   const int warp = threadIdx.x >> 5, pairs = rows * top;
-  for (int e = threadIdx.x; e < experts; e += kErThreads) counts[e] = 0;
   __syncthreads();
-  for (int m = warp; m < rows; m += kErThreads / 32)
-    choose_experts(logits + (size_t)m * ld, experts, top, score, renorm, [&](int i, int e, float w) {
+  for (int m = warp; m < rows; m += blockDim.x >> 5)
+    choose_experts<NR>(logits + (size_t)m * ld, experts, top, score, renorm, [&](int i, int e, float w) {
       const int p = m * top + i;
-      r.expert[p] = e;
-      r.weight[p] = w;
-      r.rank[p] = atomicAdd(&counts[e], 1);
+      pe[p] = (unsigned short)e;
+      pw[p] = w;
+      pk[p] = (unsigned short)atomicAdd(&counts[e], 1);
     });
   __syncthreads();
   int offset = 0;
   plan_jobs(threadIdx.x < (unsigned)experts ? counts[threadIdx.x] : 0, experts, chunk, max_jobs, r.jobs, r.n_jobs, offset);
-  if (threadIdx.x < (unsigned)experts) {
-    offs[threadIdx.x] = offset;
-    r.offsets[threadIdx.x] = offset;
-  }
+  if (threadIdx.x < (unsigned)experts) offs[threadIdx.x] = offset;
   __syncthreads();
-  for (int p = threadIdx.x; p < pairs; p += kErThreads) {
-    const int s = offs[r.expert[p]] + r.rank[p];      // (written above by this CTA, before the barriers)
+  for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
+    const int s = offs[pe[p]] + pk[p];
+    r.expert[p] = pe[p];
+    r.weight[p] = pw[p];
     r.slot[p] = s;
     r.slot_row[s] = p / top;
-    r.slot_weight[s] = r.weight[p];
+    r.slot_weight[s] = pw[p];
   }
   if (gathered) {
-    for (int i = threadIdx.x; i < pairs * row_vecs; i += kErThreads) {
+    for (int i = threadIdx.x; i < pairs * row_vecs; i += blockDim.x) {
       const int p = i / row_vecs, v = i - p * row_vecs;
-      const int s = offs[r.expert[p]] + r.rank[p];
+      const int s = offs[pe[p]] + pk[p];
       *reinterpret_cast<uint4*>(gathered + (size_t)s * ldg + 16 * (size_t)v) = *reinterpret_cast<const uint4*>(x + (size_t)(p / top) * ldx + 16 * (size_t)v);
     }
   }
 }
 
+template <int NR>
 __global__ void __launch_bounds__(256) route_choose_kernel(const float* logits, size_t ld, int rows, int experts, int top, int score, bool renorm, Routing r) {
   pdl_wait();
   pdl_launch_dependents();
   const int m = blockIdx.x * 8 + (threadIdx.x >> 5);
   if (m >= rows) return;
-  choose_experts(logits + (size_t)m * ld, experts, top, score, renorm, [&](int i, int e, float w) {
+  choose_experts<NR>(logits + (size_t)m * ld, experts, top, score, renorm, [&](int i, int e, float w) {
     const size_t p = (size_t)m * top + i;
     r.expert[p] = e;
     r.weight[p] = w;
@@ -185,15 +199,26 @@ int launch_route(tq_ctx* ctx, const float* logits, size_t ld, size_t rows, size_
   const int pairs = (int)(rows * top), mj = (int)route_max_jobs(pairs, experts, chunk), vecs = (int)(row_bytes / 16);
   const uint8_t* xb = static_cast<const uint8_t*>(x);
   uint8_t* gb = static_cast<uint8_t*>(gathered);
-  if (pairs <= (gathered ? 64 : kErSmall)) {
-    TQ_CUDA(ctx, launch_k(ctx, route_small_kernel, dim3(1), dim3(kErThreads), 0, logits, ld, (int)rows, (int)experts, (int)top, score, renorm, (int)chunk, mj,
-                          r, xb, ldx_bytes, vecs, gb, ldg_bytes));
+  auto go = [&](auto nr) -> int {
+    constexpr int NR = decltype(nr)::value;
+    if (pairs <= (gathered ? 64 : kErSmall)) {
+      int threads = (int)(experts > 32 * rows ? experts : 32 * rows);
+      threads = threads < 256 ? 256 : threads > kErThreads ? kErThreads : (threads + 31) / 32 * 32;
+      TQ_CUDA(ctx, launch_k(ctx, route_small_kernel<NR>, dim3(1), dim3((unsigned)threads), 0, logits, ld, (int)rows, (int)experts, (int)top, score, renorm,
+                            (int)chunk, mj, r, xb, ldx_bytes, vecs, gb, ldg_bytes));
+      return TQ_OK;
+    }
+    TQ_CUDA(ctx, launch_k(ctx, route_choose_kernel<NR>, dim3((unsigned)((rows + 7) / 8)), dim3(256), 0, logits, ld, (int)rows, (int)experts, (int)top, score,
+                          renorm, r));
+    TQ_CUDA(ctx, launch_k(ctx, route_plan_kernel, dim3(1), dim3(kErThreads), 0, (int)experts, (int)chunk, mj, r));
+    TQ_CUDA(ctx, launch_k(ctx, route_place_kernel, dim3((unsigned)pairs), dim3(128), 0, (int)top, r, xb, ldx_bytes, vecs, gb, ldg_bytes));
     return TQ_OK;
-  }
-  TQ_CUDA(ctx, launch_k(ctx, route_choose_kernel, dim3((unsigned)((rows + 7) / 8)), dim3(256), 0, logits, ld, (int)rows, (int)experts, (int)top, score, renorm, r));
-  TQ_CUDA(ctx, launch_k(ctx, route_plan_kernel, dim3(1), dim3(kErThreads), 0, (int)experts, (int)chunk, mj, r));
-  TQ_CUDA(ctx, launch_k(ctx, route_place_kernel, dim3((unsigned)pairs), dim3(128), 0, (int)top, r, xb, ldx_bytes, vecs, gb, ldg_bytes));
-  return TQ_OK;
+  };
+  if (experts <= 32) return go(std::integral_constant<int, 1>());
+  if (experts <= 64) return go(std::integral_constant<int, 2>());
+  if (experts <= 128) return go(std::integral_constant<int, 4>());
+  if (experts <= 256) return go(std::integral_constant<int, 8>());
+  return go(std::integral_constant<int, kErMaxExperts / 32>());
 }
 
 }  // namespace tq

@@ -163,14 +163,18 @@ int launch_add_norm(tq_ctx* ctx, const AddNorm& a, size_t rows, size_t width) {
 
 // ------------------------------------------------------------------------------------------------ query / key norm, rotation
 // One CTA per row; the row's queries and keys pass through shared memory as f32 (a pair's halves sit in different places).
-template <typename T>
-__global__ void __launch_bounds__(kRoThreads) qk_norm_rope_kernel(QkNormRope a, const int* row_pos, const int* cache_row, size_t cache_rows) {
-  extern __shared__ float qr_smem[];
-  __shared__ float red[2][kRoWarps];
-  const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, half = a.rot.dims / 2;
-  float* qs = qr_smem;
-  float* ks = qs + nq;
-  float* cs = ks + nk;             // [half] cosine, then [half] sine
+// VEC: everything in 16-byte pieces; a thread then handles one piece of a row at a time.
+constexpr int kQkMaxThreads = 640;
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kQkMaxThreads) qk_norm_rope_kernel(QkNormRope a, const int* row_pos, const int* cache_row, size_t cache_rows) {
+  extern __shared__ __align__(16) float qr_smem[];
+  __shared__ float red[2][kQkMaxThreads / 32];
+  constexpr int V = VEC ? 16 / (int)sizeof(T) : 1;
+  const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, half = a.rot.dims / 2, per = a.dim / V;
+  const int n_pieces = (nq + nk) / V;
+  float* vals = qr_smem;                     // [nq + nk]: queries, then keys
+  float* cs = vals + nq + nk;                // [half] cosine, then [half] sine
   pdl_wait();
   pdl_launch_dependents();
   const int m = blockIdx.x, crow = cache_row[m];
@@ -178,49 +182,43 @@ __global__ void __launch_bounds__(kRoThreads) qk_norm_rope_kernel(QkNormRope a, 
   T* q = static_cast<T*>(a.q) + (size_t)m * a.ldq;
   const T* raw = static_cast<const T*>(a.raw) + (size_t)crow * a.kv_heads * a.raw_pad;
   T* keys = static_cast<T*>(a.keys) + (size_t)crow * a.kv_heads * a.key_pad;
-  const float pos = (float)row_pos[m];
-  for (int i = threadIdx.x; i < half; i += kRoThreads) {
-    float s, c;
-    sincosf(pos * a.rot.freq[i], &s, &c);
-    cs[i] = c * a.rot.mult;
-    cs[half + i] = s * a.rot.mult;
-  }
-  float sq = 0.f, sk = 0.f;
-  constexpr int V = 16 / sizeof(T);
-  const bool vec = a.dim % V == 0 && a.ldq % V == 0 && a.raw_pad % V == 0 && a.key_pad % V == 0;
   auto unpack = [](const uint4& u, float (&f)[V]) {
     const uint32_t w[4] = {u.x, u.y, u.z, u.w};
 #pragma unroll
     for (int j = 0; j < V; ++j) f[j] = V == 4 ? __uint_as_float(w[j & 3]) : bf16_bits_to_float(j & 1 ? w[(j >> 1) & 3] >> 16 : w[(j >> 1) & 3] & 0xFFFFu);
   };
-  if (vec) {
-    const int per = a.dim / V;
-    for (int i = threadIdx.x; i < (nq + nk) / V; i += kRoThreads) {
-      const bool is_q = i < nq / V;
-      const int c = is_q ? i : i - nq / V;
-      float f[V];
-      unpack(*reinterpret_cast<const uint4*>(is_q ? q + c * V : raw + (c / per) * a.raw_pad + (c % per) * V), f);
-      float* dst = (is_q ? qs : ks) + c * V;
-      float s = 0.f;
+  auto load = [&](const T* p, float (&f)[V]) {
+    if constexpr (VEC) unpack(*reinterpret_cast<const uint4*>(p), f);
+    else f[0] = ro_load(p);
+  };
+  float sq = 0.f, sk = 0.f;
+  for (int i = threadIdx.x; i < n_pieces; i += blockDim.x) {
+    const bool is_q = i < nq / V;
+    const int c = is_q ? i : i - nq / V;
+    float f[V], s = 0.f;
+    if (is_q) {
+      load(q + c * V, f);
+    } else {
+      const int head = (int)((unsigned)c / (unsigned)per);
+      load(raw + head * a.raw_pad + (c - head * per) * V, f);
+    }
 #pragma unroll
-      for (int j = 0; j < V; ++j) {
-        dst[j] = f[j];
-        s += f[j] * f[j];
-      }
-      if (is_q) sq += s;
-      else sk += s;
+    for (int j = 0; j < V; ++j) s += f[j] * f[j];
+    if constexpr (VEC) {
+#pragma unroll
+      for (int j = 0; j < V; j += 4) *reinterpret_cast<float4*>(vals + (size_t)i * V + j) = make_float4(f[j], f[j + 1], f[j + 2], f[j + 3]);
+    } else {
+      vals[i] = f[0];
     }
-  } else {
-    for (int i = threadIdx.x; i < nq; i += kRoThreads) {
-      const float v = ro_load(q + i);
-      qs[i] = v;
-      sq += v * v;
-    }
-    for (int i = threadIdx.x; i < nk; i += kRoThreads) {
-      const float v = ro_load(raw + (i / a.dim) * a.raw_pad + i % a.dim);
-      ks[i] = v;
-      sk += v * v;
-    }
+    if (is_q) sq += s;
+    else sk += s;
+  }
+  const float pos = (float)row_pos[m];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf(pos * a.rot.freq[i], &s, &c);
+    cs[i] = c * a.rot.mult;
+    cs[half + i] = s * a.rot.mult;
   }
   sq = warp_sum(sq);
   sk = warp_sum(sk);
@@ -229,39 +227,62 @@ __global__ void __launch_bounds__(kRoThreads) qk_norm_rope_kernel(QkNormRope a, 
     red[1][threadIdx.x >> 5] = sk;
   }
   __syncthreads();
-  sq = sk = 0.f;
-#pragma unroll
-  for (int i = 0; i < kRoWarps; ++i) {
-    sq += red[0][i];
-    sk += red[1][i];
-  }
+  const bool has = (threadIdx.x & 31) < (blockDim.x >> 5);
+  sq = warp_sum(has ? red[0][threadIdx.x & 31] : 0.f);
+  sk = warp_sum(has ? red[1][threadIdx.x & 31] : 0.f);
   const float qi = 1.0f / sqrtf(sq / (float)nq + a.eps), ki = 1.0f / sqrtf(sk / (float)nk + a.eps);
-  const T *qg = static_cast<const T*>(a.q_gain), *kg = static_cast<const T*>(a.k_gain);
-  // value i of a row, normed and rotated
-  auto value = [&](const float* row, const T* gain, float inv, int i) -> float {
-    const int d = i % a.dim;
-    const float own = row[i] * inv * ro_load(gain + i);
-    if (d >= 2 * half) return own;
-    const bool first = d < half;
-    const int o = first ? i + half : i - half, f = first ? d : d - half;
-    const float other = row[o] * inv * ro_load(gain + o);
-    return first ? own * cs[f] - other * cs[half + f] : own * cs[f] + other * cs[half + f];
-  };
-  if (vec) {
-    const int per = a.dim / V;
-    for (int i = threadIdx.x; i < (nq + nk) / V; i += kRoThreads) {
-      const bool is_q = i < nq / V;
-      const int c = is_q ? i : i - nq / V;
-      float f[V];
+  for (int i = threadIdx.x; i < n_pieces; i += blockDim.x) {
+    const bool is_q = i < nq / V;
+    const int c = is_q ? i : i - nq / V, head = (int)((unsigned)c / (unsigned)per), d0 = (c - head * per) * V;
+    const float inv = is_q ? qi : ki;
+    const T* gain = static_cast<const T*>(is_q ? a.q_gain : a.k_gain);
+    // V values of the row from vals[at], normed
+    auto piece = [&](int at, float (&f)[V]) {
+      float gf[V];
+      load(gain + at, gf);
+      const float* src = vals + (is_q ? 0 : nq) + at;
+      if constexpr (VEC) {
 #pragma unroll
-      for (int j = 0; j < V; ++j) f[j] = is_q ? value(qs, qg, qi, c * V + j) : value(ks, kg, ki, c * V + j);
-      T* dst = is_q ? q + c * V : keys + (c / per) * a.key_pad + (c % per) * V;
-      ro_store4(dst, make_float4(f[0], f[1], f[2], f[3]));
-      if constexpr (V == 8) ro_store4(dst + 4, make_float4(f[4], f[5], f[6], f[7]));
+        for (int j = 0; j < V; j += 4) {
+          const float4 v = *reinterpret_cast<const float4*>(src + j);
+          f[j] = v.x, f[j + 1] = v.y, f[j + 2] = v.z, f[j + 3] = v.w;
+        }
+      } else {
+        f[0] = *src;
+      }
+#pragma unroll
+      for (int j = 0; j < V; ++j) f[j] *= inv * gf[j];
+    };
+    float f[V];
+    piece(c * V, f);
+    if (d0 < 2 * half) {
+      if (half % V == 0) {                   // whole pieces turn with whole pieces
+        const bool first = d0 < half;
+        const int r = first ? d0 : d0 - half;
+        float o[V];
+        piece(c * V + (first ? half : -half), o);
+#pragma unroll
+        for (int j = 0; j < V; ++j) f[j] = f[j] * cs[r + j] + (first ? -o[j] : o[j]) * cs[half + r + j];
+      } else {
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+          const int d = d0 + j;
+          if (d < 2 * half) {
+            const bool first = d < half;
+            const int shift = first ? half : -half, r = first ? d : d - half;
+            const float other = vals[i * V + j + shift] * inv * ro_load(gain + c * V + j + shift);
+            f[j] = f[j] * cs[r] + (first ? -other : other) * cs[half + r];
+          }
+        }
+      }
     }
-  } else {
-    for (int i = threadIdx.x; i < nq; i += kRoThreads) ro_store(q + i, value(qs, qg, qi, i));
-    for (int i = threadIdx.x; i < nk; i += kRoThreads) ro_store(keys + (i / a.dim) * a.key_pad + i % a.dim, value(ks, kg, ki, i));
+    T* dst = is_q ? q + c * V : keys + head * a.key_pad + d0;
+    if constexpr (VEC) {
+#pragma unroll
+      for (int j = 0; j < V; j += 4) ro_store4(dst + j, make_float4(f[j], f[j + 1], f[j + 2], f[j + 3]));
+    } else {
+      ro_store(dst, f[0]);
+    }
   }
 }
 
@@ -271,12 +292,18 @@ int launch_qk_norm_rope(tq_ctx* ctx, const QkNormRope& a, const RaggedBatch& b, 
   if (b.rows == 0) return TQ_OK;
   const size_t smem = ((size_t)(a.heads + a.kv_heads) * a.dim + a.rot.dims) * sizeof(float);
   TQ_REQUIRE(ctx, smem <= 200 * 1024, "query/key norm: %d + %d heads of %d values are too many", a.heads, a.kv_heads, a.dim);
-  auto go = [&](auto kern) -> int {
+  auto go = [&](auto kern, int v) -> int {
+    // one round of pieces when there are few rows, several rounds per thread when the rows fill the GPU anyway
+    const int pieces = (a.heads + a.kv_heads) * a.dim / v, most = b.rows >= 4 * ctx->sm_count ? 256 : kQkMaxThreads, threads = pieces >= most ? most : (pieces + 31) / 32 * 32;
     if (smem > 48 * 1024) TQ_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)b.rows), dim3(kRoThreads), smem, a, b.row_pos, b.cache_row, b.cache_rows));
+    TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)b.rows), dim3((unsigned)threads), smem, a, b.row_pos, b.cache_row, b.cache_rows));
     return TQ_OK;
   };
-  return dtype == TQ_F32 ? go(qk_norm_rope_kernel<float>) : go(qk_norm_rope_kernel<__nv_bfloat16>);
+  const int v = dtype == TQ_F32 ? 4 : 8;
+  const uintptr_t bits = (uintptr_t)a.q | (uintptr_t)a.raw | (uintptr_t)a.keys | (uintptr_t)a.q_gain | (uintptr_t)a.k_gain;
+  const bool vec = a.dim % v == 0 && a.ldq % v == 0 && a.raw_pad % v == 0 && a.key_pad % v == 0 && (bits & 15) == 0;
+  if (dtype == TQ_F32) return vec ? go(qk_norm_rope_kernel<float, true>, v) : go(qk_norm_rope_kernel<float, false>, 1);
+  return vec ? go(qk_norm_rope_kernel<__nv_bfloat16, true>, v) : go(qk_norm_rope_kernel<__nv_bfloat16, false>, 1);
 }
 
 void yarn_frequencies(int dims, double base, double factor, double original, double fast, double slow, float* freq, float* mult) {
