@@ -294,7 +294,8 @@ int launch_qk_norm_rope(tq_ctx* ctx, const QkNormRope& a, const RaggedBatch& b, 
   TQ_REQUIRE(ctx, smem <= 200 * 1024, "query/key norm: %d + %d heads of %d values are too many", a.heads, a.kv_heads, a.dim);
   auto go = [&](auto kern, int v) -> int {
     // one round of pieces when there are few rows, several rounds per thread when the rows fill the GPU anyway
-    const int pieces = (a.heads + a.kv_heads) * a.dim / v, most = b.rows >= 4 * ctx->sm_count ? 256 : kQkMaxThreads, threads = pieces >= most ? most : (pieces + 31) / 32 * 32;
+    const int pieces = (a.heads + a.kv_heads) * a.dim / v, most = b.rows >= 4 * ctx->sm_count ? 256 : kQkMaxThreads;
+    const int threads = pieces >= most ? most : (pieces + 31) / 32 * 32;
     if (smem > 48 * 1024) TQ_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)b.rows), dim3((unsigned)threads), smem, a, b.row_pos, b.cache_row, b.cache_rows));
     return TQ_OK;
