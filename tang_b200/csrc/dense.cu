@@ -431,7 +431,7 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
           float* pp = p.partial + ((size_t)z * p.m + mb) * n_pad + row;
 #pragma unroll
           for (int j = 0; j < 16; ++j)
-            if (j < n) __stcg(pp + (size_t)j * n_pad, v[j]);
+            if (j < n && dst.base) __stcg(pp + (size_t)j * n_pad, v[j]);
           continue;
         }
         if (p.epi.row_scale) {
@@ -496,25 +496,36 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
         if (*last_flag) {
           __threadfence();
           const size_t plane = (size_t)p.m * n_pad;
-          // warp (q, half): features 32q.., every other pair of rows
-          const bool upper = lane & 8;
-          for (int c0 = 4 * half; c0 < m_n; c0 += 8) {
+          // the 256 threads: F features (as many as the tile has) x 256 / F groups of four rows
+          int F = kUmmaRows;
+          while (F > 16 && ft * kUmmaRows + F / 2 >= p.epi.s[p.epi.n - 1].row_end) F >>= 1;
+          const int mrow = ft * kUmmaRows + (et & (F - 1)), rows_step = 4 * (256 / F);
+          const DenseDst md = dense_dst(p.epi, mrow);
+          const bool upper = et & 8;
+          for (int r0 = 0; r0 < m_n; r0 += rows_step) {       // (the same number of turns for every lane: they exchange below)
+            const int c0 = r0 + 4 * (et / F);
             float v[4] = {0.f, 0.f, 0.f, 0.f};
-            const int n = min(4, m_n - c0), mb = m0 + c0;
-            const float* src = p.partial + (size_t)mb * n_pad + row;
-            for (int zz = 0; zz < p.splits; ++zz) {
+            const int n = md.base ? min(4, m_n - c0) : 0, mb = m0 + c0;
+            const float* src = p.partial + (size_t)mb * n_pad + mrow;
+            for (int z0 = 0; z0 < p.splits; z0 += 4) {        // sixteen loads in flight, added in split order
+              float part[4][4];
 #pragma unroll
-              for (int j = 0; j < 4; ++j)
-                if (j < n) v[j] += __ldcg(src + (size_t)zz * plane + (size_t)j * n_pad);
+              for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) part[i][j] = z0 + i < p.splits && j < n ? __ldcg(src + (size_t)(z0 + i) * plane + (size_t)j * n_pad) : 0.f;
+#pragma unroll
+              for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) v[j] += part[i][j];
             }
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
               const float other = __shfl_xor_sync(0xffffffffu, v[j], 8);
               if (j >= n) continue;
-              if (dst.kind == DENSE_GLU) {
-                if (!upper) dense_store(p.epi, dst, mb + j, clamped_glu(v[j], other, p.epi.glu_limit, p.epi.glu_alpha));
+              if (md.kind == DENSE_GLU) {
+                if (!upper) dense_store(p.epi, md, mb + j, clamped_glu(v[j], other, p.epi.glu_limit, p.epi.glu_alpha));
               } else {
-                dense_store(p.epi, dst, mb + j, v[j]);
+                dense_store(p.epi, md, mb + j, v[j]);
               }
             }
           }
