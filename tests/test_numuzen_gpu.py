@@ -245,6 +245,16 @@ def test_other_sizes(dev, layers, width, vocab):
         model.destroy()
 
 
+def test_long_rows_split_over_k(dev):
+    """Wide enough that the router's and the mixers' products are split over k."""
+    cfg = config([attn(2, 1, 16, 20, moe(20, 3, 40)), gla(2, 16, 32, moe(3, 1, 24))], width=1100, vocab=50)
+    w = weights(cfg, 41)
+    tokens = [int(t) for t in np.random.default_rng(42).integers(0, 50, 90)]
+    model = make(dev, cfg, w, "bf16", max_slots=1, max_seq=90)
+    assert row_errors(engine(model).step([(0, tokens, range(90))]), reference(cfg, w, tokens)).max() < TOL["bf16"]
+    model.destroy()
+
+
 def greedy(cfg, w, prompt, n):
     m = N.Numuzen(cfg, w)
     st = m.new_state()

@@ -185,6 +185,17 @@ def test_edges_show_in_prompts_and_in_decoding(dev, window, keep):
             model.destroy()
 
 
+@pytest.mark.parametrize("ff", [5, 24, 130])
+def test_long_rows_split_over_k(dev, ff):
+    """Wide enough that the tcgen05 GEMM splits k over CTAs, with tiles of few features: projections, GLU and residual."""
+    cfg = config([layer(2, 1, 8, 16, 20, 1, ff=ff), layer(2, 2, 4, 8, 9, 0, ff=ff)], width=1100)
+    w = weights(cfg, 41)
+    tokens = list(np.random.default_rng(42).integers(0, cfg["vocab"], 45))
+    model = make(dev, cfg, w, "bf16", max_slots=1)
+    assert row_errors(engine(model).step([(0, tokens, range(45))]), reference(cfg, w, tokens)).max() < TOL["bf16"]
+    model.destroy()
+
+
 def test_long_decoding_crosses_windows_and_tiles(dev):
     cfg = config([layer(4, 2, 24, 32, 21, 2, ff=48), layer(4, 2, 24, 32, 100, 0, ff=48, kv_from=0)], max_positions=300)
     w = weights(cfg, 31, sharp=2.0)
