@@ -548,6 +548,27 @@ TQ_API int tq_add_norm(tq_ctx* ctx, float* x_dev, const float* y_dev_or_null, co
 TQ_API int tq_qk_norm_rope(tq_ctx* ctx, int dtype, size_t heads, size_t kv_heads, size_t dim, void* q_dev, size_t ldq, const void* raw_dev,
                            void* keys_dev, size_t cache_rows, const void* q_gain_dev, const void* k_gain_dev, size_t rot_dims,
                            const float* freq_dev, float rot_mult, float eps, const int* row_pos_dev, const int* cache_row_dev, size_t rows);
+/* Per-head norm and rotation.  Queries (head h of row m at q + m * ldq + h * q_head) are divided by the root mean square over
+ * their `dim` values and multiplied by q_gain [dim] (NULL: no norm), then rotated in place: pair i of the rot_dims dimensions from
+ * rot_first on is (i, i + rot_dims / 2), or with `interleaved` (2i, 2i + 1).  Keys (kv_heads of them, may be 0) as in
+ * tq_qk_norm_rope, with k_gain [dim]. */
+TQ_API int tq_head_norm_rope(tq_ctx* ctx, int dtype, size_t heads, size_t kv_heads, size_t dim, void* q_dev, size_t ldq, size_t q_head,
+                             const void* raw_dev_or_null, void* keys_dev_or_null, size_t cache_rows, const void* q_gain_dev_or_null,
+                             const void* k_gain_dev_or_null, size_t rot_first, size_t rot_dims, int interleaved, const float* freq_dev, float rot_mult,
+                             float eps, const int* row_pos_dev, const int* cache_row_dev, size_t rows);
+/* base^(-2i/dims) with factor > 0 stretched by wavelength: kept below original / high, divided by `factor` above original / low,
+ * blended between. */
+TQ_API int tq_banded_frequencies(size_t dims, double base, double factor, double low, double high, double original, float* freq_host);
+/* Residual streams.  x has `streams` rows of `width` per row of the batch (src_streams 1: one row that stands for all).
+ *   x'_t = sum_s mix[s * streams + t] x_s + w_out[t] y             (y NULL: x' = x, nothing is stored)
+ *   out  = rms_norm(sum_s w_in[s] x'_s) * gain                     (gain NULL: not formed);   sum = sum_s x'_s (NULL: not stored)
+ * y = sum over n_y of weight[m * n_y + i] * row (y_rows[m * n_y + i]) of y, where a negative row stands for `self` row m (of
+ * out_dtype, ld_out apart; may be `out` itself), + row m of y_more.  y_rows NULL: row m of y with weight 1. */
+TQ_API int tq_stream_mix(tq_ctx* ctx, size_t streams, size_t src_streams, const float* src_dev, float* dst_dev_or_null, const float* y_dev_or_null,
+                         const int* y_rows_dev_or_null, const float* y_weight_dev_or_null, size_t n_y, const void* self_dev_or_null,
+                         const float* y_more_dev_or_null, const float* mix_dev_or_null, const float* w_out_dev_or_null, const float* w_in_dev_or_null,
+                         const float* gain_dev_or_null, size_t rows, size_t width, float eps, void* out_dev_or_null, int out_dtype, size_t ld_out,
+                         float* sum_dev_or_null);
 /* Grouped-query attention: s = (q . k) scale, softcap * tanh(s / softcap) unless softcap is 0; weights
  * exp(s_j) / (exp(sink) + sum exp(s)) (sink -infinity: none); the query at position i sees j when 0 <= i - j < window; the
  * result times sigmoid(gate).  q [rows][ldq], gate (may be NULL) [rows][ldg], caches as in tq_diff_attention with one map. */
@@ -560,6 +581,11 @@ TQ_API int tq_window_attention(tq_ctx* ctx, const tq_window_attn_config* cfg, in
                                const void* gate_dev_or_null, size_t ldg, const void* k_cache_dev, const void* v_cache_dev, size_t cache_rows,
                                const int* seq_rows_dev_or_null, const int* row_pos_dev, const int* cache_row_dev, size_t n_seqs, size_t rows,
                                size_t max_q, size_t max_len, void* out_dev, size_t ldo);
+/* The same with a sink per head (sinks [heads] f32; NULL: cfg->sink for all). */
+TQ_API int tq_window_attention_sinks(tq_ctx* ctx, const tq_window_attn_config* cfg, const float* sinks_dev_or_null, int dtype, const void* q_dev,
+                                     size_t ldq, const void* gate_dev_or_null, size_t ldg, const void* k_cache_dev, const void* v_cache_dev,
+                                     size_t cache_rows, const int* seq_rows_dev_or_null, const int* row_pos_dev, const int* cache_row_dev,
+                                     size_t n_seqs, size_t rows, size_t max_q, size_t max_len, void* out_dev, size_t ldo);
 /* Gated linear attention: S_t = diag(alpha_t) S_(t-1) + k_t v_t^T, o_t = S_t^T (q_scale q_t), per head, with
  * alpha_t = sigmoid(a2 a1_t + bias)^(1/tau) per key channel; out = o / sqrt(mean(o^2) + eps) * norm * silu(gate).  Rows of q, k
  * (heads * dim), v, gate (heads * vdim) are `ld` elements apart, a1 [rows][ld_a1] and everything about the state is f32.
@@ -577,6 +603,11 @@ TQ_API int tq_gla(tq_ctx* ctx, const tq_gla_config* cfg, int dtype, const void* 
  * consecutive.  jobs int[.][4]: (expert, first slot, slots <= chunk, 0), at most min(pairs, experts + pairs / chunk). */
 TQ_API int tq_route(tq_ctx* ctx, const float* logits_dev, size_t rows, size_t experts, size_t top, int score, int renorm, size_t chunk,
                     int* expert_dev, float* weight_dev, int* slot_dev, int* slot_row_dev, int* jobs_dev, int* n_jobs_dev);
+/* The same with a correction [experts] (NULL: none) added to the scores for the choice but not for the weights, and `identity`
+ * experts without weights at the end of the list: a pair that chose one of them has slot -1 and is in no job. */
+TQ_API int tq_route_rule(tq_ctx* ctx, const float* logits_dev, size_t rows, size_t experts, size_t top, int score, int renorm,
+                         const float* correction_dev_or_null, size_t identity, size_t chunk, int* expert_dev, float* weight_dev, int* slot_dev,
+                         int* slot_row_dev, int* jobs_dev, int* n_jobs_dev);
 
 /* ---- Numuzen ------------------------------------------------------------------------------------
  * No reference counterpart.  A decoder with a norm before and after every sublayer (weights stored around zero),

@@ -118,8 +118,13 @@ PROTOTYPES = {
     "tq_add_norm": (_i, [_p, _p, _p, _p, _sz, _p, _p, _sz, _sz, C.c_float, _p, _i, _sz]),
     "tq_qk_norm_rope": (_i, [_p, _i, _sz, _sz, _sz, _p, _sz, _p, _p, _sz, _p, _p, _sz, _p, C.c_float, C.c_float, _p, _p, _sz]),
     "tq_window_attention": (_i, [_p, _p, _i, _p, _sz, _p, _sz, _p, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _sz, _p, _sz]),
+    "tq_window_attention_sinks": (_i, [_p, _p, _p, _i, _p, _sz, _p, _sz, _p, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _sz, _p, _sz]),
+    "tq_head_norm_rope": (_i, [_p, _i, _sz, _sz, _sz, _p, _sz, _sz, _p, _p, _sz, _p, _p, _sz, _sz, _i, _p, C.c_float, C.c_float, _p, _p, _sz]),
+    "tq_banded_frequencies": (_i, [_sz] + [C.c_double] * 5 + [_p]),
+    "tq_stream_mix": (_i, [_p, _sz, _sz, _p, _p, _p, _p, _p, _sz, _p, _p, _p, _p, _p, _p, _sz, _sz, C.c_float, _p, _i, _sz, _p]),
     "tq_gla": (_i, [_p, _p, _i, _p, _p, _p, _p, _sz, _p, _sz, _p, _p, _p, _p, _sz, _sz, _p, _p, _p, _sz, _sz, _sz, _p, _sz]),
     "tq_route": (_i, [_p, _p, _sz, _sz, _sz, _i, _i, _sz, _p, _p, _p, _p, _p, _p]),
+    "tq_route_rule": (_i, [_p, _p, _sz, _sz, _sz, _i, _i, _p, _sz, _sz, _p, _p, _p, _p, _p, _p]),
     "tq_numuzen_create": (_i, [_p, _p, _p, _pp]),
     "tq_numuzen_destroy": (_i, [_p]),
     "tq_numuzen_put": (_i, [_p, _i, _sz, _sz, _p, _i, _sz, _sz]),

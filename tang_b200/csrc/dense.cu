@@ -103,7 +103,7 @@ __global__ void __launch_bounds__(kGvThreads, 2) dgemv_kernel(const __grid_const
   }
 
   const size_t xs_stride = row_bytes + 16;   // bytes; 16 mod 32: two rows' reads, 32 bytes apart, do not meet in a bank
-  int m_rows = p.m, m_first = 0, job = -1;
+  int m_rows = p.m, m_first = 0, m_shift = 0, job = -1;
   if constexpr (!GROUPED) {
     if (p.h) {
       int wpr = kGvWarps;                        // warps per row
@@ -169,6 +169,7 @@ __global__ void __launch_bounds__(kGvThreads, 2) dgemv_kernel(const __grid_const
         job = tile / p.n_rb;
         const int4 jb = p.grp.jobs[job];
         m_first = jb.y;
+        m_shift = jb.w;
         m_rows = min(jb.z, p.grp.chunk);
         const int vpr = p.kpad / 8;
         for (int i = threadIdx.x; i < m_rows * vpr; i += kGvThreads) {
@@ -225,15 +226,15 @@ __global__ void __launch_bounds__(kGvThreads, 2) dgemv_kernel(const __grid_const
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < kGvWarps; ++w) v += red[buf][w][row * 8 + m];
-        const float scale = p.epi.row_scale ? p.epi.row_scale[m_first + m] : 1.f;
+        const float scale = p.epi.row_scale ? p.epi.row_scale[m_first + m_shift + m] : 1.f;
         v *= scale;
         if (d.kind == DENSE_GLU) {
           float up = 0.f;
 #pragma unroll
           for (int w = 0; w < kGvWarps; ++w) up += red[buf][w][(row + 8) * 8 + m];
-          v = clamped_glu(v, up * scale, p.epi.glu_limit, p.epi.glu_alpha);
+          v = dense_glu(p.epi, v, up * scale);
         }
-        dense_store(p.epi, d, m_first + m, v);
+        dense_store(p.epi, d, m_first + m_shift + m, v);
       }
     }
     buf ^= 1;
@@ -420,7 +421,7 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
       if (!good) give_up(DERR_TMEM);
       tc_fence_after();
       const int row = ft * kUmmaRows + 32 * q + lane;
-      const int m0 = x_row(tt), m_n = good ? min(p.ntok, p.grouped ? p.grp.jobs[tt].z : p.m - m0) : 0;
+      const int m0 = x_row(tt) + (p.grouped ? p.grp.jobs[tt].w : 0), m_n = good ? min(p.ntok, p.grouped ? p.grp.jobs[tt].z : p.m - m0) : 0;
       const uint32_t t_addr = tmem_d + (uint32_t)(a * p.acc_stride) + ((uint32_t)(32 * q) << 16);
       const DenseDst dst = dense_dst(p.epi, row);
       for (int c0 = 16 * half; c0 < m_n; c0 += 32) {
@@ -450,8 +451,7 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
             const float give = upper ? v[j] : v[j + 1];
             const float got = __shfl_xor_sync(0xffffffffu, give, 8);
             if (glu) {
-              const float val = upper ? clamped_glu(got, v[j + 1], p.epi.glu_limit, p.epi.glu_alpha)
-                                      : clamped_glu(v[j], got, p.epi.glu_limit, p.epi.glu_alpha);
+              const float val = upper ? dense_glu(p.epi, got, v[j + 1]) : dense_glu(p.epi, v[j], got);
               const int jj = upper ? j + 1 : j;
               if (jj < n) dense_store(p.epi, dst, mb + jj, val);
             }
@@ -523,7 +523,7 @@ dgemm_umma_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
               const float other = __shfl_xor_sync(0xffffffffu, v[j], 8);
               if (j >= n) continue;
               if (md.kind == DENSE_GLU) {
-                if (!upper) dense_store(p.epi, md, mb + j, clamped_glu(v[j], other, p.epi.glu_limit, p.epi.glu_alpha));
+                if (!upper) dense_store(p.epi, md, mb + j, dense_glu(p.epi, v[j], other));
               } else {
                 dense_store(p.epi, md, mb + j, v[j]);
               }
@@ -556,12 +556,13 @@ __global__ void __launch_bounds__(256) dgemm_f32_kernel(const float* w, int kpad
   pdl_wait();
   pdl_launch_dependents();
   const int n0 = blockIdx.x * kDfTile;
-  int m0 = blockIdx.y * kDfTile;
+  int m0 = blockIdx.y * kDfTile, shift = 0;
   if (grp.jobs) {
     if ((int)blockIdx.y >= *grp.n_jobs) return;
     const int4 job = grp.jobs[blockIdx.y];
     w += (size_t)job.x * grp.group_rows * kpad;
     m0 = job.y;
+    shift = job.w;
     m = min(m, m0 + min(job.z, kDfTile));
   }
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;      // features 4 tx.., rows 4 ty..
@@ -596,10 +597,10 @@ __global__ void __launch_bounds__(256) dgemm_f32_kernel(const float* w, int kpad
   const DenseDst d = dense_dst(epi, n0 + n);
   if (d.kind == DENSE_GLU && (n & 8)) return;
   for (int r = threadIdx.x >> 6; r < kDfTile && m0 + r < m; r += 4) {
-    const float scale = epi.row_scale ? epi.row_scale[m0 + r] : 1.f;
+    const float scale = epi.row_scale ? epi.row_scale[m0 + shift + r] : 1.f;
     float v = ys[r][n] * scale;
-    if (d.kind == DENSE_GLU) v = clamped_glu(v, ys[r][n + 8] * scale, epi.glu_limit, epi.glu_alpha);
-    dense_store(epi, d, m0 + r, v);
+    if (d.kind == DENSE_GLU) v = dense_glu(epi, v, ys[r][n + 8] * scale);
+    dense_store(epi, d, m0 + shift + r, v);
   }
 }
 
@@ -716,6 +717,13 @@ int dense_group_chunk(int dtype, size_t kpad, size_t rows, size_t n_groups) {
   return (int)(((need + jobs - 1) / jobs + 15) / 16 * 16);
 }
 
+int dense_even_chunk(int dtype, size_t kpad, size_t rows) {
+  if (dtype == TQ_F32) return kDfTile;
+  if (rows <= kGvRows && kGvRows * (kpad * 2 + 16) <= kGvSmemMax) return (int)kGvRows;
+  const size_t jobs = (rows + 255) / 256;
+  return (int)(((rows + jobs - 1) / jobs + 15) / 16 * 16);
+}
+
 int launch_dense_grouped(tq_ctx* ctx, const tq_dweight* w, const void* x, size_t ldx, size_t rows, const DenseGroups& g, const DenseEpilogue& epi) {
   if (rows == 0) return TQ_OK;
   TQ_REQUIRE(ctx, g.jobs && g.n_jobs && g.max_jobs > 0 && g.chunk > 0 && g.group_rows > 0 && g.group_rows % 16 == 0, "grouped dense linear: bad groups");
@@ -787,6 +795,32 @@ __global__ void dweight_put_kernel(const void* src, int s_dt, void* dst, int d_d
   const size_t o = dr * kpad + col0 + c;
   if (d_dt == TQ_F32) reinterpret_cast<float*>(dst)[o] = v;
   else reinterpret_cast<__nv_bfloat16*>(dst)[o] = __float2bfloat16_rn(v);
+}
+
+__global__ void dweight_put_head_t_kernel(const void* src, int s_dt, void* dst, int d_dt, size_t heads, size_t dim, size_t rank, size_t group_rows, size_t kpad) {
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= heads * dim * rank) return;
+  const size_t r = i / rank, c = i % rank, o = (r / dim * group_rows + c) * kpad + r % dim;
+  const float v = s_dt == TQ_F32 ? reinterpret_cast<const float*>(src)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(src)[i]);
+  if (d_dt == TQ_F32) reinterpret_cast<float*>(dst)[o] = v;
+  else reinterpret_cast<__nv_bfloat16*>(dst)[o] = __float2bfloat16_rn(v);
+}
+
+int dweight_put_head_transposed(tq_ctx* ctx, tq_dweight* w, const void* src, int src_dtype, size_t heads, size_t dim, size_t rank, size_t group_rows) {
+  TQ_REQUIRE(ctx, rank <= group_rows && heads * group_rows <= w->rpad && dim <= w->kpad, "dense weight: transposed heads outside the weight");
+  const size_t n = heads * dim * rank, bytes = n * dtype_size(src_dtype);
+  void* tmp = nullptr;
+  TQ_CUDA(ctx, cudaMalloc(&tmp, bytes));
+  cudaError_t e = cudaMemcpyAsync(tmp, src, bytes, cudaMemcpyDefault, ctx->stream);
+  if (e == cudaSuccess) {
+    dweight_put_head_t_kernel<<<(unsigned)((n + 255) / 256), 256, 0, ctx->stream>>>(tmp, src_dtype, w->data, w->dtype, heads, dim, rank, group_rows, w->kpad);
+    ctx->launches++;
+    e = cudaGetLastError();
+  }
+  if (e == cudaSuccess) e = cudaStreamSynchronize(ctx->stream);
+  cudaFree(tmp);
+  TQ_CUDA(ctx, e);
+  return TQ_OK;
 }
 
 __global__ void clamped_glu_kernel(const void* gate, const void* up, int dt, size_t n, float limit, float alpha, void* out, int out_dt) {

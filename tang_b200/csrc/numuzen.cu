@@ -468,7 +468,7 @@ static int expert_layer(tq_numuzen* m, const Layer& L, size_t rows) {
   g.max_jobs = (int)route_max_jobs(pairs, c.experts, g.chunk);
   // the tcgen05 kernel copies boxes of consecutive rows, the others follow the slots' row numbers
   const bool gather = !f32 && g.chunk > 8;
-  TQ_STEP(launch_route(ctx, m->logits, m->max_experts, rows, c.experts, c.top, ROUTE_SIGMOID, false, g.chunk, m->route, m->hn, hn_ld * es, up8(width) * es,
+  TQ_STEP(launch_route(ctx, m->logits, m->max_experts, rows, c.experts, c.top, RouteRule(), g.chunk, m->route, m->hn, hn_ld * es, up8(width) * es,
                        gather ? m->xs : nullptr, hn_ld * es));
   DenseEpilogue u;
   section(u, L.gu_rows, c.ff, DENSE_GLU, f32, m->act, m->act_ld);

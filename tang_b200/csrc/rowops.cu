@@ -4,6 +4,7 @@
 #include <cuda_bf16.h>
 
 #include <cmath>
+#include <type_traits>
 
 #include "common.cuh"
 
@@ -307,6 +308,173 @@ int launch_qk_norm_rope(tq_ctx* ctx, const QkNormRope& a, const RaggedBatch& b, 
   return vec ? go(qk_norm_rope_kernel<__nv_bfloat16, true>, v) : go(qk_norm_rope_kernel<__nv_bfloat16, false>, 1);
 }
 
+// ------------------------------------------------------------------------------------------------ per-head norm, rotation
+// blockIdx.x: row; the CTA's warps (and blockIdx.y's CTAs) share its heads, queries first.  A head passes through its warp's shared
+// memory as f32; the row's cosines and sines are formed once per CTA.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) head_norm_rope_kernel(HeadNormRope a, const int* row_pos, const int* cache_row, size_t cache_rows) {
+  extern __shared__ __align__(16) float hr_smem[];
+  constexpr int V = VEC ? 16 / (int)sizeof(T) : 1;
+  const QkNormRope& r = a.r;
+  const int half = r.rot.dims / 2, dim = r.dim, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  float* cs = hr_smem;                                    // [half] cosine, then [half] sine
+  float* vals = hr_smem + (2 * half + 3) / 4 * 4 + (size_t)warp * ((dim + 3) / 4 * 4);
+  pdl_wait();
+  pdl_launch_dependents();
+  const int m = blockIdx.x, crow = cache_row[m];
+  if (crow < 0 || (size_t)crow >= cache_rows) return;
+  const float pos = (float)row_pos[m];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf(pos * r.rot.freq[i], &s, &c);
+    cs[i] = c * r.rot.mult;
+    cs[half + i] = s * r.rot.mult;
+  }
+  __syncthreads();
+  for (int h = blockIdx.y * warps + warp; h < r.heads + r.kv_heads; h += warps * gridDim.y) {
+    const bool is_q = h < r.heads;
+    const int g = h - r.heads;
+    const T* src = is_q ? static_cast<const T*>(r.q) + (size_t)m * r.ldq + (size_t)h * a.q_head
+                        : static_cast<const T*>(r.raw) + ((size_t)crow * r.kv_heads + g) * r.raw_pad;
+    T* dst = is_q ? static_cast<T*>(r.q) + (size_t)m * r.ldq + (size_t)h * a.q_head : static_cast<T*>(r.keys) + ((size_t)crow * r.kv_heads + g) * r.key_pad;
+    const T* gain = static_cast<const T*>(is_q ? r.q_gain : r.k_gain);
+    float sq = 0.f;
+    for (int d = lane * V; d < dim; d += 32 * V) {
+      if constexpr (VEC) {
+        const uint4 u = *reinterpret_cast<const uint4*>(src + d);
+        const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+          const float f = V == 4 ? __uint_as_float(w[j & 3]) : bf16_bits_to_float(j & 1 ? w[(j >> 1) & 3] >> 16 : w[(j >> 1) & 3] & 0xFFFFu);
+          vals[d + j] = f;
+          sq += f * f;
+        }
+      } else {
+        vals[d] = ro_load(src + d);
+        sq += vals[d] * vals[d];
+      }
+    }
+    const float inv = gain ? 1.0f / sqrtf(warp_sum(sq) / (float)dim + r.eps) : 1.0f;
+    __syncwarp();
+    auto normed = [&](int d) { return gain ? vals[d] * inv * ro_load(gain + d) : vals[d]; };
+    for (int d0 = lane * V; d0 < dim; d0 += 32 * V) {
+      float f[V];
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        const int d = d0 + j, i = d - r.rot.first;
+        f[j] = normed(d);
+        if (i >= 0 && i < 2 * half) {
+          const bool lead = r.rot.interleaved ? !(i & 1) : i < half;
+          const int shift = r.rot.interleaved ? 1 : half, p = r.rot.interleaved ? i >> 1 : lead ? i : i - half;
+          const float other = normed(lead ? d + shift : d - shift);
+          f[j] = f[j] * cs[p] + (lead ? -other : other) * cs[half + p];
+        }
+      }
+      if constexpr (VEC) {
+#pragma unroll
+        for (int j = 0; j < V; j += 4) ro_store4(dst + d0 + j, make_float4(f[j], f[j + 1], f[j + 2], f[j + 3]));
+      } else {
+        ro_store(dst + d0, f[0]);
+      }
+    }
+    __syncwarp();
+  }
+}
+
+int launch_head_norm_rope(tq_ctx* ctx, const HeadNormRope& a0, const RaggedBatch& b, int dtype) {
+  HeadNormRope a = a0;
+  if (!a.q_head) a.q_head = (size_t)a.r.dim;
+  const QkNormRope& r = a.r;
+  TQ_REQUIRE(ctx, r.heads >= 0 && r.kv_heads >= 0 && r.heads + r.kv_heads > 0 && r.dim > 0 && r.rot.first >= 0 && r.rot.dims >= 0 && r.rot.dims % 2 == 0 &&
+                      r.rot.first + r.rot.dims <= r.dim,
+             "head norm: the rotated dimensions must be even and inside the head");
+  if (b.rows == 0) return TQ_OK;
+  const int total = r.heads + r.kv_heads;
+  int warps = total < 8 ? total : 8;
+  const size_t smem = ((size_t)r.rot.dims + 3 + (size_t)warps * ((r.dim + 3) / 4 * 4)) * sizeof(float);
+  TQ_REQUIRE(ctx, smem <= 200 * 1024, "head norm: heads of %d values are too large", r.dim);
+  int parts = 1;
+  while (parts * warps < total && (long long)b.rows * parts < 2ll * ctx->sm_count) ++parts;
+  auto go = [&](auto kern) -> int {
+    if (smem > 48 * 1024) TQ_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)b.rows, (unsigned)parts), dim3((unsigned)(32 * warps)), smem, a, b.row_pos, b.cache_row, b.cache_rows));
+    return TQ_OK;
+  };
+  const int v = dtype == TQ_F32 ? 4 : 8;
+  const uintptr_t bits = (uintptr_t)r.q | (uintptr_t)r.raw | (uintptr_t)r.keys;
+  const bool vec = r.dim % v == 0 && r.ldq % v == 0 && a.q_head % v == 0 && r.raw_pad % v == 0 && r.key_pad % v == 0 && (bits & 15) == 0;
+  if (dtype == TQ_F32) return vec ? go(head_norm_rope_kernel<float, true>) : go(head_norm_rope_kernel<float, false>);
+  return vec ? go(head_norm_rope_kernel<__nv_bfloat16, true>) : go(head_norm_rope_kernel<__nv_bfloat16, false>);
+}
+
+// ------------------------------------------------------------------------------------------------ row norm and gate
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kRoThreads) norm_gate_kernel(const float* o, size_t ld_o, const float* norm, const T* gate, size_t ldg, T* out, size_t ldo,
+                                                               const int* cache_row, int width, float eps) {
+  __shared__ float red[kRoWarps];
+  constexpr int V = VEC ? 4 : 1;
+  pdl_wait();
+  pdl_launch_dependents();
+  const size_t m = blockIdx.x;
+  if (cache_row && cache_row[m] < 0) return;
+  o += m * ld_o;
+  gate += m * ldg;
+  out += m * ldo;
+  float sq = 0.f;
+#pragma unroll 4
+  for (int d = V * threadIdx.x; d < width; d += V * kRoThreads) {
+    if constexpr (VEC) {
+      const float4 v = *reinterpret_cast<const float4*>(o + d);
+      sq += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    } else {
+      sq += o[d] * o[d];
+    }
+  }
+  const float inv = 1.0f / sqrtf(ro_block_sum(sq, red) / (float)width + eps);
+  auto open = [](float z) { return 1.0f / (1.0f + expf(-z)); };
+#pragma unroll 4
+  for (int d = V * threadIdx.x; d < width; d += V * kRoThreads) {
+    if constexpr (VEC) {
+      const float4 v = *reinterpret_cast<const float4*>(o + d), w = *reinterpret_cast<const float4*>(norm + d);
+      ro_store4(out + d, make_float4(v.x * inv * w.x * open(ro_load(gate + d)), v.y * inv * w.y * open(ro_load(gate + d + 1)),
+                                     v.z * inv * w.z * open(ro_load(gate + d + 2)), v.w * inv * w.w * open(ro_load(gate + d + 3))));
+    } else {
+      ro_store(out + d, o[d] * inv * norm[d] * open(ro_load(gate + d)));
+    }
+  }
+}
+
+int launch_norm_gate(tq_ctx* ctx, const float* o, size_t ld_o, const float* norm, const void* gate, size_t ldg, void* out, size_t ldo, const int* cache_row,
+                     size_t rows, size_t width, float eps, int dtype) {
+  if (rows == 0) return TQ_OK;
+  const bool vec = width % 4 == 0 && ld_o % 4 == 0 && ldo % 4 == 0 && (((uintptr_t)o | (uintptr_t)norm | (uintptr_t)out) & 15) == 0;
+  auto go = [&](auto kern, auto* tag) -> int {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)rows), dim3(kRoThreads), 0, o, ld_o, norm, static_cast<const T*>(gate), ldg, static_cast<T*>(out), ldo,
+                          cache_row, (int)width, eps));
+    return TQ_OK;
+  };
+  if (dtype == TQ_F32) return vec ? go(norm_gate_kernel<float, true>, (float*)nullptr) : go(norm_gate_kernel<float, false>, (float*)nullptr);
+  return vec ? go(norm_gate_kernel<__nv_bfloat16, true>, (__nv_bfloat16*)nullptr) : go(norm_gate_kernel<__nv_bfloat16, false>, (__nv_bfloat16*)nullptr);
+}
+
+void banded_frequencies(int dims, double base, double factor, double low, double high, double original, float* freq) {
+  const double pi = 3.14159265358979323846;
+  for (int i = 0; i < dims / 2; ++i) {
+    const double f = std::pow(base, -2.0 * i / dims), wave = 2 * pi / f;
+    double g = f;
+    if (factor > 0) {
+      if (wave > original / low) {
+        g = f / factor;
+      } else if (wave >= original / high) {
+        const double s = (original / wave - low) / (high - low);
+        g = (1 - s) * f / factor + s * f;
+      }
+    }
+    freq[i] = (float)g;
+  }
+}
+
 void yarn_frequencies(int dims, double base, double factor, double original, double fast, double slow, float* freq, float* mult) {
   const double pi = 3.14159265358979323846;
   *mult = factor > 0 ? (float)(0.1 * std::log(factor) + 1.0) : 1.0f;
@@ -330,6 +498,13 @@ int tq_yarn_frequencies(size_t dims, double base, double factor, double original
   if (!freq_host || !mult_host || dims % 2 || dims == 0 || !(base > 1.0)) return TQ_EINVAL;
   if (factor > 0 && !(original > 0 && fast > 0 && slow > 0)) return TQ_EINVAL;
   yarn_frequencies((int)dims, base, factor, original, fast, slow, freq_host, mult_host);
+  return TQ_OK;
+}
+
+int tq_banded_frequencies(size_t dims, double base, double factor, double low, double high, double original, float* freq_host) {
+  if (!freq_host || dims % 2 || dims == 0 || !(base > 1.0)) return TQ_EINVAL;
+  if (factor > 0 && !(original > 0 && low > 0 && high > low)) return TQ_EINVAL;
+  banded_frequencies((int)dims, base, factor, low, high, original, freq_host);
   return TQ_OK;
 }
 
@@ -380,6 +555,39 @@ int tq_qk_norm_rope(tq_ctx* ctx, int dtype, size_t heads, size_t kv_heads, size_
   b.cache_row = cache_row_dev;
   b.cache_rows = cache_rows;
   return launch_qk_norm_rope(ctx, a, b, dtype);
+}
+
+int tq_head_norm_rope(tq_ctx* ctx, int dtype, size_t heads, size_t kv_heads, size_t dim, void* q_dev, size_t ldq, size_t q_head, const void* raw_dev,
+                      void* keys_dev, size_t cache_rows, const void* q_gain_dev, const void* k_gain_dev, size_t rot_first, size_t rot_dims, int interleaved,
+                      const float* freq_dev, float rot_mult, float eps, const int* row_pos_dev, const int* cache_row_dev, size_t rows) {
+  if (int st = bind(ctx)) return st;
+  TQ_REQUIRE(ctx, dtype == TQ_F32 || dtype == TQ_BF16, "tq_head_norm_rope: dtype must be f32 or bf16");
+  TQ_REQUIRE(ctx, (q_dev || !heads) && ((raw_dev && keys_dev) || !kv_heads) && (freq_dev || rot_dims == 0) && row_pos_dev && cache_row_dev,
+             "tq_head_norm_rope: null pointer");
+  HeadNormRope a;
+  a.q_head = q_head;
+  a.r.heads = (int)heads;
+  a.r.kv_heads = (int)kv_heads;
+  a.r.dim = (int)dim;
+  a.r.raw_pad = a.r.key_pad = (int)((dim + 7) / 8 * 8);
+  a.r.q = q_dev;
+  a.r.ldq = ldq;
+  a.r.raw = raw_dev;
+  a.r.keys = keys_dev;
+  a.r.q_gain = q_gain_dev;
+  a.r.k_gain = k_gain_dev;
+  a.r.rot.first = (int)rot_first;
+  a.r.rot.dims = (int)rot_dims;
+  a.r.rot.interleaved = interleaved != 0;
+  a.r.rot.freq = freq_dev;
+  a.r.rot.mult = rot_mult;
+  a.r.eps = eps;
+  RaggedBatch b;
+  b.rows = (int)rows;
+  b.row_pos = row_pos_dev;
+  b.cache_row = cache_row_dev;
+  b.cache_rows = cache_rows;
+  return launch_head_norm_rope(ctx, a, b, dtype);
 }
 
 }  // extern "C"

@@ -1,0 +1,226 @@
+// Hyper-connections (StreamMix in rowops.cuh): one pass over a row's streams takes a sublayer's output in -- summing the rows of
+// its chosen experts on the way --, mixes the streams, forms the next sublayer's input from them and norms it.
+#include <cuda_bf16.h>
+
+#include <type_traits>
+
+#include "common.cuh"
+#include "rowops.cuh"
+
+namespace tq {
+
+constexpr int kSmMaxRows = 64;       // rows of y per row of the batch
+
+template <int V>
+struct SmVec {
+  float v[V];
+};
+template <int V>
+__device__ __forceinline__ SmVec<V> sm_load(const float* p) {
+  SmVec<V> r;
+  if constexpr (V == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    r.v[0] = f.x, r.v[1] = f.y, r.v[2] = f.z, r.v[3] = f.w;
+  } else {
+    r.v[0] = *p;
+  }
+  return r;
+}
+template <int V>
+__device__ __forceinline__ SmVec<V> sm_load(const __nv_bfloat16* p) {
+  SmVec<V> r;
+  if constexpr (V == 4) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    r.v[0] = bf16_bits_to_float(u.x & 0xFFFFu), r.v[1] = bf16_bits_to_float(u.x >> 16);
+    r.v[2] = bf16_bits_to_float(u.y & 0xFFFFu), r.v[3] = bf16_bits_to_float(u.y >> 16);
+  } else {
+    r.v[0] = __bfloat162float(*p);
+  }
+  return r;
+}
+template <int V>
+__device__ __forceinline__ void sm_store(float* p, const SmVec<V>& r) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+  else *p = r.v[0];
+}
+template <int V>
+__device__ __forceinline__ void sm_store(__nv_bfloat16* p, const SmVec<V>& r) {
+  if constexpr (V == 4) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(r.v[0], r.v[1]), b = __floats2bfloat162_rn(r.v[2], r.v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+  } else {
+    *p = __float2bfloat16_rn(r.v[0]);
+  }
+}
+
+// One CTA per row; a thread owns V columns at a time in every stream, so that the streams and `self` may be overwritten in place.
+// S: streams, or (above 4) the most of them.
+template <typename OT, int S, int V>
+__global__ void __launch_bounds__(512) stream_mix_kernel(StreamMix a, int width) {
+  extern __shared__ __align__(16) float sm_u[];           // [width] the next input before its norm
+  __shared__ float mix[S * S], w_out[S], w_in[S], red[32], yw[kSmMaxRows];
+  __shared__ int yr[kSmMaxRows];
+  const int n = S > 4 ? a.streams : S;
+  // (weights: before the wait)
+  if (a.y && (int)threadIdx.x < n * n) mix[threadIdx.x] = a.mix[threadIdx.x];
+  if ((int)threadIdx.x < n) {
+    if (a.y) w_out[threadIdx.x] = a.w_out[threadIdx.x];
+    w_in[threadIdx.x] = a.w_in ? a.w_in[threadIdx.x] : 1.f;
+  }
+  pdl_wait();
+  pdl_launch_dependents();
+  const size_t m = blockIdx.x, row = a.src_rows ? (size_t)a.src_rows[m] : m;
+  if (a.y && (int)threadIdx.x < a.n_y) {
+    yr[threadIdx.x] = a.y_rows ? a.y_rows[m * a.n_y + threadIdx.x] : (int)m;
+    yw[threadIdx.x] = a.y_weight ? a.y_weight[m * a.n_y + threadIdx.x] : 1.f;
+  }
+  __syncthreads();
+  const float* src = a.src + row * a.src_streams * width;
+  const size_t src_ld = a.src_streams == 1 ? 0 : width;
+  float* dst = a.dst + m * n * width;
+  OT* out = static_cast<OT*>(a.out) + m * a.ld_out;
+  const OT* self = static_cast<const OT*>(a.self) + m * a.ld_out;
+  float sq = 0.f;
+#pragma unroll(S > 4 ? 1 : 2)
+  for (int d = V * threadIdx.x; d < width; d += V * blockDim.x) {
+    SmVec<V> x[S], u, total;
+#pragma unroll
+    for (int s = 0; s < S; ++s)
+      if (s < n) x[s] = sm_load<V>(src + s * src_ld + d);
+    if (a.y) {
+      SmVec<V> y;
+#pragma unroll
+      for (int j = 0; j < V; ++j) y.v[j] = 0.f;
+      for (int k = 0; k < a.n_y; ++k) {
+        const int r = yr[k];
+        const float w = yw[k];
+        SmVec<V> part;
+        if (r >= 0) part = sm_load<V>(a.y + (size_t)r * width + d);
+        else if (a.self) part = sm_load<V>(self + d);
+        else continue;
+#pragma unroll
+        for (int j = 0; j < V; ++j) y.v[j] = fmaf(w, part.v[j], y.v[j]);
+      }
+      if (a.y_more) {
+        const SmVec<V> part = sm_load<V>(a.y_more + m * width + d);
+#pragma unroll
+        for (int j = 0; j < V; ++j) y.v[j] += part.v[j];
+      }
+      SmVec<V> old[S];
+#pragma unroll
+      for (int s = 0; s < S; ++s)
+        if (s < n) old[s] = x[s];
+#pragma unroll
+      for (int t = 0; t < S; ++t) {
+        if (t >= n) continue;
+#pragma unroll
+        for (int j = 0; j < V; ++j) x[t].v[j] = w_out[t] * y.v[j];
+#pragma unroll
+        for (int s = 0; s < S; ++s)
+          if (s < n) {
+#pragma unroll
+            for (int j = 0; j < V; ++j) x[t].v[j] = fmaf(mix[s * n + t], old[s].v[j], x[t].v[j]);
+          }
+        sm_store<V>(dst + (size_t)t * width + d, x[t]);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) u.v[j] = total.v[j] = 0.f;
+#pragma unroll
+    for (int s = 0; s < S; ++s)
+      if (s < n) {
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+          u.v[j] = fmaf(w_in[s], x[s].v[j], u.v[j]);
+          total.v[j] += x[s].v[j];
+        }
+      }
+    if (a.sum) sm_store<V>(a.sum + m * width + d, total);
+    if (a.gain) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) sq += u.v[j] * u.v[j];
+      sm_store<V>(sm_u + d, u);
+    }
+  }
+  if (!a.gain) return;
+  sq = warp_sum(sq);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = sq;
+  __syncthreads();
+  sq = warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? red[threadIdx.x & 31] : 0.f);
+  const float inv = 1.0f / sqrtf(sq / (float)width + a.eps);
+  for (int d = V * threadIdx.x; d < width; d += V * blockDim.x) {
+    const SmVec<V> g = sm_load<V>(a.gain + d);
+    SmVec<V> u = sm_load<V>(sm_u + d);
+#pragma unroll
+    for (int j = 0; j < V; ++j) u.v[j] *= inv * g.v[j];
+    sm_store<V>(out + d, u);
+  }
+}
+
+template <typename OT>
+static int stream_mix_typed(tq_ctx* ctx, const StreamMix& a, size_t rows, size_t width) {
+  const uintptr_t bits = (uintptr_t)a.src | (uintptr_t)a.dst | (uintptr_t)a.y | (uintptr_t)a.y_more | (uintptr_t)a.gain | (uintptr_t)a.out | (uintptr_t)a.self |
+                         (uintptr_t)a.sum;
+  const bool vec = a.streams <= 4 && width % 4 == 0 && a.ld_out % 4 == 0 && (bits & 15) == 0;
+  const size_t smem = a.gain ? width * sizeof(float) : 0;
+  size_t threads = vec ? width / 4 : width;
+  const size_t most = rows >= 2 * (size_t)ctx->sm_count ? 256 : 512, least = a.streams > 4 ? 256 : 64;
+  threads = threads > most ? most : threads < least ? least : (threads + 31) / 32 * 32;
+  auto go = [&](auto s) -> int {
+    constexpr int S = decltype(s)::value;
+    auto kern = vec ? stream_mix_kernel<OT, S, S <= 4 ? 4 : 1> : stream_mix_kernel<OT, S, 1>;
+    if (smem > 40 * 1024) TQ_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)rows), dim3((unsigned)threads), smem, a, (int)width));
+    return TQ_OK;
+  };
+  switch (a.streams) {
+    case 1: return go(std::integral_constant<int, 1>());
+    case 2: return go(std::integral_constant<int, 2>());
+    case 3: return go(std::integral_constant<int, 3>());
+    case 4: return go(std::integral_constant<int, 4>());
+    default: return go(std::integral_constant<int, kMaxStreams>());
+  }
+}
+
+int launch_stream_mix(tq_ctx* ctx, const StreamMix& a, size_t rows, size_t width) {
+  TQ_REQUIRE(ctx, a.streams >= 1 && a.streams <= kMaxStreams && (a.src_streams == 1 || a.src_streams == a.streams), "stream mix: 1 to %d streams", kMaxStreams);
+  TQ_REQUIRE(ctx, width > 0 && width <= 49152, "stream mix: rows of 1 to 49152 values");
+  TQ_REQUIRE(ctx, !a.y || (a.dst && a.mix && a.w_out && a.n_y >= 1 && a.n_y <= kSmMaxRows && !a.src_rows && (a.y_rows || a.n_y == 1)),
+             "stream mix: bad sublayer output (at most %d rows each)", kSmMaxRows);
+  TQ_REQUIRE(ctx, !a.gain || a.out, "stream mix: nowhere to put the norm");
+  if (rows == 0) return TQ_OK;
+  return a.out_dtype == TQ_F32 ? stream_mix_typed<float>(ctx, a, rows, width) : stream_mix_typed<__nv_bfloat16>(ctx, a, rows, width);
+}
+
+}  // namespace tq
+
+using namespace tq;
+
+extern "C" int tq_stream_mix(tq_ctx* ctx, size_t streams, size_t src_streams, const float* src_dev, float* dst_dev, const float* y_dev, const int* y_rows_dev,
+                             const float* y_weight_dev, size_t n_y, const void* self_dev, const float* y_more_dev, const float* mix_dev,
+                             const float* w_out_dev, const float* w_in_dev, const float* gain_dev, size_t rows, size_t width, float eps, void* out_dev,
+                             int out_dtype, size_t ld_out, float* sum_dev) {
+  if (int st = bind(ctx)) return st;
+  TQ_REQUIRE(ctx, src_dev && (out_dtype == TQ_F32 || out_dtype == TQ_BF16), "tq_stream_mix: no streams, or out is neither f32 nor bf16");
+  StreamMix a;
+  a.streams = (int)streams;
+  a.src_streams = (int)src_streams;
+  a.src = src_dev;
+  a.dst = dst_dev;
+  a.y = y_dev;
+  a.y_rows = y_rows_dev;
+  a.y_weight = y_weight_dev;
+  a.n_y = y_rows_dev ? (int)n_y : 1;
+  a.self = self_dev;
+  a.y_more = y_more_dev;
+  a.mix = mix_dev;
+  a.w_out = w_out_dev;
+  a.w_in = w_in_dev;
+  a.gain = gain_dev;
+  a.out = out_dev;
+  a.out_dtype = out_dtype;
+  a.ld_out = ld_out ? ld_out : width;
+  a.eps = eps;
+  a.sum = sum_dev;
+  return launch_stream_mix(ctx, a, rows, width);
+}

@@ -143,9 +143,9 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
   auto q_src = [&](int r) -> const __nv_bfloat16* {
     const int qi = SPLIT ? 0 : r / p.gb, hh = SPLIT ? r : r % p.gb;
     if (i0 + qi > i1 || (!SPLIT && r >= pos_per_cta * p.gb) || hh >= gb) return nullptr;
-    return p.q + (size_t)(row0 + i0 + qi) * p.ldq + (size_t)(head0 + hh) * p.a.dim;
+    return p.q + (size_t)(row0 + i0 + qi) * p.ldq + (size_t)(head0 + hh) * p.a.q_head;
   };
-  if ((p.a.dim & 7) == 0 && (p.ldq & 7) == 0) {
+  if ((p.a.dim & 7) == 0 && (p.ldq & 7) == 0 && (p.a.q_head & 7) == 0) {
     const int pm = p.a.dim / 8;
     for (int i = threadIdx.x; i < q_rows * pm; i += kThreads) {
       const int r = i / pm, c = i - r * pm;
@@ -180,11 +180,15 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
   float o[DVT][4];                                         // [columns 8j + 2t, +1] of pair g, then of pair g + 8
 #pragma unroll
   for (int j = 0; j < DVT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-  const float sink2 = p.a.sink * kLog2e;
   // one lane of a row (one warp and split of a pair) carries the sink's term
-  const bool owns_sink = t == 0 && p.a.sink > -FLT_MAX && (!SPLIT || (warp == 0 && blockIdx.x == 0));
-  float m_run[2] = {sink2, sink2}, l_run[2];
-  l_run[0] = l_run[1] = owns_sink ? 1.f : 0.f;
+  const bool owns_sink = t == 0 && (!SPLIT || (warp == 0 && blockIdx.x == 0));
+  float m_run[2], l_run[2];
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const float sink = p.a.sinks ? (live[h] ? p.a.sinks[qhead[h]] : 0.f) : p.a.sink;
+    m_run[h] = sink * kLog2e;
+    l_run[h] = owns_sink && sink > -FLT_MAX ? 1.f : 0.f;
+  }
   const CapScore cap(p.a);
   const int nks = p.dp / 16;
 
@@ -443,7 +447,7 @@ __global__ void __launch_bounds__(128) window_attention_simt_kernel(const T* q, 
   const size_t ke = (size_t)a.kv_heads * a.dim_pad, ve = (size_t)a.kv_heads * a.vdim_pad;
   const T* kb = k + seq0 * ke + (size_t)kvh * a.dim_pad;
   const T* vb = v + seq0 * ve + (size_t)kvh * a.vdim_pad;
-  for (int i = tid; i < a.dim; i += 128) qs[i] = wa_load(q + (size_t)row * ldq + (size_t)head * a.dim + i);
+  for (int i = tid; i < a.dim; i += 128) qs[i] = wa_load(q + (size_t)row * ldq + (size_t)head * a.q_head + i);
   for (int i = tid; i < a.vdim; i += 128) acc[i] = 0.f;
   __syncthreads();
   auto block_reduce = [&](float x, bool is_max) {
@@ -455,8 +459,9 @@ __global__ void __launch_bounds__(128) window_attention_simt_kernel(const T* q, 
     return r;
   };
   const int lo = max(0, pos - a.window + 1), n_vis = pos - lo + 1;
-  const bool has_sink = a.sink > -FLT_MAX;
-  float m_run = has_sink ? a.sink : -FLT_MAX, l_run = has_sink ? 1.f : 0.f;
+  const float sink = a.sinks ? a.sinks[head] : a.sink;
+  const bool has_sink = sink > -FLT_MAX;
+  float m_run = has_sink ? sink : -FLT_MAX, l_run = has_sink ? 1.f : 0.f;
   for (int c0 = 0; c0 < n_vis; c0 += 128) {
     const int c = c0 + tid, n = min(128, n_vis - c0);
     float sc = -FLT_MAX;
@@ -511,8 +516,10 @@ static int launch_mma(tq_ctx* ctx, WinParams& p, bool split, size_t smem, dim3 g
   return split ? go(window_attention_kernel<DVT, true>, 128) : go(window_attention_kernel<DVT, false>, 256);
 }
 
-int launch_window_attention(tq_ctx* ctx, const WindowAttn& a, const RaggedBatch& b, int dtype, const void* q, size_t ldq, const void* gate,
+int launch_window_attention(tq_ctx* ctx, const WindowAttn& attn, const RaggedBatch& b, int dtype, const void* q, size_t ldq, const void* gate,
                             size_t ldg, const void* k_cache, const void* v_cache, void* out, size_t ldo) {
+  WindowAttn a = attn;
+  if (!a.q_head) a.q_head = (size_t)a.dim;
   TQ_REQUIRE(ctx, a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0, "window attention: heads must be a multiple of kv_heads");
   TQ_REQUIRE(ctx, a.dim > 0 && a.vdim > 0 && a.dim_pad >= a.dim && a.vdim_pad >= a.vdim && a.dim_pad % 8 == 0 && a.vdim_pad % 8 == 0,
              "window attention: bad head sizes");
@@ -607,6 +614,14 @@ extern "C" int tq_window_attention(tq_ctx* ctx, const tq_window_attn_config* cfg
                                    size_t ldg, const void* k_cache_dev, const void* v_cache_dev, size_t cache_rows, const int* seq_rows_dev,
                                    const int* row_pos_dev, const int* cache_row_dev, size_t n_seqs, size_t rows, size_t max_q, size_t max_len,
                                    void* out_dev, size_t ldo) {
+  return tq_window_attention_sinks(ctx, cfg, nullptr, dtype, q_dev, ldq, gate_dev, ldg, k_cache_dev, v_cache_dev, cache_rows, seq_rows_dev, row_pos_dev,
+                                   cache_row_dev, n_seqs, rows, max_q, max_len, out_dev, ldo);
+}
+
+extern "C" int tq_window_attention_sinks(tq_ctx* ctx, const tq_window_attn_config* cfg, const float* sinks_dev, int dtype, const void* q_dev, size_t ldq,
+                                         const void* gate_dev, size_t ldg, const void* k_cache_dev, const void* v_cache_dev, size_t cache_rows,
+                                         const int* seq_rows_dev, const int* row_pos_dev, const int* cache_row_dev, size_t n_seqs, size_t rows,
+                                         size_t max_q, size_t max_len, void* out_dev, size_t ldo) {
   if (int st = bind(ctx)) return st;
   TQ_REQUIRE(ctx, cfg && (dtype == TQ_BF16 || dtype == TQ_F32), "tq_window_attention: dtype must be bf16 or f32");
   if (rows == 0) return TQ_OK;
@@ -623,6 +638,7 @@ extern "C" int tq_window_attention(tq_ctx* ctx, const tq_window_attn_config* cfg
   a.scale = cfg->scale;
   a.softcap = cfg->softcap;
   a.sink = cfg->sink;
+  a.sinks = sinks_dev;
   RaggedBatch b;
   b.n_seqs = (int)n_seqs;
   b.rows = (int)rows;

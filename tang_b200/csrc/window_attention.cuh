@@ -1,6 +1,6 @@
 // Grouped-query attention under a sliding window, with capped scores, a sink and an output gate:
 //     s = (q . k) * scale;  s <- softcap * tanh(s / softcap)          (softcap 0: no cap)
-//     p_j = exp(s_j) / (exp(sink) + sum exp(s))                       (sink -infinity: none; it has no value)
+//     p_j = exp(s_j) / (exp(sink) + sum exp(s))                       (one sink, or one per head; -infinity: none; it has no value)
 //     out = (sum p_j v_j) * sigmoid(gate)                             (no gate pointer: 1)
 // Mask: the query at position i sees key j when j <= i and i - j < window.
 #pragma once
@@ -15,9 +15,11 @@ struct WindowAttn {
   int heads = 0, kv_heads = 0, dim = 0, vdim = 0, dim_pad = 0, vdim_pad = 0;
   int window = 0;
   float scale = 0.f, softcap = 0.f, sink = 0.f;
+  const float* sinks = nullptr;        // [heads], instead of `sink`
+  size_t q_head = 0;                   // elements between the heads of a query row; 0: dim
 };
 
-// q [rows][ldq], head h at column h * dim; gate [rows][ldg] and out [rows][ldo], head h at column h * vdim.  dtype (TQ_BF16 or
+// q [rows][ldq], head h at column h * dim (q_head); gate [rows][ldg] and out [rows][ldo], head h at column h * vdim.  dtype (TQ_BF16 or
 // TQ_F32) is that of q, gate, caches and out; scores, weights and sums are f32, in TQ_F32 every operation is.
 int launch_window_attention(tq_ctx* ctx, const WindowAttn& a, const RaggedBatch& b, int dtype, const void* q, size_t ldq, const void* gate,
                             size_t ldg, const void* k_cache, const void* v_cache, void* out, size_t ldo);
