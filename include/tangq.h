@@ -598,6 +598,12 @@ TQ_API int tq_gla(tq_ctx* ctx, const tq_gla_config* cfg, int dtype, const void* 
                   size_t ld, const float* a1_dev, size_t ld_a1, const float* a2_dev, const float* a2_bias_dev, const float* norm_dev,
                   float* state_dev, size_t max_seq, size_t cache_rows, const int* seq_rows_dev_or_null, const int* row_pos_dev,
                   const int* cache_row_dev, size_t n_seqs, size_t rows, size_t max_q, void* out_dev, size_t ldo);
+/* Lightning attention: S_t = decay_h S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head; out = o / sqrt(mean(o^2) + eps) * norm *
+ * sigmoid(gate) over the heads' values side by side (norm [heads * vdim] f32).  Rows and states as in tq_gla. */
+TQ_API int tq_lightning(tq_ctx* ctx, int dtype, size_t heads, size_t dim, size_t vdim, float eps, const float* decay_dev, const void* q_dev,
+                        const void* k_dev, const void* v_dev, const void* gate_dev, size_t ld, const float* norm_dev, float* state_dev, size_t max_seq,
+                        size_t cache_rows, const int* seq_rows_dev_or_null, const int* row_pos_dev, const int* cache_row_dev, size_t n_seqs,
+                        size_t rows, size_t max_q, void* out_dev, size_t ldo);
 /* The `top` experts with the largest logits [rows][experts] per row (the lower index among equals) with weights sigmoid(z)
  * (score 0) or softmax (score 1), divided by their sum if renorm.  Pair p = row * top + i gets a slot; the slots of an expert are
  * consecutive.  jobs int[.][4]: (expert, first slot, slots <= chunk, 0), at most min(pairs, experts + pairs / chunk). */

@@ -4,6 +4,7 @@
 //     registers once and exchanges the sums of squares of the head norm through distributed shared memory;
 //   * gla_scan_kernel + gla_out_kernel: any number of rows, token by token, the state in shared memory: the exact f32 form;
 //   * prompts in bf16: csrc/gla_chunk.cu.
+// Lightning attention runs through the first two, which then leave f32 outputs for launch_norm_gate; prompts: csrc/lightning.cu.
 #include "gla.cuh"
 
 #include <cooperative_groups.h>
@@ -11,6 +12,7 @@
 
 #include "common.cuh"
 #include "gla_device.cuh"
+#include "rowops.cuh"
 
 namespace tq {
 
@@ -22,7 +24,7 @@ constexpr int kGdWarps = kGdThreads / 32;
 
 // blockIdx.x: head * splits + part (a cluster is one head's parts); part owns vdim / splits columns.
 template <typename T>
-__global__ void __launch_bounds__(kGdThreads) gla_decode_kernel(Gla g, GlaRows r, RaggedBatch b, int splits) {
+__global__ void __launch_bounds__(kGdThreads) gla_decode_kernel(Gla g, GlaRows r, RaggedBatch b, int splits, float* o_out) {
   extern __shared__ float gd_smem[];
   __shared__ float sums[2];
   const int cw = g.vdim / splits;
@@ -43,7 +45,7 @@ __global__ void __launch_bounds__(kGdThreads) gla_decode_kernel(Gla g, GlaRows r
     base_v = static_cast<const T*>(r.v) + row * r.ld + (size_t)head * g.vdim + c0;
     for (int d = threadIdx.x; d < g.dim; d += kGdThreads) {
       const int ch = head * g.dim + d;
-      alpha[d] = s.fresh ? 0.f : expf(gl_log_decay(gl_decay_logit(g, ch, r.a1 + row * r.ld_a1), 1.0f / g.tau));
+      alpha[d] = s.fresh ? 0.f : gl_decay(g, head, ch, r.a1 + row * r.ld_a1);
       ks[d] = gl_load(static_cast<const T*>(r.k) + row * r.ld + ch);
       qs[d] = gl_load(static_cast<const T*>(r.q) + row * r.ld + ch) * g.q_scale;
     }
@@ -84,9 +86,14 @@ __global__ void __launch_bounds__(kGdThreads) gla_decode_kernel(Gla g, GlaRows r
       float o = 0.f;
 #pragma unroll
       for (int w = 0; w < kGdWarps; ++w) o += part[w * cw + c];
+      if (g.head_decay) {
+        o_out[((size_t)s.row0 * g.heads + head) * g.vdim + c0 + c] = o;
+        continue;
+      }
       part[c] = o;              // (column c is read and written by this thread alone)
       sq += o * o;
     }
+    if (g.head_decay) return;   // (no clusters then)
     sq = warp_sum(sq);
     if (lane == 0) red[warp] = sq;
     __syncthreads();
@@ -141,7 +148,7 @@ __global__ void __launch_bounds__(kGsThreads) gla_scan_kernel(Gla g, GlaRows r, 
     for (int i = threadIdx.x; i < n * g.dim; i += kGsThreads) {
       const int t = i / g.dim, d = i - t * g.dim, ch = head * g.dim + d;
       const size_t row = s.row0 + t0 + t;
-      al[i] = expf(gl_log_decay(gl_decay_logit(g, ch, r.a1 + row * r.ld_a1), 1.0f / g.tau));
+      al[i] = gl_decay(g, head, ch, r.a1 + row * r.ld_a1);
       ks[i] = gl_load(static_cast<const T*>(r.k) + row * r.ld + ch);
       qs[i] = gl_load(static_cast<const T*>(r.q) + row * r.ld + ch) * g.q_scale;
     }
@@ -189,7 +196,7 @@ __global__ void __launch_bounds__(256) gla_out_kernel(Gla g, GlaRows r, const in
 
 // ------------------------------------------------------------------------------------------------ launch
 template <typename T>
-static int launch_decode(tq_ctx* ctx, const Gla& g, const GlaRows& r, const RaggedBatch& b) {
+static int launch_decode(tq_ctx* ctx, const Gla& g, const GlaRows& r, const RaggedBatch& b, float* o) {
   // columns over a cluster until about two CTAs per SM are busy, at least 32 columns each
   int splits = 1;
   while (splits < 8 && g.vdim % (64 * splits) == 0 && (long long)b.n_seqs * g.heads * splits < 2ll * ctx->sm_count) splits *= 2;
@@ -197,32 +204,50 @@ static int launch_decode(tq_ctx* ctx, const Gla& g, const GlaRows& r, const Ragg
   TQ_REQUIRE(ctx, smem <= 200 * 1024, "gated linear attention: head sizes %d / %d are too large", g.dim, g.vdim);
   auto kern = gla_decode_kernel<T>;
   if (smem > 48 * 1024) TQ_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  TQ_CUDA(ctx, launch_k_cluster(ctx, kern, dim3((unsigned)(g.heads * splits), (unsigned)b.n_seqs), dim3(kGdThreads), smem, splits, g, r, b, splits));
+  const dim3 grid((unsigned)(g.heads * splits), (unsigned)b.n_seqs);
+  if (g.head_decay) TQ_CUDA(ctx, launch_k(ctx, kern, grid, dim3(kGdThreads), smem, g, r, b, splits, o));
+  else TQ_CUDA(ctx, launch_k_cluster(ctx, kern, grid, dim3(kGdThreads), smem, splits, g, r, b, splits, o));
   return TQ_OK;
 }
 
 template <typename T>
-static int launch_scan(tq_ctx* ctx, const Gla& g, const GlaRows& r, const RaggedBatch& b) {
-  if (int st = ensure_scratch(ctx, (size_t)b.rows * g.heads * g.vdim * sizeof(float))) return st;
-  float* o = static_cast<float*>(ctx->scratch);
+static int launch_scan(tq_ctx* ctx, const Gla& g, const GlaRows& r, const RaggedBatch& b, float* o) {
   const size_t smem = ((size_t)g.dim * kGsCols + (size_t)3 * kGsRows * g.dim + kGsWarps * kGsRows * kGsCols) * sizeof(float);
   TQ_REQUIRE(ctx, smem <= 226 * 1024, "gated linear attention: key size %d is too large", g.dim);
   auto kern = gla_scan_kernel<T>;
   if (smem > 48 * 1024) TQ_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)b.n_seqs, (unsigned)g.heads, (unsigned)((g.vdim + kGsCols - 1) / kGsCols)), dim3(kGsThreads), smem, g,
                         r, b, o));
+  if (g.head_decay) return TQ_OK;
   TQ_CUDA(ctx, launch_k(ctx, gla_out_kernel<T>, dim3((unsigned)(((long long)b.rows * g.heads + 7) / 8)), dim3(256), 0, g, r, b.cache_row, b.rows,
                         (const float*)o));
   return TQ_OK;
 }
 
 int launch_gla(tq_ctx* ctx, const Gla& g, const GlaRows& r, const RaggedBatch& b, int dtype) {
-  TQ_REQUIRE(ctx, g.heads > 0 && g.dim > 0 && g.vdim > 0 && g.rank > 0 && g.tau > 0.f && g.max_seq > 0, "gated linear attention: bad sizes");
+  TQ_REQUIRE(ctx, g.heads > 0 && g.dim > 0 && g.vdim > 0 && (g.head_decay || (g.rank > 0 && g.tau > 0.f)) && g.max_seq > 0, "gated linear attention: bad sizes");
   if (b.rows == 0 || b.n_seqs == 0) return TQ_OK;
   TQ_REQUIRE(ctx, g.heads <= 65535 && b.n_seqs <= 65535, "gated linear attention: too many heads or sequences");
-  if (b.max_q <= 1) return dtype == TQ_F32 ? launch_decode<float>(ctx, g, r, b) : launch_decode<__nv_bfloat16>(ctx, g, r, b);
-  if (dtype == TQ_BF16 && b.max_q >= 8 && gla_chunked_supported(g, r)) return launch_gla_chunked(ctx, g, r, b);
-  return dtype == TQ_F32 ? launch_scan<float>(ctx, g, r, b) : launch_scan<__nv_bfloat16>(ctx, g, r, b);
+  const bool decode = b.max_q <= 1, prompts = dtype == TQ_BF16 && b.max_q >= 8;
+  if (!g.head_decay && prompts && gla_chunked_supported(g, r)) return launch_gla_chunked(ctx, g, r, b);
+  float* o = nullptr;
+  auto rows = [&]() -> int {
+    if (decode) return dtype == TQ_F32 ? launch_decode<float>(ctx, g, r, b, o) : launch_decode<__nv_bfloat16>(ctx, g, r, b, o);
+    return dtype == TQ_F32 ? launch_scan<float>(ctx, g, r, b, o) : launch_scan<__nv_bfloat16>(ctx, g, r, b, o);
+  };
+  const size_t width = (size_t)g.heads * g.vdim;
+  if (!g.head_decay) {
+    if (!decode) {
+      if (int st = ensure_scratch(ctx, (size_t)b.rows * width * sizeof(float))) return st;
+      o = static_cast<float*>(ctx->scratch);
+    }
+    return rows();
+  }
+  const bool chunked = prompts && lightning_chunked_supported(g, r);
+  if (int st = ensure_scratch(ctx, ((size_t)b.rows * width + (chunked ? lightning_chunk_floats(g, b) : 0)) * sizeof(float))) return st;
+  o = static_cast<float*>(ctx->scratch);
+  if (int st = chunked ? launch_lightning_chunked(ctx, g, r, b, o, o + (size_t)b.rows * width) : rows()) return st;
+  return launch_norm_gate(ctx, o, width, g.norm, r.gate, r.ld, r.out, r.ldo, b.cache_row, (size_t)b.rows, width, g.eps, dtype);
 }
 
 }  // namespace tq

@@ -23,6 +23,11 @@ __device__ __forceinline__ float gl_decay_logit(const Gla& g, int channel, const
   return z;
 }
 
+// Decay of a channel at a row whose a1 values are given (null: constant decays).
+__device__ __forceinline__ float gl_decay(const Gla& g, int head, int channel, const float* a1) {
+  return g.head_decay ? g.head_decay[head] : expf(gl_log_decay(gl_decay_logit(g, channel, a1), 1.0f / g.tau));
+}
+
 __device__ __forceinline__ float gl_silu(float x) { return x / (1.0f + expf(-x)); }
 
 // The rows of a sequence and its state; false: nothing to do.
