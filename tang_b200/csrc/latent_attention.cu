@@ -10,6 +10,7 @@
 #include <cuda_bf16.h>
 
 #include <cfloat>
+#include <type_traits>
 
 #include "attn_mma.cuh"
 #include "common.cuh"
@@ -172,7 +173,7 @@ __global__ void __launch_bounds__(kLpThreads) latent_plan_kernel(RaggedBatch b, 
   }
   if (threadIdx.x == 0) *p.n_jobs = min(base_jobs, max_jobs);
   for (int seq = 0; seq < b.n_seqs; ++seq) {
-    const int row0 = b.seq_rows ? b.seq_rows[seq] : seq, end = min(b.seq_rows ? b.seq_rows[seq + 1] : seq + 1, b.rows), off = p.off[seq];
+    const int row0 = max(b.seq_rows ? b.seq_rows[seq] : seq, 0), end = min(b.seq_rows ? b.seq_rows[seq + 1] : seq + 1, b.rows), off = p.off[seq];
     for (int m = row0 + threadIdx.x; m < end; m += kLpThreads) p.exp_row[m] = off < 0 ? -1 : off + b.row_pos[m];
   }
 }
@@ -233,3 +234,311 @@ int launch_latent_gather(tq_ctx* ctx, const RaggedBatch& b, const int* single, c
                         b.n_seqs, ld, static_cast<__nv_bfloat16*>(out)));
   return TQ_OK;
 }
+
+// ------------------------------------------------------------------------------------------------ one query per sequence
+constexpr int kLdTile = 64, kLdThreads = 128;             // positions of a cache tile; threads per head tile
+constexpr int kLdPRow = kLdTile * 2 + 16;                 // bytes of a row of weights
+constexpr int kLdMaxSplits = 64;
+
+struct LatentDecodeParams {
+  LatentDims d;
+  RaggedBatch b;
+  const int* single;
+  const __nv_bfloat16 *q_lat, *q, *cache;
+  size_t ldq;
+  __nv_bfloat16* out;
+  float scale;
+  Rotation rot;
+  int rotate, n_splits;
+  float* part_o;                                          // [n_seqs][heads][n_splits][c_pad]
+  float* part_ml;                                         // [n_seqs][heads][n_splits][2]
+};
+
+// VT: 8-column tiles of latents per warp (c_pad <= 32 VT); HT: head tiles per CTA.
+template <int VT, int HT>
+__global__ void __launch_bounds__(kLdThreads * HT) latent_decode_kernel(const __grid_constant__ LatentDecodeParams p) {
+  extern __shared__ __align__(128) uint8_t ld_smem[];
+  constexpr int kThreads = kLdThreads * HT;
+  const int row_bytes = p.d.row() * 2 + 16;               // an odd number of 16-byte groups: ldmatrix rows do not meet in a bank
+  const int ht = threadIdx.x >> 7, warp = (threadIdx.x >> 5) & 3, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  uint8_t* q_s = ld_smem + (size_t)ht * 16 * row_bytes;
+  uint8_t* kv_s = ld_smem + (size_t)HT * 16 * row_bytes;
+  uint8_t* p_s = kv_s + (size_t)2 * kLdTile * row_bytes + (size_t)ht * 2 * 16 * kLdPRow;      // [terms][16][kLdPRow]
+  float* mw = reinterpret_cast<float*>(kv_s + (size_t)2 * kLdTile * row_bytes + (size_t)HT * 2 * 16 * kLdPRow) + ht * 64;   // [4 warps][16] maxima
+  pdl_wait();
+  pdl_launch_dependents();
+  const int seq = blockIdx.z, head0 = (blockIdx.y * HT + ht) * 16;
+  const int row = p.single ? p.single[seq] : seq;
+  if (row < 0) return;
+  const int pos = p.b.row_pos[row], crow = p.b.cache_row[row];
+  if (crow < pos || (size_t)crow >= p.b.cache_rows) return;
+  const __nv_bfloat16* base = p.cache + (size_t)(crow - pos) * p.d.row();
+  const int tiles = pos / kLdTile + 1, per = (tiles + p.n_splits - 1) / p.n_splits;
+  const int t0 = min((int)blockIdx.x * per, tiles), t1 = min(t0 + per, tiles);
+  const int chunks = p.d.row() / 8;
+
+  auto load_tile = [&](int tile, int buf) {
+    for (int i = threadIdx.x; i < kLdTile * chunks; i += kThreads) {
+      const int r = i / chunks, c = i - r * chunks, key = tile * kLdTile + r;
+      cp_async16(smem_u32(kv_s + (size_t)(buf * kLdTile + r) * row_bytes + c * 16), base + (size_t)(key <= pos ? key : 0) * p.d.row() + c * 8, key <= pos);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (t0 < t1) load_tile(t0, 0);
+
+  // ---- queries: [latent | rotated part] of 16 heads
+  for (int i = threadIdx.x & 127; i < 16 * p.d.c_pad / 2; i += kLdThreads) {
+    const int r = i / (p.d.c_pad / 2), c = 2 * (i - r * (p.d.c_pad / 2));
+    uint32_t v = 0u;
+    if (head0 + r < p.d.heads) {
+      v = *reinterpret_cast<const uint32_t*>(p.q_lat + ((size_t)(head0 + r) * p.b.n_seqs + seq) * p.d.c_pad + c);
+      if (c + 1 >= p.d.rank) v = c < p.d.rank ? v & 0xFFFFu : 0u;
+    }
+    *reinterpret_cast<uint32_t*>(q_s + (size_t)r * row_bytes + 2 * c) = v;
+  }
+  for (int i = threadIdx.x & 127; i < 16 * p.d.r_pad / 2; i += kLdThreads) {
+    const int r = i / (p.d.r_pad / 2), c = 2 * (i - r * (p.d.r_pad / 2));
+    float u = 0.f, v = 0.f;
+    if (head0 + r < p.d.heads) {
+      const __nv_bfloat16* src = p.q + ((size_t)(head0 + r) * p.b.n_seqs + seq) * p.ldq + p.d.dim;
+      if (c < p.d.rot) u = __bfloat162float(src[c]);
+      if (c + 1 < p.d.rot) v = __bfloat162float(src[c + 1]);
+      if (p.rotate && c < p.rot.dims) {
+        float s, co;
+        sincosf((float)pos * p.rot.freq[c / 2], &s, &co);
+        s *= p.rot.mult;
+        co *= p.rot.mult;
+        const float x = u * co - v * s;
+        v = v * co + u * s;
+        u = x;
+      }
+    }
+    *reinterpret_cast<uint32_t*>(q_s + (size_t)r * row_bytes + 2 * (p.d.c_pad + c)) = pack_bf16(u, v);
+  }
+
+  float o[VT][4];                                         // latent columns 8 (VT warp + j) + 2t, +1; heads g, then g + 8
+#pragma unroll
+  for (int j = 0; j < VT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  float m_run[2] = {-FLT_MAX, -FLT_MAX}, l_run[2] = {0.f, 0.f};
+  const float scale2 = p.scale * kLog2e;
+  const int nks = p.d.row() / 16, col0 = 8 * VT * warp;
+  const int n_vt = max(0, min(VT, (p.d.c_pad - col0) / 8));   // this warp's tiles (an even number)
+
+  for (int tile = t0; tile < t1; ++tile) {
+    const int buf = (tile - t0) & 1;
+    if (tile + 1 < t1) {
+      load_tile(tile + 1, buf ^ 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const uint8_t* kt = kv_s + (size_t)buf * kLdTile * row_bytes;
+    const int key0 = tile * kLdTile + 16 * warp;
+    float s[2][4] = {};
+    {
+      const uint8_t* qa = q_s + (size_t)(lane & 15) * row_bytes + 16 * (lane >> 4);
+      const uint8_t* ka = kt + (size_t)(16 * warp + 8 * (lane >> 4) + (lane & 7)) * row_bytes + 16 * ((lane >> 3) & 1);
+#pragma unroll 4
+      for (int ks = 0; ks < nks; ++ks) {
+        uint32_t a[4], kb[4];
+        ldmatrix4(a, qa + 32 * ks);
+        ldmatrix4(kb, ka + 32 * ks);
+        mma_bf16_16816(s[0], a[0], a[1], a[2], a[3], kb[0], kb[1]);
+        mma_bf16_16816(s[1], a[0], a[1], a[2], a[3], kb[2], kb[3]);
+      }
+    }
+    float mx[2] = {-FLT_MAX, -FLT_MAX};
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        s[n][c] = key0 + 8 * n + 2 * t + (c & 1) <= pos ? s[n][c] * scale2 : -FLT_MAX;
+        mx[c >> 1] = fmaxf(mx[c >> 1], s[n][c]);
+      }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+    }
+    if (t == 0) {
+      mw[warp * 16 + g] = mx[0];
+      mw[warp * 16 + g + 8] = mx[1];
+    }
+    __syncthreads();
+    float alpha[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int hr = g + 8 * r;
+      const float mn = fmaxf(m_run[r], fmaxf(fmaxf(mw[hr], mw[16 + hr]), fmaxf(mw[32 + hr], mw[48 + hr])));   // (finite: a tile has a visible key)
+      alpha[r] = ex2_ftz(m_run[r] - mn);
+      m_run[r] = mn;
+      float w[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) w[i] = ex2_ftz(s[i >> 1][2 * r + (i & 1)] - mn);
+      l_run[r] = l_run[r] * alpha[r] + ((w[0] + w[1]) + (w[2] + w[3]));
+      uint32_t hi, lo;
+      uint8_t* pr = p_s + (size_t)hr * kLdPRow + 2 * (16 * warp + 2 * t);
+      split_bf16(w[0], w[1], hi, lo);
+      *reinterpret_cast<uint32_t*>(pr) = hi;
+      *reinterpret_cast<uint32_t*>(pr + 16 * kLdPRow) = lo;
+      split_bf16(w[2], w[3], hi, lo);
+      *reinterpret_cast<uint32_t*>(pr + 16) = hi;
+      *reinterpret_cast<uint32_t*>(pr + 16 * kLdPRow + 16) = lo;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int j = 0; j < VT; ++j) {
+      o[j][0] *= alpha[0];
+      o[j][1] *= alpha[0];
+      o[j][2] *= alpha[1];
+      o[j][3] *= alpha[1];
+    }
+    const uint8_t* pa = p_s + (size_t)(lane & 15) * kLdPRow + 16 * (lane >> 4);
+    const uint8_t* va = kt + (size_t)(lane & 15) * row_bytes + 16 * (lane >> 4) + 2 * col0;
+#pragma unroll
+    for (int ks = 0; ks < 4; ++ks) {
+      uint32_t ah[4], al[4];
+      ldmatrix4(ah, pa + 32 * ks);
+      ldmatrix4(al, pa + 16 * kLdPRow + 32 * ks);
+#pragma unroll
+      for (int j = 0; j < VT; j += 2) {
+        if (j < n_vt) {
+          uint32_t vb[4];
+          ldmatrix4_t(vb, va + (size_t)16 * ks * row_bytes + 16 * j);
+          mma_bf16_16816(o[j], ah[0], ah[1], ah[2], ah[3], vb[0], vb[1]);
+          mma_bf16_16816(o[j + 1], ah[0], ah[1], ah[2], ah[3], vb[2], vb[3]);
+          mma_bf16_16816(o[j], al[0], al[1], al[2], al[3], vb[0], vb[1]);
+          mma_bf16_16816(o[j + 1], al[0], al[1], al[2], al[3], vb[2], vb[3]);
+        }
+      }
+    }
+    __syncthreads();                                      // the tile's buffer and the weights may be overwritten
+  }
+  // ---- sums: lanes of a quad, then the four warps (all share the running maxima)
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
+    l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
+  }
+  if (t == 0) {
+    mw[warp * 16 + g] = l_run[0];
+    mw[warp * 16 + g + 8] = l_run[1];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int hr = g + 8 * r, head = head0 + hr;
+    if (head >= p.d.heads) continue;
+    const float L = (mw[hr] + mw[16 + hr]) + (mw[32 + hr] + mw[48 + hr]);
+    if (p.n_splits == 1) {
+      const float inv = 1.0f / L;
+      __nv_bfloat16* dst = p.out + ((size_t)head * p.b.n_seqs + seq) * p.d.c_pad + col0 + 2 * t;
+#pragma unroll
+      for (int j = 0; j < VT; ++j)
+        if (j < n_vt) *reinterpret_cast<uint32_t*>(dst + 8 * j) = pack_bf16(o[j][2 * r] * inv, o[j][2 * r + 1] * inv);
+    } else {
+      const size_t at = ((size_t)seq * p.d.heads + head) * p.n_splits + blockIdx.x;
+      float* dst = p.part_o + at * p.d.c_pad + col0 + 2 * t;
+#pragma unroll
+      for (int j = 0; j < VT; ++j)
+        if (j < n_vt) *reinterpret_cast<float2*>(dst + 8 * j) = make_float2(o[j][2 * r], o[j][2 * r + 1]);
+      if (warp == 0 && t == 0) {
+        p.part_ml[2 * at] = m_run[r];
+        p.part_ml[2 * at + 1] = L;
+      }
+    }
+  }
+}
+
+// One CTA per (head, sequence): a thread owns two columns at a time.
+__global__ void __launch_bounds__(256) latent_combine_kernel(const int* single, const int* cache_row, int n_splits, int heads, int n_seqs, int c_pad,
+                                                             const float* part_o, const float* part_ml, __nv_bfloat16* out) {
+  __shared__ float wgt[kLdMaxSplits];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int head = blockIdx.x, seq = blockIdx.y, row = single ? single[seq] : seq, lane = threadIdx.x & 31;
+  if (row < 0 || cache_row[row] < 0) return;
+  const size_t at = ((size_t)seq * heads + head) * n_splits;
+  if (threadIdx.x < 32) {
+    float m[2], l[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int s = lane + 32 * i;
+      m[i] = s < n_splits ? part_ml[2 * (at + s)] : -FLT_MAX;
+      l[i] = s < n_splits ? part_ml[2 * (at + s) + 1] : 0.f;
+    }
+    const float M = warp_max(fmaxf(m[0], m[1])), w0 = ex2_ftz(m[0] - M), w1 = ex2_ftz(m[1] - M);
+    const float f = 1.0f / warp_sum(l[0] * w0 + l[1] * w1);
+    wgt[lane] = w0 * f;
+    wgt[lane + 32] = w1 * f;
+  }
+  __syncthreads();
+  for (int c = 2 * threadIdx.x; c < c_pad; c += 512) {
+    float x = 0.f, y = 0.f;
+#pragma unroll 8
+    for (int s = 0; s < n_splits; ++s) {
+      const float2 v = *reinterpret_cast<const float2*>(part_o + (at + s) * c_pad + c);
+      x = fmaf(wgt[s], v.x, x);
+      y = fmaf(wgt[s], v.y, y);
+    }
+    *reinterpret_cast<uint32_t*>(out + ((size_t)head * n_seqs + seq) * c_pad + c) = pack_bf16(x, y);
+  }
+}
+
+static size_t decode_smem(const LatentDims& d, int ht) {
+  const size_t row_bytes = (size_t)d.row() * 2 + 16;
+  return (size_t)(16 * ht + 2 * kLdTile) * row_bytes + (size_t)ht * (2 * 16 * kLdPRow + 64 * sizeof(float));
+}
+
+bool latent_absorb_supported(const LatentDims& d) { return d.c_pad <= 512 && decode_smem(d, 2) <= 226 * 1024; }
+
+int launch_latent_decode(tq_ctx* ctx, const LatentDims& d, const RaggedBatch& b, const int* single, float scale, const Rotation& rot, bool rotate,
+                         const void* q_lat, const void* q, size_t ldq, const void* cache, void* out) {
+  TQ_REQUIRE(ctx, latent_absorb_supported(d), "latent attention: a latent of %d values is too large for the absorbed form", d.rank);
+  const int HT = d.heads > 16 ? 2 : 1, hg = (d.heads + 16 * HT - 1) / (16 * HT);
+  TQ_REQUIRE(ctx, hg <= 65535 && b.n_seqs <= 65535, "latent attention: too many heads or sequences");
+  LatentDecodeParams p;
+  p.d = d;
+  p.b = b;
+  p.single = single;
+  p.q_lat = static_cast<const __nv_bfloat16*>(q_lat);
+  p.q = static_cast<const __nv_bfloat16*>(q);
+  p.ldq = ldq;
+  p.cache = static_cast<const __nv_bfloat16*>(cache);
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.scale = scale;
+  p.rot = rot;
+  p.rotate = rotate;
+  p.part_o = p.part_ml = nullptr;
+  // about two CTAs per SM, at least two tiles each
+  const long long tiles = (b.max_len + kLdTile - 1) / kLdTile, ctas = (long long)hg * b.n_seqs;
+  long long n = (2ll * ctx->sm_count + ctas - 1) / ctas;
+  if (n > (tiles + 1) / 2) n = (tiles + 1) / 2;
+  if (n > kLdMaxSplits) n = kLdMaxSplits;
+  p.n_splits = n < 1 ? 1 : (int)n;
+  if (p.n_splits > 1) {
+    const size_t parts = (size_t)b.n_seqs * d.heads * p.n_splits;
+    if (int st = ensure_scratch(ctx, parts * (d.c_pad + 2) * sizeof(float))) return st;
+    p.part_o = static_cast<float*>(ctx->scratch);
+    p.part_ml = p.part_o + parts * d.c_pad;
+  }
+  const size_t smem = decode_smem(d, HT);
+  const dim3 grid((unsigned)p.n_splits, (unsigned)hg, (unsigned)b.n_seqs);
+  auto go = [&](auto kern) -> int {
+    if (smem > 48 * 1024) TQ_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    TQ_CUDA(ctx, launch_k(ctx, kern, grid, dim3((unsigned)(kLdThreads * HT)), smem, p));
+    return TQ_OK;
+  };
+  int st;
+  if (d.c_pad <= 128) st = HT == 2 ? go(latent_decode_kernel<4, 2>) : go(latent_decode_kernel<4, 1>);
+  else if (d.c_pad <= 256) st = HT == 2 ? go(latent_decode_kernel<8, 2>) : go(latent_decode_kernel<8, 1>);
+  else st = HT == 2 ? go(latent_decode_kernel<16, 2>) : go(latent_decode_kernel<16, 1>);
+  if (st != TQ_OK) return st;
+  if (p.n_splits > 1)
+    TQ_CUDA(ctx, launch_k(ctx, latent_combine_kernel, dim3((unsigned)d.heads, (unsigned)b.n_seqs), dim3(256), 0, single, b.cache_row, p.n_splits, d.heads, b.n_seqs,
+                          d.c_pad, (const float*)p.part_o, (const float*)p.part_ml, p.out));
+  return TQ_OK;
+}
+
+}  // namespace tq
