@@ -18,7 +18,7 @@ namespace tq {
 struct LatentDims {
   int heads = 0, dim = 0, rot = 0, vdim = 0, rank = 0;
   int c_pad = 0, r_pad = 0;
-  int row() const { return c_pad + r_pad; }
+  __host__ __device__ int row() const { return c_pad + r_pad; }
 };
 LatentDims latent_dims(int heads, int dim, int rot, int vdim, int rank);
 
