@@ -658,6 +658,58 @@ TQ_API int tq_numuzen_step(tq_numuzen* model, const int* token_ids_dev, size_t r
 TQ_API int tq_numuzen_hidden(tq_numuzen* model, float** hidden_dev);
 TQ_API int tq_numuzen_trace(tq_numuzen* model, float* streams_dev_or_null);
 
+/* ---- Dotanex ------------------------------------------------------------------------------------
+ * No reference counterpart.  A decoder with several residual streams (tq_stream_mix) around its mixers -- windowed attention
+ * (per-head query/key norm, rotation in halves with banded frequencies, a learned sink per head, the raw keys as values), latent
+ * attention (low-rank queries, keys and values from one cached latent and one rotated part per position, interleaved YaRN
+ * rotation, output gate) and lightning attention -- and its feed-forwards: gated dense, or softmax-routed experts with a choice
+ * correction, identity experts and a shared expert, both of the clamped GLU (sigmoid factor 1.702).  A layer may use another
+ * layer's weights (weights_of) with a cache and states of its own.  The model owns weights, caches, states (one slot per sequence)
+ * and workspaces.  dtype TQ_BF16: bf16 weights, activations and caches; streams, norms, scores, router, recurrences f32; TQ_F32:
+ * everything f32. */
+typedef struct tq_dotanex tq_dotanex;
+typedef struct tq_dotanex_config {
+  uint32_t n_layers, width, vocab;
+  uint32_t streams;
+  uint32_t max_seq;        /* positions per slot */
+  uint32_t max_slots;
+  int dtype;
+  float eps;
+} tq_dotanex_config;
+typedef enum tq_dotanex_mixer { TQ_DX_ATTENTION = 0, TQ_DX_LATENT = 1, TQ_DX_LIGHTNING = 2 } tq_dotanex_mixer;
+typedef enum tq_dotanex_ff { TQ_DX_NONE = 0, TQ_DX_DENSE = 1, TQ_DX_MOE = 2 } tq_dotanex_ff;
+typedef struct tq_dotanex_layer {
+  uint32_t kind;
+  int32_t weights_of;                    /* -1: tensors of its own; else the rest equals that layer's */
+  uint32_t heads, kv_heads, dim, vdim;   /* kv_heads: attention only; dim: without the rotated part of latent attention */
+  uint32_t window, rot_dims;             /* window: attention; rot_dims: attention and latent attention */
+  uint32_t q_rank, kv_rank, rot_dim;     /* latent attention */
+  uint32_t ff_kind, ff;                  /* ff: of the dense feed-forward or of an expert */
+  uint32_t experts, identity, top, shared_ff;   /* shared_ff = 0: no shared expert */
+  float scale, limit, shared_limit;
+  double rot_base, rot_factor, rot_original;    /* rot_factor = 0: no scaling */
+  double rot_low, rot_high;              /* attention: banded */
+  double rot_fast, rot_slow;             /* latent attention: YaRN */
+  const float* decay;                    /* lightning: host [heads], read by tq_dotanex_create */
+} tq_dotanex_layer;
+typedef enum tq_dotanex_tensor {
+  TQ_DX_EMBED = 0, TQ_DX_FINAL_NORM = 1, TQ_DX_HEAD = 2, TQ_DX_NORM1 = 3, TQ_DX_NORM2 = 4, TQ_DX_HC1_IN = 5, TQ_DX_HC1_OUT = 6, TQ_DX_HC1_MIX = 7,
+  TQ_DX_HC2_IN = 8, TQ_DX_HC2_OUT = 9, TQ_DX_HC2_MIX = 10, TQ_DX_Q = 11, TQ_DX_K = 12, TQ_DX_V = 13, TQ_DX_G = 14, TQ_DX_O = 15, TQ_DX_Q_NORM = 16,
+  TQ_DX_K_NORM = 17, TQ_DX_SINK = 18, TQ_DX_O_NORM = 19, TQ_DX_DQ = 20, TQ_DX_DQ_NORM = 21, TQ_DX_UQ = 22, TQ_DX_DKV = 23, TQ_DX_DKV_NORM = 24,
+  TQ_DX_UK = 25, TQ_DX_UV = 26, TQ_DX_ROUTER = 27, TQ_DX_CORRECTION = 28, TQ_DX_GATE = 29, TQ_DX_UP = 30, TQ_DX_DOWN = 31, TQ_DX_SHARED_GATE = 32,
+  TQ_DX_SHARED_UP = 33, TQ_DX_SHARED_DOWN = 34
+} tq_dotanex_tensor;
+TQ_API int tq_dotanex_create(tq_ctx* ctx, const tq_dotanex_config* cfg, const tq_dotanex_layer* layers, tq_dotanex** out);
+TQ_API int tq_dotanex_destroy(tq_dotanex* model);
+/* As tq_tofazen_put; `expert` counts for gate, up and down of routed experts.  Layers with weights_of take none. */
+TQ_API int tq_dotanex_put(tq_dotanex* model, int tensor, size_t layer, size_t expert, const void* src, int src_dtype, size_t rows, size_t cols);
+/* As tq_numuzen_step. */
+TQ_API int tq_dotanex_step(tq_dotanex* model, const int* token_ids_dev, size_t rows, const int* seq_rows_dev_or_null, const int* starts_dev,
+                           const int* slots_dev_or_null, size_t n_seqs, size_t max_q, size_t max_len, const int* logit_rows_dev_or_null,
+                           size_t n_logits, float* logits_dev);
+/* While set, every step also leaves the sum of the streams after each layer in sums [n_layers][rows][width] (NULL turns it off). */
+TQ_API int tq_dotanex_trace(tq_dotanex* model, float* sums_dev_or_null);
+
 /* ---- CUDA graphs ------------------------------------------------------------------------------
  * CudaComputeDevice::begin_capture / end_capture (crates/tang-compute/src/cuda.rs:344-356): every
  * asynchronous call made on the context between begin and end is recorded instead of run, and

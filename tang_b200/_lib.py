@@ -132,6 +132,11 @@ PROTOTYPES = {
     "tq_numuzen_step": (_i, [_p, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _p, _sz, _p]),
     "tq_numuzen_hidden": (_i, [_p, _pp]),
     "tq_numuzen_trace": (_i, [_p, _p]),
+    "tq_dotanex_create": (_i, [_p, _p, _p, _pp]),
+    "tq_dotanex_destroy": (_i, [_p]),
+    "tq_dotanex_put": (_i, [_p, _i, _sz, _sz, _p, _i, _sz, _sz]),
+    "tq_dotanex_step": (_i, [_p, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _p, _sz, _p]),
+    "tq_dotanex_trace": (_i, [_p, _p]),
     "tq_graph_begin": (_i, [_p]),
     "tq_graph_end": (_i, [_p, _pp]),
     "tq_graph_launch": (_i, [_p, _p]),

@@ -797,6 +797,30 @@ __global__ void dweight_put_kernel(const void* src, int s_dt, void* dst, int d_d
   else reinterpret_cast<__nv_bfloat16*>(dst)[o] = __float2bfloat16_rn(v);
 }
 
+// dst = src + add, to f32 or bf16.
+__global__ void put_vector_kernel(const void* src, int s_dt, void* dst, int d_dt, size_t n, float add) {
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const float v = (s_dt == TQ_F32 ? static_cast<const float*>(src)[i] : __bfloat162float(static_cast<const __nv_bfloat16*>(src)[i])) + add;
+  if (d_dt == TQ_F32) static_cast<float*>(dst)[i] = v;
+  else static_cast<__nv_bfloat16*>(dst)[i] = __float2bfloat16_rn(v);
+}
+
+int put_vector(tq_ctx* ctx, const void* src, int src_dtype, void* dst, int dst_dtype, size_t n, float add) {
+  void* tmp = nullptr;
+  TQ_CUDA(ctx, cudaMalloc(&tmp, n * dtype_size(src_dtype)));
+  cudaError_t e = cudaMemcpyAsync(tmp, src, n * dtype_size(src_dtype), cudaMemcpyDefault, ctx->stream);
+  if (e == cudaSuccess) {
+    put_vector_kernel<<<(unsigned)((n + 255) / 256), 256, 0, ctx->stream>>>(tmp, src_dtype, dst, dst_dtype, n, add);
+    ctx->launches++;
+    e = cudaGetLastError();
+  }
+  if (e == cudaSuccess) e = cudaStreamSynchronize(ctx->stream);
+  cudaFree(tmp);
+  TQ_CUDA(ctx, e);
+  return TQ_OK;
+}
+
 __global__ void dweight_put_head_t_kernel(const void* src, int s_dt, void* dst, int d_dt, size_t heads, size_t dim, size_t rank, size_t group_rows, size_t kpad) {
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= heads * dim * rank) return;

@@ -71,6 +71,18 @@ struct DenseEpilogue {
   long long ldg = 0;
 };
 
+// Appends a section of weight rows [previous end, end), of which `real` exist.
+inline DenseSection& dense_section(DenseEpilogue& e, size_t end, size_t real, int kind, int f32, void* out, size_t ld) {
+  DenseSection& s = e.s[e.n++];
+  s.row_end = (int)end;
+  s.rows = (int)real;
+  s.kind = kind;
+  s.f32 = f32;
+  s.out = out;
+  s.ld = (long long)ld;
+  return s;
+}
+
 // Where one output feature goes; constant over the activation rows.
 struct DenseDst {
   char* base;        // null: a padding row
@@ -184,6 +196,9 @@ int dense_group_chunk(int dtype, size_t kpad, size_t rows, size_t n_groups);
 int dense_even_chunk(int dtype, size_t kpad, size_t rows);
 // The epilogue's sections describe one group's rows; its row indices are activation rows (`first` + `shift` of a job onwards).
 int launch_dense_grouped(tq_ctx* ctx, const tq_dweight* w, const void* x, size_t ldx, size_t rows, const DenseGroups& groups, const DenseEpilogue& epi);
+
+// dst = src + add over a vector of n values (host or device memory, bf16 or f32); for loading weights.
+int put_vector(tq_ctx* ctx, const void* src, int src_dtype, void* dst, int dst_dtype, size_t n, float add);
 
 // Per-head transposition for absorbed products: row-major src [heads * dim][rank] becomes, group by group,
 // w[h * group_rows + c][d] = src[h * dim + d][c].

@@ -121,30 +121,6 @@ static int ensure_rows(tq_numuzen* m, size_t rows) {
   return TQ_OK;
 }
 
-// dst = src + add, to f32 or bf16.
-static __global__ void vector_put_kernel(const void* src, int s_dt, void* dst, int d_dt, size_t n, float add) {
-  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i >= n) return;
-  const float v = (s_dt == TQ_F32 ? static_cast<const float*>(src)[i] : __bfloat162float(static_cast<const __nv_bfloat16*>(src)[i])) + add;
-  if (d_dt == TQ_F32) static_cast<float*>(dst)[i] = v;
-  else static_cast<__nv_bfloat16*>(dst)[i] = __float2bfloat16_rn(v);
-}
-
-static int vector_put(tq_ctx* ctx, const void* src, int src_dtype, void* dst, int dst_dtype, size_t n, float add) {
-  void* tmp = nullptr;
-  TQ_CUDA(ctx, cudaMalloc(&tmp, n * dtype_size(src_dtype)));
-  cudaError_t e = cudaMemcpyAsync(tmp, src, n * dtype_size(src_dtype), cudaMemcpyDefault, ctx->stream);
-  if (e == cudaSuccess) {
-    vector_put_kernel<<<(unsigned)((n + 255) / 256), 256, 0, ctx->stream>>>(tmp, src_dtype, dst, dst_dtype, n, add);
-    ctx->launches++;
-    e = cudaGetLastError();
-  }
-  if (e == cudaSuccess) e = cudaStreamSynchronize(ctx->stream);
-  cudaFree(tmp);
-  TQ_CUDA(ctx, e);
-  return TQ_OK;
-}
-
 static unsigned needed(const Layer& L) {
   auto bit = [](int t) { return 1u << t; };
   unsigned n = bit(TQ_NZ_NORM1) | bit(TQ_NZ_NORM1B) | bit(TQ_NZ_Q) | bit(TQ_NZ_K) | bit(TQ_NZ_G) | bit(TQ_NZ_O);
@@ -290,7 +266,7 @@ int tq_numuzen_put(tq_numuzen* m, int which, size_t layer, size_t expert, const 
     return false;
   };
   auto vec = [&](size_t n, void* dst, int dst_dtype, float add) {
-    if (shape(1, n)) st = vector_put(ctx, src, src_dtype, dst, dst_dtype, n, add);
+    if (shape(1, n)) st = put_vector(ctx, src, src_dtype, dst, dst_dtype, n, add);
   };
   auto mat = [&](size_t r, size_t c, tq_dweight* w, size_t row0, int interleave = 0) {
     if (shape(r, c)) st = tq_dweight_put(ctx, w, src, src_dtype, r, c, row0, 0, interleave);
@@ -327,7 +303,7 @@ int tq_numuzen_put(tq_numuzen* m, int which, size_t layer, size_t expert, const 
     case TQ_NZ_O_NORM: vec(c.vdim, L.o_norm, TQ_F32, 0.f); break;
     case TQ_NZ_A1: mat(c.rank, width, L.w_in, L.a0); break;
     case TQ_NZ_A2:
-      if (shape(L.q_rows, c.rank)) st = vector_put(ctx, src, src_dtype, L.a2, TQ_F32, rows * cols, 0.f);
+      if (shape(L.q_rows, c.rank)) st = put_vector(ctx, src, src_dtype, L.a2, TQ_F32, rows * cols, 0.f);
       break;
     case TQ_NZ_A2_BIAS: vec(L.q_rows, L.a2_bias, TQ_F32, 0.f); break;
     default: mat(c.experts, width, L.router, 0); break;
@@ -353,17 +329,6 @@ int tq_numuzen_trace(tq_numuzen* m, float* streams_dev_or_null) {
 #define TQ_STEP(expr) \
   if (int st = (expr)) return st;
 
-static DenseSection& section(DenseEpilogue& e, size_t end, size_t real, int kind, int f32, void* out, size_t ld) {
-  DenseSection& s = e.s[e.n++];
-  s.row_end = (int)end;
-  s.rows = (int)real;
-  s.kind = kind;
-  s.f32 = f32;
-  s.out = out;
-  s.ld = (long long)ld;
-  return s;
-}
-
 static int attention_layer(tq_numuzen* m, const Layer& L, const RaggedBatch& b) {
   tq_ctx* ctx = m->ctx;
   const tq_numuzen_layer& c = L.c;
@@ -374,11 +339,11 @@ static int attention_layer(tq_numuzen* m, const Layer& L, const RaggedBatch& b) 
   in.x = m->hn;
   in.ldx = m->embed->kpad;
   DenseEpilogue e;
-  section(e, L.k0, L.q_rows, DENSE_ROW, f32, mix, m->mix_ld);
-  DenseSection& k = section(e, L.g0, L.k_rows, DENSE_CACHE, f32, L.v_cache, (size_t)c.kv_heads * L.dim_pad);
+  dense_section(e, L.k0, L.q_rows, DENSE_ROW, f32, mix, m->mix_ld);
+  DenseSection& k = dense_section(e, L.g0, L.k_rows, DENSE_CACHE, f32, L.v_cache, (size_t)c.kv_heads * L.dim_pad);
   k.inner = (int)c.dim;
   k.inner_pad = (int)L.dim_pad;
-  section(e, L.w_in->rpad, L.g_rows, DENSE_ROW, f32, mix + L.gc * es, m->mix_ld);
+  dense_section(e, L.w_in->rpad, L.g_rows, DENSE_ROW, f32, mix + L.gc * es, m->mix_ld);
   e.cache_row = m->cache_row;
   TQ_STEP(launch_dense(ctx, L.w_in, in, b.rows, e));
   QkNormRope n;
@@ -418,11 +383,11 @@ static int gla_layer(tq_numuzen* m, const Layer& L, const RaggedBatch& b) {
   in.x = m->hn;
   in.ldx = m->embed->kpad;
   DenseEpilogue e;
-  section(e, L.k0, L.q_rows, DENSE_ROW, f32, mix, m->mix_ld);
-  section(e, L.v0, L.k_rows, DENSE_ROW, f32, mix + L.kc * es, m->mix_ld);
-  section(e, L.g0, L.v_rows, DENSE_ROW, f32, mix + L.vc * es, m->mix_ld);
-  section(e, L.a0, L.g_rows, DENSE_ROW, f32, mix + L.gc * es, m->mix_ld);
-  section(e, L.w_in->rpad, c.rank, DENSE_ROW, 1, m->a1, m->rank_ld);
+  dense_section(e, L.k0, L.q_rows, DENSE_ROW, f32, mix, m->mix_ld);
+  dense_section(e, L.v0, L.k_rows, DENSE_ROW, f32, mix + L.kc * es, m->mix_ld);
+  dense_section(e, L.g0, L.v_rows, DENSE_ROW, f32, mix + L.vc * es, m->mix_ld);
+  dense_section(e, L.a0, L.g_rows, DENSE_ROW, f32, mix + L.gc * es, m->mix_ld);
+  dense_section(e, L.w_in->rpad, c.rank, DENSE_ROW, 1, m->a1, m->rank_ld);
   TQ_STEP(launch_dense(m->ctx, L.w_in, in, b.rows, e));
   Gla g;
   g.heads = (int)c.heads;
@@ -459,7 +424,7 @@ static int expert_layer(tq_numuzen* m, const Layer& L, size_t rows) {
   in.x = m->hn;
   in.ldx = hn_ld;
   DenseEpilogue z;
-  section(z, L.router->rpad, c.experts, DENSE_ROW, 1, m->logits, m->max_experts);
+  dense_section(z, L.router->rpad, c.experts, DENSE_ROW, 1, m->logits, m->max_experts);
   TQ_STEP(launch_dense(ctx, L.router, in, rows, z));
   DenseGroups g;
   g.jobs = m->route.jobs;
@@ -471,7 +436,7 @@ static int expert_layer(tq_numuzen* m, const Layer& L, size_t rows) {
   TQ_STEP(launch_route(ctx, m->logits, m->max_experts, rows, c.experts, c.top, RouteRule(), g.chunk, m->route, m->hn, hn_ld * es, up8(width) * es,
                        gather ? m->xs : nullptr, hn_ld * es));
   DenseEpilogue u;
-  section(u, L.gu_rows, c.ff, DENSE_GLU, f32, m->act, m->act_ld);
+  dense_section(u, L.gu_rows, c.ff, DENSE_GLU, f32, m->act, m->act_ld);
   u.glu_limit = c.limit;
   u.glu_alpha = kGluAlpha;
   u.row_scale = m->route.slot_weight;
@@ -479,7 +444,7 @@ static int expert_layer(tq_numuzen* m, const Layer& L, size_t rows) {
   g.x_rows = gather ? nullptr : m->route.slot_row;
   TQ_STEP(launch_dense_grouped(ctx, L.gate_up, gather ? m->xs : m->hn, hn_ld, pairs, g, u));
   DenseEpilogue d;
-  section(d, L.down_rows, width, DENSE_ROW, 1, m->yp, width);
+  dense_section(d, L.down_rows, width, DENSE_ROW, 1, m->yp, width);
   g.group_rows = L.down_rows;
   g.x_rows = nullptr;
   return launch_dense_grouped(ctx, L.down, m->act, m->act_ld, pairs, g, d);
@@ -533,7 +498,7 @@ extern "C" int tq_numuzen_step(tq_numuzen* m, const int* token_ids_dev, size_t r
     att.x = m->att;
     att.ldx = m->att_ld;
     DenseEpilogue o;
-    section(o, L.w_out->rpad, c.width, DENSE_ROW, 1, m->y, c.width);
+    dense_section(o, L.w_out->rpad, c.width, DENSE_ROW, 1, m->y, c.width);
     TQ_STEP(launch_dense(ctx, L.w_out, att, rows, o));
     n.y = m->y;
     n.y_rows = nullptr;
@@ -563,7 +528,7 @@ extern "C" int tq_numuzen_step(tq_numuzen* m, const int* token_ids_dev, size_t r
     h.eps = c.eps;
     h.xn_tmp = m->hn;
     DenseEpilogue e;
-    section(e, m->embed->rpad, c.vocab, DENSE_ROW, 1, logits_dev, c.vocab);
+    dense_section(e, m->embed->rpad, c.vocab, DENSE_ROW, 1, logits_dev, c.vocab);
     TQ_STEP(launch_dense(ctx, m->embed, h, n_logits, e));
   }
   return TQ_OK;
