@@ -226,3 +226,272 @@ int check_layer(tq_ctx* ctx, const tq_dotanex_config& cfg, const tq_dotanex_laye
 }
 
 }  // namespace
+
+extern "C" {
+
+int tq_dotanex_create(tq_ctx* ctx, const tq_dotanex_config* cfg, const tq_dotanex_layer* layers, tq_dotanex** out) {
+  if (int st = bind(ctx)) return st;
+  TQ_REQUIRE(ctx, cfg && layers && out, "tq_dotanex_create: null argument");
+  *out = nullptr;
+  TQ_REQUIRE(ctx, cfg->n_layers > 0 && cfg->width > 0 && cfg->width <= 49152 && cfg->vocab > 0, "tq_dotanex_create: width must be 1..49152, and there must be layers and a vocabulary");
+  TQ_REQUIRE(ctx, cfg->streams > 0 && cfg->streams <= (uint32_t)kMaxStreams, "tq_dotanex_create: 1 to %d streams", kMaxStreams);
+  TQ_REQUIRE(ctx, cfg->dtype == TQ_BF16 || cfg->dtype == TQ_F32, "tq_dotanex_create: dtype must be bf16 or f32");
+  TQ_REQUIRE(ctx, cfg->max_seq > 0 && cfg->max_slots > 0 && (size_t)cfg->max_seq * cfg->max_slots < (1ull << 31), "tq_dotanex_create: cache empty or too large");
+  for (uint32_t i = 0; i < cfg->n_layers; ++i)
+    if (int st = check_layer(ctx, *cfg, layers, i)) return st;
+  tq_dotanex* m = new (std::nothrow) tq_dotanex();
+  if (!m) return fail(ctx, TQ_ENOMEM, "out of host memory");
+  m->ctx = ctx;
+  m->cfg = *cfg;
+  m->layers.resize(cfg->n_layers);
+  const size_t es = dtype_size(cfg->dtype), tokens = (size_t)cfg->max_slots * cfg->max_seq, width = cfg->width, streams = cfg->streams;
+  int st = TQ_OK;
+  auto A = [&](auto** p, size_t bytes) {
+    if (st != TQ_OK) return;
+    st = zalloc(m, (void**)p, bytes);
+    if (st == TQ_OK) m->owned.push_back(*p);
+  };
+  auto W = [&](size_t rows, size_t cols, tq_dweight** w) {
+    if (st == TQ_OK) st = tq_dweight_create(ctx, rows, cols, cfg->dtype, w);
+  };
+  auto U = [&](float** p, const std::vector<float>& v) {
+    A(p, v.size() * 4);
+    if (st == TQ_OK && !v.empty() &&
+        (cudaMemcpyAsync(*p, v.data(), v.size() * 4, cudaMemcpyHostToDevice, ctx->stream) != cudaSuccess || cudaStreamSynchronize(ctx->stream) != cudaSuccess))
+      st = fail(ctx, TQ_ECUDA, "tq_dotanex_create: copying constants failed");
+  };
+  auto most = [](size_t& a, size_t b) { a = a > b ? a : b; };
+  size_t q_lat = 0, lqs = 0, head_jobs = 0;
+  A(&m->final_norm, width * 4);
+  W(cfg->vocab, width, &m->embed);
+  W(cfg->vocab, width, &m->head);
+  for (uint32_t i = 0; i < cfg->n_layers && st == TQ_OK; ++i) {
+    Layer& L = m->layers[i];
+    L.c = layers[i];
+    L.c.decay = nullptr;
+    const tq_dotanex_layer& c = layers[i];
+    L.src = c.weights_of < 0 ? i : (size_t)c.weights_of;
+    const bool own = c.weights_of < 0;
+    L.q_rows = (size_t)c.heads * c.dim;
+    size_t in_rows = 0;
+    if (c.kind == TQ_DX_ATTENTION) {
+      L.k_rows = (size_t)c.kv_heads * c.dim;
+      L.k0 = up16(L.q_rows);
+      in_rows = L.k0 + L.k_rows;
+      L.dim_pad = up8(c.dim);
+      A(&L.k_cache, tokens * c.kv_heads * L.dim_pad * es);
+      A(&L.v_cache, tokens * c.kv_heads * L.dim_pad * es);
+      most(m->mix_ld, up8(L.q_rows));
+      if (own) {
+        A(&L.q_gain, c.dim * es);
+        A(&L.k_gain, c.dim * es);
+        A(&L.sinks, c.heads * 4);
+        std::vector<float> f(c.rot_dims / 2);
+        banded_frequencies((int)c.rot_dims, c.rot_base, c.rot_factor, c.rot_low, c.rot_high, c.rot_original, f.data());
+        U(&L.freq, f);
+      }
+    } else if (c.kind == TQ_DX_LATENT) {
+      m->latent = true;
+      L.d = latent_dims((int)c.heads, (int)c.dim, (int)c.rot_dim, (int)c.vdim, (int)c.kv_rank);
+      L.absorb = cfg->dtype == TQ_BF16 && latent_absorb_supported(L.d);
+      L.q_rows = (size_t)c.heads * (c.dim + c.rot_dim);
+      L.k_rows = (size_t)c.kv_rank + c.rot_dim;
+      L.g_rows = (size_t)c.heads * c.vdim;
+      L.k0 = up16(c.q_rank);
+      L.g0 = L.k0 + up16(L.k_rows);
+      in_rows = L.g0 + L.g_rows;
+      L.q_ld = up8(c.dim + c.rot_dim);
+      L.key_pad = L.q_ld;
+      L.v_pad = up8(c.vdim);
+      L.ukt_rows = up16(c.kv_rank);
+      L.uv_rows = up16(c.vdim);
+      L.v0 = up16((size_t)c.heads * c.dim);                  // of w_kv
+      A(&L.k_cache, tokens * L.d.row() * es);
+      most(m->mix_ld, up8(L.g_rows));
+      most(m->low_ld, c.q_rank + L.k_rows);
+      most(m->lq_ld, c.heads * L.q_ld);
+      if (L.absorb) {
+        most(q_lat, (size_t)c.heads * L.d.c_pad);
+        most(lqs, c.heads * L.q_ld);
+        most(head_jobs, (size_t)c.heads * (cfg->max_slots / 8 + 1));
+      }
+      if (own) {
+        A(&L.dq_norm, c.q_rank * 4);
+        A(&L.c_norm, c.kv_rank * 4);
+        std::vector<float> f(c.rot_dims / 2);
+        yarn_frequencies((int)c.rot_dims, c.rot_base, c.rot_factor, c.rot_original, c.rot_fast, c.rot_slow, f.data(), &L.rot_mult);
+        U(&L.freq, f);
+        W(L.q_rows, c.q_rank, &L.w_uq);
+        W(L.v0 + L.g_rows, c.kv_rank, &L.w_kv);
+        if (L.absorb) {
+          W(c.heads * L.ukt_rows, c.dim, &L.w_ukt);
+          W(c.heads * L.uv_rows, c.kv_rank, &L.w_uv);
+        }
+        if (st == TQ_OK) most(m->cq_ld, L.w_uq->kpad);
+      }
+    } else {
+      L.k_rows = L.q_rows;
+      L.v_rows = L.g_rows = (size_t)c.heads * c.vdim;
+      L.k0 = up16(L.q_rows);
+      L.v0 = L.k0 + up16(L.k_rows);
+      L.g0 = L.v0 + up16(L.v_rows);
+      in_rows = L.g0 + L.g_rows;
+      L.kc = up8(L.q_rows);
+      L.vc = L.kc + up8(L.k_rows);
+      L.gc = L.vc + up8(L.v_rows);
+      most(m->mix_ld, L.gc + up8(L.g_rows));
+      A(&L.state, (size_t)cfg->max_slots * c.heads * c.dim * c.vdim * 4);
+      if (own) {
+        A(&L.o_norm, L.v_rows * 4);
+        U(&L.decay, std::vector<float>(c.decay, c.decay + c.heads));
+      }
+    }
+    if (c.ff_kind == TQ_DX_MOE) {
+      m->moe = true;
+      most(m->max_experts, c.experts + c.identity);
+      most(m->max_top, c.top);
+    }
+    if (!own) continue;
+    for (int q = 0; q < (c.ff_kind == TQ_DX_NONE ? 1 : 2); ++q) {
+      A(&L.norm[q], width * 4);
+      A(&L.hc_in[q], streams * 4);
+      A(&L.hc_out[q], streams * 4);
+      A(&L.hc_mix[q], streams * streams * 4);
+    }
+    W(in_rows, width, &L.w_in);
+    W(width, (size_t)c.heads * c.vdim, &L.w_out);
+    if (st == TQ_OK) most(m->att_ld, L.w_out->kpad);
+    if (c.ff_kind == TQ_DX_NONE) continue;
+    const size_t n = c.ff_kind == TQ_DX_MOE ? c.experts : 1;
+    L.gu_rows = 2 * up8(c.ff);
+    L.down_rows = up16(width);
+    L.have_expert.assign(n, 0);
+    W(n * L.gu_rows, width, &L.gate_up);
+    W(n * L.down_rows, c.ff, &L.down);
+    if (st == TQ_OK) most(m->act_ld, L.down->kpad);
+    if (c.ff_kind == TQ_DX_MOE) {
+      L.shared0 = up16(c.experts + c.identity);
+      A(&L.correction, (c.experts + c.identity) * 4);
+      W(L.shared0 + 2 * up8(c.shared_ff), width, &L.front);
+      if (c.shared_ff) {
+        W(width, c.shared_ff, &L.shared_down);
+        if (st == TQ_OK) most(m->shared_ld, L.shared_down->kpad);
+      }
+    }
+  }
+  A(&m->route.counts, m->max_experts * 4);
+  A(&m->route.offsets, m->max_experts * 4);
+  A(&m->route.n_jobs, 16);
+  if (m->latent) {
+    A(&m->plan.off, cfg->max_slots * 4);
+    A(&m->plan.single, cfg->max_slots * 4);
+    A(&m->plan.jobs, kExpandJobs * sizeof(int4));
+    A(&m->plan.n_jobs, 16);
+    A(&m->lqs, cfg->max_slots * lqs * es);
+    A(&m->q_lat, cfg->max_slots * q_lat * es);
+    A(&m->o_lat, cfg->max_slots * q_lat * es);
+    A(&m->head_jobs, head_jobs * sizeof(int4));
+    A(&m->n_head_jobs, 16);
+  }
+  if (st != TQ_OK) {
+    release(m);
+    return st;
+  }
+  *out = m;
+  return TQ_OK;
+}
+
+int tq_dotanex_destroy(tq_dotanex* m) {
+  if (!m) return TQ_OK;
+  bind(m->ctx);
+  cudaStreamSynchronize(m->ctx->stream);
+  release(m);
+  return TQ_OK;
+}
+
+int tq_dotanex_put(tq_dotanex* m, int which, size_t layer, size_t expert, const void* src, int src_dtype, size_t rows, size_t cols) {
+  if (!m) return TQ_EINVAL;
+  tq_ctx* ctx = m->ctx;
+  if (int st = bind(ctx)) return st;
+  TQ_REQUIRE(ctx, src != nullptr && (src_dtype == TQ_BF16 || src_dtype == TQ_F32), "tq_dotanex_put: the source must be bf16 or f32");
+  TQ_REQUIRE(ctx, which >= TQ_DX_EMBED && which <= TQ_DX_SHARED_DOWN, "tq_dotanex_put: unknown tensor %d", which);
+  const size_t width = m->cfg.width, streams = m->cfg.streams;
+  const int dt = m->cfg.dtype;
+  int st = TQ_OK;
+  auto shape = [&](size_t r, size_t c) -> bool {
+    if (rows == r && cols == c) return true;
+    st = fail(ctx, TQ_EINVAL, "tq_dotanex_put: tensor %d of layer %zu must be [%zu, %zu], got [%zu, %zu]", which, layer, r, c, rows, cols);
+    return false;
+  };
+  auto table = [&](size_t r, size_t c, void* dst, int dst_dtype) {
+    if (shape(r, c)) st = put_vector(ctx, src, src_dtype, dst, dst_dtype, r * c, 0.f);
+  };
+  auto vec = [&](size_t n, void* dst, int dst_dtype = TQ_F32) { table(1, n, dst, dst_dtype); };
+  auto mat = [&](size_t r, size_t c, tq_dweight* w, size_t row0, int interleave = 0) {
+    if (st == TQ_OK && shape(r, c)) st = tq_dweight_put(ctx, w, src, src_dtype, r, c, row0, 0, interleave);
+  };
+  if (which <= TQ_DX_HEAD) {
+    if (which == TQ_DX_FINAL_NORM) vec(width, m->final_norm);
+    else mat(m->cfg.vocab, width, which == TQ_DX_EMBED ? m->embed : m->head, 0);
+    if (st == TQ_OK) m->have |= bit(which);
+    return st;
+  }
+  TQ_REQUIRE(ctx, layer < m->layers.size(), "tq_dotanex_put: layer %zu out of range", layer);
+  Layer& L = m->layers[layer];
+  const tq_dotanex_layer& c = L.c;
+  TQ_REQUIRE(ctx, L.src == layer, "tq_dotanex_put: layer %zu uses the weights of layer %zu", layer, L.src);
+  if (which == TQ_DX_GATE || which == TQ_DX_UP || which == TQ_DX_DOWN) {
+    TQ_REQUIRE(ctx, expert < L.have_expert.size(), "tq_dotanex_put: layer %zu has %zu experts", layer, L.have_expert.size());
+    if (which == TQ_DX_DOWN) mat(width, c.ff, L.down, expert * L.down_rows);
+    else mat(c.ff, width, L.gate_up, expert * L.gu_rows, which == TQ_DX_GATE ? 1 : 2);
+    if (st == TQ_OK) L.have_expert[expert] |= 1u << (which - TQ_DX_GATE);
+    return st;
+  }
+  TQ_REQUIRE(ctx, needed(L) & bit(which), "tq_dotanex_put: layer %zu has no tensor %d", layer, which);
+  const size_t all = (size_t)c.experts + c.identity;
+  switch (which) {
+    case TQ_DX_NORM1: case TQ_DX_NORM2: vec(width, L.norm[which - TQ_DX_NORM1]); break;
+    case TQ_DX_HC1_IN: case TQ_DX_HC2_IN: vec(streams, L.hc_in[which == TQ_DX_HC2_IN]); break;
+    case TQ_DX_HC1_OUT: case TQ_DX_HC2_OUT: vec(streams, L.hc_out[which == TQ_DX_HC2_OUT]); break;
+    case TQ_DX_HC1_MIX: case TQ_DX_HC2_MIX: table(streams, streams, L.hc_mix[which == TQ_DX_HC2_MIX], TQ_F32); break;
+    case TQ_DX_Q: mat(L.q_rows, width, L.w_in, 0); break;
+    case TQ_DX_K: mat(L.k_rows, width, L.w_in, L.k0); break;
+    case TQ_DX_V: mat(L.v_rows, width, L.w_in, L.v0); break;
+    case TQ_DX_G: mat(L.g_rows, width, L.w_in, L.g0); break;
+    case TQ_DX_O: mat(width, (size_t)c.heads * c.vdim, L.w_out, 0); break;
+    case TQ_DX_Q_NORM: vec(c.dim, L.q_gain, dt); break;
+    case TQ_DX_K_NORM: vec(c.dim, L.k_gain, dt); break;
+    case TQ_DX_SINK: vec(c.heads, L.sinks); break;
+    case TQ_DX_O_NORM: vec(L.v_rows, L.o_norm); break;
+    case TQ_DX_DQ: mat(c.q_rank, width, L.w_in, 0); break;
+    case TQ_DX_DQ_NORM: vec(c.q_rank, L.dq_norm); break;
+    case TQ_DX_UQ: mat(L.q_rows, c.q_rank, L.w_uq, 0); break;
+    case TQ_DX_DKV: mat(L.k_rows, width, L.w_in, L.k0); break;
+    case TQ_DX_DKV_NORM: vec(c.kv_rank, L.c_norm); break;
+    case TQ_DX_UK:
+      mat((size_t)c.heads * c.dim, c.kv_rank, L.w_kv, 0);
+      if (st == TQ_OK && L.absorb) st = dweight_put_head_transposed(ctx, L.w_ukt, src, src_dtype, c.heads, c.dim, c.kv_rank, L.ukt_rows);
+      break;
+    case TQ_DX_UV:
+      mat(L.g_rows, c.kv_rank, L.w_kv, L.v0);
+      if (L.absorb)
+        for (size_t h = 0; h < c.heads && st == TQ_OK; ++h)
+          st = tq_dweight_put(ctx, L.w_uv, static_cast<const char*>(src) + h * c.vdim * c.kv_rank * dtype_size(src_dtype), src_dtype, c.vdim, c.kv_rank, h * L.uv_rows, 0, 0);
+      break;
+    case TQ_DX_ROUTER: mat(all, width, L.front, 0); break;
+    case TQ_DX_CORRECTION: vec(all, L.correction); break;
+    case TQ_DX_SHARED_GATE: mat(c.shared_ff, width, L.front, L.shared0, 1); break;
+    case TQ_DX_SHARED_UP: mat(c.shared_ff, width, L.front, L.shared0, 2); break;
+    default: mat(width, c.shared_ff, L.shared_down, 0); break;
+  }
+  if (st == TQ_OK) L.have |= bit(which);
+  return st;
+}
+
+int tq_dotanex_trace(tq_dotanex* m, float* sums_dev_or_null) {
+  if (!m) return TQ_EINVAL;
+  m->trace = sums_dev_or_null;
+  return TQ_OK;
+}
+
+}  // extern "C"
