@@ -13,6 +13,7 @@
 // own slot (cache rows of the attention layers, state of the recurrent ones).
 #include <cuda_bf16.h>
 
+#include <cmath>
 #include <new>
 #include <vector>
 
@@ -495,3 +496,397 @@ int tq_dotanex_trace(tq_dotanex* m, float* sums_dev_or_null) {
 }
 
 }  // extern "C"
+
+#define TQ_STEP(expr) \
+  if (int st = (expr)) return st;
+
+// In what follows L is the layer (its caches and state), W the layer whose weights it uses.
+
+static int attention_layer(tq_dotanex* m, const Layer& L, const Layer& W, const RaggedBatch& b) {
+  tq_ctx* ctx = m->ctx;
+  const tq_dotanex_layer& c = L.c;
+  const int dt = m->cfg.dtype, f32 = dt == TQ_F32;
+  DenseInput in;
+  in.x = m->hn;
+  in.ldx = m->embed->kpad;
+  DenseEpilogue e;
+  dense_section(e, W.k0, W.q_rows, DENSE_ROW, f32, m->mix, m->mix_ld);
+  DenseSection& k = dense_section(e, W.w_in->rpad, W.k_rows, DENSE_CACHE, f32, L.v_cache, (size_t)c.kv_heads * L.dim_pad);
+  k.inner = (int)c.dim;
+  k.inner_pad = (int)L.dim_pad;
+  e.cache_row = m->cache_row;
+  TQ_STEP(launch_dense(ctx, W.w_in, in, b.rows, e));
+  HeadNormRope n;
+  n.r.heads = (int)c.heads;
+  n.r.kv_heads = (int)c.kv_heads;
+  n.r.dim = (int)c.dim;
+  n.r.raw_pad = n.r.key_pad = (int)L.dim_pad;
+  n.r.q = m->mix;
+  n.r.ldq = m->mix_ld;
+  n.r.raw = L.v_cache;
+  n.r.keys = L.k_cache;
+  n.r.q_gain = W.q_gain;
+  n.r.k_gain = W.k_gain;
+  n.r.rot.dims = (int)c.rot_dims;
+  n.r.rot.freq = W.freq;
+  n.r.eps = m->cfg.eps;
+  TQ_STEP(launch_head_norm_rope(ctx, n, b, dt));
+  WindowAttn a;
+  a.heads = (int)c.heads;
+  a.kv_heads = (int)c.kv_heads;
+  a.dim = a.vdim = (int)c.dim;
+  a.dim_pad = a.vdim_pad = (int)L.dim_pad;
+  a.window = (int)c.window;
+  a.scale = c.scale;
+  a.sinks = W.sinks;
+  return launch_window_attention(ctx, a, b, dt, m->mix, m->mix_ld, nullptr, 0, L.k_cache, L.v_cache, m->att, m->att_ld);
+}
+
+static int lightning_layer(tq_dotanex* m, const Layer& L, const Layer& W, const RaggedBatch& b) {
+  const tq_dotanex_layer& c = L.c;
+  const int dt = m->cfg.dtype, f32 = dt == TQ_F32;
+  const size_t es = dtype_size(dt);
+  char* mix = static_cast<char*>(m->mix);
+  DenseInput in;
+  in.x = m->hn;
+  in.ldx = m->embed->kpad;
+  DenseEpilogue e;
+  dense_section(e, W.k0, W.q_rows, DENSE_ROW, f32, mix, m->mix_ld).act = DENSE_SILU;
+  dense_section(e, W.v0, W.k_rows, DENSE_ROW, f32, mix + W.kc * es, m->mix_ld).act = DENSE_SILU;
+  dense_section(e, W.g0, W.v_rows, DENSE_ROW, f32, mix + W.vc * es, m->mix_ld).act = DENSE_SILU;
+  dense_section(e, W.w_in->rpad, W.g_rows, DENSE_ROW, f32, mix + W.gc * es, m->mix_ld);
+  TQ_STEP(launch_dense(m->ctx, W.w_in, in, b.rows, e));
+  Gla g;
+  g.heads = (int)c.heads;
+  g.dim = (int)c.dim;
+  g.vdim = (int)c.vdim;
+  g.eps = m->cfg.eps;
+  g.norm = W.o_norm;
+  g.head_decay = W.decay;
+  g.state = L.state;
+  g.max_seq = (int)m->cfg.max_seq;
+  GlaRows r;
+  r.q = mix;
+  r.k = mix + W.kc * es;
+  r.v = mix + W.vc * es;
+  r.gate = mix + W.gc * es;
+  r.ld = m->mix_ld;
+  r.out = m->att;
+  r.ldo = m->att_ld;
+  return launch_gla(m->ctx, g, r, b, dt);
+}
+
+// Sequences that bring several rows (at least min_q): keys and values of their positions, then windowed attention without a window.
+static int latent_expanded(tq_dotanex* m, const Layer& L, const Layer& W, const RaggedBatch& b, int min_q, const Rotation& rot) {
+  tq_ctx* ctx = m->ctx;
+  const tq_dotanex_layer& c = L.c;
+  const int dt = m->cfg.dtype, f32 = dt == TQ_F32;
+  const size_t es = dtype_size(dt), q_head = (size_t)b.rows * L.q_ld;
+  HeadNormRope n;
+  n.r.heads = (int)c.heads;
+  n.r.dim = (int)(c.dim + c.rot_dim);
+  n.r.q = m->lq;
+  n.r.ldq = L.q_ld;
+  n.r.rot = rot;
+  n.q_head = q_head;
+  TQ_STEP(launch_head_norm_rope(ctx, n, b, dt));
+  // as many sequences at a time as fit the budget, every one as long as the longest
+  const size_t k_row = c.heads * L.key_pad * es, v_row = c.heads * L.v_pad * es;
+  const int chunk = f32 ? 64 : (int)(b.max_len >= 256 ? 256 : up16(b.max_len));
+  const size_t seq_jobs = ((size_t)b.max_len + chunk - 1) / chunk;
+  size_t per = kExpandBytes / ((k_row + v_row) * b.max_len);
+  if (per > kExpandJobs / seq_jobs) per = kExpandJobs / seq_jobs;
+  if (per > (size_t)b.n_seqs) per = b.n_seqs;
+  if (per < 1) per = 1;
+  TQ_REQUIRE(ctx, seq_jobs <= kExpandJobs, "tq_dotanex_step: sequences of %d positions are too long", b.max_len);
+  const size_t exp_rows = per * b.max_len;
+  TQ_STEP(ensure_expanded(m, exp_rows * k_row, exp_rows * v_row));
+  DenseEpilogue e;
+  DenseSection& k = dense_section(e, W.v0, (size_t)c.heads * c.dim, DENSE_ROW, f32, m->exp_k, c.heads * L.key_pad);
+  k.inner = (int)c.dim;
+  k.inner_pad = (int)L.key_pad;
+  DenseSection& v = dense_section(e, W.w_kv->rpad, W.g_rows, DENSE_ROW, f32, m->exp_v, c.heads * L.v_pad);
+  v.inner = (int)c.vdim;
+  v.inner_pad = (int)L.v_pad;
+  DenseGroups g;
+  g.jobs = m->plan.jobs;
+  g.n_jobs = m->plan.n_jobs;
+  g.max_jobs = (int)(per * seq_jobs);
+  g.chunk = chunk;
+  g.group_rows = W.w_kv->rpad;
+  WindowAttn a;
+  a.heads = a.kv_heads = (int)c.heads;
+  a.dim = (int)(c.dim + c.rot_dim);
+  a.vdim = (int)c.vdim;
+  a.dim_pad = (int)L.key_pad;
+  a.vdim_pad = (int)L.v_pad;
+  a.window = kAllKeys;
+  a.scale = c.scale;
+  a.sink = -INFINITY;
+  a.q_head = q_head;
+  RaggedBatch x = b;
+  x.cache_row = m->plan.exp_row;
+  x.cache_rows = exp_rows;
+  for (int s0 = 0; s0 < b.n_seqs; s0 += (int)per) {
+    const int s1 = s0 + (int)per < b.n_seqs ? s0 + (int)per : b.n_seqs;
+    if (m->planned != s0 || m->planned_end != s1 || m->planned_chunk != chunk || m->planned_min != min_q) {
+      TQ_STEP(launch_latent_plan(ctx, b, s0, s1, min_q, chunk, g.max_jobs, m->plan));
+      m->planned = s0;
+      m->planned_end = s1;
+      m->planned_chunk = chunk;
+      m->planned_min = min_q;
+    }
+    TQ_STEP(launch_dense_grouped(ctx, W.w_kv, L.k_cache, L.d.row(), b.cache_rows, g, e));
+    TQ_STEP(launch_latent_place(ctx, L.d, b, m->plan, L.k_cache, m->exp_k, (int)L.key_pad, dt));
+    TQ_STEP(launch_window_attention(ctx, a, x, dt, m->lq, L.q_ld, m->mix, m->mix_ld, m->exp_k, m->exp_v, m->att, m->att_ld));
+  }
+  return TQ_OK;
+}
+
+static int latent_layer(tq_dotanex* m, const Layer& L, const Layer& W, const RaggedBatch& b) {
+  tq_ctx* ctx = m->ctx;
+  const tq_dotanex_layer& c = L.c;
+  const int dt = m->cfg.dtype, f32 = dt == TQ_F32;
+  const bool all_single = b.max_q == 1, some_single = all_single || (long long)b.rows < (long long)b.n_seqs * b.max_q;
+  const bool absorb = L.absorb && some_single;
+  TQ_REQUIRE(ctx, (size_t)b.rows * L.q_ld < (1ull << 31), "tq_dotanex_step: too many rows for these heads");
+  DenseInput in;
+  in.x = m->hn;
+  in.ldx = m->embed->kpad;
+  DenseEpilogue e;
+  dense_section(e, W.k0, c.q_rank, DENSE_ROW, 1, m->low, m->low_ld);
+  dense_section(e, W.g0, W.k_rows, DENSE_ROW, 1, m->low + c.q_rank, m->low_ld);
+  dense_section(e, W.w_in->rpad, W.g_rows, DENSE_ROW, f32, m->mix, m->mix_ld);
+  TQ_STEP(launch_dense(ctx, W.w_in, in, b.rows, e));
+  Rotation rot;
+  rot.dims = (int)c.rot_dims;
+  rot.freq = W.freq;
+  rot.mult = W.rot_mult;
+  rot.interleaved = true;
+  LatentIn li;
+  li.d = L.d;
+  li.low = m->low;
+  li.ld_low = m->low_ld;
+  li.q_rank = li.c0 = (int)c.q_rank;
+  li.q_gain = W.dq_norm;
+  li.c_gain = W.c_norm;
+  li.cq = m->cq;
+  li.ld_cq = m->cq_ld;
+  li.cache = L.k_cache;
+  li.rot = rot;
+  li.eps = m->cfg.eps;
+  if (absorb) {
+    const size_t kpad = W.w_ukt->kpad > W.w_uv->kpad ? W.w_ukt->kpad : W.w_uv->kpad;
+    li.head_jobs = m->head_jobs;
+    li.n_head_jobs = m->n_head_jobs;
+    li.n_head_rows = b.n_seqs;
+    li.head_chunk = dense_even_chunk(dt, kpad, b.n_seqs);
+  }
+  TQ_STEP(launch_latent_in(ctx, li, b, dt));
+  DenseInput cq;
+  cq.x = m->cq;
+  cq.ldx = m->cq_ld;
+  DenseEpilogue q;                                           // head by head: [head][row][q_ld]
+  DenseSection& qs = dense_section(q, W.w_uq->rpad, W.q_rows, DENSE_ROW, f32, m->lq, L.q_ld);
+  qs.inner = (int)(c.dim + c.rot_dim);
+  qs.inner_pad = (int)(b.rows * L.q_ld);
+  TQ_STEP(launch_dense(ctx, W.w_uq, cq, b.rows, q));
+  rot.first = (int)c.dim;
+  if (!all_single || !L.absorb) TQ_STEP(latent_expanded(m, L, W, b, L.absorb ? 2 : 1, rot));
+  if (!absorb) return TQ_OK;
+  const int* single = all_single ? nullptr : m->plan.single;
+  const void* query = m->lq;
+  if (single) {
+    TQ_STEP(launch_latent_gather(ctx, b, single, m->lq, (int)c.heads, L.q_ld, m->lqs));
+    query = m->lqs;
+  }
+  const size_t pairs = (size_t)c.heads * b.n_seqs;
+  DenseGroups g;
+  g.jobs = m->head_jobs;
+  g.n_jobs = m->n_head_jobs;
+  g.chunk = li.head_chunk;
+  g.max_jobs = (int)(c.heads * (((size_t)b.n_seqs + g.chunk - 1) / g.chunk));
+  g.group_rows = W.ukt_rows;
+  DenseEpilogue ql;
+  dense_section(ql, W.ukt_rows, c.kv_rank, DENSE_ROW, f32, m->q_lat, L.d.c_pad);
+  TQ_STEP(launch_dense_grouped(ctx, W.w_ukt, query, L.q_ld, pairs, g, ql));
+  TQ_STEP(launch_latent_decode(ctx, L.d, b, single, c.scale, rot, single == nullptr, m->q_lat, query, L.q_ld, L.k_cache, m->o_lat));
+  DenseEpilogue o;
+  dense_section(o, W.uv_rows, c.vdim, DENSE_HEADS, f32, m->att, m->att_ld).inner_pad = (int)c.vdim;
+  o.head_rows = b.n_seqs;
+  o.head_row = single;
+  o.gate = m->mix;
+  o.ldg = (long long)m->mix_ld;
+  g.group_rows = W.uv_rows;
+  return launch_dense_grouped(ctx, W.w_uv, m->o_lat, L.d.c_pad, pairs, g, o);
+}
+
+// Leaves its output to the stream kernel: y rows and how they are summed.
+static int feed_forward(tq_dotanex* m, const Layer& W, size_t rows, StreamMix& mix) {
+  tq_ctx* ctx = m->ctx;
+  const tq_dotanex_layer& c = W.c;
+  const int dt = m->cfg.dtype, f32 = dt == TQ_F32;
+  const size_t es = dtype_size(dt), width = m->cfg.width, hn_ld = m->embed->kpad;
+  DenseInput in;
+  in.x = m->hn;
+  in.ldx = hn_ld;
+  if (c.ff_kind == TQ_DX_DENSE) {
+    DenseEpilogue u;
+    dense_section(u, W.gate_up->rpad, c.ff, DENSE_GLU, f32, m->act, m->act_ld);
+    u.glu = DENSE_GLU_SILU;
+    TQ_STEP(launch_dense(ctx, W.gate_up, in, rows, u));
+    DenseInput a;
+    a.x = m->act;
+    a.ldx = m->act_ld;
+    DenseEpilogue d;
+    dense_section(d, W.down->rpad, width, DENSE_ROW, 1, m->y, width);
+    mix.y = m->y;
+    return launch_dense(ctx, W.down, a, rows, d);
+  }
+  const size_t pairs = rows * c.top, all = (size_t)c.experts + c.identity;
+  DenseEpilogue f;
+  dense_section(f, W.shared0, all, DENSE_ROW, 1, m->logits, m->max_experts);
+  if (c.shared_ff) dense_section(f, W.front->rpad, c.shared_ff, DENSE_GLU, f32, m->shared, m->shared_ld);
+  f.glu_limit = c.shared_limit;
+  f.glu_alpha = kGluAlpha;
+  TQ_STEP(launch_dense(ctx, W.front, in, rows, f));
+  DenseGroups g;
+  g.jobs = m->route.jobs;
+  g.n_jobs = m->route.n_jobs;
+  g.chunk = dense_group_chunk(dt, W.gate_up->kpad > W.down->kpad ? W.gate_up->kpad : W.down->kpad, pairs * c.experts / all + 1, c.experts);
+  g.max_jobs = (int)route_max_jobs(pairs, c.experts, g.chunk);
+  // the tcgen05 kernel copies boxes of consecutive rows, the others follow the slots' row numbers
+  const bool gather = !f32 && g.chunk > 8;
+  RouteRule rule;
+  rule.score = ROUTE_SOFTMAX;
+  rule.renorm = true;
+  rule.correction = W.correction;
+  rule.identity = (int)c.identity;
+  TQ_STEP(launch_route(ctx, m->logits, m->max_experts, rows, all, c.top, rule, g.chunk, m->route, m->hn, hn_ld * es, up8(width) * es,
+                       gather ? m->gathered : nullptr, hn_ld * es));
+  DenseEpilogue u;
+  dense_section(u, W.gu_rows, c.ff, DENSE_GLU, f32, m->act, m->act_ld);
+  u.glu_limit = c.limit;
+  u.glu_alpha = kGluAlpha;
+  g.group_rows = W.gu_rows;
+  g.x_rows = gather ? nullptr : m->route.slot_row;
+  TQ_STEP(launch_dense_grouped(ctx, W.gate_up, gather ? m->gathered : m->hn, hn_ld, pairs, g, u));
+  DenseEpilogue d;
+  dense_section(d, W.down_rows, width, DENSE_ROW, 1, m->yp, width);
+  g.group_rows = W.down_rows;
+  g.x_rows = nullptr;
+  TQ_STEP(launch_dense_grouped(ctx, W.down, m->act, m->act_ld, pairs, g, d));
+  if (c.shared_ff) {
+    DenseInput s;
+    s.x = m->shared;
+    s.ldx = m->shared_ld;
+    DenseEpilogue y;
+    dense_section(y, W.shared_down->rpad, width, DENSE_ROW, 1, m->ys, width);
+    TQ_STEP(launch_dense(ctx, W.shared_down, s, rows, y));
+    mix.y_more = m->ys;
+  }
+  mix.y = m->yp;
+  mix.y_rows = m->route.slot;
+  mix.y_weight = m->route.weight;
+  mix.n_y = (int)c.top;
+  mix.self = m->hn;
+  return TQ_OK;
+}
+
+extern "C" int tq_dotanex_step(tq_dotanex* m, const int* token_ids_dev, size_t rows, const int* seq_rows_dev, const int* starts_dev, const int* slots_dev,
+                               size_t n_seqs, size_t max_q, size_t max_len, const int* logit_rows_dev, size_t n_logits, float* logits_dev) {
+  if (!m) return TQ_EINVAL;
+  tq_ctx* ctx = m->ctx;
+  if (int st = bind(ctx)) return st;
+  const tq_dotanex_config& c = m->cfg;
+  TQ_REQUIRE(ctx, token_ids_dev && starts_dev && rows > 0 && n_seqs > 0, "tq_dotanex_step: null pointer or empty step");
+  TQ_REQUIRE(ctx, rows < (1ull << 24), "tq_dotanex_step: too many rows");
+  TQ_REQUIRE(ctx, seq_rows_dev || rows == n_seqs, "tq_dotanex_step: without row offsets every sequence brings one row");
+  TQ_REQUIRE(ctx, max_q > 0 && max_q <= rows && (seq_rows_dev || max_q == 1), "tq_dotanex_step: max_q must bound the sequences' rows");
+  TQ_REQUIRE(ctx, n_seqs <= c.max_slots && max_len > 0 && max_len <= c.max_seq, "tq_dotanex_step: at most %u sequences of %u positions", c.max_slots, c.max_seq);
+  TQ_REQUIRE(ctx, n_logits == 0 || logits_dev, "tq_dotanex_step: null logits");
+  TQ_REQUIRE(ctx, logit_rows_dev || n_logits == 0 || n_logits == rows, "tq_dotanex_step: without a row list every row has logits");
+  TQ_REQUIRE(ctx, m->have == (bit(TQ_DX_EMBED) | bit(TQ_DX_FINAL_NORM) | bit(TQ_DX_HEAD)), "tq_dotanex_step: the embedding, the final norm or the head is missing");
+  for (size_t i = 0; i < m->layers.size(); ++i) {
+    const Layer& L = m->layers[i];
+    bool all = L.src != i || L.have == needed(L);
+    for (unsigned char e : L.have_expert) all = all && e == 7;
+    TQ_REQUIRE(ctx, all, "tq_dotanex_step: layer %zu has tensors missing", i);
+  }
+  TQ_STEP(ensure_rows(m, rows));
+  TQ_REQUIRE(ctx, n_logits <= m->ws_rows, "tq_dotanex_step: more logits than rows");
+  m->planned = -1;
+  TQ_STEP(launch_embedding_pos(ctx, m->embed->data, m->embed->kpad, nullptr, c.dtype, token_ids_dev, seq_rows_dev, starts_dev, slots_dev, (int)n_seqs, rows,
+                               (int)c.width, (int)c.vocab, (int)c.max_seq, (int)c.max_seq, (int)c.max_slots, m->x, m->row_pos, m->cache_row));
+  RaggedBatch b;
+  b.n_seqs = (int)n_seqs;
+  b.rows = (int)rows;
+  b.max_q = (int)max_q;
+  b.max_len = (int)max_len;
+  b.seq_rows = seq_rows_dev;
+  b.row_pos = m->row_pos;
+  b.cache_row = m->cache_row;
+  b.cache_rows = (size_t)c.max_slots * c.max_seq;
+  // the streams are all equal to the embedding until the first sublayer is done
+  StreamMix s;
+  s.streams = (int)c.streams;
+  s.src = m->x;
+  s.dst = m->xs;
+  s.out = m->hn;
+  s.out_dtype = c.dtype;
+  s.ld_out = m->embed->kpad;
+  s.eps = c.eps;
+  auto read = [&](StreamMix& mix, const Layer* next, int q) {
+    mix.w_in = next ? next->hc_in[q] : nullptr;
+    mix.gain = next ? next->norm[q] : nullptr;
+  };
+  auto write = [&](StreamMix& mix, const Layer& W, int q) {
+    mix.mix = W.hc_mix[q];
+    mix.w_out = W.hc_out[q];
+  };
+  read(s, &m->layers[m->layers[0].src], 0);
+  TQ_STEP(launch_stream_mix(ctx, s, rows, c.width));
+  for (size_t i = 0; i < m->layers.size(); ++i) {
+    const Layer &L = m->layers[i], &W = m->layers[L.src];
+    const Layer* next = i + 1 < m->layers.size() ? &m->layers[m->layers[i + 1].src] : nullptr;
+    const bool ff = L.c.ff_kind != TQ_DX_NONE;
+    float* sum = m->trace ? m->trace + i * rows * c.width : nullptr;
+    TQ_STEP(L.c.kind == TQ_DX_ATTENTION ? attention_layer(m, L, W, b) : L.c.kind == TQ_DX_LATENT ? latent_layer(m, L, W, b) : lightning_layer(m, L, W, b));
+    DenseInput att;
+    att.x = m->att;
+    att.ldx = m->att_ld;
+    DenseEpilogue o;
+    dense_section(o, W.w_out->rpad, c.width, DENSE_ROW, 1, m->y, c.width);
+    TQ_STEP(launch_dense(ctx, W.w_out, att, rows, o));
+    StreamMix mix = s;
+    mix.y = m->y;
+    mix.sum = ff ? nullptr : sum;
+    write(mix, W, 0);
+    read(mix, ff ? &W : next, ff ? 1 : 0);
+    TQ_STEP(launch_stream_mix(ctx, mix, rows, c.width));
+    s.src = m->xs;
+    s.src_streams = (int)c.streams;
+    if (!ff) continue;
+    StreamMix after = s;
+    TQ_STEP(feed_forward(m, W, rows, after));
+    after.sum = sum;
+    write(after, W, 1);
+    read(after, next, 0);
+    TQ_STEP(launch_stream_mix(ctx, after, rows, c.width));
+  }
+  if (n_logits) {
+    s.dst = nullptr;
+    s.src_rows = logit_rows_dev;
+    s.w_in = nullptr;
+    s.gain = m->final_norm;
+    TQ_STEP(launch_stream_mix(ctx, s, n_logits, c.width));
+    DenseInput h;
+    h.x = m->hn;
+    h.ldx = m->embed->kpad;
+    DenseEpilogue e;
+    dense_section(e, m->head->rpad, c.vocab, DENSE_ROW, 1, logits_dev, c.vocab);
+    TQ_STEP(launch_dense(ctx, m->head, h, n_logits, e));
+  }
+  return TQ_OK;
+}
+#undef TQ_STEP

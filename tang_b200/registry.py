@@ -6,11 +6,12 @@ import os
 
 from . import _lib
 from .checkpoint import read_safetensors
+from .dotanex import DotanexConfig, DotanexModel
 from .numuzen import NumuzenConfig, NumuzenModel
 from .tofazen import TofazenConfig, TofazenModel
 
 # architecture -> (configuration class, model class with ``from_tensors``)
-ARCHITECTURES = {"Tofazen": (TofazenConfig, TofazenModel), "Numuzen": (NumuzenConfig, NumuzenModel)}
+ARCHITECTURES = {"Tofazen": (TofazenConfig, TofazenModel), "Numuzen": (NumuzenConfig, NumuzenModel), "Dotanex": (DotanexConfig, DotanexModel)}
 
 DEFAULT_MAX_SEQ = 8192      # for designs without a largest position
 
