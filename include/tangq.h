@@ -680,7 +680,7 @@ typedef enum tq_dotanex_mixer { TQ_DX_ATTENTION = 0, TQ_DX_LATENT = 1, TQ_DX_LIG
 typedef enum tq_dotanex_ff { TQ_DX_NONE = 0, TQ_DX_DENSE = 1, TQ_DX_MOE = 2 } tq_dotanex_ff;
 typedef struct tq_dotanex_layer {
   uint32_t kind;
-  int32_t weights_of;                    /* -1: tensors of its own; else the rest equals that layer's */
+  int weights_of;                        /* -1: tensors of its own; else the rest equals that layer's */
   uint32_t heads, kv_heads, dim, vdim;   /* kv_heads: attention only; dim: without the rotated part of latent attention */
   uint32_t window, rot_dims;             /* window: attention; rot_dims: attention and latent attention */
   uint32_t q_rank, kv_rank, rot_dim;     /* latent attention */
