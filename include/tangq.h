@@ -604,6 +604,13 @@ TQ_API int tq_lightning(tq_ctx* ctx, int dtype, size_t heads, size_t dim, size_t
                         const void* k_dev, const void* v_dev, const void* gate_dev, size_t ld, const float* norm_dev, float* state_dev, size_t max_seq,
                         size_t cache_rows, const int* seq_rows_dev_or_null, const int* row_pos_dev, const int* cache_row_dev, size_t n_seqs,
                         size_t rows, size_t max_q, void* out_dev, size_t ldo);
+/* Latent attention of one bf16 query per sequence over cache rows [latent: rank padded to 16 | rotated part: rot padded to 16] (the
+ * padding zero): out[h] = sum_j softmax_j((q_lat[h] . c_j + q_rot[h] . r_j) scale) c_j.  q_lat and out [heads][n_seqs][rank padded
+ * to 16], q [heads][n_seqs][ldq] with the rotated part from column dim on; rotate: its first rot_dims are still to be rotated
+ * (2i with 2i + 1).  rank at most 512. */
+TQ_API int tq_latent_decode(tq_ctx* ctx, size_t heads, size_t dim, size_t rot, size_t rank, float scale, size_t rot_dims, const float* freq_dev,
+                            float rot_mult, int rotate, const void* q_lat_dev, const void* q_dev, size_t ldq, const void* cache_dev, size_t cache_rows,
+                            const int* row_pos_dev, const int* cache_row_dev, size_t n_seqs, size_t max_len, void* out_dev);
 /* The `top` experts with the largest logits [rows][experts] per row (the lower index among equals) with weights sigmoid(z)
  * (score 0) or softmax (score 1), divided by their sum if renorm.  Pair p = row * top + i gets a slot; the slots of an expert are
  * consecutive.  jobs int[.][4]: (expert, first slot, slots <= chunk, 0), at most min(pairs, experts + pairs / chunk). */

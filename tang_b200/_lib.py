@@ -124,6 +124,7 @@ PROTOTYPES = {
     "tq_stream_mix": (_i, [_p, _sz, _sz, _p, _p, _p, _p, _p, _sz, _p, _p, _p, _p, _p, _p, _sz, _sz, C.c_float, _p, _i, _sz, _p]),
     "tq_gla": (_i, [_p, _p, _i, _p, _p, _p, _p, _sz, _p, _sz, _p, _p, _p, _p, _sz, _sz, _p, _p, _p, _sz, _sz, _sz, _p, _sz]),
     "tq_lightning": (_i, [_p, _i, _sz, _sz, _sz, C.c_float, _p, _p, _p, _p, _p, _sz, _p, _p, _sz, _sz, _p, _p, _p, _sz, _sz, _sz, _p, _sz]),
+    "tq_latent_decode": (_i, [_p, _sz, _sz, _sz, _sz, C.c_float, _sz, _p, C.c_float, _i, _p, _p, _sz, _p, _sz, _p, _p, _sz, _sz, _p]),
     "tq_route": (_i, [_p, _p, _sz, _sz, _sz, _i, _i, _sz, _p, _p, _p, _p, _p, _p]),
     "tq_route_rule": (_i, [_p, _p, _sz, _sz, _sz, _i, _i, _p, _sz, _sz, _p, _p, _p, _p, _p, _p]),
     "tq_numuzen_create": (_i, [_p, _p, _p, _pp]),

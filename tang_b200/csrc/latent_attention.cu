@@ -542,3 +542,28 @@ int launch_latent_decode(tq_ctx* ctx, const LatentDims& d, const RaggedBatch& b,
 }
 
 }  // namespace tq
+
+using namespace tq;
+
+extern "C" int tq_latent_decode(tq_ctx* ctx, size_t heads, size_t dim, size_t rot, size_t rank, float scale, size_t rot_dims, const float* freq_dev,
+                                float rot_mult, int rotate, const void* q_lat_dev, const void* q_dev, size_t ldq, const void* cache_dev, size_t cache_rows,
+                                const int* row_pos_dev, const int* cache_row_dev, size_t n_seqs, size_t max_len, void* out_dev) {
+  if (int st = bind(ctx)) return st;
+  if (n_seqs == 0) return TQ_OK;
+  TQ_REQUIRE(ctx, heads > 0 && rank > 0 && max_len > 0 && rot_dims <= rot && rot_dims % 2 == 0, "tq_latent_decode: bad sizes");
+  TQ_REQUIRE(ctx, q_lat_dev && (q_dev || rot == 0) && cache_dev && row_pos_dev && cache_row_dev && out_dev && (freq_dev || rot_dims == 0 || !rotate),
+             "tq_latent_decode: null pointer");
+  RaggedBatch b;
+  b.n_seqs = b.rows = (int)n_seqs;
+  b.max_len = (int)max_len;
+  b.row_pos = row_pos_dev;
+  b.cache_row = cache_row_dev;
+  b.cache_rows = cache_rows;
+  Rotation r;
+  r.dims = (int)rot_dims;
+  r.freq = freq_dev;
+  r.mult = rot_mult;
+  r.interleaved = true;
+  return launch_latent_decode(ctx, latent_dims((int)heads, (int)dim, (int)rot, 0, (int)rank), b, nullptr, scale, r, rotate != 0, q_lat_dev, q_dev, ldq, cache_dev,
+                              out_dev);
+}
