@@ -682,6 +682,7 @@ typedef struct tq_dotanex_config {
   uint32_t max_slots;
   int dtype;
   float eps;
+  size_t expand_bytes;     /* latent attention expands keys and values of as many sequences at a time as fit (0: 1 GiB) */
 } tq_dotanex_config;
 typedef enum tq_dotanex_mixer { TQ_DX_ATTENTION = 0, TQ_DX_LATENT = 1, TQ_DX_LIGHTNING = 2 } tq_dotanex_mixer;
 typedef enum tq_dotanex_ff { TQ_DX_NONE = 0, TQ_DX_DENSE = 1, TQ_DX_MOE = 2 } tq_dotanex_ff;

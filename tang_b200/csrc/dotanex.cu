@@ -31,7 +31,7 @@ namespace {
 
 constexpr float kGluAlpha = 1.702f;
 constexpr int kAllKeys = 0x7fffffff;
-constexpr size_t kExpandBytes = 1ull << 30;      // of expanded keys and values at a time
+constexpr size_t kExpandBytes = 1ull << 30;      // of expanded keys and values at a time, unless the configuration says
 constexpr size_t kExpandJobs = 32768;
 
 size_t up16(size_t n) { return (n + 15) / 16 * 16; }
@@ -594,7 +594,7 @@ static int latent_expanded(tq_dotanex* m, const Layer& L, const Layer& W, const 
   const size_t k_row = c.heads * L.key_pad * es, v_row = c.heads * L.v_pad * es;
   const int chunk = f32 ? 64 : (int)(b.max_len >= 256 ? 256 : up16(b.max_len));
   const size_t seq_jobs = ((size_t)b.max_len + chunk - 1) / chunk;
-  size_t per = kExpandBytes / ((k_row + v_row) * b.max_len);
+  size_t per = (m->cfg.expand_bytes ? m->cfg.expand_bytes : kExpandBytes) / ((k_row + v_row) * b.max_len);
   if (per > kExpandJobs / seq_jobs) per = kExpandJobs / seq_jobs;
   if (per > (size_t)b.n_seqs) per = b.n_seqs;
   if (per < 1) per = 1;

@@ -26,7 +26,8 @@ NONE, DENSE, MOE = range(3)
 
 
 class _CConfig(C.Structure):
-    _fields_ = [(n, C.c_uint32) for n in ("n_layers", "width", "vocab", "streams", "max_seq", "max_slots")] + [("dtype", C.c_int), ("eps", C.c_float)]
+    _fields_ = [(n, C.c_uint32) for n in ("n_layers", "width", "vocab", "streams", "max_seq", "max_slots")] + [("dtype", C.c_int), ("eps", C.c_float), (
+        "expand_bytes", C.c_size_t)]
 
 
 class _CLayer(C.Structure):
@@ -188,16 +189,17 @@ def tensor_names(cfg: DotanexConfig):
 
 class DotanexModel(StepModel):
     """Weights, caches, states and the step.  `dtype` BF16: bf16 weights, activations and caches with f32 streams and states; F32:
-    all f32.  ``trace`` receives the sum of the streams after each layer."""
+    all f32.  ``trace`` receives the sum of the streams after each layer.  `expand_bytes`: see tq_dotanex_config."""
 
     abi = "tq_dotanex"
 
-    def __init__(self, dev: QuantComputeDevice, cfg: DotanexConfig, dtype: int = _lib.BF16, max_slots: int = 64, max_seq: int | None = None):
+    def __init__(self, dev: QuantComputeDevice, cfg: DotanexConfig, dtype: int = _lib.BF16, max_slots: int = 64, max_seq: int | None = None,
+                 expand_bytes: int = 0):
         from .registry import DEFAULT_MAX_SEQ
 
         self.dev, self.cfg, self.dtype, self.max_slots = dev, cfg, dtype, max_slots
         self.max_seq = max_seq or DEFAULT_MAX_SEQ
-        cc = _CConfig(len(cfg.layers), cfg.width, cfg.vocab, cfg.streams, self.max_seq, max_slots, dtype, cfg.eps)
+        cc = _CConfig(len(cfg.layers), cfg.width, cfg.vocab, cfg.streams, self.max_seq, max_slots, dtype, cfg.eps, expand_bytes)
         cl, keep = (_CLayer * len(cfg.layers))(), []
         for c, l in zip(cl, cfg.layers):
             for n in ("kind", "weights_of", "heads", "kv_heads", "dim", "vdim", "window", "q_rank", "kv_rank", "rot_dim", "scale"):
@@ -216,10 +218,10 @@ class DotanexModel(StepModel):
 
     @classmethod
     def from_tensors(cls, dev: QuantComputeDevice, config: dict, tensors: dict, dtype: int = _lib.BF16, max_slots: int = 64,
-                     max_seq: int | None = None) -> "DotanexModel":
+                     max_seq: int | None = None, expand_bytes: int = 0) -> "DotanexModel":
         """From a parsed config.json and the tensors of the checkpoint (``read_safetensors``)."""
         cfg = DotanexConfig.from_dict(config)
-        model = cls(dev, cfg, dtype, max_slots, max_seq)
+        model = cls(dev, cfg, dtype, max_slots, max_seq, expand_bytes)
         try:
             for name, tensor, layer, expert in tensor_names(cfg):
                 model.put(tensor, layer, need(tensors, name), expert)

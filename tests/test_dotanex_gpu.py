@@ -147,6 +147,24 @@ def test_large_prompt_batch(dev, refs):
     model.destroy()
 
 
+@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+def test_expansion_in_parts(dev, refs, dtype):
+    """Keys and values of the latent layers expanded for one or a few sequences at a time, among sequences that bring one row."""
+    cfg, w, tokens, want = refs["mixed"]
+    for expand_bytes in (1, 200_000):
+        model = make(dev, cfg, w, dtype, max_slots=6, max_seq=120, expand_bytes=expand_bytes)
+        e = engine(model)
+        at, got = {r: 0 for r in range(6)}, {r: [] for r in range(6)}
+        for counts in ((70, 1, 33, 5, 64, 1), (1, 40, 2, 1, 9, 30), (3, 1, 1, 60, 20, 1)):
+            out, k = e.step([(r, tokens[at[r]:at[r] + n], range(n)) for r, n in enumerate(counts)]), 0
+            for r, n in enumerate(counts):
+                got[r].append(out[k:k + n])
+                k, at[r] = k + n, at[r] + n
+        for r in range(6):
+            assert row_errors(np.concatenate(got[r]), want[:at[r]]).max() < TOL[dtype], (expand_bytes, r)
+        model.destroy()
+
+
 def _planted(mixer, n, j, i):
     """A one-layer model in which the token at position i looks for what the token at position j left; token ids carry the
     match, so that the same weights serve any pair of positions."""
