@@ -95,7 +95,7 @@ def test_streams(dev, dt, tol, streams, rows, width):
     eps, ld = 1e-4, (width + 7) // 8 * 8
     mix, wo, wi, gain = (rng.standard_normal(s) for s in ((streams, streams), streams, streams, width))
     mix_d, wo_d, wi_d, gain_d = (up(dev, a)[0] for a in (mix, wo, wi, gain))
-    mix, wo, wi, gain = (np.float64(np.float32(a)) for a in (mix, wo, wi, gain))
+    mix, wo, wi, gain = (a.astype(np.float32).astype(np.float64) for a in (mix, wo, wi, gain))
     n_y = 3
     for equal in (False, True):
         for experts in (False, True):
@@ -125,7 +125,7 @@ def test_streams(dev, dt, tol, streams, rows, width):
             assert np.array_equal(got[:, width:], hv[:, width:])
 
 
-@pytest.mark.parametrize("dt,tol", [(F32, 2e-6), (BF16, 8e-3)])
+@pytest.mark.parametrize("dt,tol", [(F32, 6e-5), (BF16, 8e-3)])      # (an f32 angle of 300 carries 1.5e-5)
 @pytest.mark.parametrize("heads,kv_heads,dim,first,rot,interleaved,norm", [
     (4, 2, 32, 0, 16, False, True), (3, 1, 33, 0, 10, False, True), (20, 4, 128, 0, 128, False, True), (5, 0, 24, 16, 8, True, False), (7, 0, 13, 7, 6, True, False),
     (33, 0, 192, 128, 64, True, False), (2, 2, 8, 0, 0, False, True)])
@@ -153,9 +153,9 @@ def test_head_norm_and_rotation(dev, dt, tol, heads, kv_heads, dim, first, rot, 
         return y
 
     for r in range(b.rows):
-        assert rel(got[:, r, :dim], want(qv[:, r, :dim], qgv, b.pos[r])) < tol * (8 if dt == F32 else 1)
+        assert rel(got[:, r, :dim], want(qv[:, r, :dim], qgv, b.pos[r])) < tol
         if kv_heads:
-            assert rel(gk[b.crow[r], :, :dim], want(rv[b.crow[r], :, :dim], kgv, b.pos[r])) < tol * (8 if dt == F32 else 1)
+            assert rel(gk[b.crow[r], :, :dim], want(rv[b.crow[r], :, :dim], kgv, b.pos[r])) < tol
     if kv_heads:
         other = np.setdiff1d(np.arange(960), b.crow)
         assert not gk[other].any()
