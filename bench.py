@@ -14,6 +14,7 @@ weak and the aggregate is the sum over ranks.
     python bench.py --impl reference        # the CPU restatement of tang-infer on the host cores
     python bench.py --tofazen               # instead: the Tofazen family beside the int4 model (one JSON line of its own)
     python bench.py --numuzen               # instead: the Numuzen family beside the Tofazen family (one JSON line of its own)
+    python bench.py --dotanex               # instead: the Dotanex family beside the Numuzen family (one JSON line of its own)
 
 The JSON line also carries: `e2e` (the same rate through the reference-shaped call q4_matvec with
 HOST vectors, copies inside the timed region), `roofline` (dominant kernel vs measured HBM peak),
@@ -1372,6 +1373,283 @@ def run_numuzen(args) -> None:
     out["clocks"] = sampler.stop(t_start, time.perf_counter())
     print(json.dumps(out))
 
+
+# ----------------------------------------------------------------------------------------------
+# --dotanex: the Dotanex family (bf16) beside the Numuzen family at equal width, head sizes, window and active feed-forward,
+# random weights: decode and prefill throughput of both, and the new kernels beside the like ones, against their rooflines.
+# ----------------------------------------------------------------------------------------------
+DOTANEX_SIZES = {
+    # of four layers: attention, lightning, latent attention, lightning; of `top` choices two thirds (8b) or four fifths (1b) fall on
+    # experts with weights, which together with the shared one are as wide as the other models' feed-forward
+    "8b": {**{k: NUMUZEN_SIZES["8b"][k] for k in ("layers", "width", "heads", "kv", "dim", "vocab")}, "lightning": (16, 128, 256), "latent": (1536, 512, 64),
+           "experts": 8, "identity": 4, "top": 3, "ff": 4096, "shared": 6144, "streams": 4},
+    "1b": {**{k: NUMUZEN_SIZES["1b"][k] for k in ("layers", "width", "heads", "kv", "dim", "vocab")}, "lightning": (8, 128, 256), "latent": (768, 512, 64),
+           "experts": 32, "identity": 8, "top": 5, "ff": 1536, "shared": 2048, "streams": 4},
+}
+
+
+def build_dotanex(dev, tb, torch, stream, s, max_seq, max_batch, window):
+    from tang_b200 import dotanex as dx
+
+    gen = torch.Generator(device="cuda").manual_seed(7)
+    mlp = dx.FeedForward(dx.MOE, s["ff"], s["experts"], s["identity"], s["top"], 7.0, s["shared"], 7.0)
+    (lh, ld, lv), (q_rank, kv_rank, rot) = s["lightning"], s["latent"]
+    banded = dx.Rotation(64, 500000.0, 4.0, 4096, low=1.0, high=4.0)
+    yarn = dx.Rotation(rot, 500000.0, 4.0, 4096, fast=32.0, slow=1.0)
+    kinds = [dx.DotanexLayer(dx.ATTENTION, s["heads"], s["dim"], s["dim"], s["dim"] ** -0.5, s["kv"], window, banded, mlp=mlp),
+             dx.DotanexLayer(dx.LIGHTNING, lh, ld, lv, decay=tuple(1 - 2.0 ** (-2 - 0.3 * h) for h in range(lh)), mlp=mlp),
+             dx.DotanexLayer(dx.LATENT, s["heads"], s["dim"], s["dim"], (s["dim"] + rot) ** -0.5, rot=yarn, q_rank=q_rank, kv_rank=kv_rank, rot_dim=rot, mlp=mlp)]
+    cfg = tb.DotanexConfig(s["vocab"], s["width"], s["streams"], 1e-6, [kinds[(0, 1, 2, 1)[i % 4]] for i in range(s["layers"])])
+    model = tb.DotanexModel(dev, cfg, tb.BF16, max_batch, max_seq)
+    d, S, n = s["width"], s["streams"], s["experts"] + s["identity"]
+    pool = {}
+    for name, tensor, i, e in dx.tensor_names(cfg):
+        l = cfg.layers[i]
+        H, G, D, V = l.heads, l.kv_heads or l.heads, l.dim, l.vdim
+        r, c = {dx.EMBED: (s["vocab"], d), dx.HEAD: (s["vocab"], d), dx.HC1_IN: (1, S), dx.HC2_IN: (1, S), dx.HC1_OUT: (1, S), dx.HC2_OUT: (1, S), dx.HC1_MIX: (S, S),
+                dx.HC2_MIX: (S, S), dx.Q: (H * D, d), dx.K: (G * D, d), dx.V: (H * V, d), dx.G: (H * V, d), dx.O: (d, H * V), dx.Q_NORM: (1, D), dx.K_NORM: (1, D),
+                dx.SINK: (1, H), dx.O_NORM: (1, H * V), dx.DQ: (q_rank, d), dx.DQ_NORM: (1, q_rank), dx.UQ: (H * (D + rot), q_rank), dx.DKV: (kv_rank + rot, d),
+                dx.DKV_NORM: (1, kv_rank), dx.UK: (H * D, kv_rank), dx.UV: (H * V, kv_rank), dx.ROUTER: (n, d), dx.CORRECTION: (1, n), dx.GATE: (s["ff"], d),
+                dx.UP: (s["ff"], d), dx.DOWN: (d, s["ff"]), dx.SHARED_GATE: (s["shared"], d), dx.SHARED_UP: (s["shared"], d),
+                dx.SHARED_DOWN: (d, s["shared"])}.get(tensor, (1, d))
+        level = {dx.HC1_IN: 1.0 / S, dx.HC2_IN: 1.0 / S, dx.HC1_OUT: 0.5, dx.HC2_OUT: 0.5, dx.HC1_MIX: 1.0 / S, dx.HC2_MIX: 1.0 / S, dx.SINK: 0.0, dx.CORRECTION: 0.0}.get(
+            tensor, 1.0 if r == 1 else 0.0)
+        key = (r, c, level, tensor == dx.ROUTER and i)
+        if key not in pool:
+            with torch.cuda.stream(stream):
+                pool[key] = (torch.randn((r, c), device="cuda", generator=gen) * (0.02 if r == 1 or r == S else c ** -0.5) + level).bfloat16()
+            stream.synchronize()
+        model.put_pointer(tensor, i, pool[key].data_ptr(), tb.BF16, r, c, e)
+    return model
+
+
+def run_dotanex(args) -> None:
+    import ctypes as C
+
+    import torch
+
+    import tang_b200 as tb
+
+    torch.cuda.set_device(0)
+    dev = tb.QuantComputeDevice(0)
+    L_ = dev._L
+    stream = torch.cuda.ExternalStream(dev.stream, device=torch.device("cuda", 0))
+    peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")) else {}
+    hbm, tf = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    ctx, window = 2048, 512
+    sampler = ClockSampler(0)
+    sampler.start()
+    t_start = time.perf_counter()
+
+    def graph_ms(fn, reps=10):
+        fn()
+        dev.sync()
+        dev.begin_capture()
+        fn()
+        g = dev.end_capture()
+        ms = _time_ms(torch, stream, dev, g.launch, reps, warm=3)
+        g.free()
+        return ms
+
+    def rand(*shape, std=1.0, dt=None):
+        with torch.cuda.stream(stream):
+            t = torch.randn(shape, device="cuda") * std
+            t = t if dt == tb.F32 else t.bfloat16()
+        stream.synchronize()
+        return t
+
+    P = lambda t: C.c_void_p(t.data_ptr() if hasattr(t, "data_ptr") else t.ptr)
+    ints = lambda a: dev.upload(np.asarray(a, np.int32).reshape(-1), tb.I32)
+    null = C.c_void_p(0)
+    touched = lambda experts, share, rows: experts * (1 - (1 - share) ** rows)      # expected number of experts that `rows` rows choose
+    out = {"metric": "dotanex_throughput", "unit": "tokens/s", "data": "synthetic", "dtype": "bf16", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf},
+           "window": window, "models": [], "kernels": []}
+    batches = [1, 2, 4, 8, 16, 64]
+
+    def time_model(size, name, model, s, decode_bytes, prefill_flops):
+        row = {"size": size, "model": name, "decode": {}, "prefill": {}}
+        for B in batches:
+            tok = ints(np.random.randint(0, s["vocab"], B))
+            pos, lg = ints(np.full(B, ctx)), dev.alloc(B * s["vocab"], tb.F32)
+            ms = graph_ms(lambda: model.decode(tok, pos, B, ctx + 1, lg))
+            row["decode"][B] = {"ms": ms, "tokens_per_s": B / ms * 1e3, "frac_of_hbm": decode_bytes(B) / ms / 1e6 / hbm}
+        for T in (512, ctx):
+            tok = ints(np.random.randint(0, s["vocab"], T))
+            cu, st, last, lg = ints([0, T]), ints([0]), ints([T - 1]), dev.alloc(s["vocab"], tb.F32)
+            ms = graph_ms(lambda: model.step(tok, T, cu, st, None, 1, T, T, last, 1, lg), 3)
+            row["prefill"][T] = {"ms": ms, "tokens_per_s": T / ms * 1e3, "frac_of_bf16": T * prefill_flops(T) / ms / 1e9 / tf}
+        out["models"].append(row)
+        model.destroy()
+        torch.cuda.empty_cache()
+
+    for size in [x for x in args.dotanex.split(",") if x in DOTANEX_SIZES]:
+        s = DOTANEX_SIZES[size]
+        d, H, D, (lh, ld, lv), (qr, kr, rot) = s["width"], s["heads"], s["dim"], s["lightning"], s["latent"]
+        n = s["experts"] + s["identity"]
+        att = d * (2 * H + s["kv"]) * D
+        rec = d * (2 * lh * ld + 3 * lh * lv)
+        lat = d * (qr + kr + rot + 2 * H * D) + qr * H * (D + rot) + 2 * kr * H * D
+        mixers = s["layers"] // 4 * (att + 2 * rec + lat)
+        one, share = 3 * d * s["ff"], s["top"] / n
+        fixed = 2 * (mixers + s["layers"] * (n * d + 3 * d * s["shared"]) + s["vocab"] * d)
+        per_row = s["layers"] // 4 * (s["kv"] * 2 * D * 2 * window + 2 * lh * ld * lv * 4 * 2 + (kr + rot) * 2 * ctx)
+        active = mixers + s["layers"] * (s["experts"] * share * one + 3 * d * s["shared"])
+        time_model(size, "dotanex", build_dotanex(dev, tb, torch, stream, s, ctx + 1, max(batches), window), s,
+                   lambda B: fixed + 2 * s["layers"] * one * touched(s["experts"], share, B) + B * per_row,
+                   lambda T: 2.0 * active + s["layers"] // 4 * H * T * (2 * D + rot))
+        if not args.dotanex_only:
+            z = NUMUZEN_SIZES[size]
+            gh, gd, gv = z["gla"]
+            zm = z["layers"] // 2 * (d * (3 * H + z["kv"]) * D + d * (2 * gh * gd + 3 * gh * gv + 16))
+            zone, zrow = 3 * d * z["ff"], z["layers"] // 2 * (z["kv"] * 2 * D * 2 * window + gh * gd * gv * 8)
+            time_model(size, "numuzen", build_numuzen(dev, tb, torch, stream, z, ctx + 1, max(batches), window), z,
+                       lambda B: 2 * (zm + z["layers"] * z["experts"] * d + z["vocab"] * d + z["layers"] * zone * touched(z["experts"], z["top"] / z["experts"], B)) + B * zrow,
+                       lambda T: 2.0 * (zm + z["layers"] * z["top"] * zone))
+
+    def kernel(name, m, us, byt=0.0, flops=0.0):
+        roof = max(byt / hbm / 1e3, flops / tf / 1e6)
+        out["kernels"].append({"kernel": name, "m": m, "us": round(us, 2), "roofline_us": round(roof, 2), "frac": round(roof / us, 3)})
+
+    # ---- decode: absorbed latent attention beside the int8 family's, lightning beside the gated recurrence
+    class Win(C.Structure):
+        _fields_ = [(k, C.c_uint32) for k in ("heads", "kv_heads", "dim", "vdim", "window")] + [(k, C.c_float) for k in ("scale", "softcap", "sink")]
+
+    class Gla(C.Structure):
+        _fields_ = [(k, C.c_uint32) for k in ("heads", "dim", "vdim", "rank")] + [(k, C.c_float) for k in ("tau", "q_scale", "eps")]
+
+    def handle(rows, cols):
+        t, h = rand(min(rows, 65536), cols, std=cols ** -0.5), C.c_void_p()
+        dev._check(L_.tq_dweight_create(dev._ctx, rows, cols, tb.BF16, C.byref(h)))
+        for r in range(0, rows, 65536):
+            dev._check(L_.tq_dweight_put(dev._ctx, h, P(t), tb.BF16, min(65536, rows - r), cols, r, 0, 0))
+        return h
+
+    H, D, R, K = 32, 128, 64, 512
+    lh, ld, lv = 16, 128, 256
+    width = 2 * lh * ld + 2 * lh * lv
+    freq, decay = rand(R // 2, dt=tb.F32), torch.full((lh,), 0.97, device="cuda")
+    norm, gnorm, a2, bias = rand(lh * lv, dt=tb.F32), rand(lv, dt=tb.F32), rand(lh * ld, 16, dt=tb.F32), rand(lh * ld, dt=tb.F32)
+    torch.cuda.synchronize()
+
+    def lightning(x, st, o, rows, n_seqs, cu, rp, cr, max_q):
+        off = lambda c: C.c_void_p(x.data_ptr() + 2 * c)
+        return L_.tq_lightning(dev._ctx, tb.BF16, lh, ld, lv, 1e-6, P(decay), off(0), off(lh * ld), off(2 * lh * ld), off(2 * lh * ld + lh * lv), width, P(norm), P(st), ctx,
+                               n_seqs * ctx, cu, P(rp), P(cr), n_seqs, rows, max_q, P(o), lh * lv)
+
+    def recurrence(x, a1, st, o, rows, n_seqs, cu, rp, cr, max_q):
+        g, off = Gla(lh, ld, lv, 16, 16.0, ld ** -0.5, 1e-6), lambda c: C.c_void_p(x.data_ptr() + 2 * c)
+        return L_.tq_gla(dev._ctx, C.byref(g), tb.BF16, off(0), off(lh * ld), off(2 * lh * ld), off(2 * lh * ld + lh * lv), width, P(a1), 16, P(a2), P(bias), P(gnorm),
+                         P(st), ctx, n_seqs * ctx, cu, P(rp), P(cr), n_seqs, rows, max_q, P(o), lh * lv)
+
+    uk, uv = [handle(H * K, D) for _ in range(16)], [handle(H * D, K) for _ in range(16)]
+    q8 = []
+    for _ in range(16):
+        with torch.cuda.stream(stream):
+            wk, wv = (torch.randint(-127, 128, (H * r, c), dtype=torch.int8, device="cuda") for r, c in ((K, D), (D, K)))
+            sk, sv = (torch.full((H * r,), 0.002, device="cuda") for r in (K, D))
+        stream.synchronize()
+        pair = []
+        for w8, s8, rows, cols in ((wk, sk, H * K, D), (wv, sv, H * D, K)):
+            h = C.c_void_p()
+            dev._check(L_.tq_qweight_from_device_arrays(dev._ctx, tb.I8_ROW, P(s8), P(w8), rows, cols, C.byref(h)))
+            pair.append(h)
+        q8.append(pair)
+    for B in (1, 16, 64):
+        n = max(2, min(16, 128 // B))                  # distinct caches per pass
+        cache = rand(n, B, ctx, K + R)
+        q, ql, qf, o = rand(H, B, D + R), rand(H, B, K), rand(B, H, K + R), torch.empty((H, B, K), dtype=torch.bfloat16, device="cuda")
+        rp, cr, lens = ints(np.full(B, ctx - 1)), ints(np.arange(B) * ctx + ctx - 1), ints(np.full(B, ctx))
+        byt, flops = B * ctx * (K + R) * 2, 2.0 * B * ctx * H * (2 * K + R)
+        us = graph_ms(lambda: [dev._check(L_.tq_latent_decode(dev._ctx, H, D, R, K, 0.07, R, P(freq), 1.0, 1, P(ql), P(q), D + R, P(cache[i]), B * ctx, P(rp), P(cr), B, ctx,
+                                                              P(o))) for i in range(n)]) / n * 1e3
+        kernel("decode latent attention", B, us, byt, flops)
+        us = graph_ms(lambda: [dev._check(L_.tq_mla_decode(dev._ctx, P(qf), P(cache[i]), P(lens), B, H, K, R, ctx * (K + R), ctx, 0.07, P(o))) for i in range(n)]) / n * 1e3
+        kernel("decode latent attention (int8 family)", B, us, byt, flops)
+        chunk = 8 if B <= 8 else (B + 15) // 16 * 16
+        jobs = ints([(h, h * B + i, min(chunk, B - i), 0) for h in range(H) for i in range(0, B, chunk)])
+        nj, o2 = ints([jobs.n // 4]), torch.empty((H * B, K), dtype=torch.bfloat16, device="cuda")
+        for what, hs, x, cols, rows in (("absorb W_uk", uk, q, D, K), ("absorb W_uv", uv, ql, K, D)):
+            ldx = D + R if what == "absorb W_uk" else K
+            us = graph_ms(lambda: [dev._check(L_.tq_dlinear_grouped(dev._ctx, h, P(x), ldx, H * B, P(jobs), P(nj), jobs.n // 4, chunk, rows, null, null, 0.0, 0.0, P(o2),
+                                                                    tb.BF16, rows)) for h in hs]) / len(hs) * 1e3
+            kernel(what, B, us, H * K * D * 2 + H * B * (K + D) * 2, 2.0 * H * B * K * D)
+        qn, qp, y = rand(B, H, D), rand(B, H, R), torch.empty((B, H, K + R), dtype=torch.bfloat16, device="cuda")
+        us = graph_ms(lambda: [dev._check(L_.tq_mla_absorb_q(dev._ctx, p[0], P(qn), P(qp), B, H, D, P(y))) for p in q8]) / len(q8) * 1e3
+        kernel("absorb W_uk (int8 family)", B, us, H * K * D + H * B * (K + D) * 2, 2.0 * H * B * K * D)
+        us = graph_ms(lambda: [dev._check(L_.tq_mla_unabsorb(dev._ctx, p[1], P(o2), B, H, D, P(y), tb.BF16)) for p in q8]) / len(q8) * 1e3
+        kernel("absorb W_uv (int8 family)", B, us, H * K * D + H * B * (K + D) * 2, 2.0 * H * B * K * D)
+        del cache
+        st = [rand(B, lh, ld, lv, dt=tb.F32) for _ in range(max(4, min(64, 128 // B)))]
+        x, a1, o = rand(B, width), rand(B, 16, dt=tb.F32), torch.empty((B, lh * lv), dtype=torch.bfloat16, device="cuda")
+        us = graph_ms(lambda: [dev._check(lightning(x, t, o, B, B, null, rp, cr, 1)) for t in st]) / len(st) * 1e3
+        kernel("decode lightning", B, us, B * lh * ld * lv * 4 * 2)
+        us = graph_ms(lambda: [dev._check(recurrence(x, a1, t, o, B, B, null, rp, cr, 1)) for t in st]) / len(st) * 1e3
+        kernel("decode gated recurrence", B, us, B * lh * ld * lv * 4 * 2)
+        del st
+        torch.cuda.empty_cache()
+
+    # ---- prompts
+    w_kv = handle(H * 2 * D, K)
+    for T in (512, 2048):
+        x, a1, st = rand(T, width), rand(T, 16, dt=tb.F32), rand(1, lh, ld, lv, dt=tb.F32)
+        cu, rp, o = ints([0, T]), ints(np.arange(T)), torch.empty((T, lh * lv), dtype=torch.bfloat16, device="cuda")
+        byt, flops = T * (width + lh * lv) * 2, 2.0 * T * lh * (32 * (ld + lv) + 2 * ld * lv)
+        kernel("prefill lightning", T, graph_ms(lambda: dev._check(lightning(x, st, o, T, 1, P(cu), rp, rp, T))) * 1e3, byt, flops)
+        kernel("prefill gated recurrence", T, graph_ms(lambda: dev._check(recurrence(x, a1, st, o, T, 1, P(cu), rp, rp, T))) * 1e3, byt, flops)
+        sinks = rand(H, dt=tb.F32)
+        for name, G, dk, dv, w, sk in (("prefill attention, expanded latents", H, D + R, D, ctx, null), ("prefill attention, all keys (grouped)", 8, D, D, ctx, null),
+                                       ("prefill attention, window and sinks", 8, D, D, window, P(sinks)), ("prefill attention, window", 8, D, D, window, null)):
+            q, k, v, o = rand(T, H * dk), rand(T, G * dk), rand(T, G * dv), torch.empty((T, H * dv), dtype=torch.bfloat16, device="cuda")
+            a = Win(H, G, dk, dv, w, dk ** -0.5, 0.0, float("-inf"))
+            us = graph_ms(lambda: dev._check(L_.tq_window_attention_sinks(dev._ctx, C.byref(a), sk, tb.BF16, P(q), H * dk, null, 0, P(k), P(v), T, P(cu), P(rp), P(rp), 1, T, T, T,
+                                                                          P(o), H * dv))) * 1e3
+            kernel(name, T, us, 0, 2.0 * H * (dk + dv) * sum(min(i + 1, w) for i in range(T)))
+        x, y, chunk = rand(T, K), torch.empty((T, H * 2 * D), dtype=torch.bfloat16, device="cuda"), min(T, 256)
+        jobs = ints([(0, i, min(chunk, T - i), 0) for i in range(0, T, chunk)])
+        nj = ints([jobs.n // 4])
+        us = graph_ms(lambda: dev._check(L_.tq_dlinear_grouped(dev._ctx, w_kv, P(x), K, T, P(jobs), P(nj), jobs.n // 4, chunk, H * 2 * D, null, null, 0.0, 0.0, P(y), tb.BF16,
+                                                               H * 2 * D))) * 1e3
+        kernel("expansion of latents", T, us, (H * 2 * D + T) * K * 2 + T * H * 2 * D * 2, 2.0 * T * K * H * 2 * D)
+        us = graph_ms(lambda: dev._check(L_.tq_dlinear(dev._ctx, w_kv, P(x), K, T, P(y), tb.BF16, H * 2 * D))) * 1e3
+        kernel("linear of the same size", T, us, (H * 2 * D + T) * K * 2 + T * H * 2 * D * 2, 2.0 * T * K * H * 2 * D)
+
+    # ---- row operators
+    G, D, n = 8, 128, 20
+    for m in (1, 64, 2048):
+        for S in (2, 4):
+            xs = [rand(m, S, 4096, dt=tb.F32) for _ in range(n if m < 2048 else 4)]
+            y, gain, h = rand(m * 3, 4096, dt=tb.F32), rand(4096, dt=tb.F32), torch.empty((m, 4096), dtype=torch.bfloat16, device="cuda")
+            mix, co, slots, wt = rand(S, S, std=0.3, dt=tb.F32), rand(S, dt=tb.F32), ints(np.random.permutation(3 * m)), rand(m, 3, dt=tb.F32)
+            us = graph_ms(lambda: [dev._check(L_.tq_stream_mix(dev._ctx, S, S, P(x), P(x), P(y), null, null, 1, null, null, P(mix), P(co), P(co), P(gain), m, 4096, 1e-6, P(h),
+                                                               tb.BF16, 4096, null)) for x in xs]) / len(xs) * 1e3
+            kernel(f"{S} streams, next norm", m, us, m * 4096 * (8 * S + 6))
+            us = graph_ms(lambda: [dev._check(L_.tq_stream_mix(dev._ctx, S, S, P(x), P(x), P(y), P(slots), P(wt), 3, P(h), P(y), P(mix), P(co), P(co), P(gain), m, 4096, 1e-6,
+                                                               P(h), tb.BF16, 4096, null)) for x in xs]) / len(xs) * 1e3
+            kernel(f"{S} streams, next norm, three experts and a shared one", m, us, m * 4096 * (8 * S + 2 + 16))
+        xs = [rand(m, 4096, dt=tb.F32) for _ in range(n if m < 2048 else 8)]
+        us = graph_ms(lambda: [dev._check(L_.tq_add_norm(dev._ctx, P(x), P(y), P(slots), 2, P(gain), P(gain), m, 4096, 1e-6, P(h), tb.BF16, 4096)) for x in xs]) / len(xs) * 1e3
+        kernel("post-norm, stream, next norm over two experts", m, us, m * 4096 * 18)
+        q, raw, keys, qg, rp, fr = rand(m, H * D), rand(m, G * D), rand(m, G * D), rand(H * D), ints(np.arange(m)), rand(32, dt=tb.F32)
+        us = graph_ms(lambda: [dev._check(L_.tq_head_norm_rope(dev._ctx, tb.BF16, H, G, D, P(q), H * D, D, P(raw), P(keys), m, P(qg), P(qg), 0, 64, 0, P(fr), 1.0, 1e-6, P(rp),
+                                                               P(rp), m)) for _ in range(n)]) / n * 1e3
+        kernel("per-head norm and rotation", m, us, m * (H + G) * D * 4)
+        us = graph_ms(lambda: [dev._check(L_.tq_qk_norm_rope(dev._ctx, tb.BF16, H, G, D, P(q), H * D, P(raw), P(keys), m, P(qg), P(qg), 64, P(fr), 1.0, 1e-6, P(rp), P(rp), m))
+                               for _ in range(n)]) / n * 1e3
+        kernel("whole-projection norm and rotation", m, us, m * (H + G) * D * 4)
+        q = rand(H, m, 192)
+        us = graph_ms(lambda: [dev._check(L_.tq_head_norm_rope(dev._ctx, tb.BF16, H, 0, 192, P(q), 192, m * 192, null, null, m, null, null, 128, 64, 1, P(fr), 1.0, 1e-6, P(rp),
+                                                               P(rp), m)) for _ in range(n)]) / n * 1e3
+        kernel("rotation of latent queries", m, us, m * H * 192 * 4)
+        z, corr = rand(m, 40, dt=tb.F32), rand(40, std=0.01, dt=tb.F32)
+        bufs = [ints(np.zeros(m * 5)) for _ in range(4)] + [ints(np.zeros(4 * (m * 5 + 40))), ints([0])]
+        us = graph_ms(lambda: [dev._check(L_.tq_route_rule(dev._ctx, P(z), m, 40, 5, 1, 1, P(corr), 8, 8, *map(P, bufs))) for _ in range(n)]) / n * 1e3
+        kernel("corrected routing, 5 of 32 + 8", m, us, m * 40 * 4)
+        us = graph_ms(lambda: [dev._check(L_.tq_route(dev._ctx, P(z), m, 40, 5, 0, 0, 8, *map(P, bufs))) for _ in range(n)]) / n * 1e3
+        kernel("routing, 5 of 40", m, us, m * 40 * 4)
+    out["clocks"] = sampler.stop(t_start, time.perf_counter())
+    print(json.dumps(out))
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1391,8 +1669,13 @@ def main() -> None:
     ap.add_argument("--tofazen", nargs="?", const="8b,1b", default="", help="time the Tofazen family instead (sizes: 8b, 1b, or none: kernels only)")
     ap.add_argument("--tofazen-only", action="store_true", help="with --tofazen: leave the int4 model out")
     ap.add_argument("--numuzen", nargs="?", const="8b,1b", default="", help="time the Numuzen family instead (sizes: 8b, 1b, or none: kernels only)")
+    ap.add_argument("--dotanex", nargs="?", const="8b,1b", default="", help="time the Dotanex family instead (sizes: 8b, 1b, or none: kernels only)")
+    ap.add_argument("--dotanex-only", action="store_true", help="with --dotanex: leave the Numuzen model out")
     ap.add_argument("--numuzen-only", action="store_true", help="with --numuzen: leave the Tofazen model out")
     args = ap.parse_args()
+    if args.dotanex:
+        run_dotanex(args)
+        return
     if args.numuzen:
         run_numuzen(args)
         return
