@@ -254,12 +254,14 @@ struct LatentDecodeParams {
   float* part_ml;                                         // [n_seqs][heads][n_splits][2]
 };
 
-// VT: 8-column tiles of latents per warp (c_pad <= 32 VT); HT: head tiles per CTA.
-template <int VT, int HT>
+// VT: 8-column tiles of latents per warp (c_pad <= 32 VT); HT: head tiles per CTA; FULL: c_pad = 32 VT; ROW: elements of a cache row (0: any).
+template <int VT, int HT, bool FULL, int ROW = 0>
 __global__ void __launch_bounds__(kLdThreads * HT) latent_decode_kernel(const __grid_constant__ LatentDecodeParams p) {
   extern __shared__ __align__(128) uint8_t ld_smem[];
+  static_assert(kLdTile * (ROW / 8) % (kLdThreads * HT) == 0, "whole rounds of copies");
   constexpr int kThreads = kLdThreads * HT;
-  const int row_bytes = p.d.row() * 2 + 16;               // an odd number of 16-byte groups: ldmatrix rows do not meet in a bank
+  const int row_el = ROW ? ROW : p.d.row();
+  const int row_bytes = row_el * 2 + 16;               // an odd number of 16-byte groups: ldmatrix rows do not meet in a bank
   const int ht = threadIdx.x >> 7, warp = (threadIdx.x >> 5) & 3, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   uint8_t* q_s = ld_smem + (size_t)ht * 16 * row_bytes;
   uint8_t* kv_s = ld_smem + (size_t)HT * 16 * row_bytes;
@@ -272,15 +274,37 @@ __global__ void __launch_bounds__(kLdThreads * HT) latent_decode_kernel(const __
   if (row < 0) return;
   const int pos = p.b.row_pos[row], crow = p.b.cache_row[row];
   if (crow < pos || (size_t)crow >= p.b.cache_rows) return;
-  const __nv_bfloat16* base = p.cache + (size_t)(crow - pos) * p.d.row();
+  const __nv_bfloat16* base = p.cache + (size_t)(crow - pos) * row_el;
   const int tiles = pos / kLdTile + 1, per = (tiles + p.n_splits - 1) / p.n_splits;
   const int t0 = min((int)blockIdx.x * per, tiles), t1 = min(t0 + per, tiles);
-  const int chunks = p.d.row() / 8;
+  const int chunks = row_el / 8;
+  const int step_r = kThreads / chunks, step_c = kThreads % chunks, first_r = threadIdx.x / chunks, first_c = threadIdx.x % chunks;
+  const uint32_t kv_u = smem_u32(kv_s);
 
   auto load_tile = [&](int tile, int buf) {
-    for (int i = threadIdx.x; i < kLdTile * chunks; i += kThreads) {
-      const int r = i / chunks, c = i - r * chunks, key = tile * kLdTile + r;
-      cp_async16(smem_u32(kv_s + (size_t)(buf * kLdTile + r) * row_bytes + c * 16), base + (size_t)(key <= pos ? key : 0) * p.d.row() + c * 8, key <= pos);
+    const int n_valid = pos + 1 - tile * kLdTile;          // rows at or beyond it become zeros
+    const __nv_bfloat16* src = base + (size_t)tile * kLdTile * row_el;
+    const uint32_t dst = kv_u + (uint32_t)(buf * kLdTile * row_bytes);
+    if constexpr (ROW != 0) {
+#pragma unroll
+      for (int i = 0; i < kLdTile * (ROW / 8) / kThreads; ++i) {
+        const int at = i * kThreads + threadIdx.x, r = at / (ROW / 8), c = at % (ROW / 8);
+        const bool ok = r < n_valid;
+        cp_async16(dst + (uint32_t)(r * row_bytes + c * 16), ok ? src + at * 8 : base, ok);
+      }
+      asm volatile("cp.async.commit_group;" ::: "memory");
+      return;
+    }
+    int r = first_r, c = first_c;
+    while (r < kLdTile) {
+      const bool ok = r < n_valid;
+      cp_async16(dst + (uint32_t)(r * row_bytes + c * 16), ok ? src + r * row_el + c * 8 : base, ok);
+      r += step_r;
+      c += step_c;
+      if (c >= chunks) {
+        c -= chunks;
+        ++r;
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -321,7 +345,7 @@ __global__ void __launch_bounds__(kLdThreads * HT) latent_decode_kernel(const __
   for (int j = 0; j < VT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
   float m_run[2] = {-FLT_MAX, -FLT_MAX}, l_run[2] = {0.f, 0.f};
   const float scale2 = p.scale * kLog2e;
-  const int nks = p.d.row() / 16, col0 = 8 * VT * warp;
+  const int nks = row_el / 16, col0 = 8 * VT * warp;
   const int n_vt = max(0, min(VT, (p.d.c_pad - col0) / 8));   // this warp's tiles (an even number)
 
   for (int tile = t0; tile < t1; ++tile) {
@@ -403,7 +427,7 @@ __global__ void __launch_bounds__(kLdThreads * HT) latent_decode_kernel(const __
       ldmatrix4(al, pa + 16 * kLdPRow + 32 * ks);
 #pragma unroll
       for (int j = 0; j < VT; j += 2) {
-        if (j < n_vt) {
+        if (FULL || j < n_vt) {
           uint32_t vb[4];
           ldmatrix4_t(vb, va + (size_t)16 * ks * row_bytes + 16 * j);
           mma_bf16_16816(o[j], ah[0], ah[1], ah[2], ah[3], vb[0], vb[1]);
@@ -436,13 +460,13 @@ __global__ void __launch_bounds__(kLdThreads * HT) latent_decode_kernel(const __
       __nv_bfloat16* dst = p.out + ((size_t)head * p.b.n_seqs + seq) * p.d.c_pad + col0 + 2 * t;
 #pragma unroll
       for (int j = 0; j < VT; ++j)
-        if (j < n_vt) *reinterpret_cast<uint32_t*>(dst + 8 * j) = pack_bf16(o[j][2 * r] * inv, o[j][2 * r + 1] * inv);
+        if (FULL || j < n_vt) *reinterpret_cast<uint32_t*>(dst + 8 * j) = pack_bf16(o[j][2 * r] * inv, o[j][2 * r + 1] * inv);
     } else {
       const size_t at = ((size_t)seq * p.d.heads + head) * p.n_splits + blockIdx.x;
       float* dst = p.part_o + at * p.d.c_pad + col0 + 2 * t;
 #pragma unroll
       for (int j = 0; j < VT; ++j)
-        if (j < n_vt) *reinterpret_cast<float2*>(dst + 8 * j) = make_float2(o[j][2 * r], o[j][2 * r + 1]);
+        if (FULL || j < n_vt) *reinterpret_cast<float2*>(dst + 8 * j) = make_float2(o[j][2 * r], o[j][2 * r + 1]);
       if (warp == 0 && t == 0) {
         p.part_ml[2 * at] = m_run[r];
         p.part_ml[2 * at + 1] = L;
@@ -496,7 +520,9 @@ bool latent_absorb_supported(const LatentDims& d) { return d.c_pad <= 512 && dec
 int launch_latent_decode(tq_ctx* ctx, const LatentDims& d, const RaggedBatch& b, const int* single, float scale, const Rotation& rot, bool rotate,
                          const void* q_lat, const void* q, size_t ldq, const void* cache, void* out) {
   TQ_REQUIRE(ctx, latent_absorb_supported(d), "latent attention: a latent of %d values is too large for the absorbed form", d.rank);
-  const int HT = d.heads > 16 ? 2 : 1, hg = (d.heads + 16 * HT - 1) / (16 * HT);
+  const long long tiles = (b.max_len + kLdTile - 1) / kLdTile;
+  // two head tiles share a CTA's cache tiles unless that leaves the GPU half empty
+  const int HT = d.heads > 16 && (d.heads + 31) / 32 * (tiles + 1) / 2 * b.n_seqs >= ctx->sm_count ? 2 : 1, hg = (d.heads + 16 * HT - 1) / (16 * HT);
   TQ_REQUIRE(ctx, hg <= 65535 && b.n_seqs <= 65535, "latent attention: too many heads or sequences");
   LatentDecodeParams p;
   p.d = d;
@@ -511,12 +537,14 @@ int launch_latent_decode(tq_ctx* ctx, const LatentDims& d, const RaggedBatch& b,
   p.rot = rot;
   p.rotate = rotate;
   p.part_o = p.part_ml = nullptr;
-  // about two CTAs per SM, at least two tiles each
-  const long long tiles = (b.max_len + kLdTile - 1) / kLdTile, ctas = (long long)hg * b.n_seqs;
+  // about two CTAs per SM
+  const long long ctas = (long long)hg * b.n_seqs;
   long long n = (2ll * ctx->sm_count + ctas - 1) / ctas;
-  if (n > (tiles + 1) / 2) n = (tiles + 1) / 2;
+  if (n > tiles) n = tiles;
   if (n > kLdMaxSplits) n = kLdMaxSplits;
-  p.n_splits = n < 1 ? 1 : (int)n;
+  if (n < 1) n = 1;
+  const long long per = (tiles + n - 1) / n;               // (no split without a tile)
+  p.n_splits = (int)((tiles + per - 1) / per);
   if (p.n_splits > 1) {
     const size_t parts = (size_t)b.n_seqs * d.heads * p.n_splits;
     if (int st = ensure_scratch(ctx, parts * (d.c_pad + 2) * sizeof(float))) return st;
@@ -531,9 +559,12 @@ int launch_latent_decode(tq_ctx* ctx, const LatentDims& d, const RaggedBatch& b,
     return TQ_OK;
   };
   int st;
-  if (d.c_pad <= 128) st = HT == 2 ? go(latent_decode_kernel<4, 2>) : go(latent_decode_kernel<4, 1>);
-  else if (d.c_pad <= 256) st = HT == 2 ? go(latent_decode_kernel<8, 2>) : go(latent_decode_kernel<8, 1>);
-  else st = HT == 2 ? go(latent_decode_kernel<16, 2>) : go(latent_decode_kernel<16, 1>);
+  if (d.c_pad <= 128) st = HT == 2 ? go(latent_decode_kernel<4, 2, false>) : go(latent_decode_kernel<4, 1, false>);
+  else if (d.c_pad < 256) st = HT == 2 ? go(latent_decode_kernel<8, 2, false>) : go(latent_decode_kernel<8, 1, false>);
+  else if (d.c_pad == 256) st = HT == 2 ? go(latent_decode_kernel<8, 2, true>) : go(latent_decode_kernel<8, 1, true>);
+  else if (d.c_pad < 512) st = HT == 2 ? go(latent_decode_kernel<16, 2, false>) : go(latent_decode_kernel<16, 1, false>);
+  else if (d.row() == 576) st = HT == 2 ? go(latent_decode_kernel<16, 2, true, 576>) : go(latent_decode_kernel<16, 1, true, 576>);
+  else st = HT == 2 ? go(latent_decode_kernel<16, 2, true>) : go(latent_decode_kernel<16, 1, true>);
   if (st != TQ_OK) return st;
   if (p.n_splits > 1)
     TQ_CUDA(ctx, launch_k(ctx, latent_combine_kernel, dim3((unsigned)d.heads, (unsigned)b.n_seqs), dim3(256), 0, single, b.cache_row, p.n_splits, d.heads, b.n_seqs,

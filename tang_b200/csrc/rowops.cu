@@ -309,8 +309,84 @@ int launch_qk_norm_rope(tq_ctx* ctx, const QkNormRope& a, const RaggedBatch& b, 
 }
 
 // ------------------------------------------------------------------------------------------------ per-head norm, rotation
-// blockIdx.x: row; the CTA's warps (and blockIdx.y's CTAs) share its heads, queries first.  A head passes through its warp's shared
-// memory as f32; the row's cosines and sines are formed once per CTA.
+// blockIdx.x: row; the CTA's warps (and blockIdx.y's CTAs) share its heads, queries first.  The row's cosines and sines are formed
+// once per CTA.  Two forms: a head's 16-byte pieces in the registers of up to 32 lanes, which pass the other half of a pair through
+// shuffles; any size and alignment, the head in its warp's shared memory.
+template <typename T>
+__global__ void __launch_bounds__(256) head_norm_rope_reg_kernel(HeadNormRope a, int lanes, const int* row_pos, const int* cache_row, size_t cache_rows) {
+  extern __shared__ __align__(16) float hr_smem[];
+  constexpr int V = 16 / (int)sizeof(T);
+  const QkNormRope& r = a.r;
+  const int half = r.rot.dims / 2, dim = r.dim, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  float* cs = hr_smem;                                    // [half rounded to 4] cosine, then sine
+  float* sn = hr_smem + (half + 3) / 4 * 4;
+  const int l = lane & (lanes - 1), d0 = l * V, i0 = d0 - r.rot.first, per_warp = 32 / lanes;
+  const bool live = d0 < dim;
+  auto unpack = [](const uint4& u, float (&f)[V]) {
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int j = 0; j < V; ++j) f[j] = V == 4 ? __uint_as_float(w[j & 3]) : bf16_bits_to_float(j & 1 ? w[(j >> 1) & 3] >> 16 : w[(j >> 1) & 3] & 0xFFFFu);
+  };
+  uint4 qg = make_uint4(0u, 0u, 0u, 0u), kg = qg;         // (weights: before the wait)
+  if (live && r.q_gain) qg = *reinterpret_cast<const uint4*>(static_cast<const T*>(r.q_gain) + d0);
+  if (live && r.k_gain) kg = *reinterpret_cast<const uint4*>(static_cast<const T*>(r.k_gain) + d0);
+  pdl_wait();
+  pdl_launch_dependents();
+  const int m = blockIdx.x, crow = cache_row[m];
+  if (crow < 0 || (size_t)crow >= cache_rows) return;
+  const float pos = (float)row_pos[m];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf(pos * r.rot.freq[i], &s, &c);
+    cs[i] = c * r.rot.mult;
+    sn[i] = s * r.rot.mult;
+  }
+  __syncthreads();
+  const bool turns = live && i0 >= 0 && i0 < 2 * half, lead = i0 < half;
+  // this lane's cosines and sines (the same for every head), and where its pairs' other halves are
+  float c[V], s[V];
+  const int other = r.rot.interleaved || !turns ? lane : lead ? lane + half / V : lane - half / V;
+#pragma unroll
+  for (int j = 0; j < V; ++j) {
+    const int p = r.rot.interleaved ? (i0 + j) >> 1 : lead ? i0 + j : i0 + j - half;
+    const bool on = turns && p < half;
+    c[j] = on ? cs[p] : 1.f;
+    s[j] = on ? ((r.rot.interleaved ? !(j & 1) : lead) ? -sn[p] : sn[p]) : 0.f;
+  }
+  const int total = r.heads + r.kv_heads;
+  for (int h0 = (blockIdx.y * warps + warp) * per_warp; h0 < total; h0 += warps * gridDim.y * per_warp) {
+    const int h = h0 + lane / lanes, g = h - r.heads;
+    const bool is_q = h < r.heads, on = live && h < total;
+    const T* src = is_q ? static_cast<const T*>(r.q) + (size_t)m * r.ldq + (size_t)h * a.q_head
+                        : static_cast<const T*>(r.raw) + ((size_t)crow * r.kv_heads + g) * r.raw_pad;
+    T* dst = is_q ? static_cast<T*>(r.q) + (size_t)m * r.ldq + (size_t)h * a.q_head : static_cast<T*>(r.keys) + ((size_t)crow * r.kv_heads + g) * r.key_pad;
+    float f[V];
+    unpack(on ? *reinterpret_cast<const uint4*>(src + d0) : make_uint4(0u, 0u, 0u, 0u), f);
+    if (is_q ? r.q_gain != nullptr : r.k_gain != nullptr) {
+      float sq = 0.f, gf[V];
+#pragma unroll
+      for (int j = 0; j < V; ++j) sq += f[j] * f[j];
+      for (int o = lanes / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      const float inv = 1.0f / sqrtf(sq / (float)dim + r.eps);
+      unpack(is_q ? qg : kg, gf);
+#pragma unroll
+      for (int j = 0; j < V; ++j) f[j] *= inv * gf[j];
+    }
+    float out[V];
+    if (r.rot.interleaved) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) out[j] = f[j] * c[j] + f[j ^ 1] * s[j];
+    } else {
+#pragma unroll
+      for (int j = 0; j < V; ++j) out[j] = f[j] * c[j] + __shfl_sync(0xffffffffu, f[j], other) * s[j];
+    }
+    if (on) {
+#pragma unroll
+      for (int j = 0; j < V; j += 4) ro_store4(dst + d0 + j, make_float4(out[j], out[j + 1], out[j + 2], out[j + 3]));
+    }
+  }
+}
+
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) head_norm_rope_kernel(HeadNormRope a, const int* row_pos, const int* cache_row, size_t cache_rows) {
   extern __shared__ __align__(16) float hr_smem[];
@@ -384,11 +460,17 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(HeadNormRope a, con
 int launch_head_norm_rope(tq_ctx* ctx, const HeadNormRope& a0, const RaggedBatch& b, int dtype) {
   HeadNormRope a = a0;
   if (!a.q_head) a.q_head = (size_t)a.r.dim;
-  const QkNormRope& r = a.r;
+  QkNormRope& r = a.r;
   TQ_REQUIRE(ctx, r.heads >= 0 && r.kv_heads >= 0 && r.heads + r.kv_heads > 0 && r.dim > 0 && r.rot.first >= 0 && r.rot.dims >= 0 && r.rot.dims % 2 == 0 &&
                       r.rot.first + r.rot.dims <= r.dim,
              "head norm: the rotated dimensions must be even and inside the head");
   if (b.rows == 0) return TQ_OK;
+  if (!r.q_gain && r.kv_heads == 0) {          // only what turns is touched
+    if (r.rot.dims == 0) return TQ_OK;
+    r.q = static_cast<char*>(r.q) + (size_t)r.rot.first * dtype_size(dtype);
+    r.dim = r.rot.dims;
+    r.rot.first = 0;
+  }
   const int total = r.heads + r.kv_heads;
   int warps = total < 8 ? total : 8;
   const size_t smem = ((size_t)r.rot.dims + 3 + (size_t)warps * ((r.dim + 3) / 4 * 4)) * sizeof(float);
@@ -403,6 +485,20 @@ int launch_head_norm_rope(tq_ctx* ctx, const HeadNormRope& a0, const RaggedBatch
   const int v = dtype == TQ_F32 ? 4 : 8;
   const uintptr_t bits = (uintptr_t)r.q | (uintptr_t)r.raw | (uintptr_t)r.keys;
   const bool vec = r.dim % v == 0 && r.ldq % v == 0 && a.q_head % v == 0 && r.raw_pad % v == 0 && r.key_pad % v == 0 && (bits & 15) == 0;
+  const bool gains = (((uintptr_t)r.q_gain | (uintptr_t)r.k_gain) & 15) == 0 && (r.kv_heads == 0 || !r.q_gain == !r.k_gain);
+  if (vec && gains && r.dim / v <= 32 && r.rot.first % v == 0 && (r.rot.interleaved || r.rot.dims % (2 * v) == 0)) {
+    int lanes = 1;
+    while (lanes < r.dim / v) lanes *= 2;
+    const int units = (total + 32 / lanes - 1) / (32 / lanes), w = units < 8 ? units : 8;      // warps of heads
+    int y = 1;
+    while (y * w < units && (long long)b.rows * y < 2ll * ctx->sm_count) ++y;
+    const size_t cs = ((size_t)r.rot.dims + 8) * sizeof(float);
+    auto reg = [&](auto kern) -> int {
+      TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)b.rows, (unsigned)y), dim3((unsigned)(32 * w)), cs, a, lanes, b.row_pos, b.cache_row, b.cache_rows));
+      return TQ_OK;
+    };
+    return dtype == TQ_F32 ? reg(head_norm_rope_reg_kernel<float>) : reg(head_norm_rope_reg_kernel<__nv_bfloat16>);
+  }
   if (dtype == TQ_F32) return vec ? go(head_norm_rope_kernel<float, true>) : go(head_norm_rope_kernel<float, false>);
   return vec ? go(head_norm_rope_kernel<__nv_bfloat16, true>) : go(head_norm_rope_kernel<__nv_bfloat16, false>);
 }
