@@ -18,7 +18,7 @@
 #include <vector>
 
 #include "dense.cuh"
-#include "expert_route.cuh"
+#include "expert_ff.cuh"
 #include "gla.cuh"
 #include "latent_attention.cuh"
 #include "ragged.h"
@@ -726,7 +726,7 @@ static int feed_forward(tq_dotanex* m, const Layer& W, size_t rows, StreamMix& m
   tq_ctx* ctx = m->ctx;
   const tq_dotanex_layer& c = W.c;
   const int dt = m->cfg.dtype, f32 = dt == TQ_F32;
-  const size_t es = dtype_size(dt), width = m->cfg.width, hn_ld = m->embed->kpad;
+  const size_t width = m->cfg.width, hn_ld = m->embed->kpad;
   DenseInput in;
   in.x = m->hn;
   in.ldx = hn_ld;
@@ -743,54 +743,39 @@ static int feed_forward(tq_dotanex* m, const Layer& W, size_t rows, StreamMix& m
     mix.y = m->y;
     return launch_dense(ctx, W.down, a, rows, d);
   }
-  const size_t pairs = rows * c.top, all = (size_t)c.experts + c.identity;
-  DenseEpilogue f;
-  dense_section(f, W.shared0, all, DENSE_ROW, 1, m->logits, m->max_experts);
-  if (c.shared_ff) dense_section(f, W.front->rpad, c.shared_ff, DENSE_GLU, f32, m->shared, m->shared_ld);
-  f.glu_limit = c.shared_limit;
-  f.glu_alpha = kGluAlpha;
-  TQ_STEP(launch_dense(ctx, W.front, in, rows, f));
-  DenseGroups g;
-  g.jobs = m->route.jobs;
-  g.n_jobs = m->route.n_jobs;
-  g.chunk = dense_group_chunk(dt, W.gate_up->kpad > W.down->kpad ? W.gate_up->kpad : W.down->kpad, pairs * c.experts / all + 1, c.experts);
-  g.max_jobs = (int)route_max_jobs(pairs, c.experts, g.chunk);
-  // the tcgen05 kernel copies boxes of consecutive rows, the others follow the slots' row numbers
-  const bool gather = !f32 && g.chunk > 8;
-  RouteRule rule;
-  rule.score = ROUTE_SOFTMAX;
-  rule.renorm = true;
-  rule.correction = W.correction;
-  rule.identity = (int)c.identity;
-  TQ_STEP(launch_route(ctx, m->logits, m->max_experts, rows, all, c.top, rule, g.chunk, m->route, m->hn, hn_ld * es, up8(width) * es,
-                       gather ? m->gathered : nullptr, hn_ld * es));
-  DenseEpilogue u;
-  dense_section(u, W.gu_rows, c.ff, DENSE_GLU, f32, m->act, m->act_ld);
-  u.glu_limit = c.limit;
-  u.glu_alpha = kGluAlpha;
-  g.group_rows = W.gu_rows;
-  g.x_rows = gather ? nullptr : m->route.slot_row;
-  TQ_STEP(launch_dense_grouped(ctx, W.gate_up, gather ? m->gathered : m->hn, hn_ld, pairs, g, u));
-  DenseEpilogue d;
-  dense_section(d, W.down_rows, width, DENSE_ROW, 1, m->yp, width);
-  g.group_rows = W.down_rows;
-  g.x_rows = nullptr;
-  TQ_STEP(launch_dense_grouped(ctx, W.down, m->act, m->act_ld, pairs, g, d));
-  if (c.shared_ff) {
-    DenseInput s;
-    s.x = m->shared;
-    s.ldx = m->shared_ld;
-    DenseEpilogue y;
-    dense_section(y, W.shared_down->rpad, width, DENSE_ROW, 1, m->ys, width);
-    TQ_STEP(launch_dense(ctx, W.shared_down, s, rows, y));
-    mix.y_more = m->ys;
-  }
-  mix.y = m->yp;
-  mix.y_rows = m->route.slot;
-  mix.y_weight = m->route.weight;
-  mix.n_y = (int)c.top;
-  mix.self = m->hn;
-  return TQ_OK;
+  ExpertFf f;
+  f.front = W.front;
+  f.gate_up = W.gate_up;
+  f.down = W.down;
+  f.shared_down = W.shared_down;
+  f.logits = (size_t)c.experts + c.identity;
+  f.logit_end = W.shared0;
+  f.experts = c.experts;
+  f.identity = c.identity;
+  f.top = c.top;
+  f.ff = c.ff;
+  f.shared_ff = c.shared_ff;
+  f.gu_rows = W.gu_rows;
+  f.down_rows = W.down_rows;
+  f.rule.score = ROUTE_SOFTMAX;
+  f.rule.renorm = true;
+  f.rule.correction = W.correction;
+  f.rule.identity = (int)c.identity;
+  f.limit = c.limit;
+  f.alpha = kGluAlpha;
+  f.shared_limit = c.shared_limit;
+  ExpertBuffers b;
+  b.logits = m->logits;
+  b.ld_logits = m->max_experts;
+  b.route = m->route;
+  b.gathered = m->gathered;
+  b.act = m->act;
+  b.act_ld = m->act_ld;
+  b.shared = m->shared;
+  b.shared_ld = m->shared_ld;
+  b.y = m->yp;
+  b.y_shared = m->ys;
+  return launch_expert_ff(ctx, f, b, m->hn, hn_ld, rows, width, dt, mix);
 }
 
 extern "C" int tq_dotanex_step(tq_dotanex* m, const int* token_ids_dev, size_t rows, const int* seq_rows_dev, const int* starts_dev, const int* slots_dev,
