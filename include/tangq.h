@@ -569,6 +569,15 @@ TQ_API int tq_stream_mix(tq_ctx* ctx, size_t streams, size_t src_streams, const 
                          const float* y_more_dev_or_null, const float* mix_dev_or_null, const float* w_out_dev_or_null, const float* w_in_dev_or_null,
                          const float* gain_dev_or_null, size_t rows, size_t width, float eps, void* out_dev_or_null, int out_dtype, size_t ld_out,
                          float* sum_dev_or_null);
+/* One stream with what a step of one row per sequence needs beside that: x' = src + w_out y, where row m of y_more is multiplied by
+ * sigmoid(y_more_gate[m * ld_gate]); sum = x'; x' += inject row m (NULL: nothing); dst = x'; h = rms_norm(x') * gain, rounded to
+ * out_dtype; out = h + conv(h) with conv_w [taps][width] f32 and conv_state [slots][taps - 1][width] of out_dtype, moved on by the row
+ * (conv_w NULL: out = h).  mix_one_dev: the value 1. */
+TQ_API int tq_stream_step(tq_ctx* ctx, const float* src_dev, float* dst_dev, const float* y_dev, const int* y_rows_dev_or_null,
+                          const float* y_weight_dev_or_null, size_t n_y, const float* y_more_dev_or_null, const float* y_more_gate_dev_or_null, size_t ld_gate,
+                          const float* inject_dev_or_null, const float* mix_one_dev, const float* w_out_dev, const float* gain_dev, size_t rows, size_t width,
+                          float eps, const float* conv_w_dev_or_null, void* conv_state_dev_or_null, size_t taps, size_t max_seq, const int* row_pos_dev,
+                          const int* cache_row_dev, void* out_dev, int out_dtype, size_t ld_out, float* sum_dev_or_null);
 /* Grouped-query attention: s = (q . k) scale, softcap * tanh(s / softcap) unless softcap is 0; weights
  * exp(s_j) / (exp(sink) + sum exp(s)) (sink -infinity: none); the query at position i sees j when 0 <= i - j < window; the
  * result times sigmoid(gate).  q [rows][ldq], gate (may be NULL) [rows][ldg], caches as in tq_diff_attention with one map. */
@@ -586,6 +595,44 @@ TQ_API int tq_window_attention_sinks(tq_ctx* ctx, const tq_window_attn_config* c
                                      size_t ldq, const void* gate_dev_or_null, size_t ldg, const void* k_cache_dev, const void* v_cache_dev,
                                      size_t cache_rows, const int* seq_rows_dev_or_null, const int* row_pos_dev, const int* cache_row_dev,
                                      size_t n_seqs, size_t rows, size_t max_q, size_t max_len, void* out_dev, size_t ldo);
+/* The same with one key and one value for each block of `pool` tokens that lies wholly before the window (0: none): the query at
+ * position i sees block b too when b pool + pool - 1 <= i - window, under the same softmax.  Pooled rows have the layout of the cache
+ * rows; block b of a slot is row slot * pool_rows + b, and a slot has max_seq cache rows.  The result is multiplied by out_scale. */
+TQ_API int tq_window_attention_pooled(tq_ctx* ctx, const tq_window_attn_config* cfg, const float* sinks_dev_or_null, int dtype, const void* q_dev,
+                                      size_t ldq, const void* gate_dev_or_null, size_t ldg, const void* k_cache_dev, const void* v_cache_dev,
+                                      size_t cache_rows, size_t pool, const void* pooled_keys_dev_or_null, const void* pooled_values_dev_or_null,
+                                      size_t pool_rows, size_t max_seq, float out_scale, const int* seq_rows_dev_or_null, const int* row_pos_dev,
+                                      const int* cache_row_dev, size_t n_seqs, size_t rows, size_t max_q, size_t max_len, void* out_dev, size_t ldo);
+/* Short causal convolutions per channel, y_t = sum_j w[j] u_(t - taps + 1 + j), zeros before a sequence's position 0.  w [taps][channels]
+ * f32; state [slots][taps - 1][channels] of `dtype` holds a slot's last inputs (slot = cache_row / max_seq) and is moved on by the
+ * step's rows.
+ * tq_conv_residual: out = x + conv(x), in another buffer. */
+TQ_API int tq_conv_residual(tq_ctx* ctx, int dtype, size_t channels, size_t taps, const float* w_dev, void* state_dev, size_t max_seq, size_t cache_rows,
+                            const void* x_dev, size_t ldx, const int* seq_rows_dev_or_null, const int* row_pos_dev, const int* cache_row_dev, size_t n_seqs,
+                            size_t rows, size_t max_q, size_t max_len, void* out_dev, size_t ldo);
+/* tq_conv_heads: rows of raw queries (heads * dim at column 0), keys (kv_heads * dim at k0) and values (kv_heads * vdim at v0).
+ * All are convolved (channels: the raw columns; w NULL: not); queries and keys are rotated (first rot_dims dimensions, in halves, freq
+ * [rot_dims / 2], cos and sin times rot_mult) and, if norm, divided by their root mean square per head.  Queries go to q, keys and
+ * values to the row's cache row ([kv_heads][dim or vdim padded to 8], zero padding).  pool > 0: the means of blocks of `pool` keys and
+ * values are left in the pooled rows (as in tq_window_attention_pooled) as soon as a later row can need them. */
+typedef struct tq_conv_heads_config {
+  uint32_t heads, kv_heads, dim, vdim;
+  uint32_t k0, v0, channels, taps;
+  uint32_t rot_dims;
+  int norm;
+  uint32_t pool, pool_rows;
+  float rot_mult, eps;
+} tq_conv_heads_config;
+TQ_API int tq_conv_heads(tq_ctx* ctx, const tq_conv_heads_config* cfg, int dtype, const void* raw_dev, size_t ld, const float* w_dev_or_null,
+                         void* state_dev_or_null, const float* freq_dev_or_null, size_t max_seq, size_t cache_rows, const int* seq_rows_dev_or_null,
+                         const int* row_pos_dev, const int* cache_row_dev, size_t n_seqs, size_t rows, size_t max_q, size_t max_len, void* q_dev,
+                         size_t ldq, void* keys_dev, void* values_dev, void* pooled_keys_dev_or_null, void* pooled_values_dev_or_null);
+/* minGRU, per channel: z = sigmoid(z_t + z_bias), u = u_t + u_bias, S_t = (1 - z) S_(t-1) + z (u >= 0 ? u + 1/2 : sigmoid(u)),
+ * out_t = S_t silu(gate_t) out_scale.  Rows of z, u and gate are `ld` elements apart (even, as ldo); biases and state [slots][width
+ * rounded up to 2] are f32; slot = cache_row / max_seq; a sequence's position 0 starts from zero. */
+TQ_API int tq_min_gru(tq_ctx* ctx, int dtype, size_t width, const void* z_dev, const void* u_dev, const void* gate_dev, size_t ld, const float* z_bias_dev,
+                      const float* u_bias_dev, float out_scale, float* state_dev, size_t max_seq, size_t cache_rows, const int* seq_rows_dev_or_null,
+                      const int* row_pos_dev, const int* cache_row_dev, size_t n_seqs, size_t rows, size_t max_q, void* out_dev, size_t ldo);
 /* Gated linear attention: S_t = diag(alpha_t) S_(t-1) + k_t v_t^T, o_t = S_t^T (q_scale q_t), per head, with
  * alpha_t = sigmoid(a2 a1_t + bias)^(1/tau) per key channel; out = o / sqrt(mean(o^2) + eps) * norm * silu(gate).  Rows of q, k
  * (heads * dim), v, gate (heads * vdim) are `ld` elements apart, a1 [rows][ld_a1] and everything about the state is f32.
@@ -621,6 +668,10 @@ TQ_API int tq_route(tq_ctx* ctx, const float* logits_dev, size_t rows, size_t ex
 TQ_API int tq_route_rule(tq_ctx* ctx, const float* logits_dev, size_t rows, size_t experts, size_t top, int score, int renorm,
                          const float* correction_dev_or_null, size_t identity, size_t chunk, int* expert_dev, float* weight_dev, int* slot_dev,
                          int* slot_row_dev, int* jobs_dev, int* n_jobs_dev);
+/* The same with rows of logits `ld` apart and a bias [experts] (NULL: 0) that is part of the logits. */
+TQ_API int tq_route_biased(tq_ctx* ctx, const float* logits_dev, size_t ld, size_t rows, size_t experts, size_t top, int score, int renorm,
+                           const float* bias_dev_or_null, const float* correction_dev_or_null, size_t identity, size_t chunk, int* expert_dev,
+                           float* weight_dev, int* slot_dev, int* slot_row_dev, int* jobs_dev, int* n_jobs_dev);
 
 /* ---- Numuzen ------------------------------------------------------------------------------------
  * No reference counterpart.  A decoder with a norm before and after every sublayer (weights stored around zero),
@@ -717,6 +768,55 @@ TQ_API int tq_dotanex_step(tq_dotanex* model, const int* token_ids_dev, size_t r
                            size_t n_logits, float* logits_dev);
 /* While set, every step also leaves the sum of the streams after each layer in sums [n_layers][rows][width] (NULL turns it off). */
 TQ_API int tq_dotanex_trace(tq_dotanex* model, float* sums_dev_or_null);
+
+/* ---- Sakinex ------------------------------------------------------------------------------------
+ * No reference counterpart.  A decoder with one residual stream, x <- x + residual_mult * sublayer(h), h = n + conv(n), n = norm(x),
+ * whose mixer runs two branches side by side on the same h,
+ *   mixer = left_scale * attention(h) + right_scale * recurrence(h),
+ * attention with short convolutions on queries, keys and values, YaRN rotation in halves, a gainless query/key norm per head behind
+ * it, a sliding window and pooled blocks before the window (tq_conv_heads, tq_window_attention_pooled), and a minGRU (tq_min_gru).
+ * Its feed-forward has experts routed by biased logits and weighed by a softmax over the chosen ones, and a shared expert behind a
+ * sigmoid gate; all of the SiLU form.  An entry of `layers` is a run of a layer: runs that repeat another's weights (weights_of)
+ * have caches and states of their own, and add_embedding adds the embedding output to the stream ahead of the run.  The model owns
+ * weights, caches, states (one slot per sequence) and workspaces.  dtype TQ_BF16: bf16 weights, activations, caches and convolution
+ * inputs; stream, norms, scores, router, recurrence f32; TQ_F32: everything f32. */
+typedef struct tq_sakinex tq_sakinex;
+typedef struct tq_sakinex_config {
+  uint32_t n_layers, width, vocab;
+  uint32_t taps;           /* of the convolution on a sublayer's input */
+  uint32_t max_seq;        /* positions per slot */
+  uint32_t max_slots;
+  int dtype;
+  float eps, residual_mult;
+} tq_sakinex_config;
+typedef struct tq_sakinex_layer {
+  int weights_of;                        /* -1: tensors of its own; else the rest equals that run's, but for add_embedding */
+  int add_embedding;
+  uint32_t heads, kv_heads, dim, vdim;   /* attention */
+  uint32_t window, pool;                 /* pool = 0: no pooled blocks */
+  uint32_t taps, rot_dims;               /* taps = 0: no convolution on queries, keys and values */
+  uint32_t state_width;                  /* recurrence */
+  uint32_t experts, top, ff, shared_ff;  /* experts = 0: no feed-forward; shared_ff = 0: no shared expert */
+  float scale, left_scale, right_scale;
+  double rot_base, rot_factor, rot_original, rot_fast, rot_slow;   /* rot_factor = 0: no scaling */
+} tq_sakinex_layer;
+typedef enum tq_sakinex_tensor {
+  TQ_SX_EMBED = 0, TQ_SX_FINAL_NORM = 1, TQ_SX_HEAD = 2, TQ_SX_NORM1 = 3, TQ_SX_NORM2 = 4, TQ_SX_CANON1 = 5, TQ_SX_CANON2 = 6, TQ_SX_Q = 7, TQ_SX_K = 8,
+  TQ_SX_V = 9, TQ_SX_Q_CONV = 10, TQ_SX_K_CONV = 11, TQ_SX_V_CONV = 12, TQ_SX_LEFT_O = 13, TQ_SX_Z = 14, TQ_SX_Z_BIAS = 15, TQ_SX_X = 16, TQ_SX_X_BIAS = 17,
+  TQ_SX_G = 18, TQ_SX_RIGHT_O = 19, TQ_SX_ROUTER = 20, TQ_SX_ROUTER_BIAS = 21, TQ_SX_GATE = 22, TQ_SX_UP = 23, TQ_SX_DOWN = 24, TQ_SX_SHARED_GATE = 25,
+  TQ_SX_SHARED_UP = 26, TQ_SX_SHARED_DOWN = 27, TQ_SX_SHARED_SWITCH = 28
+} tq_sakinex_tensor;
+TQ_API int tq_sakinex_create(tq_ctx* ctx, const tq_sakinex_config* cfg, const tq_sakinex_layer* layers, tq_sakinex** out);
+TQ_API int tq_sakinex_destroy(tq_sakinex* model);
+/* As tq_tofazen_put; `expert` counts for gate, up and down of routed experts; convolutions are [channels, taps].  Runs with weights_of
+ * take none. */
+TQ_API int tq_sakinex_put(tq_sakinex* model, int tensor, size_t layer, size_t expert, const void* src, int src_dtype, size_t rows, size_t cols);
+/* As tq_numuzen_step. */
+TQ_API int tq_sakinex_step(tq_sakinex* model, const int* token_ids_dev, size_t rows, const int* seq_rows_dev_or_null, const int* starts_dev,
+                           const int* slots_dev_or_null, size_t n_seqs, size_t max_q, size_t max_len, const int* logit_rows_dev_or_null,
+                           size_t n_logits, float* logits_dev);
+/* While set, every step also leaves the stream after each run in streams [n_layers][rows][width] (NULL turns it off). */
+TQ_API int tq_sakinex_trace(tq_sakinex* model, float* streams_dev_or_null);
 
 /* ---- CUDA graphs ------------------------------------------------------------------------------
  * CudaComputeDevice::begin_capture / end_capture (crates/tang-compute/src/cuda.rs:344-356): every

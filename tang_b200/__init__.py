@@ -12,8 +12,9 @@ from .engine import Engine
 from .registry import load_model
 from .dotanex import DotanexConfig, DotanexModel
 from .numuzen import NumuzenConfig, NumuzenModel
+from .sakinex import SakinexConfig, SakinexModel
 from .tofazen import TofazenConfig, TofazenModel
 from .moe import MoeConfig, MoeLayer, moe_router
 
-__all__ = ["Engine", "load_model", "TofazenConfig", "TofazenModel", "NumuzenConfig", "NumuzenModel", "DotanexConfig", "DotanexModel", "read_safetensors", "write_safetensors", "quantize_linear", "TensorView", "SafetensorsError", "SamplerConfig", "mla_decode", "MlaLayer", "MlaConfig", "MoeLayer", "MoeConfig", "moe_router", "LlamaModel", "LlamaConfig", "LlamaLayerWeights", "Comm", "Graph", "QuantComputeDevice", "QuantizedQ4", "QuantizedQ8", "Buffer", "QBuffer", "TangqError", "load",
+__all__ = ["Engine", "load_model", "TofazenConfig", "TofazenModel", "NumuzenConfig", "NumuzenModel", "DotanexConfig", "DotanexModel", "SakinexConfig", "SakinexModel", "read_safetensors", "write_safetensors", "quantize_linear", "TensorView", "SafetensorsError", "SamplerConfig", "mla_decode", "MlaLayer", "MlaConfig", "MoeLayer", "MoeConfig", "moe_router", "LlamaModel", "LlamaConfig", "LlamaLayerWeights", "Comm", "Graph", "QuantComputeDevice", "QuantizedQ4", "QuantizedQ8", "Buffer", "QBuffer", "TangqError", "load",
            "F32", "BF16", "F16", "I8", "U8", "I32", "F64", "Q4_F32", "Q4_F16", "Q8_F32", "I8_ROW"]

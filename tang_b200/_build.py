@@ -22,7 +22,8 @@ NVCC_FLAGS = [
 # sources of the partial libraries (name -> csrc/*.cu stems)
 COMPONENTS = {
     "dense": ["api_core", "graph", "ops", "sampler", "dense", "rowops", "expert_route", "diff_attention",
-              "window_attention", "gla", "gla_chunk", "lightning", "stream_mix", "latent_attention", "tofazen", "numuzen", "dotanex"],
+              "window_attention", "gla", "gla_chunk", "lightning", "stream_mix", "latent_attention", "short_conv", "min_gru", "expert_ff",
+              "tofazen", "numuzen", "dotanex", "sakinex"],
 }
 
 

@@ -119,6 +119,11 @@ PROTOTYPES = {
     "tq_qk_norm_rope": (_i, [_p, _i, _sz, _sz, _sz, _p, _sz, _p, _p, _sz, _p, _p, _sz, _p, C.c_float, C.c_float, _p, _p, _sz]),
     "tq_window_attention": (_i, [_p, _p, _i, _p, _sz, _p, _sz, _p, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _sz, _p, _sz]),
     "tq_window_attention_sinks": (_i, [_p, _p, _p, _i, _p, _sz, _p, _sz, _p, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _sz, _p, _sz]),
+    "tq_window_attention_pooled": (_i, [_p, _p, _p, _i, _p, _sz, _p, _sz, _p, _p, _sz, _sz, _p, _p, _sz, _sz, C.c_float, _p, _p, _p, _sz, _sz, _sz, _sz, _p, _sz]),
+    "tq_conv_residual": (_i, [_p, _i, _sz, _sz, _p, _p, _sz, _sz, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _sz, _p, _sz]),
+    "tq_conv_heads": (_i, [_p, _p, _i, _p, _sz, _p, _p, _p, _sz, _sz, _p, _p, _p, _sz, _sz, _sz, _sz, _p, _sz, _p, _p, _p, _p]),
+    "tq_min_gru": (_i, [_p, _i, _sz, _p, _p, _p, _sz, _p, _p, C.c_float, _p, _sz, _sz, _p, _p, _p, _sz, _sz, _sz, _p, _sz]),
+    "tq_stream_step": (_i, [_p, _p, _p, _p, _p, _p, _sz, _p, _p, _sz, _p, _p, _p, _p, _sz, _sz, C.c_float, _p, _p, _sz, _sz, _p, _p, _p, _i, _sz, _p]),
     "tq_head_norm_rope": (_i, [_p, _i, _sz, _sz, _sz, _p, _sz, _sz, _p, _p, _sz, _p, _p, _sz, _sz, _i, _p, C.c_float, C.c_float, _p, _p, _sz]),
     "tq_banded_frequencies": (_i, [_sz] + [C.c_double] * 5 + [_p]),
     "tq_stream_mix": (_i, [_p, _sz, _sz, _p, _p, _p, _p, _p, _sz, _p, _p, _p, _p, _p, _p, _sz, _sz, C.c_float, _p, _i, _sz, _p]),
@@ -127,6 +132,7 @@ PROTOTYPES = {
     "tq_latent_decode": (_i, [_p, _sz, _sz, _sz, _sz, C.c_float, _sz, _p, C.c_float, _i, _p, _p, _sz, _p, _sz, _p, _p, _sz, _sz, _p]),
     "tq_route": (_i, [_p, _p, _sz, _sz, _sz, _i, _i, _sz, _p, _p, _p, _p, _p, _p]),
     "tq_route_rule": (_i, [_p, _p, _sz, _sz, _sz, _i, _i, _p, _sz, _sz, _p, _p, _p, _p, _p, _p]),
+    "tq_route_biased": (_i, [_p, _p, _sz, _sz, _sz, _sz, _i, _i, _p, _p, _sz, _sz, _p, _p, _p, _p, _p, _p]),
     "tq_numuzen_create": (_i, [_p, _p, _p, _pp]),
     "tq_numuzen_destroy": (_i, [_p]),
     "tq_numuzen_put": (_i, [_p, _i, _sz, _sz, _p, _i, _sz, _sz]),
@@ -138,6 +144,11 @@ PROTOTYPES = {
     "tq_dotanex_put": (_i, [_p, _i, _sz, _sz, _p, _i, _sz, _sz]),
     "tq_dotanex_step": (_i, [_p, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _p, _sz, _p]),
     "tq_dotanex_trace": (_i, [_p, _p]),
+    "tq_sakinex_create": (_i, [_p, _p, _p, _pp]),
+    "tq_sakinex_destroy": (_i, [_p]),
+    "tq_sakinex_put": (_i, [_p, _i, _sz, _sz, _p, _i, _sz, _sz]),
+    "tq_sakinex_step": (_i, [_p, _p, _sz, _p, _p, _p, _sz, _sz, _sz, _p, _sz, _p]),
+    "tq_sakinex_trace": (_i, [_p, _p]),
     "tq_graph_begin": (_i, [_p]),
     "tq_graph_end": (_i, [_p, _pp]),
     "tq_graph_launch": (_i, [_p, _p]),

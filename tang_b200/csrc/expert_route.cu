@@ -23,7 +23,7 @@ __device__ __forceinline__ void choose_experts(const float* z, int experts, int 
 #pragma unroll
   for (int j = 0; j < NR; ++j) {
     const int e = lane + 32 * j;
-    v[j] = e < experts ? z[e] : -INFINITY;
+    v[j] = e < experts ? z[e] + (rule.bias ? rule.bias[e] : 0.f) : -INFINITY;
   }
   float mx = -INFINITY, sum = 0.f;
   if (score == ROUTE_SOFTMAX) {
@@ -242,8 +242,15 @@ using namespace tq;
 extern "C" int tq_route_rule(tq_ctx* ctx, const float* logits_dev, size_t rows, size_t experts, size_t top, int score, int renorm,
                              const float* correction_dev, size_t identity, size_t chunk, int* expert_dev, float* weight_dev, int* slot_dev,
                              int* slot_row_dev, int* jobs_dev, int* n_jobs_dev) {
+  return tq_route_biased(ctx, logits_dev, experts, rows, experts, top, score, renorm, nullptr, correction_dev, identity, chunk, expert_dev, weight_dev, slot_dev,
+                         slot_row_dev, jobs_dev, n_jobs_dev);
+}
+
+extern "C" int tq_route_biased(tq_ctx* ctx, const float* logits_dev, size_t ld, size_t rows, size_t experts, size_t top, int score, int renorm, const float* bias_dev,
+                               const float* correction_dev, size_t identity, size_t chunk, int* expert_dev, float* weight_dev, int* slot_dev,
+                               int* slot_row_dev, int* jobs_dev, int* n_jobs_dev) {
   if (int st = bind(ctx)) return st;
-  TQ_REQUIRE(ctx, score == ROUTE_SIGMOID || score == ROUTE_SOFTMAX, "tq_route: unknown score");
+  TQ_REQUIRE(ctx, (score == ROUTE_SIGMOID || score == ROUTE_SOFTMAX) && ld >= experts, "tq_route: unknown score, or rows of logits that overlap");
   if (rows == 0) return TQ_OK;
   TQ_REQUIRE(ctx, logits_dev && expert_dev && weight_dev && slot_dev && slot_row_dev && jobs_dev && n_jobs_dev, "tq_route: null pointer");
   const size_t pairs = rows * top;
@@ -263,9 +270,10 @@ extern "C" int tq_route_rule(tq_ctx* ctx, const float* logits_dev, size_t rows, 
   RouteRule rule;
   rule.score = score;
   rule.renorm = renorm != 0;
+  rule.bias = bias_dev;
   rule.correction = correction_dev;
   rule.identity = (int)identity;
-  return launch_route(ctx, logits_dev, experts, rows, experts, top, rule, chunk, r, nullptr, 0, 0, nullptr, 0);
+  return launch_route(ctx, logits_dev, ld, rows, experts, top, rule, chunk, r, nullptr, 0, 0, nullptr, 0);
 }
 
 extern "C" int tq_route(tq_ctx* ctx, const float* logits_dev, size_t rows, size_t experts, size_t top, int score, int renorm, size_t chunk,

@@ -9,13 +9,14 @@ namespace tq {
 
 enum RouteScore : int { ROUTE_SIGMOID = 0, ROUTE_SOFTMAX = 1 };
 
-// How a row's experts are chosen and weighed.  Scores are sigmoid(logit), or softmax over all experts.  The `top` experts with
+// How a row's experts are chosen and weighed.  The bias is part of the logits.  Scores are sigmoid(logit), or softmax over all experts.  The `top` experts with
 // the largest logits -- with a correction, the largest score + correction[expert] -- are chosen (the lower index among equals);
 // weights are the scores, divided by their sum if `renorm`.  The last `identity` of the experts have no weights: their pairs
 // take no slot.
 struct RouteRule {
   int score = ROUTE_SIGMOID;
   bool renorm = false;
+  const float* bias = nullptr;         // [experts]; null: 0
   const float* correction = nullptr;
   int identity = 0;
 };

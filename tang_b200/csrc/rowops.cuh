@@ -59,7 +59,8 @@ int launch_head_norm_rope(tq_ctx* ctx, const HeadNormRope& a, const RaggedBatch&
 // Hyper-connections: `streams` residual rows per row of the batch.
 //     x'_t = sum_s mix[s][t] x_s + w_out[t] y;   u = sum_s w_in[s] x'_s;   out = u / rms(u) * gain
 // y gathers a sublayer's output: the weighted rows of its chosen experts (a negative row: the sublayer's own input, `self`) and
-// one more row.
+// one more row, multiplied by a sigmoid if there is a gate.
+// Steps of one row per sequence may add a short convolution: out <- out + conv(out), whose states move on by the row.
 constexpr int kMaxStreams = 16;
 struct StreamMix {
   int streams = 1, src_streams = 1;
@@ -72,6 +73,9 @@ struct StreamMix {
   int n_y = 1;
   const void* self = nullptr;        // of out_dtype, ld_out; may be out
   const float* y_more = nullptr;
+  const float* y_more_gate = nullptr;   // row m's logit at m * ld_gate; null: no gate
+  size_t ld_gate = 0;
+  const float* inject = nullptr;     // [rows][width], added to every x' after `sum`; with y
   const float *mix = nullptr, *w_out = nullptr, *w_in = nullptr;   // w_in null: ones
   const float* gain = nullptr;       // null: no norm, no out
   void* out = nullptr;
@@ -79,6 +83,10 @@ struct StreamMix {
   size_t ld_out = 0;
   float eps = 0.f;
   float* sum = nullptr;              // [rows][width] sum of the streams
+  const float* conv_w = nullptr;     // [conv_taps][width]; null: no convolution
+  void* conv_state = nullptr;        // [slots][conv_taps - 1][width] of out_dtype
+  int conv_taps = 0, max_seq = 1;    // cache rows per slot
+  const int *row_pos = nullptr, *cache_row = nullptr;   // of the convolution
 };
 int launch_stream_mix(tq_ctx* ctx, const StreamMix& a, size_t rows, size_t width);
 

@@ -53,6 +53,29 @@ __device__ __forceinline__ void sm_store(__nv_bfloat16* p, const SmVec<V>& r) {
   }
 }
 
+template <int S, int V>
+__device__ __forceinline__ SmVec<V> sm_sum(const SmVec<V> (&x)[S], int n) {
+  SmVec<V> r;
+#pragma unroll
+  for (int j = 0; j < V; ++j) r.v[j] = 0.f;
+#pragma unroll
+  for (int s = 0; s < S; ++s)
+    if (s < n) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) r.v[j] += x[s].v[j];
+    }
+  return r;
+}
+
+// The value of an output type, as the next reader of a stored vector sees it.
+template <typename OT, int V>
+__device__ __forceinline__ void sm_round(SmVec<V>& r) {
+  if constexpr (sizeof(OT) == 2) {
+#pragma unroll
+    for (int j = 0; j < V; ++j) r.v[j] = __bfloat162float(__float2bfloat16_rn(r.v[j]));
+  }
+}
+
 // One CTA per row; a thread owns V columns at a time in every stream, so that the streams and `self` may be overwritten in place.
 // S: streams, or (above 4) the most of them.
 template <typename OT, int S, int V>
@@ -80,10 +103,11 @@ __global__ void __launch_bounds__(512) stream_mix_kernel(StreamMix a, int width)
   float* dst = a.dst + m * n * width;
   OT* out = static_cast<OT*>(a.out) + m * a.ld_out;
   const OT* self = static_cast<const OT*>(a.self) + m * a.ld_out;
+  const float more = a.y_more_gate ? 1.0f / (1.0f + expf(-a.y_more_gate[m * a.ld_gate])) : 1.f;
   float sq = 0.f;
 #pragma unroll(S > 4 ? 1 : 2)
   for (int d = V * threadIdx.x; d < width; d += V * blockDim.x) {
-    SmVec<V> x[S], u, total;
+    SmVec<V> x[S], u;
 #pragma unroll
     for (int s = 0; s < S; ++s)
       if (s < n) x[s] = sm_load<V>(src + s * src_ld + d);
@@ -104,7 +128,7 @@ __global__ void __launch_bounds__(512) stream_mix_kernel(StreamMix a, int width)
       if (a.y_more) {
         const SmVec<V> part = sm_load<V>(a.y_more + m * width + d);
 #pragma unroll
-        for (int j = 0; j < V; ++j) y.v[j] += part.v[j];
+        for (int j = 0; j < V; ++j) y.v[j] = fmaf(more, part.v[j], y.v[j]);
       }
       SmVec<V> old[S];
 #pragma unroll
@@ -121,21 +145,30 @@ __global__ void __launch_bounds__(512) stream_mix_kernel(StreamMix a, int width)
 #pragma unroll
             for (int j = 0; j < V; ++j) x[t].v[j] = fmaf(mix[s * n + t], old[s].v[j], x[t].v[j]);
           }
-        sm_store<V>(dst + (size_t)t * width + d, x[t]);
       }
+      if (a.inject) {
+        if (a.sum) sm_store<V>(a.sum + m * width + d, sm_sum<S, V>(x, n));
+        const SmVec<V> part = sm_load<V>(a.inject + m * width + d);
+#pragma unroll
+        for (int t = 0; t < S; ++t)
+          if (t < n) {
+#pragma unroll
+            for (int j = 0; j < V; ++j) x[t].v[j] += part.v[j];
+          }
+      }
+#pragma unroll
+      for (int t = 0; t < S; ++t)
+        if (t < n) sm_store<V>(dst + (size_t)t * width + d, x[t]);
     }
 #pragma unroll
-    for (int j = 0; j < V; ++j) u.v[j] = total.v[j] = 0.f;
+    for (int j = 0; j < V; ++j) u.v[j] = 0.f;
 #pragma unroll
     for (int s = 0; s < S; ++s)
       if (s < n) {
 #pragma unroll
-        for (int j = 0; j < V; ++j) {
-          u.v[j] = fmaf(w_in[s], x[s].v[j], u.v[j]);
-          total.v[j] += x[s].v[j];
-        }
+        for (int j = 0; j < V; ++j) u.v[j] = fmaf(w_in[s], x[s].v[j], u.v[j]);
       }
-    if (a.sum) sm_store<V>(a.sum + m * width + d, total);
+    if (a.sum && !a.inject) sm_store<V>(a.sum + m * width + d, sm_sum<S, V>(x, n));
     if (a.gain) {
 #pragma unroll
       for (int j = 0; j < V; ++j) sq += u.v[j] * u.v[j];
@@ -148,11 +181,35 @@ __global__ void __launch_bounds__(512) stream_mix_kernel(StreamMix a, int width)
   __syncthreads();
   sq = warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? red[threadIdx.x & 31] : 0.f);
   const float inv = 1.0f / sqrtf(sq / (float)width + a.eps);
+  const int crow = a.conv_w ? a.cache_row[m] : 0, pos = a.conv_w ? a.row_pos[m] : 0;
+  OT* st_row = static_cast<OT*>(a.conv_state) + (size_t)(crow < 0 ? 0 : crow / a.max_seq) * (a.conv_taps - 1) * width;   // (a row without a slot reads slot 0's)
   for (int d = V * threadIdx.x; d < width; d += V * blockDim.x) {
     const SmVec<V> g = sm_load<V>(a.gain + d);
     SmVec<V> u = sm_load<V>(sm_u + d);
 #pragma unroll
     for (int j = 0; j < V; ++j) u.v[j] *= inv * g.v[j];
+    if (a.conv_w) {
+      // (the state holds what a prompt's rows hold: values of the output type)
+      sm_round<OT, V>(u);
+      const SmVec<V> h = u;
+      OT* st = st_row + d;
+      for (int t = 0; t < a.conv_taps; ++t) {
+        const SmVec<V> w = sm_load<V>(a.conv_w + (size_t)t * width + d);
+        SmVec<V> in = h;
+        if (t + 1 < a.conv_taps) {
+          in = sm_load<V>(st + (size_t)t * width);
+          if (t > 0 && crow >= 0) sm_store<V>(st + (size_t)(t - 1) * width, in);
+          if (pos < a.conv_taps - 1 - t) {                 // before the sequence's start, whatever the slot still holds
+#pragma unroll
+            for (int j = 0; j < V; ++j) in.v[j] = 0.f;
+          }
+        } else if (t > 0 && crow >= 0) {
+          sm_store<V>(st + (size_t)(t - 1) * width, h);
+        }
+#pragma unroll
+        for (int j = 0; j < V; ++j) u.v[j] = fmaf(w.v[j], in.v[j], u.v[j]);
+      }
+    }
     sm_store<V>(out + d, u);
   }
 }
@@ -160,7 +217,7 @@ __global__ void __launch_bounds__(512) stream_mix_kernel(StreamMix a, int width)
 template <typename OT>
 static int stream_mix_typed(tq_ctx* ctx, const StreamMix& a, size_t rows, size_t width) {
   const uintptr_t bits = (uintptr_t)a.src | (uintptr_t)a.dst | (uintptr_t)a.y | (uintptr_t)a.y_more | (uintptr_t)a.gain | (uintptr_t)a.out | (uintptr_t)a.self |
-                         (uintptr_t)a.sum;
+                         (uintptr_t)a.sum | (uintptr_t)a.inject | (uintptr_t)a.conv_w | (uintptr_t)a.conv_state;
   const bool vec = a.streams <= 4 && width % 4 == 0 && a.ld_out % 4 == 0 && (bits & 15) == 0;
   const size_t smem = a.gain ? width * sizeof(float) : 0;
   size_t threads = vec ? width / 4 : width;
@@ -188,6 +245,8 @@ int launch_stream_mix(tq_ctx* ctx, const StreamMix& a, size_t rows, size_t width
   TQ_REQUIRE(ctx, !a.y || (a.dst && a.mix && a.w_out && a.n_y >= 1 && a.n_y <= kSmMaxRows && !a.src_rows && (a.y_rows || a.n_y == 1)),
              "stream mix: bad sublayer output (at most %d rows each)", kSmMaxRows);
   TQ_REQUIRE(ctx, !a.gain || a.out, "stream mix: nowhere to put the norm");
+  TQ_REQUIRE(ctx, !a.inject || a.y, "stream mix: rows are added to the streams together with a sublayer's output");
+  TQ_REQUIRE(ctx, !a.conv_w || (a.gain && a.row_pos && a.cache_row && a.conv_taps >= 1 && a.max_seq > 0 && (a.conv_state || a.conv_taps == 1)), "stream mix: bad convolution");
   if (rows == 0) return TQ_OK;
   return a.out_dtype == TQ_F32 ? stream_mix_typed<float>(ctx, a, rows, width) : stream_mix_typed<__nv_bfloat16>(ctx, a, rows, width);
 }
@@ -222,5 +281,41 @@ extern "C" int tq_stream_mix(tq_ctx* ctx, size_t streams, size_t src_streams, co
   a.ld_out = ld_out ? ld_out : width;
   a.eps = eps;
   a.sum = sum_dev;
+  return launch_stream_mix(ctx, a, rows, width);
+}
+
+extern "C" int tq_stream_step(tq_ctx* ctx, const float* src_dev, float* dst_dev, const float* y_dev, const int* y_rows_dev, const float* y_weight_dev, size_t n_y,
+                              const float* y_more_dev, const float* y_more_gate_dev, size_t ld_gate, const float* inject_dev, const float* mix_one_dev,
+                              const float* w_out_dev, const float* gain_dev, size_t rows, size_t width, float eps, const float* conv_w_dev, void* conv_state_dev,
+                              size_t taps, size_t max_seq, const int* row_pos_dev, const int* cache_row_dev, void* out_dev, int out_dtype, size_t ld_out,
+                              float* sum_dev) {
+  if (int st = bind(ctx)) return st;
+  TQ_REQUIRE(ctx, src_dev && dst_dev && y_dev && mix_one_dev && w_out_dev && gain_dev && out_dev && (out_dtype == TQ_F32 || out_dtype == TQ_BF16),
+             "tq_stream_step: null pointer, or out is neither f32 nor bf16");
+  StreamMix a;
+  a.src = src_dev;
+  a.dst = dst_dev;
+  a.y = y_dev;
+  a.y_rows = y_rows_dev;
+  a.y_weight = y_weight_dev;
+  a.n_y = y_rows_dev ? (int)n_y : 1;
+  a.y_more = y_more_dev;
+  a.y_more_gate = y_more_gate_dev;
+  a.ld_gate = ld_gate;
+  a.inject = inject_dev;
+  a.mix = mix_one_dev;
+  a.w_out = w_out_dev;
+  a.gain = gain_dev;
+  a.out = out_dev;
+  a.out_dtype = out_dtype;
+  a.ld_out = ld_out ? ld_out : width;
+  a.eps = eps;
+  a.sum = sum_dev;
+  a.conv_w = conv_w_dev;
+  a.conv_state = conv_state_dev;
+  a.conv_taps = (int)taps;
+  a.max_seq = (int)max_seq;
+  a.row_pos = row_pos_dev;
+  a.cache_row = cache_row_dev;
   return launch_stream_mix(ctx, a, rows, width);
 }

@@ -57,8 +57,8 @@ struct CapScore {
   }
 };
 
-// DVT: value columns / 8 (padded to 16 columns, so even).
-template <int DVT, bool SPLIT>
+// DVT: value columns / 8 (padded to 16 columns, so even).  POOL: key tiles of pooled blocks come first, then the window's.
+template <int DVT, bool SPLIT, bool POOL>
 __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 2) window_attention_kernel(const __grid_constant__ WinParams p) {
   constexpr int kThreads = SPLIT ? 128 : 256;
   constexpr int kWarps = kThreads / 32;
@@ -97,11 +97,13 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
   const __nv_bfloat16* vb = p.v + seq0 * ve + (size_t)kvh * p.a.vdim_pad;
 
   const int lo = max(0, p0 - p.a.window + 1);
+  // tiles below `lo_t` are the pooled ones, counted from lo_t - pool_t
   const int lo_t = lo / kWaKeys, hi_t = p1 / kWaKeys;
-  int t0 = lo_t, t1 = hi_t + 1;
+  const int n_pool = POOL ? min(seen_blocks(p1, p.a.window, p.a.pool), p.a.pool_rows) : 0, pool_t = (n_pool + kWaKeys - 1) / kWaKeys, first_t = lo_t - pool_t;
+  int t0 = first_t, t1 = hi_t + 1;
   if constexpr (SPLIT) {
-    const int per = (hi_t - lo_t + p.n_splits) / p.n_splits;
-    t0 = min(lo_t + (int)blockIdx.x * per, hi_t + 1);
+    const int per = (hi_t - first_t + p.n_splits) / p.n_splits;
+    t0 = min(first_t + (int)blockIdx.x * per, hi_t + 1);
     t1 = min(t0 + per, hi_t + 1);
   }
 
@@ -119,15 +121,22 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
   const int row_first = threadIdx.x / per_row, pc = threadIdx.x - row_first * per_row;
   const bool copies = row_first < row_step, is_v = pc >= kcm;
   const __nv_bfloat16* src_c = is_v ? vb + (pc - kcm) * 8 : kb + pc * 8;
+  const __nv_bfloat16* pool_c = nullptr;
+  if constexpr (POOL) {
+    const size_t row = seq0 / (size_t)p.a.max_seq * p.a.pool_rows;
+    pool_c = is_v ? static_cast<const __nv_bfloat16*>(p.a.pooled_values) + row * ve + (size_t)kvh * p.a.vdim_pad + (pc - kcm) * 8
+                  : static_cast<const __nv_bfloat16*>(p.a.pooled_keys) + row * ke + (size_t)kvh * p.a.dim_pad + pc * 8;
+  }
   const size_t src_ld = is_v ? ve : ke;
   const int dst_ld = is_v ? v_row : k_row;
   const uint32_t dst_c = smem_u32(is_v ? v_s + (pc - kcm) * 16 : k_s + pc * 16);
   auto load_tile = [&](int tile, int buf) {
-    const int key0 = tile * kWaKeys;
+    const bool pooled = POOL && tile < lo_t;
+    const int key0 = (pooled ? tile - first_t : tile) * kWaKeys;
     if (copies) {
-      const __nv_bfloat16* src = src_c + (size_t)(key0 + row_first) * src_ld;
+      const __nv_bfloat16* src = (pooled ? pool_c : src_c) + (size_t)(key0 + row_first) * src_ld;
       uint32_t dst = dst_c + (uint32_t)((buf * kWaKeys + row_first) * dst_ld);
-      const int n_valid = p1 + 1 - key0;                   // rows at or beyond it become zeros
+      const int n_valid = (pooled ? n_pool : p1 + 1) - key0;   // rows at or beyond it become zeros
 #pragma unroll 4
       for (int row = row_first; row < kWaKeys; row += row_step) {
         cp_async16(dst, row < n_valid ? src : src_c, row < n_valid);
@@ -191,6 +200,13 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
   }
   const CapScore cap(p.a);
   const int nks = p.dp / 16;
+  int seen[2] = {0, 0}, w_seen_first = 0, w_seen_last = 0;   // pooled blocks that the two pairs, the warp's first and its last one see
+  if constexpr (POOL) {
+    seen[0] = seen_blocks(qpos[0], p.a.window, p.a.pool);
+    seen[1] = seen_blocks(qpos[1], p.a.window, p.a.pool);
+    w_seen_first = seen_blocks(w_first, p.a.window, p.a.pool);
+    w_seen_last = seen_blocks(w_last, p.a.window, p.a.pool);
+  }
 
   for (int tile = t0; tile < t1; ++tile) {
     const int buf = p.stages == 2 ? (tile - t0) & 1 : 0;
@@ -203,8 +219,9 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
     __syncthreads();
     for (int sub = 0; sub < kSub; ++sub) {
       const int w0 = SPLIT ? 16 * warp : 8 * NT * sub;     // first key of the tile for this warp's step
-      const int key0 = tile * kWaKeys + w0;
-      if (!w_live || key0 > w_last || w_first - (key0 + 8 * NT - 1) >= p.a.window) continue;
+      const bool pooled = POOL && tile < lo_t;
+      const int key0 = (pooled ? tile - first_t : tile) * kWaKeys + w0;
+      if (!w_live || (pooled ? key0 >= w_seen_last : key0 > w_last || w_first - (key0 + 8 * NT - 1) >= p.a.window)) continue;
       const uint8_t* kt = k_s + (buf * kWaKeys + w0) * k_row;
       const uint8_t* vt = v_s + (buf * kWaKeys + w0) * v_row;
       float s[NT][4];
@@ -222,7 +239,7 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
         for (int n = 0; n < NT; ++n) mma_bf16_16816(s[n], qf[0], qf[1], qf[2], qf[3], kf[n >> 1][2 * (n & 1)], kf[n >> 1][2 * (n & 1) + 1]);
       }
       // a step whose keys every pair of the warp sees needs no mask (rows without a query are never stored)
-      const bool full = key0 + 8 * NT - 1 <= w_first && w_last - key0 < p.a.window;
+      const bool full = pooled ? key0 + 8 * NT <= w_seen_first : key0 + 8 * NT - 1 <= w_first && w_last - key0 < p.a.window;
       float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int n = 0; n < NT; ++n)
@@ -231,7 +248,7 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
           float v = cap(s[n][c]);
           if (!full) {
             const int key = key0 + 8 * n + 2 * t + (c & 1);
-            const bool ok = live[c >> 1] && key <= qpos[c >> 1] && qpos[c >> 1] - key < p.a.window;
+            const bool ok = live[c >> 1] && (pooled ? key < seen[c >> 1] : key <= qpos[c >> 1] && qpos[c >> 1] - key < p.a.window);
             v = ok ? v : -INFINITY;
           }
           s[n][c] = v;
@@ -302,7 +319,7 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       if (!live[h]) continue;
-      const float inv = 1.0f / l_run[h];
+      const float inv = p.a.out_scale / l_run[h];
       __nv_bfloat16* dst = p.out + (size_t)qrow[h] * p.ldo + (size_t)qhead[h] * vd;
       const __nv_bfloat16* gate = p.gate ? p.gate + (size_t)qrow[h] * p.ldg + (size_t)qhead[h] * vd : nullptr;
 #pragma unroll
@@ -373,7 +390,7 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
           p.part_ml[pi * 2 + 1] = L;
         }
       } else {
-        const float inv = 1.0f / L;
+        const float inv = p.a.out_scale / L;
         __nv_bfloat16* dst = p.out + (size_t)row0 * p.ldo + (size_t)(head0 + h) * vd;
         const __nv_bfloat16* gate = p.gate ? p.gate + (size_t)row0 * p.ldg + (size_t)(head0 + h) * vd : nullptr;
 #pragma unroll
@@ -388,8 +405,8 @@ __global__ void __launch_bounds__(SPLIT ? 128 : 256, DVT > 16 ? 1 : SPLIT ? 3 : 
 
 // Merges the splits of one (row, head).  One CTA per head, a thread per column.
 __global__ void __launch_bounds__(256) window_combine_kernel(const float* part_o, const float* part_ml, int n_splits, int W, int heads, int vdim,
-                                                             const int* cache_row, const __nv_bfloat16* gate, long long ldg, __nv_bfloat16* out,
-                                                             long long ldo) {
+                                                             const int* cache_row, float out_scale, const __nv_bfloat16* gate, long long ldg,
+                                                             __nv_bfloat16* out, long long ldo) {
   __shared__ float wgt[kWaMaxSplits];
   pdl_wait();
   pdl_launch_dependents();
@@ -408,7 +425,7 @@ __global__ void __launch_bounds__(256) window_combine_kernel(const float* part_o
     }
     const float M = warp_max(fmaxf(m[0], m[1]));
     const float w0 = exp2f(m[0] - M), w1 = exp2f(m[1] - M);
-    const float f = 1.0f / warp_sum(l[0] * w0 + l[1] * w1);
+    const float f = out_scale / warp_sum(l[0] * w0 + l[1] * w1);
     wgt[lane] = w0 * f;
     wgt[lane + 32] = w1 * f;
   }
@@ -458,7 +475,13 @@ __global__ void __launch_bounds__(128) window_attention_simt_kernel(const T* q, 
     __syncthreads();
     return r;
   };
-  const int lo = max(0, pos - a.window + 1), n_vis = pos - lo + 1;
+  const int lo = max(0, pos - a.window + 1);
+  const int n_pool = a.pool ? min(seen_blocks(pos, a.window, a.pool), a.pool_rows) : 0, n_vis = n_pool + pos - lo + 1;   // pooled blocks first
+  const size_t pool0 = a.pool ? seq0 / (size_t)a.max_seq * a.pool_rows : 0;
+  const T* pk = static_cast<const T*>(a.pooled_keys) + pool0 * ke + (size_t)kvh * a.dim_pad;
+  const T* pv = static_cast<const T*>(a.pooled_values) + pool0 * ve + (size_t)kvh * a.vdim_pad;
+  auto key_row = [&](int c) { return c < n_pool ? pk + (size_t)c * ke : kb + (size_t)(lo + c - n_pool) * ke; };
+  auto value_row = [&](int c) { return c < n_pool ? pv + (size_t)c * ve : vb + (size_t)(lo + c - n_pool) * ve; };
   const float sink = a.sinks ? a.sinks[head] : a.sink;
   const bool has_sink = sink > -FLT_MAX;
   float m_run = has_sink ? sink : -FLT_MAX, l_run = has_sink ? 1.f : 0.f;
@@ -466,7 +489,7 @@ __global__ void __launch_bounds__(128) window_attention_simt_kernel(const T* q, 
     const int c = c0 + tid, n = min(128, n_vis - c0);
     float sc = -FLT_MAX;
     if (c < n_vis) {
-      const T* kr = kb + (size_t)(lo + c) * ke;
+      const T* kr = key_row(c);
       float s = 0.f;
       for (int d = 0; d < a.dim; ++d) s = fmaf(qs[d], wa_load(kr + d), s);
       s *= a.scale;
@@ -480,13 +503,13 @@ __global__ void __launch_bounds__(128) window_attention_simt_kernel(const T* q, 
     l_run = l_run * alpha + block_reduce(w, false);   // (its barriers also publish pr)
     for (int d = tid; d < a.vdim; d += 128) {
       float x = acc[d] * alpha;
-      for (int j = 0; j < n; ++j) x = fmaf(pr[j], wa_load(vb + (size_t)(lo + c0 + j) * ve + d), x);
+      for (int j = 0; j < n; ++j) x = fmaf(pr[j], wa_load(value_row(c0 + j) + d), x);
       acc[d] = x;
     }
     __syncthreads();
   }
   for (int d = tid; d < a.vdim; d += 128) {
-    float o = acc[d] / l_run;
+    float o = acc[d] / l_run * a.out_scale;
     if (gate) o *= sigmoid_gate(wa_load(gate + (size_t)row * ldg + (size_t)head * a.vdim + d));
     wa_store(out + (size_t)row * ldo + (size_t)head * a.vdim + d, o);
   }
@@ -513,7 +536,8 @@ static int launch_mma(tq_ctx* ctx, WinParams& p, bool split, size_t smem, dim3 g
     TQ_CUDA(ctx, launch_k(ctx, kern, grid, dim3((unsigned)threads), smem, p));
     return TQ_OK;
   };
-  return split ? go(window_attention_kernel<DVT, true>, 128) : go(window_attention_kernel<DVT, false>, 256);
+  if (p.a.pool) return split ? go(window_attention_kernel<DVT, true, true>, 128) : go(window_attention_kernel<DVT, false, true>, 256);
+  return split ? go(window_attention_kernel<DVT, true, false>, 128) : go(window_attention_kernel<DVT, false, false>, 256);
 }
 
 int launch_window_attention(tq_ctx* ctx, const WindowAttn& attn, const RaggedBatch& b, int dtype, const void* q, size_t ldq, const void* gate,
@@ -524,6 +548,7 @@ int launch_window_attention(tq_ctx* ctx, const WindowAttn& attn, const RaggedBat
   TQ_REQUIRE(ctx, a.dim > 0 && a.vdim > 0 && a.dim_pad >= a.dim && a.vdim_pad >= a.vdim && a.dim_pad % 8 == 0 && a.vdim_pad % 8 == 0,
              "window attention: bad head sizes");
   TQ_REQUIRE(ctx, a.window > 0 && a.softcap >= 0.f, "window attention: bad window or cap");
+  TQ_REQUIRE(ctx, a.pool >= 0 && (a.pool == 0 || (a.pooled_keys && a.pooled_values && a.max_seq > 0 && a.pool_rows >= 0)), "window attention: bad pooled blocks");
   if (b.rows == 0 || b.n_seqs == 0) return TQ_OK;
   if (dtype == TQ_F32) return launch_simt<float>(ctx, a, b, q, ldq, gate, ldg, k_cache, v_cache, out, ldo);
   if (a.dim > 256 || a.vdim > 256) return launch_simt<__nv_bfloat16>(ctx, a, b, q, ldq, gate, ldg, k_cache, v_cache, out, ldo);
@@ -573,6 +598,7 @@ int launch_window_attention(tq_ctx* ctx, const WindowAttn& attn, const RaggedBat
     long long tiles = (b.max_len + kWaKeys - 1) / kWaKeys;
     const long long win_tiles = ((long long)a.window - 1 + kWaKeys - 1) / kWaKeys + 1;
     if (win_tiles < tiles) tiles = win_tiles;
+    if (a.pool) tiles += (seen_blocks(b.max_len - 1, a.window, a.pool) + kWaKeys - 1) / kWaKeys;
     const long long ctas = (long long)a.kv_heads * p.n_hb * b.n_seqs;
     long long n = (4ll * ctx->sm_count + ctas - 1) / ctas;
     if (n > tiles / 2) n = tiles / 2;
@@ -602,7 +628,7 @@ int launch_window_attention(tq_ctx* ctx, const WindowAttn& attn, const RaggedBat
   if (st != TQ_OK) return st;
   if (p.n_splits > 1)
     TQ_CUDA(ctx, launch_k(ctx, window_combine_kernel, dim3((unsigned)((size_t)b.rows * a.heads)), dim3((unsigned)((a.vdim + 31) / 32 * 32)), 0,
-                          (const float*)p.part_o, (const float*)p.part_ml, p.n_splits, W, a.heads, a.vdim, b.cache_row, p.gate, p.ldg, p.out, p.ldo));
+                          (const float*)p.part_o, (const float*)p.part_ml, p.n_splits, W, a.heads, a.vdim, b.cache_row, a.out_scale, p.gate, p.ldg, p.out, p.ldo));
   return TQ_OK;
 }
 
@@ -622,6 +648,15 @@ extern "C" int tq_window_attention_sinks(tq_ctx* ctx, const tq_window_attn_confi
                                          const void* gate_dev, size_t ldg, const void* k_cache_dev, const void* v_cache_dev, size_t cache_rows,
                                          const int* seq_rows_dev, const int* row_pos_dev, const int* cache_row_dev, size_t n_seqs, size_t rows,
                                          size_t max_q, size_t max_len, void* out_dev, size_t ldo) {
+  return tq_window_attention_pooled(ctx, cfg, sinks_dev, dtype, q_dev, ldq, gate_dev, ldg, k_cache_dev, v_cache_dev, cache_rows, 0, nullptr, nullptr, 0, 0, 1.f,
+                                    seq_rows_dev, row_pos_dev, cache_row_dev, n_seqs, rows, max_q, max_len, out_dev, ldo);
+}
+
+extern "C" int tq_window_attention_pooled(tq_ctx* ctx, const tq_window_attn_config* cfg, const float* sinks_dev, int dtype, const void* q_dev, size_t ldq,
+                                          const void* gate_dev, size_t ldg, const void* k_cache_dev, const void* v_cache_dev, size_t cache_rows,
+                                          size_t pool, const void* pooled_keys_dev, const void* pooled_values_dev, size_t pool_rows, size_t max_seq,
+                                          float out_scale, const int* seq_rows_dev, const int* row_pos_dev, const int* cache_row_dev, size_t n_seqs,
+                                          size_t rows, size_t max_q, size_t max_len, void* out_dev, size_t ldo) {
   if (int st = bind(ctx)) return st;
   TQ_REQUIRE(ctx, cfg && (dtype == TQ_BF16 || dtype == TQ_F32), "tq_window_attention: dtype must be bf16 or f32");
   if (rows == 0) return TQ_OK;
@@ -639,6 +674,12 @@ extern "C" int tq_window_attention_sinks(tq_ctx* ctx, const tq_window_attn_confi
   a.softcap = cfg->softcap;
   a.sink = cfg->sink;
   a.sinks = sinks_dev;
+  a.out_scale = out_scale;
+  a.pool = (int)pool;
+  a.pool_rows = (int)pool_rows;
+  a.max_seq = (int)max_seq;
+  a.pooled_keys = pooled_keys_dev;
+  a.pooled_values = pooled_values_dev;
   RaggedBatch b;
   b.n_seqs = (int)n_seqs;
   b.rows = (int)rows;

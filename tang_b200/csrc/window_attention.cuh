@@ -3,6 +3,10 @@
 //     p_j = exp(s_j) / (exp(sink) + sum exp(s))                       (one sink, or one per head; -infinity: none; it has no value)
 //     out = (sum p_j v_j) * sigmoid(gate)                             (no gate pointer: 1)
 // Mask: the query at position i sees key j when j <= i and i - j < window.
+//
+// Pooled blocks (pool > 0): beside these, it sees one key and one value for each block of `pool` tokens that lies wholly before its
+// window -- block b of the sequence when b pool + pool - 1 <= i - window -- under the same softmax.  Tokens that have left the
+// window and whose block is not there yet are not seen.
 #pragma once
 
 #include "internal.h"
@@ -17,7 +21,13 @@ struct WindowAttn {
   float scale = 0.f, softcap = 0.f, sink = 0.f;
   const float* sinks = nullptr;        // [heads], instead of `sink`
   size_t q_head = 0;                   // elements between the heads of a query row; 0: dim
+  float out_scale = 1.f;               // factor on the result
+  int pool = 0, pool_rows = 0, max_seq = 0;            // pooled rows and cache rows per slot
+  const void *pooled_keys = nullptr, *pooled_values = nullptr;   // [slot * pool_rows + block], rows as in the caches
 };
+
+// Pooled blocks that the query at position `pos` sees.
+__host__ __device__ inline int seen_blocks(int pos, int window, int pool) { return pos >= window ? (pos - window + 1) / pool : 0; }
 
 // q [rows][ldq], head h at column h * dim (q_head); gate [rows][ldg] and out [rows][ldo], head h at column h * vdim.  dtype (TQ_BF16 or
 // TQ_F32) is that of q, gate, caches and out; scores, weights and sums are f32, in TQ_F32 every operation is.

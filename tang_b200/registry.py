@@ -8,10 +8,12 @@ from . import _lib
 from .checkpoint import read_safetensors
 from .dotanex import DotanexConfig, DotanexModel
 from .numuzen import NumuzenConfig, NumuzenModel
+from .sakinex import SakinexConfig, SakinexModel
 from .tofazen import TofazenConfig, TofazenModel
 
 # architecture -> (configuration class, model class with ``from_tensors``)
-ARCHITECTURES = {"Tofazen": (TofazenConfig, TofazenModel), "Numuzen": (NumuzenConfig, NumuzenModel), "Dotanex": (DotanexConfig, DotanexModel)}
+ARCHITECTURES = {"Tofazen": (TofazenConfig, TofazenModel), "Numuzen": (NumuzenConfig, NumuzenModel), "Dotanex": (DotanexConfig, DotanexModel),
+                 "Sakinex": (SakinexConfig, SakinexModel)}
 
 DEFAULT_MAX_SEQ = 8192      # for designs without a largest position
 

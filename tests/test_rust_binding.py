@@ -41,7 +41,8 @@ def test_every_exported_symbol_is_declared_with_its_arity():
     names = {n for n, _ in structs}
     assert names == {"tq_sampler_config", "tq_llama_config", "tq_moe_config", "tq_mla_config", "tq_diff_attn_config",
                      "tq_tofazen_config", "tq_tofazen_layer", "tq_window_attn_config", "tq_gla_config",
-                     "tq_numuzen_config", "tq_numuzen_layer", "tq_dotanex_config", "tq_dotanex_layer"}
+                     "tq_numuzen_config", "tq_numuzen_layer", "tq_dotanex_config", "tq_dotanex_layer", "tq_conv_heads_config",
+                     "tq_sakinex_config", "tq_sakinex_layer"}
     cfg = dict(structs)["tq_llama_config"]
     assert [f for f, _ in cfg] == ["n_layers", "d_model", "n_heads", "n_kv_heads", "head_dim", "ffn", "vocab", "max_seq",
                                    "max_batch", "eps", "rope_base"]
