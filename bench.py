@@ -15,6 +15,7 @@ weak and the aggregate is the sum over ranks.
     python bench.py --tofazen               # instead: the Tofazen family beside the int4 model (one JSON line of its own)
     python bench.py --numuzen               # instead: the Numuzen family beside the Tofazen family (one JSON line of its own)
     python bench.py --dotanex               # instead: the Dotanex family beside the Numuzen family (one JSON line of its own)
+    python bench.py --sakinex               # instead: the Sakinex family beside the Numuzen family (one JSON line of its own)
 
 The JSON line also carries: `e2e` (the same rate through the reference-shaped call q4_matvec with
 HOST vectors, copies inside the timed region), `roofline` (dominant kernel vs measured HBM peak),
@@ -1650,6 +1651,259 @@ def run_dotanex(args) -> None:
     print(json.dumps(out))
 
 
+# ----------------------------------------------------------------------------------------------
+# --sakinex: the Sakinex family (bf16) beside the Numuzen family at equal width, head sizes, window and active feed-forward,
+# random weights: decode and prefill throughput of both, and the new kernels beside the like ones, against their rooflines.
+# ----------------------------------------------------------------------------------------------
+SAKINEX_SIZES = {
+    # `top` experts of ff values and the shared one together are as wide as the other models' feed-forward
+    "8b": {**{k: NUMUZEN_SIZES["8b"][k] for k in ("layers", "width", "heads", "kv", "dim", "vocab")}, "state": 2048, "pool": 16, "taps": 4, "experts": 8, "top": 2,
+           "ff": 4096, "shared": 6144},
+    "1b": {**{k: NUMUZEN_SIZES["1b"][k] for k in ("layers", "width", "heads", "kv", "dim", "vocab")}, "state": 1024, "pool": 16, "taps": 4, "experts": 32, "top": 4,
+           "ff": 1536, "shared": 2048},
+}
+
+
+def build_sakinex(dev, tb, torch, stream, s, max_seq, max_batch, window):
+    from tang_b200 import sakinex as sx
+
+    gen = torch.Generator(device="cuda").manual_seed(7)
+    H, G, D, R, d, taps = s["heads"], s["kv"], s["dim"], s["state"], s["width"], s["taps"]
+    layer = sx.SakinexLayer(H, G, D, D, D ** -0.5, R, window, s["pool"], taps, sx.Rotation(64, 500000.0, 4.0, 4096, 32.0, 1.0), 0.7, 1.1,
+                            sx.Experts(s["experts"], s["top"], s["ff"], s["shared"]))
+    cfg = tb.SakinexConfig(s["vocab"], d, 1e-6, 0.5, taps, [layer] * s["layers"])
+    model = tb.SakinexModel(dev, cfg, tb.BF16, max_batch, max_seq)
+    shapes = {sx.EMBED: (s["vocab"], d), sx.HEAD: (s["vocab"], d), sx.CANON1: (d, taps), sx.CANON2: (d, taps), sx.Q: (H * D, d), sx.K: (G * D, d), sx.V: (G * D, d),
+              sx.Q_CONV: (H * D, taps), sx.K_CONV: (G * D, taps), sx.V_CONV: (G * D, taps), sx.LEFT_O: (d, H * D), sx.Z: (R, d), sx.Z_BIAS: (1, R), sx.X: (R, d),
+              sx.X_BIAS: (1, R), sx.G: (R, d), sx.RIGHT_O: (d, R), sx.ROUTER: (s["experts"], d), sx.ROUTER_BIAS: (1, s["experts"]), sx.GATE: (s["ff"], d),
+              sx.UP: (s["ff"], d), sx.DOWN: (d, s["ff"]), sx.SHARED_GATE: (s["shared"], d), sx.SHARED_UP: (s["shared"], d), sx.SHARED_DOWN: (d, s["shared"])}
+    pool = {}
+    for name, tensor, i, e in sx.tensor_names(cfg):
+        r, c = shapes.get(tensor, (1, d))
+        level = 1.0 if tensor in (sx.NORM1, sx.NORM2, sx.FINAL_NORM) else 0.0
+        key = (r, c, level, tensor == sx.ROUTER and i)
+        if key not in pool:
+            with torch.cuda.stream(stream):
+                pool[key] = (torch.randn((r, c), device="cuda", generator=gen) * (0.02 if r == 1 else 0.3 if c == taps else c ** -0.5) + level).bfloat16()
+            stream.synchronize()
+        model.put_pointer(tensor, i, pool[key].data_ptr(), tb.BF16, r, c, e)
+    return model
+
+
+def run_sakinex(args) -> None:
+    import ctypes as C
+
+    import torch
+
+    import tang_b200 as tb
+
+    torch.cuda.set_device(0)
+    dev = tb.QuantComputeDevice(0)
+    L_ = dev._L
+    stream = torch.cuda.ExternalStream(dev.stream, device=torch.device("cuda", 0))
+    peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")) else {}
+    hbm, tf = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    ctx, window = 2048, 512
+    sampler = ClockSampler(0)
+    sampler.start()
+    t_start = time.perf_counter()
+
+    def graph_ms(fn, reps=10):
+        fn()
+        dev.sync()
+        dev.begin_capture()
+        fn()
+        g = dev.end_capture()
+        ms = _time_ms(torch, stream, dev, g.launch, reps, warm=3)
+        g.free()
+        return ms
+
+    def rand(*shape, std=1.0, dt=None):
+        with torch.cuda.stream(stream):
+            t = torch.randn(shape, device="cuda") * std
+            t = t if dt == tb.F32 else t.bfloat16()
+        stream.synchronize()
+        return t
+
+    P = lambda t: C.c_void_p(t.data_ptr() if hasattr(t, "data_ptr") else t.ptr)
+    ints = lambda a: dev.upload(np.asarray(a, np.int32).reshape(-1), tb.I32)
+    null = C.c_void_p(0)
+    touched = lambda experts, top, rows: experts * (1 - (1 - top / experts) ** rows)      # expected number of experts that `rows` rows choose
+    out = {"metric": "sakinex_throughput", "unit": "tokens/s", "data": "synthetic", "dtype": "bf16", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf},
+           "window": window, "models": [], "kernels": []}
+    batches = [1, 2, 4, 8, 16, 64]
+
+    def time_model(size, name, model, s, decode_bytes, prefill_flops):
+        row = {"size": size, "model": name, "decode": {}, "prefill": {}}
+        for B in batches:
+            tok = ints(np.random.randint(0, s["vocab"], B))
+            pos, lg = ints(np.full(B, ctx)), dev.alloc(B * s["vocab"], tb.F32)
+            ms = graph_ms(lambda: model.decode(tok, pos, B, ctx + 1, lg))
+            row["decode"][B] = {"ms": ms, "tokens_per_s": B / ms * 1e3, "frac_of_hbm": decode_bytes(B) / ms / 1e6 / hbm}
+        for T in (512, ctx):
+            tok = ints(np.random.randint(0, s["vocab"], T))
+            cu, st, last, lg = ints([0, T]), ints([0]), ints([T - 1]), dev.alloc(s["vocab"], tb.F32)
+            ms = graph_ms(lambda: model.step(tok, T, cu, st, None, 1, T, T, last, 1, lg), 3)
+            row["prefill"][T] = {"ms": ms, "tokens_per_s": T / ms * 1e3, "frac_of_bf16": T * prefill_flops(T) / ms / 1e9 / tf}
+        out["models"].append(row)
+        model.destroy()
+        torch.cuda.empty_cache()
+
+    for size in [x for x in args.sakinex.split(",") if x in SAKINEX_SIZES]:
+        s = SAKINEX_SIZES[size]
+        d, H, G, D, R = s["width"], s["heads"], s["kv"], s["dim"], s["state"]
+        mixers, one = s["layers"] * d * ((2 * H + 2 * G) * D + 4 * R), 3 * d * s["ff"]
+        fixed = 2 * (mixers + s["layers"] * d * ((s["experts"] + 1) + 3 * s["shared"]) + s["vocab"] * d)
+        seen = window + (ctx - window + 1) // s["pool"]
+        per_row = s["layers"] * (G * 2 * D * 2 * seen + R * 8 + (s["taps"] - 1) * 2 * (2 * d + (H + 2 * G) * D) * 2)
+        active = mixers + s["layers"] * (s["top"] * one + 3 * d * s["shared"])
+        time_model(size, "sakinex", build_sakinex(dev, tb, torch, stream, s, ctx + 1, max(batches), window), s,
+                   lambda B: fixed + 2 * s["layers"] * one * touched(s["experts"], s["top"], B) + B * per_row, lambda T: 2.0 * active)
+        if not args.sakinex_only:
+            z = NUMUZEN_SIZES[size]
+            gh, gd, gv = z["gla"]
+            zm = z["layers"] // 2 * (d * (3 * H + z["kv"]) * D + d * (2 * gh * gd + 3 * gh * gv + 16))
+            zone, zrow = 3 * d * z["ff"], z["layers"] // 2 * (z["kv"] * 2 * D * 2 * window + gh * gd * gv * 8)
+            time_model(size, "numuzen", build_numuzen(dev, tb, torch, stream, z, ctx + 1, max(batches), window), z,
+                       lambda B: 2 * (zm + z["layers"] * z["experts"] * d + z["vocab"] * d + z["layers"] * zone * touched(z["experts"], z["top"], B)) + B * zrow,
+                       lambda T: 2.0 * (zm + z["layers"] * z["top"] * zone))
+
+    def kernel(name, m, us, byt=0.0, flops=0.0):
+        roof = max(byt / hbm / 1e3, flops / tf / 1e6)
+        out["kernels"].append({"kernel": name, "m": m, "us": round(us, 2), "roofline_us": round(roof, 2), "frac": round(roof / us, 3)})
+
+    class Win(C.Structure):
+        _fields_ = [(k, C.c_uint32) for k in ("heads", "kv_heads", "dim", "vdim", "window")] + [(k, C.c_float) for k in ("scale", "softcap", "sink")]
+
+    class Gla(C.Structure):
+        _fields_ = [(k, C.c_uint32) for k in ("heads", "dim", "vdim", "rank")] + [(k, C.c_float) for k in ("tau", "q_scale", "eps")]
+
+    class Heads(C.Structure):
+        _fields_ = [(n, C.c_uint32) for n in ("heads", "kv_heads", "dim", "vdim", "k0", "v0", "channels", "taps", "rot_dims")] + [("norm", C.c_int)] + [
+            (n, C.c_uint32) for n in ("pool", "pool_rows")] + [(n, C.c_float) for n in ("rot_mult", "eps")]
+
+    H, G, D, d, pool, taps = 32, 8, 128, 4096, 16, 4
+    prow, span = ctx // pool, (H + 2 * G) * D
+    lh, ld, lv, R = 16, 128, 256, 4096
+    gw = 2 * lh * ld + 2 * lh * lv
+    a2, a2b, gnorm = rand(lh * ld, 16, dt=tb.F32), rand(lh * ld, dt=tb.F32), rand(lv, dt=tb.F32)
+    zb, ub, freq, cw = rand(R, dt=tb.F32), rand(R, dt=tb.F32), rand(32, dt=tb.F32), rand(taps, span, std=0.4, dt=tb.F32)
+    dw, gain = rand(taps, d, std=0.3, dt=tb.F32), rand(d, dt=tb.F32)
+
+    def attention(pooled, w, q, k, v, pk, pv, o, B, rows, n_seqs, cu, rp, cr, max_q):
+        a = Win(H, G, D, D, w, D ** -0.5, 0.0, float("-inf"))
+        tail = (cu, P(rp), P(cr), n_seqs, rows, max_q, ctx, P(o), H * D)
+        if pooled:
+            return L_.tq_window_attention_pooled(dev._ctx, C.byref(a), null, tb.BF16, P(q), H * D, null, 0, P(k), P(v), B * ctx, pool, P(pk), P(pv), prow, ctx, 1.0, *tail)
+        return L_.tq_window_attention(dev._ctx, C.byref(a), tb.BF16, P(q), H * D, null, 0, P(k), P(v), B * ctx, *tail)
+
+    def min_gru(x, st, o, rows, n_seqs, cu, rp, cr, max_q):
+        off = lambda c: C.c_void_p(x.data_ptr() + 2 * c)
+        return L_.tq_min_gru(dev._ctx, tb.BF16, R, off(0), off(R), off(2 * R), 3 * R, P(zb), P(ub), 1.0, P(st), ctx, n_seqs * ctx, cu, P(rp), P(cr), n_seqs, rows, max_q, P(o), R)
+
+    def recurrence(x, a1, st, o, rows, n_seqs, cu, rp, cr, max_q):
+        g, off = Gla(lh, ld, lv, 16, 16.0, ld ** -0.5, 1e-6), lambda c: C.c_void_p(x.data_ptr() + 2 * c)
+        return L_.tq_gla(dev._ctx, C.byref(g), tb.BF16, off(0), off(lh * ld), off(2 * lh * ld), off(2 * lh * ld + lh * lv), gw, P(a1), 16, P(a2), P(a2b), P(gnorm),
+                         P(st), ctx, n_seqs * ctx, cu, P(rp), P(cr), n_seqs, rows, max_q, P(o), lh * lv)
+
+    def heads(x, st, q, k, v, pk, pv, rows, n_seqs, cu, rp, cr, max_q, max_len):
+        a = Heads(H, G, D, D, H * D, (H + G) * D, span, taps, 64, 1, pool, prow, 1.1, 1e-6)
+        return L_.tq_conv_heads(dev._ctx, C.byref(a), tb.BF16, P(x), span, P(cw), P(st), P(freq), ctx, n_seqs * ctx, cu, P(rp), P(cr), n_seqs, rows, max_q, max_len, P(q),
+                                H * D, P(k), P(v), P(pk), P(pv))
+
+    seen = window + (ctx - window) // pool
+    one, fac = torch.ones(1, device="cuda"), torch.full((1,), 0.5, device="cuda")
+    torch.cuda.synchronize()
+    # ---- one row per sequence
+    for B in (1, 16, 64):
+        n = max(2, min(16, 128 // B))                  # distinct caches per pass
+        k, v, pk, pv = rand(n, B, ctx, G * D), rand(n, B, ctx, G * D), rand(n, B, prow, G * D), rand(n, B, prow, G * D)
+        q, o = rand(B, H * D), torch.empty((B, H * D), dtype=torch.bfloat16, device="cuda")
+        rp, cr = ints(np.full(B, ctx - 1)), ints(np.arange(B) * ctx + ctx - 1)
+        for name, pooled, w, rows in (("pooled blocks and window", 1, window, seen), ("window", 0, window, window), ("window of as many keys", 0, seen, seen)):
+            us = graph_ms(lambda: [dev._check(attention(pooled, w, q, k[i], v[i], pk[i], pv[i], o, B, B, B, null, rp, cr, 1)) for i in range(n)]) / n * 1e3
+            kernel(f"decode attention, {name}", B, us, B * rows * G * D * 2 * 2)
+        N = 24
+        xs, sts = [rand(B, span) for _ in range(N)], [rand(B, taps - 1, span) for _ in range(N)]
+        us = graph_ms(lambda: [dev._check(heads(x, t, q, k[0], v[0], pk[0], pv[0], B, B, null, rp, cr, 1, ctx)) for x, t in zip(xs, sts)]) / N * 1e3
+        kernel("convolved heads", B, us, B * span * 2 * (2 + 2 * (taps - 1)))
+        rp16 = ints(np.full(B, ctx - pool))
+        cr16 = ints(np.arange(B) * ctx + ctx - pool)
+        us = graph_ms(lambda: [dev._check(heads(x, t, q, k[0], v[0], pk[0], pv[0], B, B, null, rp16, cr16, 1, ctx)) for x, t in zip(xs, sts)]) / N * 1e3
+        kernel("convolved heads, a block is complete", B, us, B * (span * 2 * (2 + 2 * (taps - 1)) + 2 * G * D * 2 * (pool + 1)))
+        qg = rand(D)
+        us = graph_ms(lambda: [dev._check(L_.tq_head_norm_rope(dev._ctx, tb.BF16, H, G, D, P(x), span, D, P(k[0]), P(v[0]), B * ctx, P(qg), P(qg), 0, 64, 0, P(freq), 1.0, 1e-6,
+                                                               P(rp), P(cr), B)) for x in xs]) / N * 1e3
+        kernel("per-head norm and rotation", B, us, B * (H + G) * D * 4)
+        del k, v, pk, pv
+        x, st = rand(B, 3 * R), [rand(B, R, dt=tb.F32) for _ in range(32)]
+        o = torch.empty((B, R), dtype=torch.bfloat16, device="cuda")
+        us = graph_ms(lambda: [dev._check(min_gru(x, t, o, B, B, null, rp, cr, 1)) for t in st]) / len(st) * 1e3
+        kernel("decode minGRU", B, us, B * R * (3 * 2 + 2 + 8))
+        st = [rand(B, lh, ld, lv, dt=tb.F32) for _ in range(max(4, min(64, 128 // B)))]
+        x, a1, o = rand(B, gw), rand(B, 16, dt=tb.F32), torch.empty((B, lh * lv), dtype=torch.bfloat16, device="cuda")
+        us = graph_ms(lambda: [dev._check(recurrence(x, a1, t, o, B, B, null, rp, cr, 1)) for t in st]) / len(st) * 1e3
+        kernel("decode gated recurrence", B, us, B * lh * ld * lv * 4 * 2)
+        del st
+        xs, h = [rand(B, d, dt=tb.F32) for _ in range(N)], torch.empty((B, d), dtype=torch.bfloat16, device="cuda")
+        y, slots, wt, cs, gate = rand(2 * B, d, dt=tb.F32), ints(np.random.permutation(2 * B)), rand(B, 2, dt=tb.F32), [rand(B, taps - 1, d) for _ in range(N)], rand(B, dt=tb.F32)
+        for name, experts in (("stream, next norm and convolution", 0), ("stream, next norm and convolution over two experts and a gated one", 1)):
+            us = graph_ms(lambda: [dev._check(L_.tq_stream_step(dev._ctx, P(x), P(x), P(y), P(slots) if experts else null, P(wt) if experts else null, 2, P(y) if experts else null,
+                                                                P(gate) if experts else null, 1, null, P(one), P(fac), P(gain), B, d, 1e-6, P(dw), P(t), taps, ctx, P(rp),
+                                                                P(cr), P(h), tb.BF16, d, null)) for x, t in zip(xs, cs)]) / N * 1e3
+            kernel(name, B, us, B * d * (14 + 4 * (taps - 1) + 8 * experts))
+        for name, r_, n_, byt in (("post-norm, stream, next norm", null, 1, 14), ("post-norm, stream, next norm over two experts", P(slots), 2, 18)):
+            us = graph_ms(lambda: [dev._check(L_.tq_add_norm(dev._ctx, P(x), P(y), r_, n_, P(gain), P(gain), B, d, 1e-6, P(h), tb.BF16, d)) for x in xs]) / N * 1e3
+            kernel(name, B, us, B * d * byt)
+        torch.cuda.empty_cache()
+
+    # ---- prompts
+    for T in (512, 2048):
+        cu, rp = ints([0, T]), ints(np.arange(T))
+        q, k, v, pk, pv = rand(T, H * D), rand(ctx, G * D), rand(ctx, G * D), rand(prow, G * D), rand(prow, G * D)
+        o = torch.empty((T, H * D), dtype=torch.bfloat16, device="cuda")
+        for w in (128, window):
+            for name, pooled in (("pooled blocks and window", 1), ("window", 0)):
+                us = graph_ms(lambda: dev._check(attention(pooled, w, q, k, v, pk, pv, o, 1, T, 1, P(cu), rp, rp, T))) * 1e3
+                kernel(f"prefill attention, {name} {w}", T, us, 0, 4.0 * H * D * sum(min(i + 1, w) + (max(0, i - w + 1) // pool if pooled else 0) for i in range(T)))
+        N = 8 if T == 512 else 4
+        xs, st = [rand(T, span) for _ in range(N)], rand(1, taps - 1, span)
+        us = graph_ms(lambda: [dev._check(heads(x, st, q, k, v, pk, pv, T, 1, P(cu), rp, rp, T, T)) for x in xs]) / N * 1e3
+        kernel("convolved heads, pooled blocks, states (3 kernels)", T, us, T * span * 4)
+        qg = rand(D)
+        us = graph_ms(lambda: [dev._check(L_.tq_head_norm_rope(dev._ctx, tb.BF16, H, G, D, P(x), span, D, P(k), P(v), ctx, P(qg), P(qg), 0, 64, 0, P(freq), 1.0, 1e-6, P(rp),
+                                                               P(rp), T)) for x in xs]) / N * 1e3
+        kernel("per-head norm and rotation", T, us, T * (H + G) * D * 4)
+        xs, st, o = [rand(T, 3 * R) for _ in range(N)], rand(1, R, dt=tb.F32), torch.empty((T, R), dtype=torch.bfloat16, device="cuda")
+        us = graph_ms(lambda: [dev._check(min_gru(x, st, o, T, 1, P(cu), rp, rp, T)) for x in xs]) / N * 1e3
+        kernel("prefill minGRU", T, us, T * R * 8)
+        x, a1, st = rand(T, gw), rand(T, 16, dt=tb.F32), rand(1, lh, ld, lv, dt=tb.F32)
+        us = graph_ms(lambda: dev._check(recurrence(x, a1, st, o, T, 1, P(cu), rp, rp, T))) * 1e3
+        kernel("prefill gated recurrence", T, us, T * (gw + lh * lv) * 2, 2.0 * T * lh * (32 * (ld + lv) + 2 * ld * lv))
+        xs, st, h = [rand(T, d) for _ in range(2 * N)], rand(1, taps - 1, d), torch.empty((T, d), dtype=torch.bfloat16, device="cuda")
+        us = graph_ms(lambda: [dev._check(L_.tq_conv_residual(dev._ctx, tb.BF16, d, taps, P(dw), P(st), ctx, ctx, P(x), d, P(cu), P(rp), P(rp), 1, T, T, T, P(h), d))
+                               for x in xs]) / len(xs) * 1e3
+        kernel("input convolution, states (2 kernels)", T, us, T * d * 4)
+        xs = [rand(T, d, dt=tb.F32) for _ in range(N)]
+        us = graph_ms(lambda: [dev._check(L_.tq_rms_norm(dev._ctx, P(x), tb.F32, null, P(gain), tb.F32, T, d, 1e-6, P(h), tb.BF16, null)) for x in xs]) / N * 1e3
+        kernel("plain norm", T, us, T * d * 6)
+        y, slots, wt, gate = rand(2 * T, d, dt=tb.F32), ints(np.random.permutation(2 * T)), rand(T, 2, dt=tb.F32), rand(T, dt=tb.F32)
+        us = graph_ms(lambda: [dev._check(L_.tq_stream_step(dev._ctx, P(x), P(x), P(y), P(slots), P(wt), 2, P(y), P(gate), 1, null, P(one), P(fac), P(gain), T, d, 1e-6, null, null,
+                                                            0, 1, P(rp), P(rp), P(h), tb.BF16, d, null)) for x in xs]) / N * 1e3
+        kernel("stream, next norm over two experts and a gated one", T, us, T * d * 22)
+        us = graph_ms(lambda: [dev._check(L_.tq_add_norm(dev._ctx, P(x), P(y), P(slots), 2, P(gain), P(gain), T, d, 1e-6, P(h), tb.BF16, d)) for x in xs]) / N * 1e3
+        kernel("post-norm, stream, next norm over two experts", T, us, T * d * 18)
+    for m in (1, 64, 2048):
+        z, bias = rand(m, 33, dt=tb.F32), rand(32, std=0.1, dt=tb.F32)
+        bufs = [ints(np.zeros(m * 4)) for _ in range(4)] + [ints(np.zeros(4 * (m * 4 + 32))), ints([0])]
+        us = graph_ms(lambda: [dev._check(L_.tq_route_biased(dev._ctx, P(z), 33, m, 32, 4, 1, 1, P(bias), null, 0, 8, *map(P, bufs))) for _ in range(20)]) / 20 * 1e3
+        kernel("biased routing, 4 of 32", m, us, m * 33 * 4)
+        us = graph_ms(lambda: [dev._check(L_.tq_route(dev._ctx, P(z), m, 32, 4, 0, 0, 8, *map(P, bufs))) for _ in range(20)]) / 20 * 1e3
+        kernel("routing, 4 of 32", m, us, m * 32 * 4)
+    out["clocks"] = sampler.stop(t_start, time.perf_counter())
+    print(json.dumps(out))
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1671,8 +1925,13 @@ def main() -> None:
     ap.add_argument("--numuzen", nargs="?", const="8b,1b", default="", help="time the Numuzen family instead (sizes: 8b, 1b, or none: kernels only)")
     ap.add_argument("--dotanex", nargs="?", const="8b,1b", default="", help="time the Dotanex family instead (sizes: 8b, 1b, or none: kernels only)")
     ap.add_argument("--dotanex-only", action="store_true", help="with --dotanex: leave the Numuzen model out")
+    ap.add_argument("--sakinex", nargs="?", const="8b,1b", default="", help="time the Sakinex family instead (sizes: 8b, 1b, or none: kernels only)")
+    ap.add_argument("--sakinex-only", action="store_true", help="with --sakinex: leave the Numuzen model out")
     ap.add_argument("--numuzen-only", action="store_true", help="with --numuzen: leave the Tofazen model out")
     args = ap.parse_args()
+    if args.sakinex:
+        run_sakinex(args)
+        return
     if args.dotanex:
         run_dotanex(args)
         return
