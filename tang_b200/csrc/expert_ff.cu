@@ -52,7 +52,7 @@ int launch_expert_ff(tq_ctx* ctx, const ExpertFf& f, const ExpertBuffers& b, con
   mix.y_rows = b.route.slot;
   mix.y_weight = b.route.weight;
   mix.n_y = (int)f.top;
-  mix.self = x;
+  if (f.identity) mix.self = x;
   return TQ_OK;
 }
 

@@ -33,7 +33,7 @@ struct ExpertBuffers {
   float *y = nullptr, *y_shared = nullptr;   // [rows * top][width], [rows][width]
 };
 
-// x rows of `width` values, ldx apart, of `dtype`; fills y, y_rows, y_weight, n_y, y_more and self of `mix`.
+// x rows of `width` values, ldx apart, of `dtype`; fills y, y_rows, y_weight, n_y, y_more and, for identity experts, self of `mix`.
 int launch_expert_ff(tq_ctx* ctx, const ExpertFf& f, const ExpertBuffers& b, const void* x, size_t ldx, size_t rows, size_t width, int dtype, StreamMix& mix);
 
 }  // namespace tq

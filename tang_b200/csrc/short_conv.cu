@@ -89,83 +89,148 @@ __device__ __forceinline__ void sc_push(const ShortConv& c, int col, int crow, c
   sc_store<T, V>(st + (size_t)(c.taps - 2) * c.channels, cur);
 }
 
-// Convolution along consecutive rows for V channels of one thread.  TAPS > 0: weights and the last inputs in registers; 0: any
-// number of taps, inputs read again for every row.
-template <typename T, int V, int TAPS>
-struct ConvRun {
-  float w[TAPS ? TAPS : 1][V], hist[TAPS > 1 ? TAPS - 1 : 1][V];
-  int last = -1;                       // cache row of the row before; -1: the window has to be filled
-
-  __device__ __forceinline__ void weights(const ShortConv& c, int col, bool live) {
-    if constexpr (TAPS > 0) {
+// y = conv at row m for V channels, whose input is cur; any number of taps, every input read again.
+template <typename T, int V>
+__device__ __forceinline__ void conv_any(const ShortConv& c, const T* x, size_t ldx, int col, int m, int pos, int crow, const int* cache_row, const float (&cur)[V],
+                                         float (&y)[V]) {
 #pragma unroll
-      for (int t = 0; t < TAPS; ++t)
-        sc_weights<V>(c.w + (size_t)t * c.channels + col, live, w[t]);
+  for (int j = 0; j < V; ++j) y[j] = 0.f;
+  for (int t = 0; t < c.taps; ++t) {
+    float f[V], wt[V];
+    if (t == c.taps - 1) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) f[j] = cur[j];
+    } else {
+      sc_before<T, V>(c, x, ldx, col, m, c.taps - 1 - t, pos, crow, cache_row, f);
+    }
+    sc_weights<V>(c.w + (size_t)t * c.channels + col, true, wt);
+#pragma unroll
+    for (int j = 0; j < V; ++j) y[j] = fmaf(wt[j], f[j], y[j]);
+  }
+}
+
+// Up to kMaxFixedTaps taps: R consecutive rows and the TAPS - 1 rows ahead of them, V channels per thread, all loaded at once.  STEP:
+// one row per sequence, whose predecessors are all in the state.
+//   cr[TAPS - 1 + r]: cache row of row r of the run, cr[TAPS - 2 - k] of the row k + 1 before the run; impossible values where there is none
+template <typename T, int V, int TAPS, int R, bool STEP>
+struct ConvWindow {
+  static constexpr int H = TAPS - 1, N = STEP ? 1 : R + H;      // rows of x in registers
+  float w[TAPS][V];
+  uint4 x[N];
+
+  __device__ __forceinline__ void weights(const ShortConv& c, int col, bool on) {
+#pragma unroll
+    for (int t = 0; t < TAPS; ++t) sc_weights<V>(c.w + (size_t)t * c.channels + col, on, w[t]);
+  }
+  // (rows of the batch that are no predecessors are loaded all the same, rows outside it are not)
+  __device__ __forceinline__ void load(const T* src, size_t ld, int col, int m0, int rows, bool on) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const int m = m0 + i - (STEP ? 0 : H);
+      x[i] = on && m >= 0 && m < rows ? *reinterpret_cast<const uint4*>(src + (size_t)m * ld + col) : make_uint4(0u, 0u, 0u, 0u);
     }
   }
-
-  // y = conv at row m, whose input is cur
-  __device__ __forceinline__ void step(const ShortConv& c, const T* x, size_t ldx, int col, int m, int pos, int crow, const int* cache_row, const float (&cur)[V],
-                                       float (&y)[V]) {
-    if constexpr (TAPS > 0) {
-      if (TAPS > 1 && (last < 0 || last != crow - 1 || pos == 0)) {
+  static __device__ __forceinline__ void unpack(const uint4& u, float (&f)[V]) {
+    const uint32_t b[4] = {u.x, u.y, u.z, u.w};
 #pragma unroll
-        for (int t = 0; t < TAPS - 1; ++t) sc_before<T, V>(c, x, ldx, col, m, TAPS - 1 - t, pos, crow, cache_row, hist[t]);
+    for (int j = 0; j < V; ++j) f[j] = V == 4 ? __uint_as_float(b[j & 3]) : bf16_bits_to_float(j & 1 ? b[(j >> 1) & 3] >> 16 : b[(j >> 1) & 3] & 0xFFFFu);
+  }
+  // Row r's input and convolution; STEP moves the state on.
+  __device__ __forceinline__ void row(const ShortConv& c, int col, int r, int pos, const int* cr, bool on, float (&cur)[V], float (&y)[V]) {
+    unpack(x[STEP ? 0 : r + H], cur);
+#pragma unroll
+    for (int j = 0; j < V; ++j) y[j] = w[H][j] * cur[j];
+    const int crow = cr[r + H];
+    uint4 old[H ? H : 1];
+    uint4* st = nullptr;
+    int n = 0;                                           // predecessors in the batch
+    if constexpr (H > 0) {
+      if constexpr (!STEP) {
+        while (n < H && cr[r + H - 1 - n] == crow - 1 - n) ++n;
+        if (n > pos) n = pos;
       }
-      last = crow;
+      st = reinterpret_cast<uint4*>(static_cast<T*>(c.state) + (size_t)(crow / c.max_seq) * H * c.channels + col);
+      if (n < H) {
 #pragma unroll
-      for (int j = 0; j < V; ++j) {
-        float s = 0.f;
-#pragma unroll
-        for (int t = 0; t < TAPS - 1; ++t) s = fmaf(w[t][j], hist[t][j], s);
-        y[j] = fmaf(w[TAPS - 1][j], cur[j], s);
-      }
-#pragma unroll
-      for (int t = 0; t < TAPS - 1; ++t)
-#pragma unroll
-        for (int j = 0; j < V; ++j) hist[t][j] = t + 1 < TAPS - 1 ? hist[t + 1][j] : cur[j];
-    } else {
-#pragma unroll
-      for (int j = 0; j < V; ++j) y[j] = 0.f;
-      for (int t = 0; t < c.taps; ++t) {
-        float f[V];
-        if (t == c.taps - 1) {
-#pragma unroll
-          for (int j = 0; j < V; ++j) f[j] = cur[j];
-        } else {
-          sc_before<T, V>(c, x, ldx, col, m, c.taps - 1 - t, pos, crow, cache_row, f);
+        for (int t = 0; t < H; ++t) {
+          const int k = H - t;                           // rows before row r
+          old[t] = on && k > n && pos >= k ? st[(size_t)(H - (k - n)) * (c.channels / V)] : make_uint4(0u, 0u, 0u, 0u);
         }
-        float wt[V];
-        sc_weights<V>(c.w + (size_t)t * c.channels + col, true, wt);
+      }
 #pragma unroll
-        for (int j = 0; j < V; ++j) y[j] = fmaf(wt[j], f[j], y[j]);
+      for (int t = 0; t < H; ++t) {
+        const int k = H - t;
+        float f[V];
+        if (STEP) unpack(old[t], f);
+        else unpack(k <= n ? x[r + t] : old[t], f);
+#pragma unroll
+        for (int j = 0; j < V; ++j) y[j] = fmaf(w[t][j], f[j], y[j]);
+      }
+      if (STEP && on) {
+#pragma unroll
+        for (int t = 0; t + 1 < H; ++t) st[(size_t)t * (c.channels / V)] = old[t + 1];
+        st[(size_t)(H - 1) * (c.channels / V)] = x[0];
       }
     }
   }
 };
 
-// A thread owns V channels of `run` consecutive rows.
-template <typename T, int V, int TAPS>
-__global__ void __launch_bounds__(kScThreads) conv_residual_kernel(ShortConv c, RaggedBatch b, int run, int push, const T* x, size_t ldx, T* out, size_t ldo) {
+// The metadata of a run of R rows: cache rows (see ConvWindow) and positions; rows that are skipped have a negative cache row.
+template <int R, int H>
+__device__ __forceinline__ void run_rows(const RaggedBatch& b, int m0, int* cr, int* pos) {
+  const int i = threadIdx.x;
+  if (i < R + H) {
+    const int m = m0 + i - H;
+    int c = m >= 0 && m < b.rows ? b.cache_row[m] : -1;
+    if (c < 0 || (size_t)c >= b.cache_rows) c = -0x40000000;
+    cr[i] = c;
+    if (i >= H) pos[i - H] = m < b.rows ? b.row_pos[m] : 0;
+  }
+}
+
+constexpr int kScRun = 8;           // rows per thread in prompts
+
+// A thread owns V channels of R consecutive rows.
+template <typename T, int TAPS, int R, bool STEP>
+__global__ void __launch_bounds__(kScThreads) conv_residual_kernel(ShortConv c, RaggedBatch b, const T* x, size_t ldx, T* out, size_t ldo) {
+  constexpr int V = 16 / (int)sizeof(T), H = TAPS - 1;
+  __shared__ int cr[R + H], ps[R];
   const int col = (blockIdx.y * kScThreads + threadIdx.x) * V;
-  if (col >= c.channels) return;
-  ConvRun<T, V, TAPS> r;
-  r.weights(c, col, true);
+  const bool on = col < c.channels;
+  ConvWindow<T, V, TAPS, R, STEP> win;
+  win.weights(c, on ? col : 0, on);
   pdl_wait();
   pdl_launch_dependents();
-  const int m0 = blockIdx.x * run, m1 = min(m0 + run, b.rows);
-#pragma unroll 4
-  for (int m = m0; m < m1; ++m) {
-    const int crow = b.cache_row[m], pos = b.row_pos[m];
-    if (crow < 0 || (size_t)crow >= b.cache_rows) continue;
+  const int m0 = blockIdx.x * R;
+  win.load(x, ldx, col, m0, b.rows, on);
+  run_rows<R, H>(b, m0, cr, ps);
+  __syncthreads();
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    if (cr[r + H] < 0) continue;
     float cur[V], y[V];
-    sc_load<T, V>(x + (size_t)m * ldx + col, cur);
-    r.step(c, x, ldx, col, m, pos, crow, b.cache_row, cur, y);
+    win.row(c, col, r, ps[r], cr, on, cur, y);
 #pragma unroll
     for (int j = 0; j < V; ++j) y[j] += cur[j];
-    sc_store<T, V>(out + (size_t)m * ldo + col, y);
-    if (push) sc_push<T, V>(c, col, crow, cur);
+    if (on) sc_store<T, V>(out + (size_t)(m0 + r) * ldo + col, y);
   }
+}
+
+// The same for any number of taps, size and alignment; a thread per V channels of a row.
+template <typename T, int V>
+__global__ void __launch_bounds__(kScThreads) conv_residual_any_kernel(ShortConv c, RaggedBatch b, int push, const T* x, size_t ldx, T* out, size_t ldo) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int col = (blockIdx.y * kScThreads + threadIdx.x) * V, m = blockIdx.x;
+  const int crow = b.cache_row[m], pos = b.row_pos[m];
+  if (col >= c.channels || crow < 0 || (size_t)crow >= b.cache_rows) return;
+  float cur[V], y[V];
+  sc_load<T, V>(x + (size_t)m * ldx + col, cur);
+  conv_any<T, V>(c, x, ldx, col, m, pos, crow, b.cache_row, cur, y);
+#pragma unroll
+  for (int j = 0; j < V; ++j) y[j] += cur[j];
+  sc_store<T, V>(out + (size_t)m * ldo + col, y);
+  if (push) sc_push<T, V>(c, col, crow, cur);
 }
 
 // Mean over the block's cache rows, one V-piece of one cache (keys, then values) per thread and turn.
@@ -193,61 +258,76 @@ __device__ __forceinline__ void pool_block(const ConvHeads& a, size_t seq0, size
   }
 }
 
-// Cosines and sines of the CTA's rows: cs [run][half] cosine, then sine.
-__device__ __forceinline__ void row_angles(const Rotation& rot, const int* row_pos, int m0, int m1, float* cs, float* sn) {
+// Cosines and sines of `n` rows: [row][half] each.
+__device__ __forceinline__ void row_angles(const Rotation& rot, const int* pos, int n, float* cs, float* sn) {
   const int half = rot.dims / 2;
-  for (int i = threadIdx.x; i < (m1 - m0) * half; i += blockDim.x) {
+  for (int i = threadIdx.x; i < n * half; i += blockDim.x) {
     const int r = i / half, d = i - r * half;
     float s, c;
-    sincosf((float)row_pos[m0 + r] * rot.freq[d], &s, &c);
+    sincosf((float)pos[r] * rot.freq[d], &s, &c);
     cs[i] = c * rot.mult;
     sn[i] = s * rot.mult;
   }
 }
 
-// blockIdx.x: `run` consecutive rows; the CTA's lane groups (and blockIdx.y's CTAs) share the heads: queries, keys, values.  A head's
+// blockIdx.x: R consecutive rows; the CTA's lane groups (and blockIdx.y's CTAs) share the heads: queries, keys, values.  A head's
 // 16-byte pieces sit in the registers of up to 32 lanes, which pass the other half of a pair through shuffles.
-template <typename T, int TAPS>
-__global__ void __launch_bounds__(256) conv_heads_reg_kernel(ConvHeads a, RaggedBatch b, int run, int push, int lanes) {
+template <typename T, int TAPS, int R, bool STEP>
+__global__ void __launch_bounds__(256) conv_heads_reg_kernel(ConvHeads a, RaggedBatch b, int lanes) {
   extern __shared__ __align__(16) float sc_smem[];
-  constexpr int V = 16 / (int)sizeof(T);
+  constexpr int V = 16 / (int)sizeof(T), H = TAPS - 1;
+  __shared__ int cr[R + H], ps[R];
   const int half = a.rot.dims / 2, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
-  float *cs = sc_smem, *sn = sc_smem + run * half;
-  const int l = lane & (lanes - 1), d0 = l * V, per_warp = 32 / lanes;
+  float *cs = sc_smem, *sn = sc_smem + R * half;
+  const int l = lane & (lanes - 1), d0 = l * V, per_warp = 32 / lanes, total = a.heads + 2 * a.kv_heads, stride = warps * gridDim.y * per_warp;
+  const int m0 = blockIdx.x * R;
+  const T* raw = static_cast<const T*>(a.raw);
+  const bool turns = d0 < 2 * half, lead = d0 < half;
+  const int other = !turns ? lane : lead ? lane + half / V : lane - half / V, p0 = !turns ? 0 : lead ? d0 : d0 - half;
+  ConvWindow<T, V, TAPS, R, STEP> win;
+  // the lane's head, its kind, its number among the kind, and its first raw column
+  int h = (blockIdx.y * warps + warp) * per_warp + lane / lanes;
+  bool is_q, is_v, on;
+  int g, col;
+  auto locate = [&]() {
+    is_q = h < a.heads;
+    is_v = h >= a.heads + a.kv_heads;
+    on = h < total && d0 < (is_v ? a.vdim : a.dim);
+    g = is_q ? h : is_v ? h - a.heads - a.kv_heads : h - a.heads;
+    col = !on ? 0 : is_q ? g * a.dim + d0 : is_v ? a.v0 + g * a.vdim + d0 : a.k0 + g * a.dim + d0;
+  };
+  locate();
+  win.weights(a.conv, col, on);
   pdl_wait();
   pdl_launch_dependents();
-  const int m0 = blockIdx.x * run, m1 = min(m0 + run, b.rows);
-  row_angles(a.rot, b.row_pos, m0, m1, cs, sn);
+  win.load(raw, a.ld, col, m0, b.rows, on);
+  run_rows<R, H>(b, m0, cr, ps);
   __syncthreads();
-  const bool turns = d0 < 2 * half, lead = d0 < half;
-  const int other = !turns ? lane : lead ? lane + half / V : lane - half / V, p0 = lead ? d0 : d0 - half;
-  const int total = a.heads + 2 * a.kv_heads;
-  for (int h0 = (blockIdx.y * warps + warp) * per_warp; h0 < total; h0 += warps * gridDim.y * per_warp) {
-    const int h = h0 + lane / lanes;
-    const bool is_q = h < a.heads, is_v = h >= a.heads + a.kv_heads, on = h < total && d0 < (is_v ? a.vdim : a.dim);
-    const int g = is_q ? h : is_v ? h - a.heads - a.kv_heads : h - a.heads;
-    const int col = is_q ? g * a.dim + d0 : is_v ? a.v0 + g * a.vdim + d0 : a.k0 + g * a.dim + d0;
-    const T* raw = static_cast<const T*>(a.raw);
-    ConvRun<T, V, TAPS> r;
-    r.weights(a.conv, col, on);
-    for (int m = m0; m < m1; ++m) {
-      const int crow = b.cache_row[m], pos = b.row_pos[m];
-      if (crow < 0 || (size_t)crow >= b.cache_rows) continue;
-      float cur[V], y[V];
+  row_angles(a.rot, ps, R, cs, sn);
+  __syncthreads();
+  for (int first = h - lane / lanes; first < total; first += stride) {     // (the same number of turns for every lane)
+    if (first != h - lane / lanes) {
+      h = first + lane / lanes;
+      locate();
+      win.weights(a.conv, col, on);
+      win.load(raw, a.ld, col, m0, b.rows, on);
+    }
 #pragma unroll
-      for (int j = 0; j < V; ++j) cur[j] = y[j] = 0.f;
-      if (on) {
-        sc_load<T, V>(raw + (size_t)m * a.ld + col, cur);
-        r.step(a.conv, raw, a.ld, col, m, pos, crow, b.cache_row, cur, y);
-        if (push) sc_push<T, V>(a.conv, col, crow, cur);
-      }
-      float out[V], sq = 0.f;
+    for (int r = 0; r < R; ++r) {
+      const int crow = cr[r + H];
+      if (crow < 0) continue;
+      float cur[V], y[V], out[V], sq = 0.f;
+      win.row(a.conv, col, r, ps[r], cr, on, cur, y);
 #pragma unroll
-      for (int j = 0; j < V; ++j) {
-        const float o = __shfl_sync(0xffffffffu, y[j], other);
-        const int p = (m - m0) * half + p0 + j;
-        out[j] = turns && !is_v ? y[j] * cs[p] + (lead ? -o : o) * sn[p] : y[j];
-        sq += out[j] * out[j];
+      for (int j = 0; j < V; j += 4) {
+        const float4 c4 = *reinterpret_cast<const float4*>(cs + r * half + p0 + j), s4 = *reinterpret_cast<const float4*>(sn + r * half + p0 + j);
+        const float c[4] = {c4.x, c4.y, c4.z, c4.w}, s[4] = {s4.x, s4.y, s4.z, s4.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float o = __shfl_sync(0xffffffffu, y[j + i], other);
+          out[j + i] = turns && !is_v ? y[j + i] * c[i] + (lead ? -o : o) * s[i] : y[j + i];
+          sq += out[j + i] * out[j + i];
+        }
       }
       if (a.norm) {
         for (int o = lanes / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
@@ -256,18 +336,16 @@ __global__ void __launch_bounds__(256) conv_heads_reg_kernel(ConvHeads a, Ragged
         for (int j = 0; j < V; ++j) out[j] *= inv;
       }
       if (on) {
-        T* dst = is_q ? static_cast<T*>(a.q) + (size_t)m * a.ldq + (size_t)g * a.dim
+        T* dst = is_q ? static_cast<T*>(a.q) + (size_t)(m0 + r) * a.ldq + (size_t)g * a.dim
                       : is_v ? static_cast<T*>(a.values) + ((size_t)crow * a.kv_heads + g) * a.val_pad : static_cast<T*>(a.keys) + ((size_t)crow * a.kv_heads + g) * a.key_pad;
         sc_store<T, V>(dst + d0, out);
       }
     }
   }
-  if (push && a.pool) {                                   // (one row per sequence)
-    for (int m = m0; m < m1; ++m) {
-      const int crow = b.cache_row[m], pos = b.row_pos[m];
-      if (crow < 0 || (size_t)crow >= b.cache_rows || pos == 0 || pos % a.pool) continue;
+  if constexpr (STEP) {
+    const int crow = cr[H], pos = ps[0];
+    if (a.pool && crow >= 0 && pos > 0 && pos % a.pool == 0)
       pool_block<T, V>(a, (size_t)(crow - pos), (size_t)(crow / a.conv.max_seq), pos / a.pool - 1, blockIdx.y * blockDim.x + threadIdx.x, gridDim.y * blockDim.x);
-    }
   }
 }
 
@@ -282,7 +360,7 @@ __global__ void __launch_bounds__(256) conv_heads_kernel(ConvHeads a, RaggedBatc
   pdl_launch_dependents();
   const int m = blockIdx.x, crow = b.cache_row[m], pos = b.row_pos[m];
   if (crow < 0 || (size_t)crow >= b.cache_rows) return;
-  row_angles(a.rot, b.row_pos, m, m + 1, cs, sn);
+  row_angles(a.rot, b.row_pos + m, 1, cs, sn);
   __syncthreads();
   const T* raw = static_cast<const T*>(a.raw);
   for (int h = blockIdx.y * warps + warp; h < a.heads + 2 * a.kv_heads; h += warps * gridDim.y) {
@@ -294,8 +372,7 @@ __global__ void __launch_bounds__(256) conv_heads_kernel(ConvHeads a, RaggedBatc
       float cur[1], y[1];
       sc_load<T, 1>(raw + (size_t)m * a.ld + col0 + d, cur);
       if (a.conv.w) {
-        ConvRun<T, 1, 0> r;
-        r.step(a.conv, raw, a.ld, col0 + d, m, pos, crow, b.cache_row, cur, y);
+        conv_any<T, 1>(a.conv, raw, a.ld, col0 + d, m, pos, crow, b.cache_row, cur, y);
         if (push) sc_push<T, 1>(a.conv, col0 + d, crow, cur);
       } else {
         y[0] = cur[0];
@@ -377,26 +454,31 @@ __global__ void put_conv_kernel(const void* src, int s_dt, float* w, size_t chan
 
 template <typename T>
 int conv_residual_typed(tq_ctx* ctx, const ShortConv& c, const RaggedBatch& b, const void* x, size_t ldx, void* out, size_t ldo) {
-  constexpr int VV = 16 / (int)sizeof(T);
+  constexpr int V = 16 / (int)sizeof(T);
   const uintptr_t bits = (uintptr_t)x | (uintptr_t)out | (uintptr_t)c.state;
-  const bool vec = c.channels % VV == 0 && ldx % VV == 0 && ldo % VV == 0 && (bits & 15) == 0;
-  auto go = [&](auto kern, int v) -> int {
-    const int cols = (c.channels / v + (c.channels % v != 0) + kScThreads - 1) / kScThreads;
-    const long long per_row = cols;
-    // as long as there are a few CTAs per SM, a thread walks several rows
-    int run = 1;
-    while (run < 32 && b.max_q > 1 && (long long)(b.rows / (2 * run)) * per_row >= 4ll * ctx->sm_count) run *= 2;
-    TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)((b.rows + run - 1) / run), (unsigned)cols), dim3(kScThreads), 0, c, b, run, (int)(b.max_q <= 1),
-                          static_cast<const T*>(x), ldx, static_cast<T*>(out), ldo));
+  const bool vec = c.channels % V == 0 && ldx % V == 0 && ldo % V == 0 && (bits & 15) == 0, step = b.max_q <= 1;
+  auto cols = [&](int v) { return (unsigned)((c.channels + v * kScThreads - 1) / (v * kScThreads)); };
+  if (!vec || c.taps > kMaxFixedTaps) {
+    auto any = [&](auto kern, int v) -> int {
+      TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)b.rows, cols(v)), dim3(kScThreads), 0, c, b, (int)step, static_cast<const T*>(x), ldx, static_cast<T*>(out), ldo));
+      return TQ_OK;
+    };
+    return vec ? any(conv_residual_any_kernel<T, V>, V) : any(conv_residual_any_kernel<T, 1>, 1);
+  }
+  // a few CTAs per SM before a thread takes several rows
+  const bool run = !step && (long long)b.rows / kScRun * cols(V) >= ctx->sm_count;
+  auto go = [&](auto taps) -> int {
+    constexpr int N = decltype(taps)::value;
+    auto kern = step ? conv_residual_kernel<T, N, 1, true> : run ? conv_residual_kernel<T, N, kScRun, false> : conv_residual_kernel<T, N, 1, false>;
+    const int rows = run ? kScRun : 1;
+    TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)((b.rows + rows - 1) / rows), cols(V)), dim3(kScThreads), 0, c, b, static_cast<const T*>(x), ldx, static_cast<T*>(out), ldo));
     return TQ_OK;
   };
-  if (!vec) return go(conv_residual_kernel<T, 1, 0>, 1);
   switch (c.taps) {
-    case 1: return go(conv_residual_kernel<T, VV, 1>, VV);
-    case 2: return go(conv_residual_kernel<T, VV, 2>, VV);
-    case 3: return go(conv_residual_kernel<T, VV, 3>, VV);
-    case 4: return go(conv_residual_kernel<T, VV, 4>, VV);
-    default: return go(conv_residual_kernel<T, VV, 0>, VV);
+    case 1: return go(std::integral_constant<int, 1>());
+    case 2: return go(std::integral_constant<int, 2>());
+    case 3: return go(std::integral_constant<int, 3>());
+    default: return go(std::integral_constant<int, 4>());
   }
 }
 
@@ -410,23 +492,24 @@ int conv_heads_typed(tq_ctx* ctx, const ConvHeads& a, const RaggedBatch& b) {
   if (vec) {
     int lanes = 1;
     while (lanes < widest / V) lanes *= 2;
-    const int units = (total + 32 / lanes - 1) / (32 / lanes), warps = units < 8 ? units : 8;
-    int run = 1;
-    while (run < 8 && !push && (long long)(b.rows / (2 * run)) * ((units + warps - 1) / warps) >= 2ll * ctx->sm_count) run *= 2;
-    const long long blocks = (b.rows + run - 1) / run;
-    int y = 1;
+    const int units = (total + 32 / lanes - 1) / (32 / lanes);
+    const bool run = !push && (long long)b.rows / kScRun * units >= 8ll * ctx->sm_count;
+    const int rows = run ? kScRun : 1, warps = units < 8 ? units : 8;
+    const long long blocks = (b.rows + rows - 1) / rows;
+    int y = 1;                                            // a head per warp when the rows alone do not fill the GPU
     while (y * warps < units && blocks * y < 4ll * ctx->sm_count) ++y;
-    const size_t smem = ((size_t)run * a.rot.dims + 4) * sizeof(float);
-    auto go = [&](auto kern) -> int {
-      if (smem > 48 * 1024) TQ_CUDA(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-      TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)blocks, (unsigned)y), dim3((unsigned)(32 * warps)), smem, a, b, run, push, lanes));
+    const size_t smem = ((size_t)rows * a.rot.dims + V) * sizeof(float);
+    auto go = [&](auto taps) -> int {
+      constexpr int N = decltype(taps)::value;
+      auto kern = push ? conv_heads_reg_kernel<T, N, 1, true> : run ? conv_heads_reg_kernel<T, N, kScRun, false> : conv_heads_reg_kernel<T, N, 1, false>;
+      TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)blocks, (unsigned)y), dim3((unsigned)(32 * warps)), smem, a, b, lanes));
       return TQ_OK;
     };
     switch (a.conv.taps) {
-      case 1: return go(conv_heads_reg_kernel<T, 1>);
-      case 2: return go(conv_heads_reg_kernel<T, 2>);
-      case 3: return go(conv_heads_reg_kernel<T, 3>);
-      default: return go(conv_heads_reg_kernel<T, 4>);
+      case 1: return go(std::integral_constant<int, 1>());
+      case 2: return go(std::integral_constant<int, 2>());
+      case 3: return go(std::integral_constant<int, 3>());
+      default: return go(std::integral_constant<int, 4>());
     }
   }
   const int warps = total < 8 ? total : 8;

@@ -214,11 +214,168 @@ __global__ void __launch_bounds__(512) stream_mix_kernel(StreamMix a, int width)
   }
 }
 
+// A decode step's form of one stream with a convolution: the row, its norm's gain, the convolution's weights and inputs in registers,
+// NV vectors of four columns per thread.  Weights are read before the wait, everything else right behind it.
+template <typename OT>
+using SmRaw = std::conditional_t<sizeof(OT) == 2, uint2, float4>;
+__device__ __forceinline__ SmVec<4> sm_unpack(uint2 u) {
+  SmVec<4> r;
+  r.v[0] = bf16_bits_to_float(u.x & 0xFFFFu), r.v[1] = bf16_bits_to_float(u.x >> 16);
+  r.v[2] = bf16_bits_to_float(u.y & 0xFFFFu), r.v[3] = bf16_bits_to_float(u.y >> 16);
+  return r;
+}
+__device__ __forceinline__ SmVec<4> sm_unpack(float4 f) {
+  SmVec<4> r;
+  r.v[0] = f.x, r.v[1] = f.y, r.v[2] = f.z, r.v[3] = f.w;
+  return r;
+}
+
+constexpr int kSmStepThreads = 512;
+
+template <typename OT, int NV, int TAPS>
+__global__ void __launch_bounds__(kSmStepThreads) stream_step_kernel(StreamMix a, int width) {
+  using Raw = SmRaw<OT>;
+  __shared__ float red[32];
+  SmVec<4> gain[NV], w[TAPS][NV], x[NV];
+  const int n_thr = blockDim.x;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = 4 * (threadIdx.x + i * n_thr);
+    const bool on = d < width;
+    gain[i] = on ? sm_load<4>(a.gain + d) : SmVec<4>{};
+#pragma unroll
+    for (int t = 0; t < TAPS; ++t) w[t][i] = on ? sm_load<4>(a.conv_w + (size_t)t * width + d) : SmVec<4>{};
+  }
+  const float keep = a.y ? a.mix[0] : 1.f, mult = a.y ? a.w_out[0] : 0.f;
+  pdl_wait();
+  pdl_launch_dependents();
+  const size_t m = blockIdx.x;
+  const int crow = a.cache_row[m], pos = a.row_pos[m];
+  const float logit = a.y_more_gate ? a.y_more_gate[m * a.ld_gate] : 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = 4 * (threadIdx.x + i * n_thr);
+    x[i] = d < width ? sm_load<4>(a.src + m * width + d) : SmVec<4>{};
+  }
+  Raw* st = static_cast<Raw*>(a.conv_state) + ((size_t)(crow < 0 ? 0 : crow / a.max_seq) * (TAPS - 1) * width) / 4;   // (a row without a slot reads slot 0's)
+  Raw hist[TAPS > 1 ? TAPS - 1 : 1][NV];
+#pragma unroll
+  for (int t = 0; t < TAPS - 1; ++t)
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int v = threadIdx.x + i * n_thr;
+      if (4 * v < width) hist[t][i] = st[(size_t)t * (width / 4) + v];
+      else hist[t][i] = Raw{};
+    }
+  if (a.y) {
+    SmVec<4> y[NV] = {};
+    for (int k0 = 0; k0 < a.n_y; k0 += 4) {
+      int r[4];
+      float wy[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const bool on = k0 + k < a.n_y;
+        r[k] = !on ? -1 : a.y_rows ? a.y_rows[m * a.n_y + k0 + k] : (int)m;
+        wy[k] = on && a.y_weight ? a.y_weight[m * a.n_y + k0 + k] : 1.f;
+      }
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int d = 4 * (threadIdx.x + i * n_thr);
+        SmVec<4> part[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) part[k] = r[k] >= 0 && d < width ? sm_load<4>(a.y + (size_t)r[k] * width + d) : SmVec<4>{};
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) y[i].v[j] = fmaf(wy[k], part[k].v[j], y[i].v[j]);
+      }
+    }
+    const float more = a.y_more_gate ? 1.0f / (1.0f + expf(-logit)) : 1.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = 4 * (threadIdx.x + i * n_thr);
+      if (d >= width) continue;
+      if (a.y_more) {
+        const SmVec<4> part = sm_load<4>(a.y_more + m * width + d);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[i].v[j] = fmaf(more, part.v[j], y[i].v[j]);
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) x[i].v[j] = fmaf(keep, x[i].v[j], mult * y[i].v[j]);
+      if (a.sum) sm_store<4>(a.sum + m * width + d, x[i]);
+      if (a.inject) {
+        const SmVec<4> part = sm_load<4>(a.inject + m * width + d);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) x[i].v[j] += part.v[j];
+      }
+      sm_store<4>(a.dst + m * width + d, x[i]);
+    }
+  }
+  const float u_mult = a.w_in ? a.w_in[0] : 1.f;
+  float sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      x[i].v[j] *= u_mult;
+      sq += x[i].v[j] * x[i].v[j];
+    }
+  sq = warp_sum(sq);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = sq;
+  __syncthreads();
+  sq = warp_sum((threadIdx.x & 31) < (blockDim.x >> 5) ? red[threadIdx.x & 31] : 0.f);
+  const float inv = 1.0f / sqrtf(sq / (float)width + a.eps);
+  OT* out = static_cast<OT*>(a.out) + m * a.ld_out;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int v = threadIdx.x + i * n_thr, d = 4 * v;
+    if (d >= width) continue;
+    SmVec<4> h;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) h.v[j] = x[i].v[j] * inv * gain[i].v[j];
+    sm_round<OT, 4>(h);
+    SmVec<4> o = h;
+#pragma unroll
+    for (int t = 0; t < TAPS - 1; ++t) {
+      const SmVec<4> in = sm_unpack(hist[t][i]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) o.v[j] = fmaf(w[t][i].v[j], pos < TAPS - 1 - t ? 0.f : in.v[j], o.v[j]);
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o.v[j] = fmaf(w[TAPS - 1][i].v[j], h.v[j], o.v[j]);
+    sm_store<4>(out + d, o);
+    if (TAPS > 1 && crow >= 0) {
+#pragma unroll
+      for (int t = 0; t + 2 < TAPS; ++t) st[(size_t)t * (width / 4) + v] = hist[t + 1][i];
+      sm_store<4>(reinterpret_cast<OT*>(st + (size_t)(TAPS - 2) * (width / 4) + v), h);
+    }
+  }
+}
+
+template <typename OT>
+static int stream_step_typed(tq_ctx* ctx, const StreamMix& a, size_t rows, size_t width) {
+  auto go = [&](auto taps) -> int {
+    constexpr int T = decltype(taps)::value;
+    const size_t vecs = width / 4;
+    auto kern = vecs <= kSmStepThreads ? stream_step_kernel<OT, 1, T> : stream_step_kernel<OT, 2, T>;
+    const size_t per = vecs <= kSmStepThreads ? vecs : (vecs + 1) / 2;
+    TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)rows), dim3((unsigned)((per + 31) / 32 * 32)), 0, a, (int)width));
+    return TQ_OK;
+  };
+  switch (a.conv_taps) {
+    case 1: return go(std::integral_constant<int, 1>());
+    case 2: return go(std::integral_constant<int, 2>());
+    case 3: return go(std::integral_constant<int, 3>());
+    default: return go(std::integral_constant<int, 4>());
+  }
+}
+
 template <typename OT>
 static int stream_mix_typed(tq_ctx* ctx, const StreamMix& a, size_t rows, size_t width) {
   const uintptr_t bits = (uintptr_t)a.src | (uintptr_t)a.dst | (uintptr_t)a.y | (uintptr_t)a.y_more | (uintptr_t)a.gain | (uintptr_t)a.out | (uintptr_t)a.self |
                          (uintptr_t)a.sum | (uintptr_t)a.inject | (uintptr_t)a.conv_w | (uintptr_t)a.conv_state;
   const bool vec = a.streams <= 4 && width % 4 == 0 && a.ld_out % 4 == 0 && (bits & 15) == 0;
+  if (vec && a.conv_w && a.conv_taps <= 4 && a.streams == 1 && !a.self && !a.src_rows && width <= 8 * (size_t)kSmStepThreads) return stream_step_typed<OT>(ctx, a, rows, width);
   const size_t smem = a.gain ? width * sizeof(float) : 0;
   size_t threads = vec ? width / 4 : width;
   const size_t most = rows >= 2 * (size_t)ctx->sm_count ? 256 : 512, least = a.streams > 4 ? 256 : 64;
