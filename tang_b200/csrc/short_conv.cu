@@ -135,41 +135,46 @@ struct ConvWindow {
 #pragma unroll
     for (int j = 0; j < V; ++j) f[j] = V == 4 ? __uint_as_float(b[j & 3]) : bf16_bits_to_float(j & 1 ? b[(j >> 1) & 3] >> 16 : b[(j >> 1) & 3] & 0xFFFFu);
   }
+  __device__ __forceinline__ void add(int t, const uint4& u, float (&y)[V]) {
+    float f[V];
+    unpack(u, f);
+#pragma unroll
+    for (int j = 0; j < V; ++j) y[j] = fmaf(w[t][j], f[j], y[j]);
+  }
   // Row r's input and convolution; STEP moves the state on.
   __device__ __forceinline__ void row(const ShortConv& c, int col, int r, int pos, const int* cr, bool on, float (&cur)[V], float (&y)[V]) {
     unpack(x[STEP ? 0 : r + H], cur);
 #pragma unroll
     for (int j = 0; j < V; ++j) y[j] = w[H][j] * cur[j];
-    const int crow = cr[r + H];
-    uint4 old[H ? H : 1];
-    uint4* st = nullptr;
-    int n = 0;                                           // predecessors in the batch
     if constexpr (H > 0) {
+      const int crow = cr[r + H];
+      int n = 0;                                         // predecessors in the batch
       if constexpr (!STEP) {
         while (n < H && cr[r + H - 1 - n] == crow - 1 - n) ++n;
         if (n > pos) n = pos;
-      }
-      st = reinterpret_cast<uint4*>(static_cast<T*>(c.state) + (size_t)(crow / c.max_seq) * H * c.channels + col);
-      if (n < H) {
+        if (n == H) {
 #pragma unroll
-        for (int t = 0; t < H; ++t) {
-          const int k = H - t;                           // rows before row r
-          old[t] = on && k > n && pos >= k ? st[(size_t)(H - (k - n)) * (c.channels / V)] : make_uint4(0u, 0u, 0u, 0u);
+          for (int t = 0; t < H; ++t) add(t, x[r + t], y);
+          return;
         }
+      }
+      uint4* st = reinterpret_cast<uint4*>(static_cast<T*>(c.state) + (size_t)(crow / c.max_seq) * H * c.channels + col);
+      const int ld = c.channels / V;
+      uint4 old[H];
+#pragma unroll
+      for (int t = 0; t < H; ++t) {
+        const int k = H - t;                             // rows before row r
+        old[t] = on && k > n && pos >= k ? st[(H - (k - n)) * ld] : make_uint4(0u, 0u, 0u, 0u);
       }
 #pragma unroll
       for (int t = 0; t < H; ++t) {
-        const int k = H - t;
-        float f[V];
-        if (STEP) unpack(old[t], f);
-        else unpack(k <= n ? x[r + t] : old[t], f);
-#pragma unroll
-        for (int j = 0; j < V; ++j) y[j] = fmaf(w[t][j], f[j], y[j]);
+        if constexpr (STEP) add(t, old[t], y);
+        else add(t, H - t <= n ? x[r + t] : old[t], y);
       }
       if (STEP && on) {
 #pragma unroll
-        for (int t = 0; t + 1 < H; ++t) st[(size_t)t * (c.channels / V)] = old[t + 1];
-        st[(size_t)(H - 1) * (c.channels / V)] = x[0];
+        for (int t = 0; t + 1 < H; ++t) st[t * ld] = old[t + 1];
+        st[(H - 1) * ld] = x[0];
       }
     }
   }
@@ -188,7 +193,7 @@ __device__ __forceinline__ void run_rows(const RaggedBatch& b, int m0, int* cr, 
   }
 }
 
-constexpr int kScRun = 8;           // rows per thread in prompts
+constexpr int kScRun = 8, kScShortRun = 4;     // rows per thread in prompts, when there are many and when there are some
 
 // A thread owns V channels of R consecutive rows.
 template <typename T, int TAPS, int R, bool STEP>
@@ -245,12 +250,19 @@ __device__ __forceinline__ void pool_block(const ConvHeads& a, size_t seq0, size
     float s[V];
 #pragma unroll
     for (int j = 0; j < V; ++j) s[j] = 0.f;
-#pragma unroll 8
-    for (int t = 0; t < a.pool; ++t) {
-      float f[V];
-      sc_load<T, V>(src + (size_t)t * w * V, f);
+    for (int t0 = 0; t0 < a.pool; t0 += 8) {              // eight rows in flight
+      float f[8][V];
 #pragma unroll
-      for (int j = 0; j < V; ++j) s[j] += f[j];
+      for (int t = 0; t < 8; ++t) {
+        if (t0 + t < a.pool) sc_load<T, V>(src + (size_t)(t0 + t) * w * V, f[t]);
+        else
+#pragma unroll
+          for (int j = 0; j < V; ++j) f[t][j] = 0.f;
+      }
+#pragma unroll
+      for (int t = 0; t < 8; ++t)
+#pragma unroll
+        for (int j = 0; j < V; ++j) s[j] += f[t][j];
     }
 #pragma unroll
     for (int j = 0; j < V; ++j) s[j] *= inv;
@@ -282,19 +294,24 @@ __global__ void __launch_bounds__(256) conv_heads_reg_kernel(ConvHeads a, Ragged
   const int l = lane & (lanes - 1), d0 = l * V, per_warp = 32 / lanes, total = a.heads + 2 * a.kv_heads, stride = warps * gridDim.y * per_warp;
   const int m0 = blockIdx.x * R;
   const T* raw = static_cast<const T*>(a.raw);
+  const float inv_dim = 1.0f / (float)a.dim;
   const bool turns = d0 < 2 * half, lead = d0 < half;
   const int other = !turns ? lane : lead ? lane + half / V : lane - half / V, p0 = !turns ? 0 : lead ? d0 : d0 - half;
   ConvWindow<T, V, TAPS, R, STEP> win;
   // the lane's head, its kind, its number among the kind, and its first raw column
   int h = (blockIdx.y * warps + warp) * per_warp + lane / lanes;
   bool is_q, is_v, on;
-  int g, col;
+  int col;
+  T* dst;                                                 // of row 0 (queries) or cache row 0
+  size_t dst_ld;
   auto locate = [&]() {
     is_q = h < a.heads;
     is_v = h >= a.heads + a.kv_heads;
     on = h < total && d0 < (is_v ? a.vdim : a.dim);
-    g = is_q ? h : is_v ? h - a.heads - a.kv_heads : h - a.heads;
+    const int g = is_q ? h : is_v ? h - a.heads - a.kv_heads : h - a.heads;
     col = !on ? 0 : is_q ? g * a.dim + d0 : is_v ? a.v0 + g * a.vdim + d0 : a.k0 + g * a.dim + d0;
+    dst = d0 + (is_q ? static_cast<T*>(a.q) + (size_t)g * a.dim : is_v ? static_cast<T*>(a.values) + (size_t)g * a.val_pad : static_cast<T*>(a.keys) + (size_t)g * a.key_pad);
+    dst_ld = is_q ? a.ldq : (size_t)a.kv_heads * (is_v ? a.val_pad : a.key_pad);
   };
   locate();
   win.weights(a.conv, col, on);
@@ -316,6 +333,7 @@ __global__ void __launch_bounds__(256) conv_heads_reg_kernel(ConvHeads a, Ragged
     for (int r = 0; r < R; ++r) {
       const int crow = cr[r + H];
       if (crow < 0) continue;
+      const bool rotates = turns && !is_v;
       float cur[V], y[V], out[V], sq = 0.f;
       win.row(a.conv, col, r, ps[r], cr, on, cur, y);
 #pragma unroll
@@ -325,21 +343,17 @@ __global__ void __launch_bounds__(256) conv_heads_reg_kernel(ConvHeads a, Ragged
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const float o = __shfl_sync(0xffffffffu, y[j + i], other);
-          out[j + i] = turns && !is_v ? y[j + i] * c[i] + (lead ? -o : o) * s[i] : y[j + i];
+          out[j + i] = rotates ? fmaf(o, lead ? -s[i] : s[i], y[j + i] * c[i]) : y[j + i];
           sq += out[j + i] * out[j + i];
         }
       }
       if (a.norm) {
         for (int o = lanes / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
-        const float inv = is_v ? 1.0f : 1.0f / sqrtf(sq / (float)a.dim + a.eps);
+        const float inv = is_v ? 1.0f : rsqrtf(sq * inv_dim + a.eps);
 #pragma unroll
         for (int j = 0; j < V; ++j) out[j] *= inv;
       }
-      if (on) {
-        T* dst = is_q ? static_cast<T*>(a.q) + (size_t)(m0 + r) * a.ldq + (size_t)g * a.dim
-                      : is_v ? static_cast<T*>(a.values) + ((size_t)crow * a.kv_heads + g) * a.val_pad : static_cast<T*>(a.keys) + ((size_t)crow * a.kv_heads + g) * a.key_pad;
-        sc_store<T, V>(dst + d0, out);
-      }
+      if (on) sc_store<T, V>(dst + (size_t)(is_q ? m0 + r : crow) * dst_ld, out);
     }
   }
   if constexpr (STEP) {
@@ -466,11 +480,12 @@ int conv_residual_typed(tq_ctx* ctx, const ShortConv& c, const RaggedBatch& b, c
     return vec ? any(conv_residual_any_kernel<T, V>, V) : any(conv_residual_any_kernel<T, 1>, 1);
   }
   // a few CTAs per SM before a thread takes several rows
-  const bool run = !step && (long long)b.rows / kScRun * cols(V) >= ctx->sm_count;
+  auto fills = [&](int rows) { return !step && (long long)b.rows / rows * cols(V) >= 2ll * ctx->sm_count; };
+  const int rows = fills(kScRun) ? kScRun : fills(kScShortRun) ? kScShortRun : 1;
   auto go = [&](auto taps) -> int {
     constexpr int N = decltype(taps)::value;
-    auto kern = step ? conv_residual_kernel<T, N, 1, true> : run ? conv_residual_kernel<T, N, kScRun, false> : conv_residual_kernel<T, N, 1, false>;
-    const int rows = run ? kScRun : 1;
+    auto kern = step ? conv_residual_kernel<T, N, 1, true> : rows == kScRun ? conv_residual_kernel<T, N, kScRun, false>
+                : rows == kScShortRun ? conv_residual_kernel<T, N, kScShortRun, false> : conv_residual_kernel<T, N, 1, false>;
     TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)((b.rows + rows - 1) / rows), cols(V)), dim3(kScThreads), 0, c, b, static_cast<const T*>(x), ldx, static_cast<T*>(out), ldo));
     return TQ_OK;
   };
@@ -493,15 +508,17 @@ int conv_heads_typed(tq_ctx* ctx, const ConvHeads& a, const RaggedBatch& b) {
     int lanes = 1;
     while (lanes < widest / V) lanes *= 2;
     const int units = (total + 32 / lanes - 1) / (32 / lanes);
-    const bool run = !push && (long long)b.rows / kScRun * units >= 8ll * ctx->sm_count;
-    const int rows = run ? kScRun : 1, warps = units < 8 ? units : 8;
+    auto fills = [&](int n, int per_sm) { return !push && (long long)b.rows / n * units >= (long long)per_sm * ctx->sm_count; };
+    const int rows = fills(kScRun, 8) ? kScRun : fills(kScShortRun, 6) ? kScShortRun : 1;
+    const int parts = (units + 7) / 8, warps = (units + parts - 1) / parts;      // up to eight warps, all of them with heads
     const long long blocks = (b.rows + rows - 1) / rows;
     int y = 1;                                            // a head per warp when the rows alone do not fill the GPU
     while (y * warps < units && blocks * y < 4ll * ctx->sm_count) ++y;
     const size_t smem = ((size_t)rows * a.rot.dims + V) * sizeof(float);
     auto go = [&](auto taps) -> int {
       constexpr int N = decltype(taps)::value;
-      auto kern = push ? conv_heads_reg_kernel<T, N, 1, true> : run ? conv_heads_reg_kernel<T, N, kScRun, false> : conv_heads_reg_kernel<T, N, 1, false>;
+      auto kern = push ? conv_heads_reg_kernel<T, N, 1, true> : rows == kScRun ? conv_heads_reg_kernel<T, N, kScRun, false>
+                  : rows == kScShortRun ? conv_heads_reg_kernel<T, N, kScShortRun, false> : conv_heads_reg_kernel<T, N, 1, false>;
       TQ_CUDA(ctx, launch_k(ctx, kern, dim3((unsigned)blocks, (unsigned)y), dim3((unsigned)(32 * warps)), smem, a, b, lanes));
       return TQ_OK;
     };
