@@ -595,8 +595,8 @@ TQ_API int tq_window_attention_sinks(tq_ctx* ctx, const tq_window_attn_config* c
                                      size_t ldq, const void* gate_dev_or_null, size_t ldg, const void* k_cache_dev, const void* v_cache_dev,
                                      size_t cache_rows, const int* seq_rows_dev_or_null, const int* row_pos_dev, const int* cache_row_dev,
                                      size_t n_seqs, size_t rows, size_t max_q, size_t max_len, void* out_dev, size_t ldo);
-/* The same with one key and one value for each block of `pool` tokens that lies wholly before the window (0: none): the query at
- * position i sees block b too when b pool + pool - 1 <= i - window, under the same softmax.  Pooled rows have the layout of the cache
+/* The same with an averaged key and value per block of `pool` older tokens (0: none): once the window of the query at position i has
+ * moved past all of block b, b pool + pool - 1 <= i - window, the block is one more term of its softmax.  Pooled rows have the layout of the cache
  * rows; block b of a slot is row slot * pool_rows + b, and a slot has max_seq cache rows.  The result is multiplied by out_scale. */
 TQ_API int tq_window_attention_pooled(tq_ctx* ctx, const tq_window_attn_config* cfg, const float* sinks_dev_or_null, int dtype, const void* q_dev,
                                       size_t ldq, const void* gate_dev_or_null, size_t ldg, const void* k_cache_dev, const void* v_cache_dev,
@@ -612,7 +612,7 @@ TQ_API int tq_conv_residual(tq_ctx* ctx, int dtype, size_t channels, size_t taps
                             size_t rows, size_t max_q, size_t max_len, void* out_dev, size_t ldo);
 /* tq_conv_heads: rows of raw queries (heads * dim at column 0), keys (kv_heads * dim at k0) and values (kv_heads * vdim at v0).
  * All are convolved (channels: the raw columns; w NULL: not); queries and keys are rotated (first rot_dims dimensions, in halves, freq
- * [rot_dims / 2], cos and sin times rot_mult) and, if norm, divided by their root mean square per head.  Queries go to q, keys and
+ * [rot_dims / 2], cos and sin times rot_mult) and, if norm, rms-normed per head.  Queries go to q, keys and
  * values to the row's cache row ([kv_heads][dim or vdim padded to 8], zero padding).  pool > 0: the means of blocks of `pool` keys and
  * values are left in the pooled rows (as in tq_window_attention_pooled) as soon as a later row can need them. */
 typedef struct tq_conv_heads_config {
@@ -771,7 +771,7 @@ TQ_API int tq_dotanex_trace(tq_dotanex* model, float* sums_dev_or_null);
 
 /* ---- Sakinex ------------------------------------------------------------------------------------
  * No reference counterpart.  A decoder with one residual stream, x <- x + residual_mult * sublayer(h), h = n + conv(n), n = norm(x),
- * whose mixer runs two branches side by side on the same h,
+ * whose mixer has two branches on the same h,
  *   mixer = left_scale * attention(h) + right_scale * recurrence(h),
  * attention with short convolutions on queries, keys and values, YaRN rotation in halves, a gainless query/key norm per head behind
  * it, a sliding window and pooled blocks before the window (tq_conv_heads, tq_window_attention_pooled), and a minGRU (tq_min_gru).

@@ -1,4 +1,4 @@
-// minGRU: a gated recurrence per channel whose gates read only the current row,
+// minGRU: per channel, a leaky average whose rate and input depend on the current row alone,
 //     z = sigmoid(z_t + z_bias);  u = u_t + u_bias;  c = u + 1/2 where u >= 0, sigmoid(u) where u < 0
 //     S_t = (1 - z) S_(t-1) + z c;   out_t = S_t * silu(gate_t) * out_scale
 // The state starts at zero with a sequence's position 0 and is kept in f32 from step to step, one per cache slot.

@@ -1,5 +1,5 @@
 // Sakinex: a decoder with one residual stream whose mixers run windowed attention (convolved queries, keys and values, pooled blocks
-// before the window) and a minGRU side by side on the same input, each followed by routed experts with a gated shared one; every
+// behind the window) and a minGRU on the same input, each followed by routed experts with a gated shared one; every
 // sublayer's input passes a short convolution, and a stretch of layers may run several times (include/tangq.h, tq_sakinex_*).
 //
 // A run of a layer is

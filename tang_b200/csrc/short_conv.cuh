@@ -28,8 +28,8 @@ int put_conv_weights(tq_ctx* ctx, const void* src, int src_dtype, float* w, size
 int launch_conv_residual(tq_ctx* ctx, const ShortConv& c, const RaggedBatch& b, int dtype, const void* x, size_t ldx, void* out, size_t ldo);
 
 // What follows the projections of attention: raw rows hold queries, keys and values at columns 0, k0 and v0 (the convolution's
-// channels are the raw columns); queries and keys are convolved, rotated, and divided by their root mean square per head (no
-// gain; norm false: not); values are only convolved.  Queries go to q, keys and values to the row's cache row.
+// channels are the raw columns); queries and keys are convolved, rotated and rms-normed per head (no gain; norm
+// false: not); values are only convolved.  Queries go to q, keys and values to the row's cache row.
 // Blocks of `pool` tokens (0: none) get one pooled row each, the mean of their keys and of their values as the cache holds them.
 // A step forms the rows of the blocks whose last position is at least its first one minus 1 and lies before its last one: a
 // block is complete in the cache one row before any query behind it can see it.

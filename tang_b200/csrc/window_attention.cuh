@@ -4,9 +4,9 @@
 //     out = (sum p_j v_j) * sigmoid(gate)                             (no gate pointer: 1)
 // Mask: the query at position i sees key j when j <= i and i - j < window.
 //
-// Pooled blocks (pool > 0): beside these, it sees one key and one value for each block of `pool` tokens that lies wholly before its
-// window -- block b of the sequence when b pool + pool - 1 <= i - window -- under the same softmax.  Tokens that have left the
-// window and whose block is not there yet are not seen.
+// Pooled blocks (pool > 0): positions b pool .. b pool + pool - 1 have an averaged key and value, which are one more term of the
+// softmax once the window has moved past all of them, b pool + pool - 1 <= i - window.  Until then the positions that the window
+// has dropped count for nothing.
 #pragma once
 
 #include "internal.h"

@@ -1,8 +1,8 @@
 """Sakinex (``tq_sakinex_*`` in include/tangq.h): configuration, weight loading and the model.
 
-A small decoder whose mixers run attention and a minGRU side by side on the same input.  The attention convolves its queries, keys
-and values over the last few tokens, rotates them (YaRN), norms queries and keys per head behind the rotation, and sees a sliding
-window and one pooled key and value per block of tokens before it.  Every sublayer's input passes a short convolution; the
+A small decoder whose mixers run attention and a minGRU on the same input.  The attention convolves its queries, keys and values
+over the last few tokens, rotates them (YaRN), norms queries and keys per head behind the rotation, and sees a sliding window and
+averages over blocks of older tokens.  Every sublayer's input passes a short convolution; the
 feed-forwards are routed experts with a gated shared one; a stretch of layers may run several times with the same weights, each
 pass with caches and states of its own.  No counterpart in the reference.
 """

@@ -58,7 +58,7 @@ def seen_tokens(i, size):
 
 
 def seen_blocks(i, size, pool):
-    """Blocks of `pool` tokens that lie wholly before its window."""
+    """Blocks that its window has moved past."""
     return [b for b in range(i // pool + 1) if b * pool + pool - 1 <= i - size]
 
 

@@ -37,7 +37,7 @@ def test_a_loop_equals_its_layers_written_out():
 
 def test_numpy_mechanisms_by_hand():
     assert X.seen_tokens(9, 3) == [7, 8, 9] and X.seen_tokens(1, 3) == [0, 1]
-    # blocks of 4 before a window of 3 at position 9: the window starts at 7, so 0..3 is wholly before it and 4..7 is not
+    # blocks of 4 before a window of 3 at position 9: the window starts at 7, so it has passed 0..3 and still touches 4..7
     assert X.seen_blocks(9, 3, 4) == [0] and X.seen_blocks(10, 3, 4) == [0, 1] and X.seen_blocks(6, 3, 4) == [0] and X.seen_blocks(5, 3, 4) == []
     assert X.seen_blocks(2, 1, 1) == [0, 1]
     q, k, v = np.array([2.0]), np.array([[1.0], [3.0], [0.5]]), np.array([[1.0], [2.0], [5.0]])
